@@ -48,6 +48,10 @@ int      llava_dequantize(const void* in, int type, uint32_t model_version, floa
 
 /* ---- llava_context (llava_context.h:21-42) */
 void*    llava_context_open(const char* model_path, int device);   /* NULL on failure */
+/* a ggjt file or a model folder (config.json, model.safetensors); f32 != 0: 32-bit arithmetic where the model leaves the
+ * choice (model folders), else bfloat16 */
+void*    llava_context_open_dtype(const char* model_path, int device, int f32);
+const char* llava_context_architecture(void* ctx);                 /* name of the model's design */
 /* the model file only (vocabulary, tensor table), no device: serves the front end's session-independent requests */
 void*    llava_context_open_model_only(const char* model_path);
 /* tensor-parallel: this process is rank `rank` of `n_ranks`, one GPU each; nccl_id = the 128 bytes
@@ -69,6 +73,10 @@ int      llava_context_run(int argc, char** argv);                  /* the comma
 
 /* ---- llava_session (llava_session.h:44-62) */
 void*    llava_session_create(void* ctx);
+/* a session that may hold max_context tokens (0: the default); NULL when the model or the memory does not allow it */
+void*    llava_session_create_sized(void* ctx, uint32_t max_context);
+/* evaluates the pushed tokens and returns the logits [n][vocab] of the wanted ones (indexes into the token buffer) */
+int      llava_session_evaluate_pending(void* session, const uint32_t* wanted, uint32_t n, float* logits);
 void     llava_session_destroy(void* session);
 int      llava_session_set_text(void* session, const char* text, size_t len);
 int      llava_session_add_text(void* session, const char* text, size_t len);

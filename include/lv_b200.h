@@ -45,7 +45,9 @@ enum { LV_TYPE_F32 = 0, LV_TYPE_F16 = 1, LV_TYPE_Q4_0 = 2, LV_TYPE_Q8_0 = 8,
         * elements 2j (low nibble) and 2j+1 (high); accepted by lv_gemv, lv_norm_gemv, lv_gemv_silu,
         * lv_norm_gate_up_silu, lv_norm_qkv_kvappend and lv_dequant_rows (the shaders matmul_dim.comp /
         * matmul_silu_ff.comp without the _fp16 suffix).  Not a GGML code: such files say "q4_0" too. */
-       LV_TYPE_Q4_0_V1 = 258 };
+       LV_TYPE_Q4_0_V1 = 258,
+       /* bfloat16 and 32-bit integers of safetensors files, under GGML's codes */
+       LV_TYPE_I32 = 26, LV_TYPE_BF16 = 30 };
 
 typedef struct lv_ctx lv_ctx;
 typedef struct lv_graph lv_graph;
@@ -182,7 +184,7 @@ int lv_argmax_advance(lv_ctx* ctx, const float* v, uint32_t n, uint32_t* config,
  * std::mt19937; here the cumulative distribution of the same candidates (in index order) is inverted at a uniform
  * variate from a counter-based generator (Philox 4x32-10) keyed by state[1] and counted in state[2]; a
  * forced_uniform in [0, 1) replaces the generator (tests).  All pointers are device memory:
- *   logits f32 [n_vocab] (16-byte aligned, n_vocab <= 32768); token_log u32, *n_tokens tokens of history;
+ *   logits f32 [n_vocab] (16-byte aligned, n_vocab <= 2^24); token_log u32, *n_tokens tokens of history;
  *   state u32 [4] = {mu as f32 bits, seed, draws so far, unused}, updated;
  *   feed_token_log (may be null): the drawn token is also stored to feed_token_log[*n_tokens], where a recorded
  *   step that follows reads its input token (index checked against log_capacity);
@@ -386,6 +388,108 @@ int lv_step_plan_read_trace(lv_step_plan* plan, uint64_t* out, size_t max_words,
  * host_token: pinned host word or null.  logits (f32 [vocab]) may be null without the head. */
 int lv_decode_step(lv_ctx* ctx, const lv_step_plan* plan, uint32_t* config, uint32_t* token_log, uint32_t log_capacity,
                    float* logits, uint32_t* argmax_out, uint32_t* host_token, int with_head);
+
+/* ---- mechanisms of decoders with bfloat16 weights (no counterpart in the reference) -------------
+ *
+ * Matrices are bfloat16 [rows][ld] with ld a multiple of 8 (rows padded with zeros), 16-byte aligned.  Sums, norms,
+ * scores, softmax, recurrences and the residual stream are f32.  `pos` is the device word with the number of tokens
+ * already evaluated (config[0] of lv_argmax_advance), token t of a launch is at position *pos + t and its id in
+ * token_log[*pos + t]. */
+
+/* The boundary between two sublayers in one launch: residual add of the normalised output of the finished sublayer, an
+ * optional vector added to the stream, the next norm, and a causal convolution over time on its result.
+ *   y_t  = (1 / y_rows) sum_s y[y_index[t * y_rows + s]]   (y[t] without y_index); y null: no sublayer yet
+ *   x_t  = x[t] + mult * y_t / rms(y_t) * (1 + post_w)     -> trace[t] (may be null)
+ *   x_t += step (may be null)                              -> x_out[t] (may be null; may equal x for batch 1)
+ *   h_t  = x_t / rms(x_t) * (1 + pre_w),  rms(v) = sqrt(mean(v^2) + eps)
+ *   out  = h_t + sum_{j < taps} conv_w[j] * h_{t - taps + 1 + j}   (taps 0: out = h_t)
+ * for the tokens first .. batch - 1.  history f32 [taps - 1][width] holds h of the last taps - 1 positions, oldest first,
+ * and is updated (entries of positions before 0 are never read).  With out_index, out row out_index[t * out_copies + s]
+ * is written for every s < out_copies, else row t - first.  x null: rows of the bfloat16 embedding table. */
+typedef struct lv_norm_conv_args {
+    const float* x;
+    const void* embed;
+    uint32_t embed_ld, vocab;
+    const uint32_t* token_log;
+    const uint32_t* pos;
+    const float* y;
+    const uint32_t* y_index;
+    uint32_t y_rows;
+    float mult, eps;
+    const float* post_w;
+    const float* step;
+    float* trace;
+    float* x_out;
+    const float* pre_w;
+    const float* conv_w;            /* [taps][width] */
+    float* history;
+    uint32_t taps;
+    void* out;
+    int out_type;                   /* LV_TYPE_F32 or LV_TYPE_BF16 */
+    uint32_t out_ld;
+    const uint32_t* out_index;
+    uint32_t out_copies;
+    uint32_t width, first, batch;
+} lv_norm_conv_args;
+int lv_norm_conv(lv_ctx* ctx, const lv_norm_conv_args* args);
+
+/* out[t][r] = factor * sum_k W[r][k] x[t][k] in f32 arithmetic (weights are exact in f32).  One pass over the weights per
+ * token. */
+int lv_gemv_bf16(lv_ctx* ctx, float* out, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols, const float* x,
+                 uint32_t x_ld, uint32_t batch, float factor);
+
+/* minGRU for one token: z = sigmoid(Wz x + bz), u = Wx x + bx, c = u + 1/2 (u >= 0) or sigmoid(u),
+ * state = (1 - z) state + z c (0 at position 0), out = state * silu(Wg x). */
+int lv_gemv_bf16_mingru(lv_ctx* ctx, float* out, const void* wz, const void* wx, const void* wg, uint32_t ld, uint32_t channels, uint32_t cols,
+                        const float* bz, const float* bx, const float* x, float* state, const uint32_t* pos);
+/* The same recurrence for `batch` tokens from the three products raw[t] = {Wz x, Wx x, Wg x} (f32, each `channels` long). */
+int lv_mingru_scan(lv_ctx* ctx, void* out, int out_type, uint32_t out_ld, const float* raw, uint32_t raw_ld, uint32_t channels,
+                   const float* bz, const float* bx, float* state, const uint32_t* pos, uint32_t batch);
+
+/* Feed-forward experts chosen by token id: table u32 [vocab][top] gives every id its experts.  w0 (and w1) are the experts'
+ * matrices stacked, [experts * rows][ld].
+ *   gate_up: out[t * top + s] = silu(gate_e x[t]) * (up_e x[t]), e = table[id_t][s] (w0 gate, w1 up; rows = ff, cols = width)
+ *   down:    out[t] = (1 / top) sum_s down_e x[t * top + s]                        (w0 down; rows = width, cols = ff) */
+typedef struct lv_expert_args {
+    const void* w0;
+    const void* w1;
+    uint32_t ld, rows, cols, experts, top, vocab;
+    const uint32_t* table;
+    const uint32_t* token_log;
+    const uint32_t* pos;
+} lv_expert_args;
+int lv_gemv_bf16_expert_gate_up(lv_ctx* ctx, float* out, uint32_t out_ld, const lv_expert_args* a, const float* x, uint32_t x_ld, uint32_t batch);
+int lv_gemv_bf16_expert_down(lv_ctx* ctx, float* out, uint32_t out_ld, const lv_expert_args* a, const float* x, uint32_t x_ld, uint32_t batch);
+
+/* Causal attention with grouped key/value heads: query and key RMS norm per head (plain weights), scores
+ * (q . k) * scale - r1_h ln(1 + r2_h (i - j)), softmax with `sink` (0 or 1) added to the denominator.
+ * qkv f32 [batch][qkv_ld]: heads * dim queries, kv_heads * dim keys, kv_heads * vdim values of each token, as projected.
+ * Caches [kv_heads][ctx_rows][dim rounded up to 8] (values: vdim), cache_type bfloat16 or f32.  dim, vdim <= 256. */
+typedef struct lv_gqa_args {
+    const float* qkv;
+    uint32_t qkv_ld, heads, kv_heads, dim, vdim;
+    float scale, eps;
+    const float* q_norm;            /* [dim] */
+    const float* k_norm;
+    const float* r1;                /* [heads] */
+    const float* r2;
+    int sink;
+    void* k_cache;
+    void* v_cache;
+    int cache_type;
+    uint32_t ctx_rows;
+    const uint32_t* pos;
+    void* out;
+    int out_type;
+    uint32_t out_ld;
+} lv_gqa_args;
+/* normalised keys and values of `batch` tokens to the caches */
+int lv_qk_norm_append(lv_ctx* ctx, const lv_gqa_args* a, uint32_t batch);
+/* The attention of `batch` tokens over their caches.  append != 0 (batch 1): the token's own key and value are appended by
+ * the same launch.  capacity: upper bound of *pos + batch, sizes the grid.  scratch: lv_gqa_scratch_bytes for the largest
+ * batch and capacity used, zero-filled once. */
+size_t lv_gqa_scratch_bytes(lv_ctx* ctx, const lv_gqa_args* a, uint32_t batch, uint32_t capacity);
+int lv_attention_gqa(lv_ctx* ctx, const lv_gqa_args* a, void* scratch, size_t scratch_bytes, uint32_t batch, uint32_t capacity, int append);
 
 /* ---- multi-GPU: one process per GPU, one communicator per context.  The
  *      reference is single-device (llava_context.cpp:264-279 takes one queue of

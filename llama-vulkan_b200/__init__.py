@@ -25,11 +25,34 @@ LV_ERR_COMM = 103
 
 TYPE_F32, TYPE_F16, TYPE_Q4_0, TYPE_Q8_0 = 0, 1, 2, 8
 TYPE_Q4_0_V1 = 258
+TYPE_I32, TYPE_BF16 = 26, 30
 
 _p = C.c_void_p
 _u32 = C.c_uint32
 _sz = C.c_size_t
 _int = C.c_int
+_f32 = C.c_float
+
+
+class NormConvArgs(C.Structure):
+    """lv_norm_conv_args"""
+    _fields_ = [("x", _p), ("embed", _p), ("embed_ld", _u32), ("vocab", _u32), ("token_log", _p), ("pos", _p), ("y", _p), ("y_index", _p),
+                ("y_rows", _u32), ("mult", _f32), ("eps", _f32), ("post_w", _p), ("step", _p), ("trace", _p), ("x_out", _p), ("pre_w", _p),
+                ("conv_w", _p), ("history", _p), ("taps", _u32), ("out", _p), ("out_type", _int), ("out_ld", _u32), ("out_index", _p),
+                ("out_copies", _u32), ("width", _u32), ("first", _u32), ("batch", _u32)]
+
+
+class ExpertArgs(C.Structure):
+    """lv_expert_args"""
+    _fields_ = [("w0", _p), ("w1", _p), ("ld", _u32), ("rows", _u32), ("cols", _u32), ("experts", _u32), ("top", _u32), ("vocab", _u32),
+                ("table", _p), ("token_log", _p), ("pos", _p)]
+
+
+class GqaArgs(C.Structure):
+    """lv_gqa_args"""
+    _fields_ = [("qkv", _p), ("qkv_ld", _u32), ("heads", _u32), ("kv_heads", _u32), ("dim", _u32), ("vdim", _u32), ("scale", _f32), ("eps", _f32),
+                ("q_norm", _p), ("k_norm", _p), ("r1", _p), ("r2", _p), ("sink", _int), ("k_cache", _p), ("v_cache", _p), ("cache_type", _int),
+                ("ctx_rows", _u32), ("pos", _p), ("out", _p), ("out_type", _int), ("out_ld", _u32)]
 
 # name -> (restype, argtypes); mirrors include/lv_b200.h
 KERNEL_API = {
@@ -106,6 +129,15 @@ KERNEL_API = {
     "lv_step_plan_set_trace": (_int, [_p, _int]),
     "lv_step_plan_read_trace": (_int, [_p, _p, _sz, _p, _p, _p]),
     "lv_decode_step": (_int, [_p, _p, _p, _p, _u32, _p, _p, _p, _int]),
+    "lv_norm_conv": (_int, [_p, C.POINTER(NormConvArgs)]),
+    "lv_gemv_bf16": (_int, [_p, _p, _u32, _p, _u32, _u32, _u32, _p, _u32, _u32, _f32]),
+    "lv_gemv_bf16_mingru": (_int, [_p, _p, _p, _p, _p, _u32, _u32, _u32, _p, _p, _p, _p, _p]),
+    "lv_mingru_scan": (_int, [_p, _p, _int, _u32, _p, _u32, _u32, _p, _p, _p, _p, _u32]),
+    "lv_gemv_bf16_expert_gate_up": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _u32, _u32]),
+    "lv_gemv_bf16_expert_down": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _u32, _u32]),
+    "lv_qk_norm_append": (_int, [_p, C.POINTER(GqaArgs), _u32]),
+    "lv_gqa_scratch_bytes": (_sz, [_p, C.POINTER(GqaArgs), _u32, _u32]),
+    "lv_attention_gqa": (_int, [_p, C.POINTER(GqaArgs), _p, _sz, _u32, _u32, _int]),
 }
 
 _kernels = None
@@ -233,6 +265,8 @@ HOST_API = {
     "ggml_file_token": (_u32, [_p, _u32, C.c_char_p, _u32, _f32p]),
     "llava_dequantize": (_int, [_p, _int, _u32, _p, _u32]),
     "llava_context_open": (_p, [C.c_char_p, _int]),
+    "llava_context_open_dtype": (_p, [C.c_char_p, _int, _int]),
+    "llava_context_architecture": (C.c_char_p, [_p]),
     "llava_context_open_model_only": (_p, [C.c_char_p]),
     "llava_context_open_sharded": (_p, [C.c_char_p, _int, _u32, _u32, _p]),
     "llava_context_peer_window_create": (_int, [_p, _p]),
@@ -243,6 +277,8 @@ HOST_API = {
     "llava_context_lv": (_p, [_p]),
     "llava_context_run": (_int, [_int, C.POINTER(C.c_char_p)]),
     "llava_session_create": (_p, [_p]),
+    "llava_session_create_sized": (_p, [_p, _u32]),
+    "llava_session_evaluate_pending": (_int, [_p, _p, _u32, _p]),
     "llava_session_destroy": (None, [_p]),
     "llava_session_set_text": (_int, [_p, C.c_char_p, _sz]),
     "llava_session_add_text": (_int, [_p, C.c_char_p, _sz]),
@@ -386,12 +422,15 @@ class ModelFile:
 class HostContext:
     """llava_context: model + device + uploaded layers."""
 
-    def __init__(self, model_path, device=0, rank=0, n_ranks=1, nccl_id=None):
+    def __init__(self, model_path, device=0, rank=0, n_ranks=1, nccl_id=None, dtype="bfloat16"):
+        """model_path: a ggjt file or a model folder; dtype: arithmetic of model folders (bfloat16 or float32)."""
         self.lib = load_host()
+        if dtype not in ("bfloat16", "float32"):
+            raise ValueError(dtype)
         if device is None:            # the model file only: no device context, no sessions
             self.handle = self.lib.llava_context_open_model_only(os.fsencode(model_path))
         elif n_ranks == 1:
-            self.handle = self.lib.llava_context_open(os.fsencode(model_path), device)
+            self.handle = self.lib.llava_context_open_dtype(os.fsencode(model_path), device, int(dtype == "float32"))
         else:
             buf = (C.c_uint8 * 128).from_buffer_copy(bytes(nccl_id))
             self.handle = self.lib.llava_context_open_sharded(os.fsencode(model_path), device, rank, n_ranks, buf)
@@ -418,8 +457,12 @@ class HostContext:
         if not self.lib.llava_context_peer_connect(self.handle, buf):
             raise RuntimeError("peer connect failed: " + (load_kernels().lv_last_error_string() or b"").decode("utf-8", "replace"))
 
-    def session(self):
-        return Session(self)
+    def architecture(self):
+        return self.lib.llava_context_architecture(self.handle).decode()
+
+    def session(self, max_context=0):
+        """max_context: tokens the session may hold (0: the default)."""
+        return Session(self, max_context)
 
     def set_exact_batched_products(self, on):
         """Batched (prompt) q4_0 products with the exact hi/lo weight planes instead of one fp16 plane (lv_gemm_tc_set_exact).
@@ -430,10 +473,12 @@ class HostContext:
 class Session:
     """llava_session."""
 
-    def __init__(self, ctx):
+    def __init__(self, ctx, max_context=0):
         self.lib = ctx.lib
         self.ctx = ctx
-        self.handle = self.lib.llava_session_create(ctx.handle)
+        self.handle = self.lib.llava_session_create_sized(ctx.handle, max_context)
+        if not self.handle:
+            raise RuntimeError("cannot create the session")
 
     def close(self):
         if self.handle:
@@ -520,6 +565,15 @@ class Session:
         out = np.empty(vocab, np.float32)
         if not self.lib.llava_session_get_logits(self.handle, out.ctypes.data_as(_p), vocab):
             raise RuntimeError("get_logits failed")
+        return out
+
+    def evaluate_pending(self, wanted, vocab):
+        """Evaluates the pushed tokens; logits [len(wanted)][vocab] of the wanted ones (indexes into the token buffer)."""
+        import numpy as np
+        idx = (_u32 * max(len(wanted), 1))(*wanted)
+        out = np.empty((len(wanted), vocab), np.float32)
+        if not self.lib.llava_session_evaluate_pending(self.handle, idx, len(wanted), out.ctypes.data_as(_p)):
+            raise RuntimeError("evaluate_pending failed: " + (load_kernels().lv_last_error_string() or b"").decode("utf-8", "replace"))
         return out
 
     def backlog_size(self):

@@ -3,7 +3,7 @@
     python llama-vulkan_b200/build.py [--force]
 
 Outputs (next to this file): liblv_b200.so (sm_100a kernels + C ABI),
-libllava_host.so (C++ host surface) and the vulkan_llama command-line tool.
+libllava_host.so (C++ host surface) and the command-line tools vulkan_llama and trace_run.
 """
 import os
 import shutil
@@ -14,6 +14,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 ROOT = os.path.dirname(HERE)
 CSRC = os.path.join(HERE, "csrc")
 HOST = os.path.join(HERE, "host")
+PROGRAMS = [("main.cpp", "vulkan_llama"), ("trace_run.cpp", "trace_run")]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -71,7 +72,7 @@ def build_kernels(force=False, verbose_ptxas=False):
 def build_host(force=False):
     if not os.path.isdir(HOST):
         return None
-    cpp = [f for f in _glob(HOST, (".cpp",)) if not f.endswith("main.cpp")] + _glob(os.path.join(HOST, "server"), (".cpp",))
+    cpp = [f for f in _glob(HOST, (".cpp",)) if os.path.basename(f) not in [p[0] for p in PROGRAMS]] + _glob(os.path.join(HOST, "server"), (".cpp",))
     if not cpp:
         return None
     deps = cpp + _glob(HOST, (".h",)) + _glob(os.path.join(HOST, "server"), (".h",)) + [os.path.join(ROOT, "include", "lv_b200.h"), os.path.join(ROOT, "include", "llava_host.h")]
@@ -81,11 +82,12 @@ def build_host(force=False):
     if force or _newer(out, deps):
         _run([cxx, "-std=c++20", "-O2", "-fPIC", "-shared", "-pthread", "-Wall", "-o", out] + cpp +
              ["-L" + HERE, "-llv_b200", "-Wl,-rpath,$ORIGIN", "-Wl,-Bsymbolic"])
-    main = os.path.join(HOST, "main.cpp")
-    exe = os.path.join(HERE, "vulkan_llama")
-    if os.path.exists(main) and (force or _newer(exe, [main, out])):
-        _run([cxx, "-std=c++20", "-O2", "-pthread", "-o", exe, main, "-L" + HERE, "-lllava_host", "-llv_b200",
-              "-Wl,-rpath,$ORIGIN"])
+    for source, program in PROGRAMS:
+        main = os.path.join(HOST, source)
+        exe = os.path.join(HERE, program)
+        if force or _newer(exe, [main, out]):
+            _run([cxx, "-std=c++20", "-O2", "-pthread", "-o", exe, main, "-L" + HERE, "-lllava_host", "-llv_b200",
+                  "-Wl,-rpath,$ORIGIN"])
     return out
 
 
@@ -96,4 +98,9 @@ def build_all(force=False):
 
 
 if __name__ == "__main__":
+    if "--locked" in sys.argv:          # programs that build on demand: one builder at a time
+        import fcntl
+        os.makedirs(os.path.join(HERE, "build"), exist_ok=True)
+        lock = open(os.path.join(HERE, "build", ".lock"), "w")
+        fcntl.flock(lock, fcntl.LOCK_EX)
     build_all(force="--force" in sys.argv)

@@ -1,0 +1,362 @@
+// Causal attention with grouped key/value heads, query/key norm, a distance bias and an optional sink, on CUDA cores in f32.
+//
+//   q'_h = scale * rmsnorm(q_h) * qw,  k'_g = rmsnorm(k_g) * kw
+//   s_ij = q'_i . k'_j - r1_h ln(1 + r2_h (i - j)),  j <= i
+//   p_ij = exp(s_ij) / (sink + sum_j exp(s_ij)),     sink = 1 or 0
+//
+// One CTA serves up to eight query heads of one key/value head for one token and walks its share of the keys in chunks of
+// 128 with an online softmax.  A decoded token spreads the chunks over several CTAs (the last to arrive combines their
+// partial sums through scratch) and its own key and value are normalised and appended to the caches by the same launch;
+// tokens of a prompt are appended first (lv_qk_norm_append).  Caches are [kv head][ctx_rows][padded dim], bfloat16 or f32.
+#include <cuda_bf16.h>
+#include <math.h>
+
+#include "attention_gqa.cuh"
+#include "common.cuh"
+#include "ctx.h"
+
+namespace lv {
+
+constexpr size_t kGqaCounterBytes = 4096;   // arrival counters at the start of the scratch (kept zero between launches)
+constexpr int kGqaThreads = 256, kGqaWarps = 8, kGqaChunk = 128, kGqaHeads = 8;
+
+struct GqaParams {
+    lv_gqa_args a;
+    uint32_t dim_p, vdim_p;         // padded to 8
+    uint32_t head_blocks;           // CTAs per key/value head
+    uint32_t splits;
+    uint32_t out_bf16;
+    float* scratch;                 // splits > 1: [token][head][split][vdim_p + 2]
+    uint32_t* counters;             // [token][kv head * head_blocks]
+    uint32_t* err;
+};
+
+template <typename CT> struct Cache8;
+template <> struct Cache8<__nv_bfloat16> {
+    static __device__ __forceinline__ void load(float (&v)[8], const __nv_bfloat16* p) {
+        const uint4 w = *reinterpret_cast<const uint4*>(p);
+        const uint32_t q[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { v[2 * i] = __uint_as_float(q[i] << 16); v[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u); }
+    }
+    static __device__ __forceinline__ __nv_bfloat16 cast(float v) { return __float2bfloat16_rn(v); }
+    static __device__ __forceinline__ float back(__nv_bfloat16 v) { return __bfloat162float(v); }
+};
+template <> struct Cache8<float> {
+    static __device__ __forceinline__ void load(float (&v)[8], const float* p) {
+        const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    }
+    static __device__ __forceinline__ float cast(float v) { return v; }
+    static __device__ __forceinline__ float back(float v) { return v; }
+};
+
+// Appends the normalised key and the value of token t (one warp per key/value head).
+template <typename CT>
+__global__ void __launch_bounds__(128) qk_norm_append_kernel(const GqaParams p, uint32_t n_tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const lv_gqa_args& a = p.a;
+    const uint32_t job = blockIdx.x * 4u + (threadIdx.x >> 5), lane = threadIdx.x & 31u;
+    if (job >= n_tokens * a.kv_heads) return;
+    const uint32_t t = job / a.kv_heads, g = job - t * a.kv_heads;
+    const uint32_t row = *a.pos + t;
+    if (row >= a.ctx_rows) {
+        if (lane == 0) atomicOr(p.err, ERR_BAD_INDEX);
+        return;
+    }
+    const float* k = a.qkv + size_t(t) * a.qkv_ld + a.heads * a.dim + g * a.dim;
+    const float* v = a.qkv + size_t(t) * a.qkv_ld + (a.heads + a.kv_heads) * a.dim + g * a.vdim;
+    const float r = gqa_rms_factor(k, a.dim, a.eps);
+    CT* kd = static_cast<CT*>(a.k_cache) + (size_t(g) * a.ctx_rows + row) * p.dim_p;
+    CT* vd = static_cast<CT*>(a.v_cache) + (size_t(g) * a.ctx_rows + row) * p.vdim_p;
+    for (uint32_t i = lane; i < p.dim_p; i += 32) kd[i] = Cache8<CT>::cast(i < a.dim ? k[i] * r * a.k_norm[i] : 0.f);
+    for (uint32_t i = lane; i < p.vdim_p; i += 32) vd[i] = Cache8<CT>::cast(i < a.vdim ? v[i] : 0.f);
+}
+
+// HB: query heads of this CTA, rounded up.  LPK: lanes that share a key, VU: threads that share a value row.
+template <typename CT, int HB, bool APPEND>
+__global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) uint8_t smem_raw[];
+    const lv_gqa_args& a = p.a;
+    const uint32_t group = a.heads / a.kv_heads;
+    const uint32_t g = blockIdx.x / p.head_blocks, hb = blockIdx.x - g * p.head_blocks;
+    const uint32_t h0 = g * group + hb * kGqaHeads, nh = min(uint32_t(kGqaHeads), group - hb * kGqaHeads);
+    const uint32_t t = blockIdx.z;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    uint32_t vu = 1;
+    while (vu * 8 < p.vdim_p) vu *= 2;                     // threads across a value row (power of two, <= 32)
+    uint32_t lpk = 8;
+    while (lpk * 8 < p.dim_p) lpk *= 2;                    // lanes across a key (>= the heads of a CTA)
+    float* s_q = reinterpret_cast<float*>(smem_raw);      // [HB][dim_p]
+    float* s_sc = s_q + HB * p.dim_p;                      // [HB][chunk]
+    float* s_red = s_sc + HB * kGqaChunk;                  // [warps][HB][vu * 8]
+    float* s_m = s_red + kGqaWarps * HB * vu * 8;          // [HB] running maximum
+    float* s_l = s_m + HB;                                 // [HB] running sum
+    float* s_c = s_l + HB;                                 // [HB] factor of this chunk
+    CT* s_k = reinterpret_cast<CT*>(s_c + 2 * HB);         // (16-byte aligned) APPEND: the token's own key and value as the cache holds them
+    CT* s_v = s_k + p.dim_p;
+    __shared__ uint32_t s_last;
+
+    pdl_wait();
+    const uint32_t P = *a.pos + t;
+    if (P >= a.ctx_rows) {
+        if (threadIdx.x == 0) atomicOr(p.err, ERR_BAD_INDEX);
+        return;
+    }
+    const float* raw = a.qkv + size_t(t) * a.qkv_ld;
+    if (warp < int(nh)) {
+        const float* q = raw + (h0 + warp) * a.dim;
+        const float r = gqa_rms_factor(q, a.dim, a.eps) * a.scale;
+        for (uint32_t i = lane; i < p.dim_p; i += 32) s_q[warp * p.dim_p + i] = i < a.dim ? q[i] * r * a.q_norm[i] : 0.f;
+    } else if (warp < HB) {
+        for (uint32_t i = lane; i < p.dim_p; i += 32) s_q[warp * p.dim_p + i] = 0.f;
+    }
+    const uint32_t own_chunk = P / kGqaChunk;
+    const bool own = APPEND && own_chunk % p.splits == blockIdx.y;
+    CT* kc = static_cast<CT*>(a.k_cache) + size_t(g) * a.ctx_rows * p.dim_p;
+    CT* vc = static_cast<CT*>(a.v_cache) + size_t(g) * a.ctx_rows * p.vdim_p;
+    if (own && warp == kGqaWarps - 1) {
+        const float* k = raw + a.heads * a.dim + g * a.dim;
+        const float* v = raw + (a.heads + a.kv_heads) * a.dim + g * a.vdim;
+        const float r = gqa_rms_factor(k, a.dim, a.eps);
+        for (uint32_t i = lane; i < p.dim_p; i += 32) {
+            const CT e = Cache8<CT>::cast(i < a.dim ? k[i] * r * a.k_norm[i] : 0.f);
+            s_k[i] = e;
+            if (hb == 0) kc[size_t(P) * p.dim_p + i] = e;
+        }
+        for (uint32_t i = lane; i < p.vdim_p; i += 32) {
+            const CT e = Cache8<CT>::cast(i < a.vdim ? v[i] : 0.f);
+            s_v[i] = e;
+            if (hb == 0) vc[size_t(P) * p.vdim_p + i] = e;
+        }
+    }
+    if (threadIdx.x < HB) { s_m[threadIdx.x] = -INFINITY; s_l[threadIdx.x] = 0.f; }
+    const uint32_t sub = lane & (lpk - 1), key_in_warp = lane / lpk, keys_per_warp = 32 / lpk;
+    const float r1 = sub < nh ? a.r1[h0 + sub] : 0.f, r2 = sub < nh ? a.r2[h0 + sub] : 0.f;
+    const uint32_t vcol = (threadIdx.x & (vu - 1)) * 8, vgroup = threadIdx.x / vu, vgroups = kGqaThreads / vu;
+    float acc[HB][8];
+#pragma unroll
+    for (int h = 0; h < HB; ++h)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) acc[h][i] = 0.f;
+    __syncthreads();
+
+    for (uint32_t c = blockIdx.y; c <= own_chunk; c += p.splits) {
+        const uint32_t k0 = c * kGqaChunk, n = min(uint32_t(kGqaChunk), P + 1 - k0);
+        // scores: lpk lanes share a key
+#pragma unroll 2
+        for (uint32_t kk = warp * keys_per_warp + key_in_warp; kk < kGqaChunk; kk += kGqaWarps * keys_per_warp) {
+            const uint32_t j = k0 + kk;
+            const bool live = kk < n && sub * 8 < p.dim_p;
+            float kv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (live) Cache8<CT>::load(kv, (APPEND && j == P) ? s_k + sub * 8 : kc + size_t(j) * p.dim_p + sub * 8);
+            float mine = 0.f;
+#pragma unroll
+            for (int h = 0; h < HB; ++h) {
+                float s = 0.f;
+                if (live) {
+                    float qv[8];
+                    Cache8<float>::load(qv, s_q + h * p.dim_p + sub * 8);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) s = fmaf(qv[i], kv[i], s);
+                }
+                for (uint32_t o = lpk >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+                if (sub == uint32_t(h)) mine = s;
+            }
+            if (sub < HB) s_sc[sub * kGqaChunk + kk] = (kk < n && sub < nh) ? mine - r1 * log1pf(r2 * float(P - j)) : -INFINITY;
+        }
+        __syncthreads();
+        // online softmax: warp h takes head h
+        if (warp < HB) {
+            float* sc = s_sc + warp * kGqaChunk;
+            float m = -INFINITY;
+            for (int i = lane; i < kGqaChunk; i += 32) m = fmaxf(m, sc[i]);
+            const float m_old = s_m[warp], m_new = fmaxf(m_old, warp_max(m));
+            float l = 0.f;
+            for (int i = lane; i < kGqaChunk; i += 32) {
+                const float e = m_new == -INFINITY ? 0.f : expf(sc[i] - m_new);
+                sc[i] = e;
+                l += e;
+            }
+            l = warp_sum(l);
+            if (lane == 0) {
+                const float f = m_new == -INFINITY ? 1.f : expf(m_old - m_new);
+                s_c[warp] = f;
+                s_m[warp] = m_new;
+                s_l[warp] = s_l[warp] * f + l;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int h = 0; h < HB; ++h) {
+            const float f = s_c[h];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc[h][i] *= f;
+        }
+        if (vcol < p.vdim_p) {
+#pragma unroll 4
+            for (uint32_t kk = vgroup; kk < n; kk += vgroups) {
+                const uint32_t j = k0 + kk;
+                float vv[8];
+                Cache8<CT>::load(vv, (APPEND && j == P) ? s_v + vcol : vc + size_t(j) * p.vdim_p + vcol);
+#pragma unroll
+                for (int h = 0; h < HB; ++h) {
+                    const float pr = s_sc[h * kGqaChunk + kk];
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) acc[h][i] = fmaf(pr, vv[i], acc[h][i]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    // value groups of a warp, then of the CTA, in a fixed order
+#pragma unroll
+    for (int h = 0; h < HB; ++h)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            float v = acc[h][i];
+            for (uint32_t o = vu; o < 32; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+            if (lane < int(vu)) s_red[(warp * HB + h) * vu * 8 + vcol + i] = v;
+        }
+    __syncthreads();
+    const uint32_t vw = vu * 8;
+    const uint32_t part = p.vdim_p + 2;
+    for (uint32_t e = threadIdx.x; e < nh * p.vdim_p; e += kGqaThreads) {
+        const uint32_t h = e / p.vdim_p, col = e - h * p.vdim_p;
+        float v = 0.f;
+        for (int w = 0; w < kGqaWarps; ++w) v += s_red[(w * HB + h) * vw + col];
+        const float m = s_m[h], l = s_l[h];
+        if (p.splits == 1) {
+            if (col < a.vdim) {
+                const float M = a.sink ? fmaxf(m, 0.f) : m, f = expf(m - M);
+                gqa_store_out(a.out, p.out_bf16, size_t(t) * a.out_ld + (h0 + h) * a.vdim + col, v * f / (l * f + (a.sink ? expf(-M) : 0.f)));
+            }
+        } else {
+            float* dst = p.scratch + ((size_t(t) * a.heads + h0 + h) * p.splits + blockIdx.y) * part;
+            dst[2 + col] = v;
+            if (col == 0) { dst[0] = m; dst[1] = l; }
+        }
+    }
+    if (p.splits == 1) return;
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        uint32_t* counter = p.counters + size_t(t) * gridDim.x + blockIdx.x;
+        s_last = atomicAdd(counter, 1u) == p.splits - 1 ? 1u : 0u;
+        if (s_last) *counter = 0u;
+    }
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    for (uint32_t e = threadIdx.x; e < nh * a.vdim; e += kGqaThreads) {
+        const uint32_t h = e / a.vdim, col = e - h * a.vdim;
+        const float* src = p.scratch + (size_t(t) * a.heads + h0 + h) * p.splits * part;
+        float M = a.sink ? 0.f : -INFINITY;
+        for (uint32_t s = 0; s < p.splits; ++s) M = fmaxf(M, __ldcg(src + s * part));
+        float num = 0.f, den = a.sink ? expf(-M) : 0.f;
+        for (uint32_t s = 0; s < p.splits; ++s) {
+            const float f = expf(__ldcg(src + s * part) - M);
+            num = fmaf(f, __ldcg(src + s * part + 2 + col), num);
+            den = fmaf(f, __ldcg(src + s * part + 1), den);
+        }
+        gqa_store_out(a.out, p.out_bf16, size_t(t) * a.out_ld + (h0 + h) * a.vdim + col, num / den);
+    }
+}
+
+static uint32_t pad8(uint32_t n) { return (n + 7) / 8 * 8; }
+
+static uint32_t gqa_head_blocks(const lv_gqa_args& a) { return (a.heads / a.kv_heads + kGqaHeads - 1) / kGqaHeads; }
+
+// CTAs that share a token's keys: enough to fill the SMs about twice, at most one per chunk of the capacity
+static uint32_t gqa_splits(const lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch, uint32_t capacity) {
+    const uint32_t ctas = a.kv_heads * gqa_head_blocks(a) * batch, chunks = (capacity + kGqaChunk - 1) / kGqaChunk;
+    const uint32_t want = (2u * uint32_t(ctx->sm_count) + ctas - 1) / ctas;
+    return want < 1 ? 1 : (want > chunks ? chunks : want);
+}
+
+static int gqa_check(const lv_gqa_args* a, uint32_t batch) {
+    LV_REQUIRE(a && a->qkv && a->q_norm && a->k_norm && a->r1 && a->r2 && a->k_cache && a->v_cache && a->pos && batch && batch <= 65535, "bad attention arguments");
+    LV_REQUIRE(a->heads && a->kv_heads && a->heads % a->kv_heads == 0 && a->dim && a->vdim && a->dim <= 256 && a->vdim <= 256, "attention: unsupported head sizes");
+    LV_REQUIRE(a->qkv_ld >= (a->heads + a->kv_heads) * a->dim + a->kv_heads * a->vdim && a->ctx_rows, "attention: bad strides");
+    LV_REQUIRE(a->cache_type == LV_TYPE_F32 || a->cache_type == LV_TYPE_BF16, "attention: cache type");
+    return LV_OK;
+}
+
+template <typename CT, bool APPEND>
+static int gqa_launch(lv_ctx* ctx, const GqaParams& p, uint32_t batch) {
+    const lv_gqa_args& a = p.a;
+    const uint32_t group = a.heads / a.kv_heads;
+    const int HB = group >= 5 ? 8 : group >= 3 ? 4 : int(group);
+    uint32_t vu = 1;
+    while (vu * 8 < p.vdim_p) vu *= 2;
+    const size_t smem = sizeof(float) * (size_t(HB) * p.dim_p + HB * kGqaChunk + size_t(kGqaWarps) * HB * vu * 8 + 4 * HB) + sizeof(CT) * (p.dim_p + p.vdim_p) + 16;
+    LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "attention: head sizes need too much shared memory");
+    const dim3 grid(a.kv_heads * p.head_blocks, p.splits, batch);
+    auto go = [&](auto kernel) -> cudaError_t {
+        if (smem > 48 * 1024) {
+            const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+            if (e != cudaSuccess) return e;
+        }
+        return launch_pdl(ctx, kernel, grid, dim3(kGqaThreads), smem, p);
+    };
+    if (HB == 8) LV_CUDA(go(gqa_kernel<CT, 8, APPEND>));
+    else if (HB == 4) LV_CUDA(go(gqa_kernel<CT, 4, APPEND>));
+    else if (HB == 2) LV_CUDA(go(gqa_kernel<CT, 2, APPEND>));
+    else LV_CUDA(go(gqa_kernel<CT, 1, APPEND>));
+    return LV_OK;
+}
+
+}  // namespace lv
+
+using namespace lv;
+
+extern "C" size_t lv_gqa_scratch_bytes(lv_ctx* ctx, const lv_gqa_args* a, uint32_t batch, uint32_t capacity) {
+    if (!ctx || !a || !batch || !capacity || !a->kv_heads) return 0;
+    size_t most = 0;
+    for (uint32_t n = 1; n <= batch; n *= 2) {             // splits shrink as the batch grows; every size in between needs no more than 2x
+        const size_t bytes = 2 * size_t(n) * a->heads * gqa_splits(ctx, *a, n, capacity) * (pad8(a->vdim) + 2) * 4;
+        most = bytes > most ? bytes : most;
+    }
+    return most + kGqaCounterBytes;
+}
+
+extern "C" int lv_qk_norm_append(lv_ctx* ctx, const lv_gqa_args* a, uint32_t batch) {
+    LV_ENTER(ctx);
+    if (const int rc = gqa_check(a, batch)) return rc;
+    GqaParams p{};
+    p.a = *a;
+    p.dim_p = pad8(a->dim);
+    p.vdim_p = pad8(a->vdim);
+    p.err = ctx->d_err;
+    const dim3 grid((batch * a->kv_heads + 3) / 4);
+    if (a->cache_type == LV_TYPE_F32) LV_CUDA(launch_pdl(ctx, qk_norm_append_kernel<float>, grid, dim3(128), 0, p, batch));
+    else LV_CUDA(launch_pdl(ctx, qk_norm_append_kernel<__nv_bfloat16>, grid, dim3(128), 0, p, batch));
+    return LV_OK;
+}
+
+extern "C" int lv_attention_gqa(lv_ctx* ctx, const lv_gqa_args* a, void* scratch, size_t scratch_bytes, uint32_t batch, uint32_t capacity, int append) {
+    LV_ENTER(ctx);
+    if (const int rc = gqa_check(a, batch)) return rc;
+    LV_REQUIRE(a->out && a->out_ld >= a->heads * a->vdim && (a->out_type == LV_TYPE_F32 || a->out_type == LV_TYPE_BF16), "attention: bad output");
+    LV_REQUIRE(capacity && capacity <= a->ctx_rows && (!append || batch == 1), "attention: bad capacity");
+    GqaParams p{};
+    p.a = *a;
+    p.dim_p = pad8(a->dim);
+    p.vdim_p = pad8(a->vdim);
+    p.head_blocks = gqa_head_blocks(*a);
+    p.splits = gqa_splits(ctx, *a, batch, capacity);
+    p.out_bf16 = a->out_type == LV_TYPE_BF16;
+    p.err = ctx->d_err;
+    if (p.splits > 1) {
+        // fewer than two CTAs per SM would run unsplit, so the counters of a split launch always fit
+        LV_REQUIRE(size_t(batch) * a->kv_heads * p.head_blocks * 4 <= kGqaCounterBytes, "attention: too many arrival counters");
+        const size_t need = kGqaCounterBytes + size_t(batch) * a->heads * p.splits * (p.vdim_p + 2) * 4;
+        LV_REQUIRE(scratch && scratch_bytes >= need, "attention: scratch too small");
+        p.counters = static_cast<uint32_t*>(scratch);
+        p.scratch = reinterpret_cast<float*>(static_cast<uint8_t*>(scratch) + kGqaCounterBytes);
+    }
+    if (a->cache_type == LV_TYPE_F32) return append ? gqa_launch<float, true>(ctx, p, batch) : gqa_launch<float, false>(ctx, p, batch);
+    return append ? gqa_launch<__nv_bfloat16, true>(ctx, p, batch) : gqa_launch<__nv_bfloat16, false>(ctx, p, batch);
+}

@@ -1,0 +1,22 @@
+// Pieces shared by the attention kernels with query/key norm.
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace lv {
+
+// 1 / rms of one head's vector, computed by a warp (every lane gets it)
+__device__ __forceinline__ float gqa_rms_factor(const float* v, uint32_t dim, float eps) {
+    float part = 0.f;
+    for (uint32_t i = threadIdx.x & 31u; i < dim; i += 32) part = fmaf(v[i], v[i], part);
+    return 1.f / sqrtf(warp_sum(part) / float(dim) + eps);
+}
+
+__device__ __forceinline__ void gqa_store_out(void* out, uint32_t bf16, size_t at, float v) {
+    if (bf16) static_cast<__nv_bfloat16*>(out)[at] = __float2bfloat16_rn(v);
+    else static_cast<float*>(out)[at] = v;
+}
+
+}  // namespace lv

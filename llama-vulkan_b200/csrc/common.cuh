@@ -11,7 +11,7 @@ namespace lv {
 // GGML tensor type codes as they appear in ggjt files.
 // T_Q4_0_V1: the q4_0 blocks of ggjt version 1 files -- f32 scale, byte j holding elements 2j (low nibble) and 2j+1 (high);
 // not a GGML code: the file says "q4_0" and its version says which block layout that is.
-enum : int { T_F32 = 0, T_F16 = 1, T_Q4_0 = 2, T_Q8_0 = 8, T_Q4_0_V1 = 258 };
+enum : int { T_F32 = 0, T_F16 = 1, T_Q4_0 = 2, T_Q8_0 = 8, T_BF16 = 30, T_Q4_0_V1 = 258 };
 
 constexpr int kBlockElems = 32;   // weights per quantisation block
 constexpr int kQ4BlockBytes = 18; // f16 scale + 16 nibble bytes (ggjt v3)
@@ -199,6 +199,19 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 
 __device__ __forceinline__ float half_bits_to_float(uint32_t h16) {
     return __half2float(__ushort_as_half(static_cast<unsigned short>(h16)));
+}
+
+__device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu_f32(float z) { return z / (1.f + expf(-z)); }
+
+// One token of one channel of the minGRU recurrence: S = (1 - sigmoid(z)) S + sigmoid(z) c(u) with c(u) = u + 1/2 for
+// u >= 0 and sigmoid(u) below; returns S * silu(gate).
+__device__ __forceinline__ float mingru_candidate(float u) { return u >= 0.f ? u + 0.5f : sigmoid_f32(u); }
+__device__ __forceinline__ float mingru_step(float z, float u, float gate, float S, float* S_out) {
+    const float k = sigmoid_f32(z);
+    const float next = fmaf(1.f - k, S, k * mingru_candidate(u));
+    *S_out = next;
+    return next * silu_f32(gate);
 }
 
 }  // namespace lv

@@ -18,7 +18,6 @@
 namespace lv {
 
 constexpr int kSampleThreads = 1024;
-constexpr int kSamplePerThread = 32;        // consecutive logits per thread: 32768 >= any vocabulary accepted here
 constexpr uint32_t kNoToken = 0xffffffffu;
 
 // sampler constants, llava_session.h:70-76
@@ -68,7 +67,9 @@ __global__ void __launch_bounds__(kSampleThreads) sample_mirostat_kernel(const f
         count13 = __syncthreads_count(count13 != 0u);
     }
 
-    const uint32_t base = threadIdx.x * kSamplePerThread;
+    // consecutive logits per thread, whole groups of four
+    const uint32_t per_thread = (n + 4 * kSampleThreads - 1) / (4 * kSampleThreads) * 4;
+    const uint32_t base = threadIdx.x * per_thread;
     // exp(logit / temp) of four consecutive tokens, with the penalty on token 13; recomputed in each of the three
     // passes below (the logits stay in L1) rather than held in 32 registers per thread
     auto weights4 = [&](uint32_t i) -> float4 {
@@ -94,7 +95,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_mirostat_kernel(const f
     };
     float local = 0.f;
 #pragma unroll 2
-    for (int k = 0; k < kSamplePerThread; k += 4) {
+    for (uint32_t k = 0; k < per_thread; k += 4) {
         const float4 v = weights4(base + k);
         local += v.x; local += v.y; local += v.z; local += v.w;
     }
@@ -115,7 +116,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_mirostat_kernel(const f
     float kept_local = 0.f;
     uint32_t kept_n = 0, last_kept = kNoToken;
 #pragma unroll 2
-    for (int k = 0; k < kSamplePerThread; k += 4) {
+    for (uint32_t k = 0; k < per_thread; k += 4) {
         const float4 v = weights4(base + k);
         const float q[4] = {v.x / total, v.y / total, v.z / total, v.w / total};
 #pragma unroll
@@ -162,7 +163,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_mirostat_kernel(const f
     uint32_t mine = kNoToken;
     if (kept_n != 0u) {
 #pragma unroll 2
-        for (int k = 0; k < kSamplePerThread; k += 4) {
+        for (uint32_t k = 0; k < per_thread; k += 4) {
             const float4 v = weights4(base + k);
             const float q[4] = {v.x / total, v.y / total, v.z / total, v.w / total};
 #pragma unroll
@@ -179,7 +180,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_mirostat_kernel(const f
     uint32_t pick = s_pick;
     if (pick == kNoToken && s_last_kept != 0u) pick = s_last_kept - 1u;       // rounding left the target at or beyond the total: the last kept token
     // the owner of the drawn token knows its probability
-    if (pick != kNoToken && pick >= base && pick < base + kSamplePerThread) {
+    if (pick != kNoToken && pick >= base && pick < base + per_thread) {
         const float4 v = weights4(pick & ~3u);
         const float w4[4] = {v.x, v.y, v.z, v.w};
         const float q = w4[pick & 3u] / total;
@@ -213,7 +214,7 @@ extern "C" int lv_sample_mirostat(lv_ctx* ctx, const float* logits, uint32_t n_v
                                   uint32_t* host_token, uint32_t* report) {
     LV_ENTER(ctx);
     LV_REQUIRE(logits && token_log && n_tokens && state && n_vocab, "bad sampler arguments");
-    LV_REQUIRE(n_vocab <= uint32_t(kSampleThreads * kSamplePerThread), "vocabulary larger than 32768");
+    LV_REQUIRE(n_vocab <= (1u << 24), "vocabulary larger than 16777216");
     LV_REQUIRE((reinterpret_cast<uintptr_t>(logits) & 15u) == 0, "logits must be 16-byte aligned");
     LV_CUDA(launch_pdl(ctx, sample_mirostat_kernel, dim3(1), dim3(kSampleThreads), 0, logits, n_vocab, token_log, n_tokens, state, forced_uniform,
                        feed_token_log, log_capacity, out_token, static_cast<volatile uint32_t*>(host_token), report, ctx->d_err));

@@ -144,6 +144,18 @@ void* llava_context_open(const char* model_path, int device) {
     return c;
 }
 
+void* llava_context_open_dtype(const char* model_path, int device, int f32) {
+    auto* c = new llava_context();
+    c->set_compute_type(f32 ? compute_type::f32 : compute_type::bf16);
+    if (!c->open(model_path, device)) {
+        delete c;
+        return nullptr;
+    }
+    return c;
+}
+
+const char* llava_context_architecture(void* ctx) { return static_cast<llava_context*>(ctx)->architecture()->name(); }
+
 void* llava_context_open_model_only(const char* model_path) {
     auto* c = new llava_context();
     if (!c->open_model_only(model_path)) {
@@ -192,6 +204,20 @@ int llava_context_run(int argc, char** argv) {
 }
 
 void* llava_session_create(void* ctx) { return new llava_session(static_cast<llava_context*>(ctx)); }
+void* llava_session_create_sized(void* ctx, uint32_t max_context) {
+    auto* s = new llava_session(static_cast<llava_context*>(ctx), max_context);
+    if (!s->is_valid()) {
+        delete s;
+        return nullptr;
+    }
+    return s;
+}
+int llava_session_evaluate_pending(void* session, const uint32_t* wanted, uint32_t n, float* logits) {
+    std::vector<float> v;
+    if (!S(session)->evaluate_pending(std::vector<u32>(wanted, wanted + n), &v)) return 0;
+    if (n) std::memcpy(logits, v.data(), v.size() * sizeof(float));
+    return 1;
+}
 void llava_session_destroy(void* session) { delete S(session); }
 int llava_session_set_text(void* s, const char* text, size_t len) { return S(s)->set_text(std::string(text, len)) ? 1 : 0; }
 int llava_session_add_text(void* s, const char* text, size_t len) { return S(s)->add_text(std::string(text, len)) ? 1 : 0; }

@@ -1,0 +1,383 @@
+#include "hybrid_architecture.h"
+
+#include <algorithm>
+#include <iostream>
+
+#include "hybrid_session_state.h"
+#include "llava_buffer.h"
+#include "llava_command_buffer.h"
+#include "llava_context.h"
+#include "llava_device_memory.h"
+#include "llava_session.h"
+#include "model_folder.h"
+
+using namespace std;
+
+// ---- configuration ---------------------------------------------------------------------------
+
+namespace {
+bool need_u32(const json_value* at, const char* key, u32* out, string* error, u32 least = 1) {
+    const json_value* v = at ? at->find(key) : nullptr;
+    if (v && v->as_u32(out) && *out >= least) return true;
+    *error = string(key) + " missing or out of range";
+    return false;
+}
+
+bool need_float(const json_value* at, const char* key, float* out, string* error) {
+    const json_value* v = at ? at->find(key) : nullptr;
+    if (v && v->as_float(out)) return true;
+    *error = string(key) + " missing or not a number";
+    return false;
+}
+}  // namespace
+
+bool parse_sonuzen_config(const json_value& config, hybrid_config* out, string* error) {
+    hybrid_config& c = *out;
+    if (!need_u32(&config, "width", &c.width, error) || !need_u32(&config, "vocab", &c.vocab, error) ||
+        !need_float(config.find("norm"), "eps", &c.eps, error) || !need_float(&config, "residual_mult", &c.residual_mult, error) ||
+        !need_float(&config, "logit_scale", &c.logit_scale, error) || !need_u32(config.find("canon"), "taps", &c.taps, error))
+        return false;
+    const json_value* layers = config.find("layers");
+    if (!layers || !layers->is_array() || layers->items().empty()) {
+        *error = "layers missing";
+        return false;
+    }
+    for (const json_value& l : layers->items()) {
+        hybrid_layer_spec spec;
+        const json_value *type = l.find("type"), *mixer = l.find("mixer"), *mlp = l.find("mlp");
+        hybrid_mixer& m = spec.mixer;
+        if (type && type->text() == "attention") {
+            m.type = hybrid_mixer::kind::attention;
+            m.sink = true;
+            if (!need_u32(mixer, "heads", &m.heads, error) || !need_u32(mixer, "kv_heads", &m.kv_heads, error) || !need_u32(mixer, "dim", &m.dim, error) ||
+                !need_u32(mixer, "vdim", &m.vdim, error) || !need_float(mixer, "scale", &m.scale, error))
+                return false;
+            if (m.heads % m.kv_heads != 0) {
+                *error = "heads must be a multiple of kv_heads";
+                return false;
+            }
+        } else if (type && type->text() == "mingru") {
+            m.type = hybrid_mixer::kind::mingru;
+            if (!need_u32(mixer, "width", &m.width, error)) return false;
+        } else {
+            *error = "unknown layer type";
+            return false;
+        }
+        if (mlp && !mlp->is_null()) {
+            const json_value* kind = mlp->find("kind");
+            if (kind && kind->text() != "moe") {
+                *error = "unknown feed-forward " + kind->text();
+                return false;
+            }
+            const json_value* router = mlp->find("router");
+            if (!need_u32(mlp->find("expert"), "ff", &spec.mlp.ff, error) || !need_u32(router, "experts", &spec.mlp.experts, error) ||
+                !need_u32(router, "top", &spec.mlp.top, error))
+                return false;
+            if (spec.mlp.top > spec.mlp.experts) {
+                *error = "top exceeds experts";
+                return false;
+            }
+        }
+        c.layers.push_back(spec);
+    }
+    if (const json_value* loop = config.find("loop"); loop && !loop->is_null()) {
+        if (!need_u32(loop, "start", &c.loop_start, error, 0) || !need_u32(loop, "stop", &c.loop_stop, error) || !need_u32(loop, "times", &c.loop_times, error)) return false;
+        if (c.loop_start >= c.loop_stop || c.loop_stop > c.layers.size()) {
+            *error = "loop outside the layers";
+            return false;
+        }
+    }
+    return true;
+}
+
+// ---- model -----------------------------------------------------------------------------------
+
+hybrid_architecture::~hybrid_architecture() {
+    for (llava_buffer* b : tensors) delete b;
+}
+
+bool hybrid_architecture::check(const model_file& model, u32 n_ranks) {
+    string error;
+    const auto* folder = dynamic_cast<const model_folder*>(&model);
+    if (folder == nullptr || !parse_(folder->get_config(), &cfg, &error)) {
+        cerr << "[!] " << name_ << ": bad configuration: " << error << endl;
+        return false;
+    }
+    if (n_ranks != 1) {
+        cerr << "[!] " << name_ << " models run on one GPU" << endl;
+        return false;
+    }
+    for (const hybrid_layer_spec& l : cfg.layers)
+        if (l.mixer.type == hybrid_mixer::kind::attention && (l.mixer.dim > 256 || l.mixer.vdim > 256)) {
+            cerr << "[!] " << name_ << ": heads of more than 256 values are not supported" << endl;
+            return false;
+        }
+    if (cfg.width > 16384 || cfg.taps > 16) {
+        cerr << "[!] " << name_ << ": width above 16384 or more than 16 taps" << endl;
+        return false;
+    }
+    const u32 n = u32(cfg.layers.size());
+    const u32 first = cfg.loop_times ? cfg.loop_start : n, last = cfg.loop_times ? cfg.loop_stop : n;
+    for (u32 i = 0; i < first; ++i) runs.push_back({i, -1});
+    for (u32 t = 0; t < cfg.loop_times; ++t)
+        for (u32 i = first; i < last; ++i) runs.push_back({i, i == first ? int(t) : -1});
+    for (u32 i = last; i < n; ++i) runs.push_back({i, -1});
+    return true;
+}
+
+bool hybrid_architecture::build(llava_context* ctx) {
+    const model_file* model = ctx->get_model();
+    bool ok = true;
+    auto find = [&](const string& name, u32 rows, u32 cols, weight_form form) -> const ggml_data_descriptor* {
+        const ggml_data_descriptor* d = model->find_buffer_descriptor(name);
+        const bool ints = form == weight_form::ids_u32, matrix = form == weight_form::rows_bf16;
+        if (d && d->shape1 == rows && d->shape2 == cols &&
+            (ints ? d->ftype == ggml_value_type::i32 : d->ftype == ggml_value_type::bf16 || (!matrix && d->ftype == ggml_value_type::f32)))
+            return d;
+        cerr << "[!] tensor " << name << (d ? " has another shape or type" : " missing") << endl;
+        ok = false;
+        return nullptr;
+    };
+    auto stack = [&](const vector<pair<string, u32>>& names_rows, u32 cols, weight_form form) -> llava_buffer* {
+        vector<const ggml_data_descriptor*> parts;
+        for (const auto& [name, rows] : names_rows)
+            if (const ggml_data_descriptor* d = find(name, rows, cols, form)) parts.push_back(d);
+        if (parts.size() != names_rows.size()) return nullptr;
+        tensors.push_back(new llava_buffer(ctx, parts, form, ctx->weights_memory()));
+        return tensors.back();
+    };
+    auto matrix = [&](const string& name, u32 rows, u32 cols) { return stack({{name, rows}}, cols, weight_form::rows_bf16); };
+    auto values = [&](const string& name, u32 rows, u32 cols = 1) { return stack({{name, rows}}, cols, weight_form::vector_f32); };
+
+    embed = matrix("embed", cfg.vocab, cfg.width);
+    head = matrix("head", cfg.vocab, cfg.width);
+    final_norm = values("final.norm", cfg.width);
+    if (cfg.loop_times) loop_step = values("loop.step", cfg.loop_times, cfg.width);
+    for (u32 i = 0; i < cfg.layers.size(); ++i) {
+        const hybrid_layer_spec& spec = cfg.layers[i];
+        const hybrid_mixer& m = spec.mixer;
+        const string p = "l" + to_string(i) + ".", mix = p + "mix.", mlp = p + "mlp.";
+        hybrid_layer l;
+        auto taps = [&](const string& name) { return stack({{name, cfg.width}}, cfg.taps, weight_form::columns_f32); };
+        l.norm1 = values(p + "norm1", cfg.width);
+        l.norm1b = values(p + "norm1b", cfg.width);
+        l.canon1 = taps(p + "canon1");
+        l.out = matrix(mix + "o", cfg.width, m.out_size());
+        if (m.type == hybrid_mixer::kind::attention) {
+            l.in = stack({{mix + "q", m.heads * m.dim}, {mix + "k", m.kv_heads * m.dim}, {mix + "v", m.kv_heads * m.vdim}}, cfg.width, weight_form::rows_bf16);
+            l.q_norm = values(mix + "q.norm", m.dim);
+            l.k_norm = values(mix + "k.norm", m.dim);
+            l.r1 = values(mix + "r1", m.heads);
+            l.r2 = values(mix + "r2", m.heads);
+        } else {
+            l.in = stack({{mix + "z", m.width}, {mix + "x", m.width}, {mix + "g", m.width}}, cfg.width, weight_form::rows_bf16);
+            l.z_bias = values(mix + "z.b", m.width);
+            l.x_bias = values(mix + "x.b", m.width);
+        }
+        if (spec.mlp.experts) {
+            l.norm2 = values(p + "norm2", cfg.width);
+            l.norm2b = values(p + "norm2b", cfg.width);
+            l.canon2 = taps(p + "canon2");
+            vector<pair<string, u32>> gate, up, down;
+            for (u32 e = 0; e < spec.mlp.experts; ++e) {
+                const string x = mlp + "e" + to_string(e) + ".";
+                gate.emplace_back(x + "gate", spec.mlp.ff);
+                up.emplace_back(x + "up", spec.mlp.ff);
+                down.emplace_back(x + "down", cfg.width);
+            }
+            l.gate = stack(gate, cfg.width, weight_form::rows_bf16);
+            l.up = stack(up, cfg.width, weight_form::rows_bf16);
+            l.down = stack(down, spec.mlp.ff, weight_form::rows_bf16);
+            l.table = stack({{mlp + "table", cfg.vocab}}, spec.mlp.top, weight_form::ids_u32);
+        }
+        layers.push_back(l);
+    }
+    return ok;
+}
+
+bool hybrid_architecture::upload(llava_context* ctx) {
+    for (llava_buffer* b : tensors)
+        if (ctx->pop_signal() || !b->load_to_gpu()) {
+            cerr << "[!] cannot upload " << b->backing_buffer_name << ": " << lv_last_error_string() << endl;
+            return false;
+        }
+    return true;
+}
+
+unique_ptr<session_state> hybrid_architecture::make_session_state(llava_session* session) { return make_unique<hybrid_session_state>(session, this); }
+
+// ---- one step --------------------------------------------------------------------------------
+
+// Records the operations of a step.  The output of a sublayer is added to the residual stream by the launch that begins the
+// next one (lv_norm_conv), which therefore carries the finished sublayer's norm along.
+struct hybrid_recorder {
+    const hybrid_architecture& arch;
+    const hybrid_config& cfg;
+    llava_command_buffer* cb;
+    llava_session* s;
+    hybrid_session_state* st;
+    lv_ctx* lv;
+    u32 T;
+    const u32* pos;
+    const u32* log;
+    // residual stream; null until the embedding rows have been read
+    float* x = nullptr;
+    // the sublayer that the next norm_conv finishes
+    const float* y = nullptr;
+    const llava_buffer* post = nullptr;
+    int finished_run = -1;               // the layer run that ends with it, for traces
+
+    static float* f32(const llava_buffer* b) { return b ? static_cast<float*>(b->device_ptr()) : nullptr; }
+
+    void norm_conv(const llava_buffer* pre, const llava_buffer* conv, llava_buffer* history, const float* step, u32 first = 0) {
+        lv_norm_conv_args a{};
+        a.x = x;
+        a.embed = arch.embed->device_ptr();
+        a.embed_ld = arch.embed->leading();
+        a.vocab = cfg.vocab;
+        a.token_log = log;
+        a.pos = pos;
+        a.y = y;
+        a.y_rows = 1;
+        a.mult = cfg.residual_mult;
+        a.eps = cfg.eps;
+        a.post_w = f32(post);
+        a.step = step;
+        if (finished_run >= 0 && !st->trace.empty()) a.trace = f32(st->trace[finished_run]);
+        a.x_out = (x == f32(st->stream_a) && T > 1) ? f32(st->stream_b) : f32(st->stream_a);
+        a.pre_w = f32(pre);
+        if (conv) {
+            a.conv_w = f32(conv);
+            a.taps = cfg.taps;
+            a.history = f32(history);
+        }
+        a.out = f32(st->normed);
+        a.out_type = LV_TYPE_F32;
+        a.out_ld = (cfg.width + 7) / 8 * 8;
+        a.width = cfg.width;
+        a.first = first;
+        a.batch = T;
+        cb->note(lv_norm_conv(lv, &a));
+        x = a.x_out;
+        y = nullptr;
+        post = nullptr;
+        finished_run = -1;
+    }
+
+    void product(llava_buffer* out, u32 out_ld, const llava_buffer* w, llava_buffer* in, u32 in_ld, u32 batch, float factor = 1.0f) {
+        cb->note(lv_gemv_bf16(lv, f32(out), out_ld, w->device_ptr(), w->shape.first, w->leading(), w->shape.second, f32(in), in_ld, batch, factor));
+    }
+
+    void attention(const hybrid_layer& l, const hybrid_mixer& m, const hybrid_run_state& r) {
+        const u32 ld = (cfg.width + 7) / 8 * 8, raw_ld = m.raw_size(), out_ld = (m.out_size() + 7) / 8 * 8;
+        product(st->raw, raw_ld, l.in, st->normed, ld, T);
+        lv_gqa_args a{};
+        a.qkv = f32(st->raw);
+        a.qkv_ld = raw_ld;
+        a.heads = m.heads;
+        a.kv_heads = m.kv_heads;
+        a.dim = m.dim;
+        a.vdim = m.vdim;
+        a.scale = m.scale;
+        a.eps = cfg.eps;
+        a.q_norm = f32(l.q_norm);
+        a.k_norm = f32(l.k_norm);
+        a.r1 = f32(l.r1);
+        a.r2 = f32(l.r2);
+        a.sink = m.sink;
+        a.k_cache = r.k_cache->device_ptr();
+        a.v_cache = r.v_cache->device_ptr();
+        a.cache_type = st->f32 ? LV_TYPE_F32 : LV_TYPE_BF16;
+        a.ctx_rows = s->max_context;
+        a.pos = pos;
+        a.out = f32(st->mixed);
+        a.out_type = LV_TYPE_F32;
+        a.out_ld = out_ld;
+        if (T > 1) cb->note(lv_qk_norm_append(lv, &a, T));
+        cb->note(lv_attention_gqa(lv, &a, st->attn_scratch->device_ptr(), st->attn_scratch->byte_size(), T, cb->backlog_size, T == 1));
+        product(st->sub, cfg.width, l.out, st->mixed, out_ld, T);
+    }
+
+    void mingru(const hybrid_layer& l, const hybrid_mixer& m, const hybrid_run_state& r) {
+        const u32 ld = (cfg.width + 7) / 8 * 8, out_ld = (m.width + 7) / 8 * 8;
+        if (T == 1) {
+            const u16* w = static_cast<const u16*>(l.in->device_ptr());
+            const size_t each = size_t(m.width) * l.in->leading();
+            cb->note(lv_gemv_bf16_mingru(lv, f32(st->mixed), w, w + each, w + 2 * each, l.in->leading(), m.width, cfg.width, f32(l.z_bias), f32(l.x_bias),
+                                         f32(st->normed), f32(r.gru_state), pos));
+        } else {
+            product(st->raw, m.raw_size(), l.in, st->normed, ld, T);
+            cb->note(lv_mingru_scan(lv, f32(st->mixed), LV_TYPE_F32, out_ld, f32(st->raw), m.raw_size(), m.width, f32(l.z_bias), f32(l.x_bias),
+                                    f32(r.gru_state), pos, T));
+        }
+        product(st->sub, cfg.width, l.out, st->mixed, out_ld, T);
+    }
+
+    void experts(const hybrid_layer& l, const hybrid_experts& e) {
+        const u32 ld = (cfg.width + 7) / 8 * 8, act_ld = (e.ff + 7) / 8 * 8;
+        lv_expert_args a{};
+        a.w0 = l.gate->device_ptr();
+        a.w1 = l.up->device_ptr();
+        a.ld = l.gate->leading();
+        a.rows = e.ff;
+        a.cols = cfg.width;
+        a.experts = e.experts;
+        a.top = e.top;
+        a.vocab = cfg.vocab;
+        a.table = static_cast<const u32*>(l.table->device_ptr());
+        a.token_log = log;
+        a.pos = pos;
+        cb->note(lv_gemv_bf16_expert_gate_up(lv, f32(st->act), act_ld, &a, f32(st->normed), ld, T));
+        a.w0 = l.down->device_ptr();
+        a.w1 = nullptr;
+        a.ld = l.down->leading();
+        a.rows = cfg.width;
+        a.cols = e.ff;
+        cb->note(lv_gemv_bf16_expert_down(lv, f32(st->sub), cfg.width, &a, f32(st->act), act_ld, T));
+    }
+
+    void finish_sublayer(const llava_buffer* norm) {
+        y = f32(st->sub);
+        post = norm;
+    }
+
+    void step() {
+        const auto& runs = arch.runs_in_order();
+        for (size_t i = 0; i < runs.size(); ++i) {
+            const hybrid_layer& l = arch.layer(runs[i].layer);
+            const hybrid_layer_spec& spec = cfg.layers[runs[i].layer];
+            const hybrid_run_state& r = st->runs[i];
+            norm_conv(l.norm1, l.canon1, r.history1, runs[i].begins_pass >= 0 ? f32(arch.loop_step) + size_t(runs[i].begins_pass) * cfg.width : nullptr);
+            if (spec.mixer.type == hybrid_mixer::kind::attention) attention(l, spec.mixer, r);
+            else mingru(l, spec.mixer, r);
+            finish_sublayer(l.norm1b);
+            if (spec.mlp.experts) {
+                norm_conv(l.norm2, l.canon2, r.history2, nullptr);
+                experts(l, spec.mlp);
+                finish_sublayer(l.norm2b);
+            }
+            finished_run = int(i);
+        }
+        const u32 ld = (cfg.width + 7) / 8 * 8;
+        if (cb->row_logits) {
+            norm_conv(arch.final_norm, nullptr, nullptr, nullptr);
+            product(st->logits_rows, cfg.vocab, arch.head, st->normed, ld, T, cfg.logit_scale);
+        } else if (cb->with_head) {
+            // only the last row's logits are wanted (a trace wants the last layer's stream of every row)
+            const u32 first = st->trace.empty() ? T - 1 : 0;
+            norm_conv(arch.final_norm, nullptr, nullptr, nullptr, first);
+            cb->note(lv_gemv_bf16(lv, f32(s->output_probs), cfg.vocab, arch.head->device_ptr(), cfg.vocab, arch.head->leading(), cfg.width,
+                                  f32(st->normed) + size_t(T - 1 - first) * ld, ld, 1, cfg.logit_scale));
+        }
+        cb->finish_step();
+    }
+};
+
+void hybrid_architecture::record(llava_command_buffer* cb) {
+    llava_session* s = cb->session;
+    auto* st = static_cast<hybrid_session_state*>(s->state.get());
+    if (!cb->expect(st != nullptr && cb->batch_size <= s->max_batch, "session state")) return;
+    hybrid_recorder r{*this, cfg, cb, s, st, s->ctx->lv(), cb->batch_size, static_cast<const u32*>(s->config_buffer->device_ptr()),
+                      static_cast<const u32*>(s->token_log->device_ptr())};
+    r.step();
+}

@@ -1,0 +1,146 @@
+#include "hybrid_session_state.h"
+
+#include <algorithm>
+#include <cstring>
+#include <string>
+
+#include "llava_buffer.h"
+#include "llava_context.h"
+#include "llava_device_memory.h"
+#include "llava_session.h"
+
+using namespace std;
+
+namespace {
+u32 pad8(u32 n) { return (n + 7) / 8 * 8; }
+}  // namespace
+
+hybrid_session_state::hybrid_session_state(llava_session* _session, const hybrid_architecture* _arch)
+    : session(_session), arch(_arch), f32(_session->ctx->get_compute_type() == compute_type::f32) {
+    const hybrid_config& c = arch->config();
+    llava_context* ctx = session->ctx;
+    const auto F = ggml_value_type::f32, C = f32 ? ggml_value_type::f32 : ggml_value_type::bf16;
+    lasting = new llava_device_memory(ctx);
+    for (const hybrid_run& r : arch->runs_in_order()) {
+        const hybrid_layer_spec& spec = c.layers[r.layer];
+        hybrid_run_state s;
+        if (spec.mixer.type == hybrid_mixer::kind::attention) {
+            s.k_cache = new llava_buffer(ctx, C, spec.mixer.kv_heads * session->max_context, pad8(spec.mixer.dim), lasting, "k_cache");
+            s.v_cache = new llava_buffer(ctx, C, spec.mixer.kv_heads * session->max_context, pad8(spec.mixer.vdim), lasting, "v_cache");
+        } else {
+            s.gru_state = new llava_buffer(ctx, F, spec.mixer.width, 1, lasting, "gru_state");
+        }
+        if (c.taps > 1) {
+            s.history1 = new llava_buffer(ctx, F, c.width, c.taps - 1, lasting, "history1");
+            if (spec.mlp.experts) s.history2 = new llava_buffer(ctx, F, c.width, c.taps - 1, lasting, "history2");
+        }
+        runs.push_back(s);
+    }
+    lasting->freeze();
+}
+
+hybrid_session_state::~hybrid_session_state() {
+    drop_scratch();
+    for (hybrid_run_state& s : runs)
+        for (llava_buffer* b : {s.k_cache, s.v_cache, s.gru_state, s.history1, s.history2}) delete b;
+    delete lasting;
+}
+
+void hybrid_session_state::drop_scratch() {
+    for (llava_buffer** b : {&stream_a, &stream_b, &normed, &raw, &mixed, &act, &sub, &attn_scratch, &logits_rows}) {
+        delete *b;
+        *b = nullptr;
+    }
+    for (llava_buffer* b : trace) delete b;
+    trace.clear();
+    delete scratch;
+    scratch = nullptr;
+    scratch_batch = 0;
+}
+
+bool hybrid_session_state::resize() {
+    if (!lasting->is_frozen()) return false;
+    const u32 B = session->max_batch;
+    const bool want_trace = session->is_tracing_enabled(), want_rows = session->want_row_logits;
+    if (scratch_batch == B && scratch_trace == want_trace && scratch_rows == want_rows) return true;
+    drop_scratch();
+    const hybrid_config& c = arch->config();
+    llava_context* ctx = session->ctx;
+    u32 raw_size = 8, mixed_size = 8, act_size = 8, copies = 1;
+    size_t attention_bytes = 0;
+    for (const hybrid_layer_spec& l : c.layers) {
+        raw_size = max(raw_size, l.mixer.raw_size());
+        mixed_size = max(mixed_size, pad8(l.mixer.out_size()));
+        if (l.mlp.experts) {
+            act_size = max(act_size, l.mlp.top * pad8(l.mlp.ff));
+            copies = max(copies, l.mlp.top);
+        }
+        if (l.mixer.type == hybrid_mixer::kind::attention) {
+            lv_gqa_args a{};
+            a.heads = l.mixer.heads;
+            a.kv_heads = l.mixer.kv_heads;
+            a.dim = l.mixer.dim;
+            a.vdim = l.mixer.vdim;
+            attention_bytes = max(attention_bytes, lv_gqa_scratch_bytes(ctx->lv(), &a, B, session->max_context));
+        }
+    }
+    const auto F = ggml_value_type::f32;
+    scratch = new llava_device_memory(ctx);
+    stream_a = new llava_buffer(ctx, F, c.width, B, scratch);
+    stream_b = new llava_buffer(ctx, F, c.width, B, scratch);
+    normed = new llava_buffer(ctx, F, pad8(c.width) * copies, B, scratch);
+    raw = new llava_buffer(ctx, F, raw_size, B, scratch);
+    mixed = new llava_buffer(ctx, F, mixed_size, B, scratch);
+    act = new llava_buffer(ctx, F, act_size, B, scratch);
+    sub = new llava_buffer(ctx, F, c.width * copies, B, scratch);
+    if (attention_bytes) attn_scratch = new llava_buffer(ctx, F, u32((attention_bytes + 3) / 4), 1, scratch);
+    if (want_rows) logits_rows = new llava_buffer(ctx, F, c.vocab, B, scratch);
+    if (want_trace)
+        for (size_t r = 0; r < runs.size(); ++r) {            // numbered so that frames list them in order
+            const string n = to_string(r);
+            trace.push_back(new llava_buffer(ctx, F, c.width, B, scratch, "run." + string(4 - min<size_t>(4, n.size()), '0') + n + ".residual"));
+        }
+    if (!scratch->freeze() || !scratch->zero(0, scratch->get_size())) return false;
+    scratch_batch = B;
+    scratch_trace = want_trace;
+    scratch_rows = want_rows;
+    return true;
+}
+
+void hybrid_session_state::dump_frame(int fd) {
+    if (scratch) scratch->dump_buffers(fd, "step");
+}
+
+// Per layer run: the first n rows of every key head, then of every value head, or the recurrent state; then the histories.
+size_t hybrid_session_state::snapshot_bytes(u32 n) const {
+    size_t total = 0;
+    for (const hybrid_run_state& s : runs) {
+        for (const llava_buffer* b : {s.k_cache, s.v_cache})
+            if (b) total += size_t(b->shape.first / session->max_context) * n * b->shape.second * cache_bytes();
+        for (const llava_buffer* b : {s.gru_state, s.history1, s.history2})
+            if (b) total += b->byte_size();
+    }
+    return total;
+}
+
+bool hybrid_session_state::transfer(u8* dst, const u8* src, u32 n) {
+    size_t at = 0;
+    bool ok = true;
+    auto move = [&](llava_buffer* b, size_t offset, size_t bytes) {
+        if (bytes != 0) ok = ok && (dst ? b->read_raw(offset, dst + at, bytes) : b->write_raw(offset, src + at, bytes));
+        at += bytes;
+    };
+    for (hybrid_run_state& s : runs) {
+        for (llava_buffer* b : {s.k_cache, s.v_cache}) {
+            if (b == nullptr) continue;
+            const size_t row = size_t(b->shape.second) * cache_bytes();
+            for (u32 g = 0; g < b->shape.first / session->max_context; ++g) move(b, size_t(g) * session->max_context * row, n * row);
+        }
+        for (llava_buffer* b : {s.gru_state, s.history1, s.history2})
+            if (b) move(b, 0, b->byte_size());
+    }
+    return ok;
+}
+
+bool hybrid_session_state::read_snapshot(u8* dst, u32 n) { return transfer(dst, nullptr, n); }
+bool hybrid_session_state::write_snapshot(const u8* src, u32 n) { return transfer(nullptr, src, n); }

@@ -1,0 +1,53 @@
+// What a session of a hybrid decoder keeps on the device: per layer run the key/value caches or the recurrent state and the
+// histories of its two convolutions, which live as long as the session, and scratch for a step, which follows max_batch.
+// No cache or state needs clearing: kernels take a state before position 0 as zero and read cache rows up to the position.
+#ifndef LLAVA_B200_HYBRID_SESSION_STATE_H
+#define LLAVA_B200_HYBRID_SESSION_STATE_H
+
+#include <vector>
+
+#include "hybrid_architecture.h"
+
+struct hybrid_run_state {
+    llava_buffer *k_cache = nullptr, *v_cache = nullptr;      // attention: [kv_heads][max_context][padded dim]
+    llava_buffer *gru_state = nullptr;                        // mingru: f32 [width]
+    llava_buffer *history1 = nullptr, *history2 = nullptr;    // f32 [taps - 1][width]
+};
+
+class hybrid_session_state : public session_state {
+public:
+    hybrid_session_state(llava_session* session, const hybrid_architecture* arch);
+    ~hybrid_session_state() override;
+    bool resize() override;
+    size_t snapshot_bytes(u32 n) const override;
+    bool read_snapshot(u8* dst, u32 n) override;
+    bool write_snapshot(const u8* src, u32 n) override;
+    void dump_frame(int fd) override;
+    llava_buffer* row_logits() const override { return logits_rows; }
+
+    llava_session* const session;
+    const hybrid_architecture* const arch;
+    std::vector<hybrid_run_state> runs;
+    // scratch of one step
+    llava_buffer *stream_a = nullptr, *stream_b = nullptr;    // residual stream, f32 [batch][width]
+    llava_buffer *normed = nullptr;                           // input of a sublayer, one row per token or per chosen expert
+    llava_buffer *raw = nullptr;                              // input projections, f32
+    llava_buffer *mixed = nullptr;                            // mixer output before its output projection
+    llava_buffer *act = nullptr;                              // expert activations
+    llava_buffer *sub = nullptr;                              // output of a sublayer, f32
+    llava_buffer *attn_scratch = nullptr;
+    llava_buffer *logits_rows = nullptr;                      // f32 [batch][vocab], only for evaluate_pending
+    std::vector<llava_buffer*> trace;                         // per layer run: the residual stream after it, only when tracing
+    u32 cache_bytes() const { return f32 ? 4 : 2; }
+    bool const f32;                                           // 32-bit arithmetic: activations and caches are f32
+
+private:
+    void drop_scratch();
+    bool transfer(u8* dst, const u8* src, u32 n);
+    llava_device_memory* lasting = nullptr;
+    llava_device_memory* scratch = nullptr;
+    u32 scratch_batch = 0;
+    bool scratch_trace = false, scratch_rows = false;
+};
+
+#endif

@@ -69,6 +69,23 @@ llava_buffer::llava_buffer(llava_context* _context, const ggml_data_descriptor& 
     if (!device_memory_is_shared) device_memory->freeze();
 }
 
+static std::pair<u32, u32> stacked_shape(const vector<const ggml_data_descriptor*>& parts) {
+    u32 rows = 0;
+    for (const ggml_data_descriptor* p : parts) rows += p->shape1;
+    return {rows, parts[0]->shape2};
+}
+
+llava_buffer::llava_buffer(llava_context* _context, const vector<const ggml_data_descriptor*>& parts, weight_form _form, llava_device_memory* _device_memory)
+    : context(_context), backing_buffer_name(parts[0]->name),
+      type(_form == weight_form::rows_bf16 ? ggml_value_type::bf16 : _form == weight_form::ids_u32 ? ggml_value_type::i32 : ggml_value_type::f32),
+      shape(stacked_shape(parts)), device_memory_is_shared(true), device_memory(_device_memory), model_version(0), file_shape(shape), form(_form),
+      used_cols(shape.second) {
+    device_memory->register_llava_buffer(this);
+    for (const ggml_data_descriptor* p : parts) part_names.push_back(p->name);
+    bytes = form == weight_form::rows_bf16 ? size_t(shape.first) * leading() * 2 : size_t(shape.first) * shape.second * 4;
+    offset = device_memory->register_buffer(kBufferAlignment, bytes);
+}
+
 llava_buffer::~llava_buffer() {
     device_memory->forget_llava_buffer(this);
     if (!device_memory_is_shared) delete device_memory;
@@ -150,7 +167,8 @@ bool llava_buffer::write_full(const void* in_buf, ggml_value_type intype, u32 ve
 bool llava_buffer::load_to_gpu() {
     if (backing_buffer_name.empty()) return true;
     if (!is_allocated()) return false;
-    const ggml_file* model = context->get_model();
+    if (form != weight_form::file) return load_parts();
+    const model_file* model = context->get_model();
     const ggml_data_descriptor& table = model->get_buffer_descriptor(backing_buffer_name);
     if (split == tp_split::none) return context->upload_from_host(device_ptr(), model->data() + table.offset, table.size);
     if (bytes == 0) return false;                      // the tensor cannot be split this way
@@ -159,6 +177,45 @@ bool llava_buffer::load_to_gpu() {
     std::vector<u8> packed(bytes);
     return tp_pack(model->data() + table.offset, type, file_shape.first, file_shape.second, split, tp_rank, tp_ranks, packed.data()) &&
            context->upload_from_host(device_ptr(), packed.data(), bytes);
+}
+
+// Tensors of a model folder in this buffer's form (see weight_form).
+bool llava_buffer::load_parts() {
+    const model_file* model = context->get_model();
+    size_t row = 0;
+    vector<u8> staged;
+    for (const string& part : part_names) {
+        const ggml_data_descriptor& t = model->get_buffer_descriptor(part);
+        const u8* src = model->data() + t.offset;
+        const size_t rows = t.shape1, cols = t.shape2;
+        if (form == weight_form::rows_bf16) {
+            const size_t ld = leading();
+            u8* dst = device_memory->device_base() + offset + row * ld * 2;
+            if (ld != cols) {
+                staged.assign(rows * ld * 2, 0);
+                for (size_t r = 0; r < rows; ++r) memcpy(staged.data() + r * ld * 2, src + r * cols * 2, cols * 2);
+                src = staged.data();
+            }
+            if (!context->upload_from_host(dst, src, rows * ld * 2)) return false;
+        } else {
+            staged.resize(rows * cols * 4);
+            for (size_t i = 0; i < rows * cols; ++i) {
+                u32 word = 0;
+                if (t.ftype == ggml_value_type::bf16) {
+                    u16 h;
+                    memcpy(&h, src + i * 2, 2);
+                    word = u32(h) << 16;                        // bfloat16 is the upper half of an f32
+                } else {
+                    memcpy(&word, src + i * 4, 4);
+                }
+                const size_t at = form == weight_form::columns_f32 ? (i % cols) * rows + i / cols : i;
+                memcpy(staged.data() + at * 4, &word, 4);
+            }
+            if (!context->upload_from_host(device_memory->device_base() + offset + row * cols * 4, staged.data(), staged.size())) return false;
+        }
+        row += rows;
+    }
+    return true;
 }
 
 void llava_buffer::dump_raw(int out_fd, const string& name) {

@@ -7,10 +7,18 @@
 
 #include <string>
 #include <utility>
+#include <vector>
 
-#include "ggml_file.h"
+#include "model_file.h"
 #include "tp_shard.h"
 #include "types.h"
+
+// How tensors of a model folder lie on the device.
+//   rows_bf16    matrices stacked by rows, bfloat16 [rows][leading()], leading() = columns rounded up to 8, padding zero
+//   vector_f32   the elements in file order, widened to f32
+//   columns_f32  f32 [columns][rows]: the transpose
+//   ids_u32      32-bit integers as they are
+enum class weight_form : u32 { file = 0, rows_bf16, vector_f32, columns_f32, ids_u32 };
 
 class llava_buffer {
 public:
@@ -22,6 +30,8 @@ public:
     // shard of a file matrix for rank `rank` of `n_ranks` (see tp_shard.h); shape = local shape
     llava_buffer(llava_context* context, const ggml_data_descriptor& table, llava_device_memory* device_memory,
                  tp_split how, u32 rank, u32 n_ranks);
+    // tensors of a model folder, stacked by rows (all of the first one's column count), in the given form
+    llava_buffer(llava_context* context, const std::vector<const ggml_data_descriptor*>& parts, weight_form form, llava_device_memory* device_memory);
     ~llava_buffer();
     llava_buffer(const llava_buffer&) = delete;
     llava_buffer& operator=(const llava_buffer&) = delete;
@@ -56,9 +66,13 @@ public:
     const tp_split split = tp_split::none;
     const u32 tp_rank = 0, tp_ranks = 1;
     const std::pair<u32, u32> file_shape;      // shape of the whole tensor in the file
+    const weight_form form = weight_form::file;
+    u32 leading() const { return (shape.second + 7) / 8 * 8; }      // rows_bf16: elements from row to row
     u32 cols_used() const { return used_cols; }   // local columns that carry weights (< shape.second when padded)
 
 private:
+    bool load_parts();
+    std::vector<std::string> part_names;
     u32 used_cols = 0;
     size_t bytes = 0;
     size_t offset = 0;

@@ -7,12 +7,13 @@
 #include "llava_layer.h"
 #include "llava_layer_session_data.h"
 #include "llava_session.h"
+#include "model_architecture.h"
 
 using namespace std;
 
-llava_command_buffer::llava_command_buffer(llava_session* _session, u32 _batch_size, bool _with_head, bool _sample)
+llava_command_buffer::llava_command_buffer(llava_session* _session, u32 _batch_size, bool _with_head, bool _sample, bool _row_logits)
     : session(_session), backlog_size(_session->backlog_size), workgroup_size(_session->ctx->workgroup_size),
-      batch_size(_batch_size), with_head(_with_head), sample(_sample && _with_head) {}
+      batch_size(_batch_size), with_head(_with_head), sample(_sample && _with_head), row_logits(_row_logits) {}
 
 llava_command_buffer::~llava_command_buffer() {
     wait_idle();
@@ -62,63 +63,17 @@ void llava_command_buffer::record_sampler() {
     u32* config = static_cast<u32*>(s->config_buffer->device_ptr());
     u32* log = static_cast<u32*>(s->token_log->device_ptr());
     note(lv_sample_mirostat(lv(), static_cast<float*>(s->output_probs->device_ptr()), s->model->get_header().vocab_size, log, config,
-                            static_cast<u32*>(s->sampler_state->device_ptr()), -1.0f, log, max_backlog_size + 1,
-                            static_cast<u32*>(s->argmax_result->device_ptr()) + 1, s->pinned + max_backlog_size + 5, nullptr));
+                            static_cast<u32*>(s->sampler_state->device_ptr()), -1.0f, log, s->log_capacity(),
+                            static_cast<u32*>(s->argmax_result->device_ptr()) + 1, s->sample_word(), nullptr));
 }
 
 bool llava_command_buffer::record_execution() {
     if (graph) return false;
-    llava_session* s = session;
-    llava_context* c = s->ctx;
-    const ggml_header& h = s->model->get_header();
-    if (!expect(s->get_layer_data().size() == c->get_layers().size(), "one layer data per layer")) return false;
     if (lv_graph_begin_capture(lv()) != LV_OK) {
         note(LV_ERR_CUDA);
         return false;
     }
-    u32* config = static_cast<u32*>(s->config_buffer->device_ptr());
-    u32* log = static_cast<u32*>(s->token_log->device_ptr());
-    if (batch_size == 1 && s->step_plan != nullptr && !s->is_tracing_enabled()) {
-        // a single token: the whole list below as one persistent kernel
-        note(lv_decode_step(lv(), s->step_plan, config, log, max_backlog_size + 1, static_cast<float*>(s->output_probs->device_ptr()),
-                            static_cast<u32*>(s->argmax_result->device_ptr()), s->pinned + max_backlog_size + 4, with_head ? 1 : 0));
-        if (sample) record_sampler();
-        lv_graph* g1 = nullptr;
-        note(lv_graph_end_capture(lv(), &g1));
-        if (first_error != LV_OK) {
-            lv_graph_destroy(g1);
-            return false;
-        }
-        graph = g1;
-        return true;
-    }
-    // embedding rows of the tokens at positions config.token_count .. + batch (the reference
-    // dequantises them on the host, llava_session.cpp:219-223)
-    note(lv_dequant_rows(lv(), static_cast<float*>(s->current_thought->device_ptr()), c->tok_embeddings->device_ptr(),
-                         c->tok_embeddings->kernel_type(), log, config, h.dim, h.vocab_size, batch_size));
-    llava_buffer* current = s->current_thought;
-    for (u32 i = 0; i < c->get_layers().size(); ++i) current = c->get_layers()[i]->execute(this, s->get_layer_data()[i], current);
-    if (with_head) {
-        // final norm + output matrix on the last row only (llava_command_buffer.cpp:38-39; the
-        // reference computes every row and reads the last, llava_session.cpp:129-135)
-        const float* last = static_cast<const float*>(current->device_ptr()) + size_t(batch_size - 1) * h.dim;
-        float* logits = static_cast<float*>(s->output_probs->device_ptr());
-        // sharded with fused exchanges: the last layer's w2 pushed its partial rows; the head's
-        // normalisation takes residual + the ranks' sum
-        if (c->tp_size() > 1 && c->fused_exchange() && !use_tensor_cores(c->get_layers()[0]->wq()))
-            tp_arm_pull(2 * u32(c->get_layers().size()) - 1, h.dim, current == s->current_thought ? s->current_thought_sublayer : s->current_thought);
-        note(lv_norm_gemv(lv(), logits, c->output_w->device_ptr(), c->output_w->kernel_type(), last,
-                          static_cast<const float*>(c->norm_w->device_ptr()), h.vocab_size, h.dim, 1));
-        // greedy choice, token log and position word in one launch; the kernel stores the token
-        // into the pinned staging word itself
-        u32* am = static_cast<u32*>(s->argmax_result->device_ptr());
-        note(lv_argmax_advance(lv(), logits, h.vocab_size, config, log, batch_size, max_backlog_size + 1, am,
-                               s->pinned + max_backlog_size + 4));
-        if (sample) record_sampler();
-    } else {
-        // leading chunk of a prompt: only the position advances
-        note(lv_decode_advance(lv(), config, nullptr, nullptr, batch_size, 0));
-    }
+    session->ctx->architecture()->record(this);
     lv_graph* g = nullptr;
     const int rc = lv_graph_end_capture(lv(), &g);
     note(rc);
@@ -128,6 +83,21 @@ bool llava_command_buffer::record_execution() {
     }
     graph = g;
     return true;
+}
+
+// Greedy choice, token log and position words in one launch when the step has the logits of its last row (the kernel
+// stores the token into the pinned staging word itself), and the draw of a sampled step; else only the position advances.
+void llava_command_buffer::finish_step() {
+    llava_session* s = session;
+    u32* config = static_cast<u32*>(s->config_buffer->device_ptr());
+    if (!with_head) {
+        note(lv_decode_advance(lv(), config, nullptr, nullptr, batch_size, 0));
+        return;
+    }
+    note(lv_argmax_advance(lv(), static_cast<float*>(s->output_probs->device_ptr()), s->model->get_header().vocab_size, config,
+                           static_cast<u32*>(s->token_log->device_ptr()), batch_size, s->log_capacity(),
+                           static_cast<u32*>(s->argmax_result->device_ptr()), s->argmax_word()));
+    if (sample) record_sampler();
 }
 
 static inline float* f32(llava_buffer* b) { return static_cast<float*>(b->device_ptr()); }

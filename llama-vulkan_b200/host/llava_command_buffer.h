@@ -14,7 +14,8 @@ public:
     // with_head: record the final norm + output matrix + argmax (not needed for
     // the leading chunks of a long prompt)
     // sample: after the head, draw the next token on the device (the reference's sampler) as part of the step
-    llava_command_buffer(llava_session* session, u32 batch_size, bool with_head, bool sample = false);
+    // row_logits: also produce the logits of every row of the batch (architectures that have_row_logits)
+    llava_command_buffer(llava_session* session, u32 batch_size, bool with_head, bool sample = false, bool row_logits = false);
     ~llava_command_buffer();
     llava_command_buffer(const llava_command_buffer&) = delete;
     llava_command_buffer& operator=(const llava_command_buffer&) = delete;
@@ -24,6 +25,9 @@ public:
     bool wait_idle() const;
     u32 kernel_launches() const;       // kernel nodes of the recorded graph
     void record_sampler();
+    void finish_step();                // last launches of every step: token choice and position words
+    void note(int rc);                 // keeps the first error of the recording
+    bool expect(bool cond, const char* what);
 
     // the reference's op set (llava_command_buffer.h:30-38)
     void normalize_logit(llava_buffer* outbuf, llava_buffer* inbuf, llava_buffer* weights);
@@ -69,10 +73,9 @@ public:
     u32 const batch_size;
     bool const with_head;
     bool const sample;
+    bool const row_logits;
 
 private:
-    void note(int rc);
-    bool expect(bool cond, const char* what);
     lv_ctx* lv() const;
     lv_graph* graph = nullptr;
     int first_error = LV_OK;

@@ -21,6 +21,7 @@
 #include "llava_device_memory.h"
 #include "llava_layer.h"
 #include "llava_session.h"
+#include "model_architecture.h"
 #include "server/tlv_server.h"
 #include "synth_ggjt.h"
 
@@ -37,6 +38,7 @@ void llava_context::close_all() {
     delete norm_w;
     delete output_w;
     tok_embeddings = norm_w = output_w = nullptr;
+    arch.reset();                // its tensors live in shared_memory
     if (rope_table && lv_context) lv_arena_free(lv_context, rope_table);
     rope_table = nullptr;
     delete shared_memory;
@@ -69,7 +71,7 @@ bool llava_context::open_sharded(const string& model_path, int device, u32 rank,
 
 bool llava_context::peer_window_create(u8* handle64) {
     if (lv_context == nullptr || model == nullptr) return false;
-    return lv_peer_window_create(lv_context, int(n_ranks_), model->get_header().dim * llava_session::max_batch_limit, handle64) == LV_OK;
+    return lv_peer_window_create(lv_context, int(n_ranks_), model->get_header().dim * 64, handle64) == LV_OK;
 }
 
 bool llava_context::peer_connect(const u8* handles) {
@@ -79,8 +81,10 @@ bool llava_context::peer_connect(const u8* handles) {
 
 bool llava_context::open_model_only(const string& model_path) {
     close_all();
-    model = new ggml_file(model_path.c_str());
-    return model->is_open();
+    model = open_model(model_path).release();
+    if (!model->is_open()) return false;
+    arch = make_architecture(model->architecture());
+    return arch != nullptr;
 }
 
 bool llava_context::open(const string& model_path, int device) {
@@ -88,62 +92,24 @@ bool llava_context::open(const string& model_path, int device) {
     close_all();
     rank_ = keep_rank;
     n_ranks_ = keep_ranks;
-    model = new ggml_file(model_path.c_str());
+    model = open_model(model_path).release();
     if (!model->is_open()) return false;
-    const ggml_header& h = model->get_header();
-    if (h.n_heads % n_ranks_ != 0 || (h.dim / 32) % n_ranks_ != 0 || (model->get_ff_size() / 32) % n_ranks_ != 0 ||
-        model->get_ff_size() % (2 * n_ranks_) != 0) {
-        cerr << "[!] heads, dim and ff must divide evenly over " << n_ranks_ << " ranks" << endl;
+    arch = make_architecture(model->architecture());
+    if (!arch) {
+        cerr << "[!] unknown architecture " << model->architecture() << "; known:";
+        for (const string& a : known_architectures()) cerr << " " << a;
+        cerr << endl;
         return false;
     }
-    // the kernels are specialised for the reference's geometries (llava_session.cpp:357-375:
-    // dim 4096 or 5120, ff 11008 or 13824) and for heads of 128
-    if (h.rot != 128 || h.dim % 256 != 0 || model->get_ff_size() % 256 != 0) {
-        cerr << "[!] unsupported geometry: need head size 128 and dim, ff multiples of 256" << endl;
-        return false;
-    }
+    if (!arch->check(*model, n_ranks_)) return false;
     if (lv_ctx_create(device, &lv_context) != LV_OK) {
         cerr << "[!] cannot create the CUDA context: " << lv_last_error_string() << endl;
         return false;
     }
-    const ggml_data_descriptor* emb = model->find_buffer_descriptor("tok_embeddings");
-    const ggml_data_descriptor* norm = model->find_buffer_descriptor("norm");
-    const ggml_data_descriptor* out = model->find_buffer_descriptor("output");
-    if (!emb || !norm || !out) {
-        cerr << "[!] tok_embeddings / norm / output missing from the model" << endl;
-        return false;
-    }
     shared_memory = new llava_device_memory(this);
-    tok_embeddings = new llava_buffer(this, *emb, shared_memory);
-    norm_w = new llava_buffer(this, *norm, shared_memory);
-    output_w = new llava_buffer(this, *out, shared_memory);
-    if (norm_w->type != ggml_value_type::f32 || !output_w->weight_buffer_is_quantised() || emb->shape1 != h.vocab_size ||
-        !(tok_embeddings->weight_buffer_is_quantised() || tok_embeddings->type == ggml_value_type::f32)) {
-        cerr << "[!] unsupported tensor types for tok_embeddings / norm / output" << endl;
-        return false;
-    }
-
-    void* table = nullptr;
-    if (lv_arena_create(lv_context, size_t(max_backlog_size) * h.rot * sizeof(float), &table) != LV_OK) return false;
-    rope_table = static_cast<float*>(table);
-    if (lv_rope_table_build(lv_context, rope_table, max_backlog_size, h.rot) != LV_OK) return false;
-
-    layers.reserve(h.n_layers);
-    for (u32 i = 0; i < h.n_layers; ++i) {
-        layers.push_back(new llava_layer(this, i));
-        if (!layers.back()->is_valid()) return false;
-    }
+    if (!arch->build(this)) return false;
     // every tensor has registered its size: one allocation for the whole model
-    if (!shared_memory->freeze()) return false;
-    if (!tok_embeddings->load_to_gpu() || !norm_w->load_to_gpu() || !output_w->load_to_gpu()) return false;
-    for (llava_layer* l : layers) {
-        if (sigfd >= 0 && pop_signal()) return false;
-        if (!l->freeze_storage() || !l->load_to_gpu()) {
-            cerr << "[!] cannot upload layer " << l->layer_id << ": " << lv_last_error_string() << endl;
-            return false;
-        }
-    }
-    return true;
+    return shared_memory->freeze() && arch->upload(this);
 }
 
 bool llava_context::setup_signal_handling() {
@@ -201,14 +167,15 @@ bool rendezvous_wait(const tp_rendezvous* rv, const std::atomic<u32>& counter, u
 // Flags of the reference (llava_context.cpp:163-200) that still mean something, plus the
 // ones its CLI lacks: --greedy, --tokens, --n-predict, --ignore-eos, --seed, --device,
 // --gpus N (tensor-parallel over devices D..D+N-1, one forked process each), --on-device, --prompt-batch N (prompt tokens
-// per recorded step, 6..64 run on the tensor cores; default 1), --exact-prompt (batched prompt products with exact weight tiles), --write-synthetic, and --port / --bind for --server.
+// per recorded step, 6..64 run on the tensor cores; default 1), --context N (tokens a session may hold) and --dtype (arithmetic
+// of models that leave the choice; model folders only), --exact-prompt (batched prompt products with exact weight tiles), --write-synthetic, and --port / --bind for --server.
 int llava_context::run(int argc, char** argv) {
     bool server_mode = false, only_print_header = false, greedy = false, ignore_eos = false, on_device = false;
     bool model_path_provided = false, have_seed = false, exact_prompt = false;
     string model_path, tokens_path, synth_spec, bind_address = "0.0.0.0";
     u32 server_port = 1337;
     string prompt = "The ten best monuments to see in Paris are";
-    u32 n_predict = 0, seed = 0, gpus = 1, prompt_batch = 1;
+    u32 n_predict = 0, seed = 0, gpus = 1, prompt_batch = 1, context_tokens = 0;
     int device = 0;
 
     auto need_value = [&](int& i) -> const char* {
@@ -231,7 +198,7 @@ int llava_context::run(int argc, char** argv) {
         } else if (streq(a, "--help") || streq(a, "-h")) {
             cout << (argc ? argv[0] : "./vulkan_llama")
                  << " [-h] [-m model.bin] [--server [--port P] [--bind ADDR]] [--greedy] [--n-predict N] [--ignore-eos] [--tokens ids.txt] [--seed S]"
-                    " [--device D] [--gpus N] [--on-device] [--prompt-batch N] [--exact-prompt] [--print_header] [--write-synthetic 7b|13b|tiny[:q8][:layers=N]] [prompt]"
+                    " [--device D] [--gpus N] [--context N] [--dtype bfloat16|float32] [--on-device] [--prompt-batch N] [--exact-prompt] [--print_header] [--write-synthetic 7b|13b|tiny[:q8][:layers=N]] [prompt]"
                  << endl;
             exit(0);
         } else if (streq(a, "--verbose") || streq(a, "-v")) {
@@ -259,6 +226,12 @@ int llava_context::run(int argc, char** argv) {
             prompt_batch = u32(strtoul(need_value(i), nullptr, 10));
         } else if (streq(a, "--tokens")) {
             tokens_path = need_value(i);
+        } else if (streq(a, "--context")) {
+            context_tokens = u32(strtoul(need_value(i), nullptr, 10));
+        } else if (streq(a, "--dtype")) {
+            const char* v = need_value(i);
+            if (streq(v, "float32")) compute = compute_type::f32;
+            else if (!streq(v, "bfloat16")) { cerr << "[!] --dtype takes bfloat16 or float32" << endl; exit(1); }
         } else if (streq(a, "--n-predict")) {
             n_predict = u32(strtoul(need_value(i), nullptr, 10));
         } else if (streq(a, "--seed")) {
@@ -315,9 +288,9 @@ int llava_context::run(int argc, char** argv) {
     }
 
     if (only_print_header) {
-        ggml_file f(model_path.c_str());
-        if (!f.is_open()) return 1;
-        f.print_info();
+        const auto f = open_model(model_path);
+        if (!f->is_open()) return 1;
+        f->print_info();
         return 0;
     }
     // --gpus N: the process forks N-1 times before anything touches CUDA; rank r drives device D + r, rank 0 (the
@@ -418,12 +391,16 @@ int llava_context::run(int argc, char** argv) {
     }
 
     // generation loop, llava_context.cpp:336-373
-    const u32 eos_id = 2;
-    llava_session session(this);
+    const u32 eos_id = model->eos_token();
+    llava_session session(this, context_tokens);
+    if (!session.is_valid()) {
+        cerr << "[!] --context takes up to " << arch->max_context_limit() << " tokens" << endl;
+        return finish(1);
+    }
     session.set_deterministic(greedy);
     if (have_seed) session.set_seed(seed);
     if (prompt_batch > 1 && !session.set_max_batch(prompt_batch)) {
-        cerr << "[!] --prompt-batch takes 1.." << llava_session::max_batch_limit << " (sharded: 6 or more, where the shard shapes fit the tiles)" << endl;
+        cerr << "[!] --prompt-batch takes 1.." << arch->max_batch_limit() << " (sharded: 6 or more, where the shard shapes fit the tiles)" << endl;
         return finish(1);
     }
     if (!tokens_path.empty()) {

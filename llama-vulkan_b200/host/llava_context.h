@@ -5,12 +5,14 @@
 #ifndef LLAVA_B200_CONTEXT_H
 #define LLAVA_B200_CONTEXT_H
 
+#include <memory>
 #include <mutex>
 #include <string>
 #include <vector>
 
 #include "../../include/lv_b200.h"
-#include "ggml_file.h"
+#include "model_architecture.h"
+#include "model_file.h"
 #include "types.h"
 
 class llava_context {
@@ -45,7 +47,11 @@ public:
     lv_ctx* lv() const { return lv_context; }
     // the one device arena that holds every weight tensor of the model
     llava_device_memory* weights_memory() const { return shared_memory; }
-    const ggml_file* get_model() const { return model; }
+    const model_file* get_model() const { return model; }
+    model_architecture* architecture() const { return arch.get(); }
+    // arithmetic of models that leave the choice (see model_architecture.h); set before open()
+    void set_compute_type(compute_type t) { compute = t; }
+    compute_type get_compute_type() const { return compute; }
     std::vector<llava_layer*>& get_layers() { return layers; }
     bool upload_from_host(void* device_dst, const void* host_src, size_t bytes);
     bool signal_debug_on() const { return signal_debug; }
@@ -68,7 +74,9 @@ private:
     bool fused_exchange_enabled = true;
     bool setup_signal_handling();
     void close_all();
-    ggml_file* model = nullptr;
+    model_file* model = nullptr;
+    std::unique_ptr<model_architecture> arch;
+    compute_type compute = compute_type::bf16;
     lv_ctx* lv_context = nullptr;
     llava_device_memory* shared_memory = nullptr;
     std::vector<llava_layer*> layers;

@@ -15,7 +15,7 @@ llava_layer::llava_layer(llava_context* _context, u32 _layer_id) : layer_id(_lay
     // every layer's tensors go into the context's one weight arena (the reference gives each layer a
     // device memory of its own, llava_layer.cpp:10-12); see llava_buffer.cpp for why
     layer_allocation = context->weights_memory();
-    const ggml_file* model = context->get_model();
+    const model_file* model = context->get_model();
     const string prefix = "layers." + to_string(layer_id) + ".";
     bool ok = true;
     const u32 rank = context->tp_rank(), n_ranks = context->tp_size();

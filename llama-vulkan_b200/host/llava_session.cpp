@@ -17,6 +17,7 @@
 #include "llava_layer.h"
 #include "tp_shard.h"
 #include "llava_layer_session_data.h"
+#include "model_architecture.h"
 #include "utils.h"
 
 using namespace std;
@@ -28,15 +29,26 @@ constexpr u32 kArgmaxWord = 4;    // argmax written by the recorded step
 constexpr u32 kSampleWord = 5;    // token drawn by the device sampler
 constexpr u32 kStateWords = 8;    // 4 words: sampler state to upload / read back
 constexpr u32 kPinnedExtra = 16;
+constexpr size_t kMaxRecordedSteps = 64;      // prompts of many lengths record many batch sizes
+
+// designs whose session buffers are sized here take any number of tokens, LLaMA sessions always cover the reference's 2048
+u32 session_context(const model_architecture* arch, u32 wanted) {
+    if (wanted > arch->max_context_limit()) return wanted;                       // refused by the constructor
+    if (!arch->has_session_state()) return arch->max_context_limit();
+    return wanted == 0 ? min(max_backlog_size, arch->max_context_limit()) : max(wanted, min_backlog_size);
+}
 }  // namespace
 
-llava_session::llava_session(llava_context* _ctx)
+llava_session::llava_session(llava_context* _ctx, u32 _max_context)
     : ctx(_ctx), model(_ctx->get_model()), rng(u32(time(nullptr))), mirostat_mu(2 * mirostat_tau), sampler_seed(u32(time(nullptr))),
-      backlog_size(min_backlog_size) {
+      max_batch(_ctx->architecture()->default_batch()), backlog_size(min_backlog_size),
+      max_context(session_context(_ctx->architecture(), _max_context)) {
     void* p = nullptr;
-    if (lv_host_alloc(ctx->lv(), size_t(max_backlog_size + kPinnedExtra) * 4, &p) == LV_OK) {
+    if (max_context > ctx->architecture()->max_context_limit()) {
+        failed = true;
+    } else if (lv_host_alloc(ctx->lv(), size_t(max_context + kPinnedExtra) * 4, &p) == LV_OK) {
         pinned = static_cast<u32*>(p);
-        memset(pinned, 0, size_t(max_backlog_size + kPinnedExtra) * 4);
+        memset(pinned, 0, size_t(max_context + kPinnedExtra) * 4);
     } else {
         failed = true;
     }
@@ -47,6 +59,7 @@ llava_session::~llava_session() {
     drop_command_buffers();
     lv_step_plan_destroy(step_plan);
     for (auto* x : layer_data) delete x;
+    state.reset();
     reset_main_buffers();
     if (pinned) lv_host_free(ctx->lv(), pinned);
 }
@@ -59,7 +72,7 @@ void llava_session::drop_command_buffers() {
 
 bool llava_session::ensure_buffers_created() {
     if (failed) return false;
-    if (layer_data.empty()) {
+    if (layer_data.empty() && !ctx->get_layers().empty()) {
         layer_data.reserve(ctx->get_layers().size());
         for (u32 i = 0; i < ctx->get_layers().size(); ++i) layer_data.push_back(new llava_layer_session_data(this));
     }
@@ -117,42 +130,20 @@ void llava_session::ensure_step_plan() {
 
 bool llava_session::recreate_buffers() {
     reset_main_buffers();
-    const ggml_header& h = model->get_header();
-    const u32 dim = h.dim, ff = model->get_ff_size(), B = max_batch;
-    const u32 ranks = ctx->tp_size(), rank = ctx->tp_rank();
-    // per-rank sizes: heads (and with them Q, K, V, the attention output) and the FFN width are
-    // split; the inputs of the column-sharded wo and w2 are padded like their shards
-    const u32 local_dim = dim / ranks;
-    const auto Wt = ctx->output_w->type;
-    const u32 vout_len = ranks == 1 ? dim : tp_shape(Wt, dim, dim, tp_split::columns, rank, ranks).cols;
-    const u32 ff_len = ranks == 1 ? ff : tp_shape(Wt, dim, ff, tp_split::columns, rank, ranks).cols;
     const auto F = ggml_value_type::f32;
     main_buffer_memory = new llava_device_memory(ctx);
     llava_device_memory* m = main_buffer_memory;
-    current_thought = new llava_buffer(ctx, F, dim, B, m);
-    current_thought_sublayer = new llava_buffer(ctx, F, dim, B, m);
-    current_thought_middle_normd = new llava_buffer(ctx, F, dim, B, m);
-    main_ff_result = new llava_buffer(ctx, F, ff_len, B, m);
-    current_Q = new llava_buffer(ctx, F, local_dim, B, m);
-    current_K = new llava_buffer(ctx, F, local_dim, B, m);
-    current_V = new llava_buffer(ctx, F, local_dim, B, m);
-    current_Vout = new llava_buffer(ctx, F, vout_len, B, m);
-    if (ranks > 1) tp_partial = new llava_buffer(ctx, F, dim, B, m);
-    if (is_tracing_enabled()) main_attn_result = new llava_buffer(ctx, F, backlog_size, h.n_heads * B, m);
+    if (!ctx->architecture()->make_scratch(this)) return false;
     config_buffer = new llava_buffer(ctx, F, 4, 1, m);
-    output_probs = new llava_buffer(ctx, F, h.vocab_size, 1, m);
-    token_log = new llava_buffer(ctx, F, max_backlog_size + kPinnedExtra, 1, m);
+    output_probs = new llava_buffer(ctx, F, model->get_header().vocab_size, 1, m);
+    token_log = new llava_buffer(ctx, F, max_context + kPinnedExtra, 1, m);
     argmax_result = new llava_buffer(ctx, F, 4, 1, m);
     sampler_state = new llava_buffer(ctx, F, 4, 1, m);
     sampler_state_dirty = true;
-    const size_t scratch = lv_attention_scratch_bytes(h.n_heads / ranks, h.rot, max_backlog_size, B);
-    if (scratch == 0) return false;
-    attn_scratch = new llava_buffer(ctx, F, u32((scratch + 3) / 4), 1, m);
-    if (B >= llava_command_buffer::kTensorCoreMinBatch)
-        act_split = new llava_buffer(ctx, F, u32(lv_act_split_bytes(max(max(dim, ff_len), vout_len), B) / 4), 1, m);
     if (!m->freeze() || !m->zero(0, m->get_size())) return false;
     device_pos = ~0U;
-    return true;
+    if (!state && ctx->architecture()->has_session_state()) state = ctx->architecture()->make_session_state(this);
+    return !state || state->resize();
 }
 
 void llava_session::reset_main_buffers() {
@@ -193,7 +184,7 @@ float llava_session::get_mirostat_mu() {
 bool llava_session::upload_sampler_state() {
     if (!sampler_state_dirty) return true;
     if (lv_stream_sync(ctx->lv(), 0) != LV_OK) return false;
-    u32* w = pinned + max_backlog_size + kStateWords;
+    u32* w = pinned + max_context + kStateWords;
     memcpy(&w[0], &mirostat_mu, 4);
     w[1] = sampler_seed;
     w[2] = 0;
@@ -203,12 +194,13 @@ bool llava_session::upload_sampler_state() {
     return true;
 }
 
-llava_command_buffer* llava_session::get_command_buffer(u32 batch, bool with_head) {
+llava_command_buffer* llava_session::get_command_buffer(u32 batch, bool with_head, bool row_logits) {
     const bool sample = with_head && sampling_on_device();
-    const u32 key = batch | (with_head ? 1u << 16 : 0u) | (sample ? 1u << 17 : 0u);
+    const u32 key = batch | (with_head ? 1u << 16 : 0u) | (sample ? 1u << 17 : 0u) | (row_logits ? 1u << 18 : 0u);
     auto it = command_buffers.find(key);
     if (it != command_buffers.end()) return it->second;
-    auto* cb = new llava_command_buffer(this, batch, with_head, sample);
+    if (command_buffers.size() >= kMaxRecordedSteps) drop_command_buffers();
+    auto* cb = new llava_command_buffer(this, batch, with_head, sample, row_logits);
     if (!cb->record_execution()) {
         delete cb;
         return nullptr;
@@ -226,8 +218,8 @@ bool llava_session::sync_device_position(u32 pos) {
     if (device_pos == pos) return true;
     // rare (first step, rewind, restore): drain the stream so the staging words are free
     if (lv_stream_sync(ctx->lv(), 0) != LV_OK) return false;
-    for (u32 i = 0; i < 4; ++i) pinned[max_backlog_size + kCfgWords + i] = pos;      // llava_session.cpp:224-225
-    if (lv_upload_async(ctx->lv(), config_buffer->device_ptr(), pinned + max_backlog_size + kCfgWords, 16) != LV_OK) return false;
+    for (u32 i = 0; i < 4; ++i) pinned[max_context + kCfgWords + i] = pos;      // llava_session.cpp:224-225
+    if (lv_upload_async(ctx->lv(), config_buffer->device_ptr(), pinned + max_context + kCfgWords, 16) != LV_OK) return false;
     device_pos = pos;
     return true;
 }
@@ -261,6 +253,54 @@ bool llava_session::start_next_token_prediction() {
         to_process -= n;
     }
     return true;
+}
+
+bool llava_session::evaluate_pending(const vector<u32>& wanted, vector<float>* logits) {
+    if (!ensure_buffers_created()) return false;
+    const u32 vocab = model->get_header().vocab_size, end = u32(token_buffer.size());
+    for (size_t i = 0; i < wanted.size(); ++i)
+        if (wanted[i] < current_tokens_in_gpu || wanted[i] >= end) return false;
+    if (end > backlog_size) return false;
+    logits->assign(wanted.size() * size_t(vocab), 0.0f);
+    const bool rows = !wanted.empty() && ctx->architecture()->has_row_logits();
+    if (rows && !want_row_logits) {
+        lv_stream_sync(ctx->lv(), 0);
+        drop_command_buffers();
+        want_row_logits = true;
+        if (state && !state->resize()) return false;
+    }
+    lock_guard<mutex> guard(ctx->queue_mutex);
+    if (!sync_device_position(current_tokens_in_gpu)) return false;
+    if (current_tokens_in_gpu < end && !upload_pending_tokens(current_tokens_in_gpu, end - current_tokens_in_gpu)) return false;
+    while (current_tokens_in_gpu < end) {
+        const u32 at = current_tokens_in_gpu;
+        u32 n = min(end - at, max_batch);
+        // without row logits a step ends at the next wanted token and gives the logits of that one
+        if (!rows)
+            for (u32 w : wanted)
+                if (w >= at) n = min(n, w - at + 1);
+        if (ctx->tp_size() > 1 && n < llava_command_buffer::kTensorCoreMinBatch) n = 1;
+        bool any = false, last = false;
+        for (u32 w : wanted) {
+            any = any || (w >= at && w < at + n);
+            last = last || w == at + n - 1;
+        }
+        llava_command_buffer* cb = get_command_buffer(n, !rows && last, rows && any);
+        if (cb == nullptr || !cb->run()) return false;
+        batch_size = n;
+        last_command_buffer = cb;
+        current_tokens_in_gpu += n;
+        device_pos += n;
+        if (!any) continue;
+        if (!cb->wait_idle()) return false;
+        for (size_t i = 0; i < wanted.size(); ++i) {
+            if (wanted[i] < at || wanted[i] >= at + n) continue;
+            const bool ok = rows ? state->row_logits()->read_raw(size_t(wanted[i] - at) * vocab * 4, logits->data() + i * vocab, size_t(vocab) * 4)
+                                 : wanted[i] != at + n - 1 || output_probs->read_raw(0, logits->data() + i * vocab, size_t(vocab) * 4);
+            if (!ok) return false;
+        }
+    }
+    return last_command_buffer == nullptr || last_command_buffer->wait_idle();
 }
 
 u32 llava_session::finish_next_token_prediction() {
@@ -303,9 +343,9 @@ u32 llava_session::get_last_predicted_token(bool want_deterministic) {
     if (last_command_buffer && !last_command_buffer->wait_idle()) return ~0U;
     if (want_deterministic) {
         // first index of the largest logit (llava_session.cpp:144-152), computed on the device
-        return pinned[max_backlog_size + kArgmaxWord];
+        return pinned[max_context + kArgmaxWord];
     }
-    if (!host_sampler) return pinned[max_backlog_size + kSampleWord];      // drawn by the recorded step (lv_sample_mirostat)
+    if (!host_sampler) return pinned[max_context + kSampleWord];      // drawn by the recorded step (lv_sample_mirostat)
     vector<float> logits;
     if (!get_logits(&logits)) return ~0U;
     for (float x : logits) {
@@ -362,8 +402,9 @@ bool llava_session::enqueue_greedy_on_device(u32 n) {
     if (!ensure_buffers_created()) return false;
     if (token_buffer.empty() || token_buffer.size() - current_tokens_in_gpu != 1) return false;
     u32 need = backlog_size;
-    while (token_buffer.size() + n > need) need <<= 1;
-    if (need > max_backlog_size || !set_backlog_size(need)) return false;
+    while (need < max_context && token_buffer.size() + n > need) need <<= 1;
+    need = min(need, max_context);
+    if (token_buffer.size() + n > need || !set_backlog_size(need)) return false;
     lock_guard<mutex> guard(ctx->queue_mutex);
     if (!sync_device_position(current_tokens_in_gpu)) return false;
     if (sampling_on_device() && !upload_sampler_state()) return false;
@@ -396,8 +437,8 @@ bool llava_session::set_text(const string& new_text) {
     vector<u32> fresh;
     model->tokenize(fresh, new_text, true);
     u32 next_backlog_size = backlog_size;
-    while (fresh.size() > next_backlog_size) next_backlog_size <<= 1;        // llava_session.cpp:260-266
-    if (next_backlog_size > max_backlog_size) return false;
+    if (fresh.size() > max_context) return false;
+    while (fresh.size() > next_backlog_size) next_backlog_size = min(next_backlog_size * 2, max_context);        // llava_session.cpp:260-266
     if (!set_backlog_size(next_backlog_size)) return false;
     // keep the evaluated prefix that the new token sequence shares with the old one (the
     // reference compares token ids with characters of the text here, llava_session.cpp:271,
@@ -407,7 +448,7 @@ bool llava_session::set_text(const string& new_text) {
            token_buffer[max_prefix] == fresh[max_prefix])
         max_prefix++;
     token_buffer = fresh;
-    current_tokens_in_gpu = max_prefix;
+    if (max_prefix < current_tokens_in_gpu) current_tokens_in_gpu = ctx->architecture()->can_rewind() ? max_prefix : 0;
     return true;
 }
 
@@ -418,15 +459,15 @@ bool llava_session::add_text(const string& s) {
 bool llava_session::push_token(u32 new_token) {
     if (new_token >= model->get_tokens().size()) return false;
     if (token_buffer.size() == backlog_size) {                              // llava_session.cpp:286-294
-        if (backlog_size == max_backlog_size) return false;
-        if (!set_backlog_size(backlog_size * 2)) return false;
+        if (backlog_size == max_context) return false;
+        if (!set_backlog_size(min(backlog_size * 2, max_context))) return false;
     }
     token_buffer.push_back(new_token);
     return true;
 }
 
 bool llava_session::set_backlog_size(u32 new_size) {
-    if (new_size > max_backlog_size) return false;                          // llava_session.cpp:303-315
+    if (new_size > max_context) return false;                               // llava_session.cpp:303-315
     if (new_size == backlog_size) return true;
     if (new_size < min_backlog_size) return false;
     if (new_size < current_tokens_in_gpu) return false;
@@ -446,7 +487,7 @@ bool llava_session::tensor_core_shapes_ok() const {
 }
 
 bool llava_session::set_max_batch(u32 n) {
-    if (n < 1 || n > max_batch_limit) return false;
+    if (n < 1 || n > ctx->architecture()->max_batch_limit()) return false;
     // sharded sessions evaluate prompt batches on the tensor cores (one exchange per sub-block for the whole batch) or,
     // where the shard shapes do not fit the tiles, token by token
     if (n > 1 && ctx->tp_size() > 1 && (n < llava_command_buffer::kTensorCoreMinBatch || !tensor_core_shapes_ok())) return false;
@@ -467,7 +508,7 @@ bool llava_session::flush_layers_data_buffers() {
 void llava_session::rewind(u32 n) {
     if (n < token_buffer.size()) {                                          // llava_session.cpp:390-395
         token_buffer.resize(n);
-        current_tokens_in_gpu = min(n, current_tokens_in_gpu);
+        if (n < current_tokens_in_gpu) current_tokens_in_gpu = ctx->architecture()->can_rewind() ? n : 0;
     }
 }
 
@@ -489,6 +530,7 @@ ReturnCode llava_session::save_frame(const string& path) {
         perror("open");
         return ReturnCode::nok;
     }
+    if (state) state->dump_frame(fd);
     u32 i = 0;
     for (llava_layer_session_data* l : layer_data) l->dump_tracing_layers(fd, "layer." + to_string(i++));
     ::close(fd);
@@ -504,6 +546,7 @@ ReturnCode llava_session::save_frame(const string& path) {
 ReturnCode llava_session::snapshot(const string& path) {
     if (!ensure_buffers_created()) return ReturnCode::nok;
     if (last_command_buffer) last_command_buffer->wait_idle();
+    if (state) return snapshot_state(path);
     const u32 n = current_tokens_in_gpu, dim = model->get_header().dim, ranks = ctx->tp_size(), width = dim / ranks;
     const size_t per_layer = size_t(2) * n * dim * 2, local = size_t(2) * n * width * 2;
     const int fd = ::open(path.c_str(), ranks > 1 ? (O_WRONLY | O_CREAT) : (O_WRONLY | O_CREAT | O_TRUNC), 0644);
@@ -532,6 +575,22 @@ ReturnCode llava_session::snapshot(const string& path) {
     return ok ? ReturnCode::ok : ReturnCode::nok;
 }
 
+// The file of a session whose design keeps its own state: {u32 n; u32 tokens[n]; the state after those tokens}.
+ReturnCode llava_session::snapshot_state(const string& path) {
+    const u32 n = current_tokens_in_gpu;
+    vector<u8> bytes(state->snapshot_bytes(n));
+    if (!state->read_snapshot(bytes.data(), n)) return ReturnCode::nok;
+    const int fd = ::open(path.c_str(), O_WRONLY | O_CREAT | O_TRUNC, 0644);
+    if (fd < 0) {
+        perror("open");
+        return ReturnCode::nok;
+    }
+    bool ok = write_noshort(fd, &n, 4) == 4 && write_noshort(fd, token_buffer.data(), size_t(n) * 4) == size_t(n) * 4 &&
+              write_noshort(fd, bytes.data(), bytes.size()) == bytes.size();
+    if (::close(fd) < 0) ok = false;
+    return ok ? ReturnCode::ok : ReturnCode::nok;
+}
+
 ReturnCode llava_session::restore(const string& path) {
     if (!ensure_buffers_created()) return ReturnCode::nok;
     const int fd = ::open(path.c_str(), O_RDONLY);
@@ -548,19 +607,25 @@ ReturnCode llava_session::restore(const string& path) {
     };
     if (::fstat(fd, &st) < 0 || !S_ISREG(st.st_mode)) return bail("Expected a regular file");
     if (st.st_size < 4 || read_noshort(fd, &n, 4) != 4) return bail("File too short");
-    if (n > max_backlog_size) return bail("Too many tokens");                      // llava_session.cpp:543
+    if (n > max_context) return bail("Too many tokens");                           // llava_session.cpp:543
     const u32 dim = model->get_header().dim;
     const size_t per_layer = size_t(2) * n * dim * 2;
-    const size_t expected = layer_data.size() * per_layer + size_t(4) * n + 4;        // llava_session.cpp:559
+    const size_t expected = (state ? state->snapshot_bytes(n) : layer_data.size() * per_layer) + size_t(4) * n + 4;        // llava_session.cpp:559
     if (expected != size_t(st.st_size)) return bail("File size mismatch");
     u32 needed = min_backlog_size;
     while (needed < n) needed <<= 1;
+    needed = min(needed, max_context);
     vector<u32> toks(n);
     if (read_noshort(fd, toks.data(), size_t(n) * 4) != size_t(n) * 4) return bail("Short read");
     for (u32 t : toks) if (t >= model->get_tokens().size()) return bail("Token id out of range");
     lv_stream_sync(ctx->lv(), 0);
     rewind(0);
     if (!set_backlog_size(needed)) return bail("Cannot set backlog size");
+    if (state) {
+        vector<u8> bytes(state->snapshot_bytes(n));
+        if (pread_noshort(fd, bytes.data(), bytes.size(), 4 + 4ll * n) != bytes.size()) return bail("Short read");
+        if (!state->write_snapshot(bytes.data(), n)) return bail("Cannot upload the session state");
+    }
     // a tensor-parallel rank takes its column slice of every row (see snapshot)
     const u32 ranks = ctx->tp_size(), width = dim / ranks;
     const size_t row_bytes = size_t(width) * 2;

@@ -6,24 +6,32 @@
 #define LLAVA_B200_SESSION_H
 
 #include <map>
+#include <memory>
 #include <random>
 #include <string>
 #include <vector>
 
 #include "../../include/lv_b200.h"
-#include "ggml_file.h"
+#include "model_architecture.h"
+#include "model_file.h"
 #include "types.h"
 
 const u32 min_backlog_size = 128;     // llava_session.cpp:23
-const u32 max_backlog_size = 2048;    // llava_session.cpp:24
+const u32 max_backlog_size = 2048;    // llava_session.cpp:24; longer sessions where the architecture has no such limit
 
 class llava_session {
     friend class llava_layer;
     friend class llava_layer_session_data;
     friend class llava_command_buffer;
     friend class llava_session_group;
+    friend class llama_architecture;
+    friend class hybrid_architecture;
+    friend struct hybrid_recorder;
+    friend class hybrid_session_state;
 public:
-    explicit llava_session(llava_context* ctx);
+    // max_context: tokens the session may hold (0: max_backlog_size, or the architecture's limit if that is lower)
+    explicit llava_session(llava_context* ctx, u32 max_context = 0);
+    bool is_valid() const { return !failed; }
     ~llava_session();
     llava_session(const llava_session&) = delete;
     llava_session& operator=(const llava_session&) = delete;
@@ -55,7 +63,7 @@ public:
     void set_host_sampler(bool on);
     float get_mirostat_mu();
     // tokens evaluated per recorded step while a prompt is ingested (1 ..
-    // max_batch_limit); the reference evaluates the whole prompt as one batch
+    // the architecture's max_batch_limit); the reference evaluates the whole prompt as one batch
     bool set_max_batch(u32 n);
     // whether the batched (tensor-core) products can take this context's matrices: always on one GPU; sharded, the
     // rank's rows of wq / wk / wv must fill 128-row tiles and its rows of w3 / w1 64-row halves
@@ -69,6 +77,9 @@ public:
     // collect waits for them and appends the n tokens.
     bool enqueue_greedy_on_device(u32 n);
     bool collect_greedy_on_device(std::vector<u32>* out);
+    // Evaluates every pending token, as start_next_token_prediction does, and returns the logits of the wanted ones
+    // (indexes into the token buffer, in any order): [wanted][vocab].  Chooses no next token.
+    bool evaluate_pending(const std::vector<u32>& wanted, std::vector<float>* logits);
     // logits of the last evaluated token (vocab floats)
     bool get_logits(std::vector<float>* out);
     u32 get_backlog_size() const { return backlog_size; }
@@ -78,10 +89,8 @@ public:
     bool read_step_trace(std::vector<u64>* out, u32* n_ops, u32* n_ctas, u32* n_points);
     u32 step_kernel_launches() const;          // kernel launches of one replay of the step evaluated last
 
-    static constexpr u32 max_batch_limit = 64;
-
     llava_context* const ctx;
-    ggml_file const* const model;
+    model_file const* const model;
 
 private:
     std::mt19937 rng;
@@ -119,11 +128,18 @@ private:
     llava_buffer* sampler_state = nullptr;        // device sampler: {mu, seed, draws, -}
     llava_buffer* act_split = nullptr;            // max_batch >= 6: fp16 (hi, lo) planes of a batch of activations
     llava_buffer* tp_partial = nullptr;           // tensor-parallel only: this rank's partial wo / w2 product
-    std::vector<llava_layer_session_data*> layer_data;
+    std::vector<llava_layer_session_data*> layer_data;      // LLaMA layers; other designs keep theirs in `state`
+    std::unique_ptr<session_state> state;
 
     u32 batch_size = 0;           // batch of the step recorded last
-    u32 max_batch = 1;
+    u32 max_batch;
     u32 backlog_size;
+    const u32 max_context;        // tokens the session may hold: rows of its caches
+    bool want_row_logits = false; // steps may produce the logits of all their rows (evaluate_pending)
+    u32 log_capacity() const { return max_context + 1; }
+    u32* argmax_word() const { return pinned + max_context + 4; }
+    u32* sample_word() const { return pinned + max_context + 5; }
+    ReturnCode snapshot_state(const std::string& path);
     u32 get_last_predicted_token(bool deterministic);
     u32 sample_from_logits(std::vector<float>& logits);
 
@@ -132,21 +148,21 @@ private:
     bool set_backlog_size(u32 new_size);
     bool ensure_buffers_created();
     void drop_command_buffers();
-    llava_command_buffer* get_command_buffer(u32 batch, bool with_head);
+    llava_command_buffer* get_command_buffer(u32 batch, bool with_head, bool row_logits = false);
     bool sampling_on_device() const { return !deterministic && !host_sampler; }
 public:
     bool samples_on_host() const { return !deterministic && host_sampler; }
 private:
     bool upload_sampler_state();
 
-    // key: batch | with_head << 16 | device sampler << 17
+    // key: batch | with_head << 16 | device sampler << 17 | row logits << 18
     std::map<u32, llava_command_buffer*> command_buffers;
     llava_command_buffer* last_command_buffer = nullptr;
 
     std::vector<u32> token_buffer;
     u32 current_tokens_in_gpu = 0;
     u32 device_pos = ~0U;         // value of config_buffer on the device as far as the host knows
-    u32* pinned = nullptr;        // [max_backlog] token staging + [8] config/argmax words
+    u32* pinned = nullptr;        // [max_context] token staging + [8] config/argmax words
     bool upload_pending_tokens(u32 first, u32 count);
     bool sync_device_position(u32 pos);
 

@@ -21,7 +21,7 @@ float* f32(llava_buffer* b) { return static_cast<float*>(b->device_ptr()); }
 
 llava_session_group::llava_session_group(llava_context* _ctx, vector<llava_session*> _members) : ctx(_ctx), members(std::move(_members)) {
     const u32 k = u32(members.size());
-    if (ctx == nullptr || ctx->lv() == nullptr || ctx->tp_size() != 1 || k < 2 || k > llava_session::max_batch_limit) return;
+    if (ctx == nullptr || ctx->lv() == nullptr || !ctx->architecture()->can_group() || ctx->tp_size() != 1 || k < 2 || k > max_members) return;
     for (llava_session* s : members)
         if (s == nullptr || s->ctx != ctx || s->is_tracing_enabled()) return;
     for (u32 i = 0; i < k; ++i)

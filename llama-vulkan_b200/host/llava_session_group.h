@@ -27,6 +27,7 @@ public:
     llava_session_group(const llava_session_group&) = delete;
     llava_session_group& operator=(const llava_session_group&) = delete;
 
+    static constexpr u32 max_members = 64;
     bool is_valid() const { return valid; }
     u32 size() const { return u32(members.size()); }
     // Every member must hold exactly one token that is not evaluated yet (the one pushed last).  Evaluates it for all

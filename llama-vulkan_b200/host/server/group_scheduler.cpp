@@ -63,7 +63,7 @@ void group_scheduler::forget(llava_session* session) {
 u32 group_scheduler::evaluate(llava_session* session) {
     // what a group step cannot serve goes through the session's own step
     const bool groupable = session->get_token_count() - session->get_tokens_in_gpu() == 1 && !session->samples_on_host() &&
-                           !session->is_tracing_enabled() && ctx->tp_size() == 1;
+                           !session->is_tracing_enabled() && ctx->tp_size() == 1 && ctx->architecture()->can_group();
     if (!groupable) {
         settle(session);
         return session->predict_next_token();
@@ -91,7 +91,7 @@ u32 group_scheduler::evaluate(llava_session* session) {
 void group_scheduler::lead(unique_lock<mutex>& lock) {
     const auto t_begin = chrono::steady_clock::now();
     const auto deadline = t_begin + kWindow;
-    cv_leader.wait_until(lock, deadline, [&]() { return waiting.size() >= max<u32>(runners, 1u) || waiting.size() >= llava_session::max_batch_limit; });
+    cv_leader.wait_until(lock, deadline, [&]() { return waiting.size() >= max<u32>(runners, 1u) || waiting.size() >= llava_session_group::max_members; });
     const auto t_collected = chrono::steady_clock::now();
     us_collect += u64(chrono::duration_cast<chrono::microseconds>(t_collected - t_begin).count());
     struct device_timer {
@@ -101,9 +101,9 @@ void group_scheduler::lead(unique_lock<mutex>& lock) {
     } timer{us_device, t_collected};
     vector<llava_session*> round;
     round.swap(waiting);
-    if (round.size() > llava_session::max_batch_limit) {          // the rest forms the next round
-        waiting.assign(round.begin() + llava_session::max_batch_limit, round.end());
-        round.resize(llava_session::max_batch_limit);
+    if (round.size() > llava_session_group::max_members) {          // the rest forms the next round
+        waiting.assign(round.begin() + llava_session_group::max_members, round.end());
+        round.resize(llava_session_group::max_members);
     }
     vector<u32> tokens(round.size(), ~0U);
     vector<llava_session*> key = round;
