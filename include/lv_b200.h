@@ -461,6 +461,32 @@ typedef struct lv_expert_args {
 int lv_gemv_bf16_expert_gate_up(lv_ctx* ctx, float* out, uint32_t out_ld, const lv_expert_args* a, const float* x, uint32_t x_ld, uint32_t batch);
 int lv_gemv_bf16_expert_down(lv_ctx* ctx, float* out, uint32_t out_ld, const lv_expert_args* a, const float* x, uint32_t x_ld, uint32_t batch);
 
+/* Products of a batch on the tensor cores: x and W bfloat16, f32 sums, one pass over the weights for up to 128 tokens.
+ * x [batch][x_ld] with x_ld a multiple of 8; out f32 or bfloat16 [batch][out_ld]. */
+int lv_gemm_bf16(lv_ctx* ctx, void* out, int out_type, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols,
+                 const void* x, uint32_t x_ld, uint32_t batch, float factor);
+/* The experts of a batch.  lv_expert_route sorts the (token, choice) pairs of each job's layer by expert: index[t * top + s] =
+ * row of choice s of token t, and lists tiles of up to tile_rows = lv_expert_tile_rows(batch, top, experts) rows of one expert
+ * (max_tiles = lv_expert_max_tiles entries, unused ones with rows 0).  The products below read and write rows in that order.
+ * jobs: device array. */
+typedef struct lv_expert_tile { uint32_t expert, row0, rows; } lv_expert_tile;
+typedef struct lv_route_job {
+    const uint32_t* table;
+    uint32_t experts, top;
+    uint32_t* index;
+    lv_expert_tile* tiles;
+    uint32_t max_tiles, unused;
+} lv_route_job;
+uint32_t lv_expert_tile_rows(uint32_t batch, uint32_t top, uint32_t experts);
+uint32_t lv_expert_max_tiles(uint32_t batch, uint32_t top, uint32_t experts);
+int lv_expert_route(lv_ctx* ctx, const lv_route_job* jobs, uint32_t n_jobs, uint32_t max_experts, const uint32_t* token_log,
+                    const uint32_t* pos, uint32_t vocab, uint32_t batch);
+/* out bfloat16 [batch * top][out_ld] = silu(gate_e x) * (up_e x);  out f32 [batch * top][out_ld] = down_e x */
+int lv_gemm_bf16_expert_gate_up(lv_ctx* ctx, void* out, uint32_t out_ld, const lv_expert_args* a, const lv_expert_tile* tiles, const void* x,
+                                uint32_t x_ld, uint32_t batch);
+int lv_gemm_bf16_expert_down(lv_ctx* ctx, float* out, uint32_t out_ld, const lv_expert_args* a, const lv_expert_tile* tiles, const void* x,
+                             uint32_t x_ld, uint32_t batch);
+
 /* Causal attention with grouped key/value heads: query and key RMS norm per head (plain weights), scores
  * (q . k) * scale - r1_h ln(1 + r2_h (i - j)), softmax with `sink` (0 or 1) added to the denominator.
  * qkv f32 [batch][qkv_ld]: heads * dim queries, kv_heads * dim keys, kv_heads * vdim values of each token, as projected.

@@ -135,6 +135,12 @@ KERNEL_API = {
     "lv_mingru_scan": (_int, [_p, _p, _int, _u32, _p, _u32, _u32, _p, _p, _p, _p, _u32]),
     "lv_gemv_bf16_expert_gate_up": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _u32, _u32]),
     "lv_gemv_bf16_expert_down": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _u32, _u32]),
+    "lv_gemm_bf16": (_int, [_p, _p, _int, _u32, _p, _u32, _u32, _u32, _p, _u32, _u32, _f32]),
+    "lv_expert_tile_rows": (_u32, [_u32, _u32, _u32]),
+    "lv_expert_max_tiles": (_u32, [_u32, _u32, _u32]),
+    "lv_expert_route": (_int, [_p, _p, _u32, _u32, _p, _p, _u32, _u32]),
+    "lv_gemm_bf16_expert_gate_up": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _p, _u32, _u32]),
+    "lv_gemm_bf16_expert_down": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _p, _u32, _u32]),
     "lv_qk_norm_append": (_int, [_p, C.POINTER(GqaArgs), _u32]),
     "lv_gqa_scratch_bytes": (_sz, [_p, C.POINTER(GqaArgs), _u32, _u32]),
     "lv_attention_gqa": (_int, [_p, C.POINTER(GqaArgs), _p, _sz, _u32, _u32, _int]),

@@ -67,6 +67,7 @@ extern "C" int lv_ctx_create(int device, lv_ctx** out) {
     int rc = gemv_configure(ctx);
     if (rc == LV_OK) rc = attention_configure(ctx);
     if (rc == LV_OK) rc = gemm_tc_configure(ctx);
+    if (rc == LV_OK) rc = gemm_bf16_configure(ctx);
     if (rc != LV_OK) {
         lv_ctx_destroy(ctx);
         return rc;
@@ -82,6 +83,7 @@ extern "C" int lv_ctx_destroy(lv_ctx* ctx) {
     if (ctx->comm) lv_comm_destroy(ctx);
     if (ctx->stream) { cudaStreamSynchronize(ctx->stream); cudaStreamDestroy(ctx->stream); }
     gemm_tc_release(ctx);
+    gemm_bf16_release(ctx);
     if (ctx->d_err) cudaFree(ctx->d_err);
     if (ctx->h_err) cudaFreeHost(ctx->h_err);
     delete ctx;

@@ -24,6 +24,8 @@ struct lv_ctx {
     bool peer_ready = false;
     void* tc_scratch = nullptr;       // partial accumulators of the K-split tensor-core products
     void* tc_counters = nullptr;
+    void* bg_scratch = nullptr;       // the same for the bfloat16 products
+    void* bg_counters = nullptr;
     bool tc_exact = false;            // batched q4_0 products with the exact hi/lo weight planes instead of one fp16 plane
     // exchange roles that lv_tp_arm_push / lv_tp_arm_pull set for the next GEMV-family launch
     struct {
@@ -42,6 +44,8 @@ int gemv_configure(lv_ctx* ctx);
 int attention_configure(lv_ctx* ctx);
 int gemm_tc_configure(lv_ctx* ctx);
 void gemm_tc_release(lv_ctx* ctx);
+int gemm_bf16_configure(lv_ctx* ctx);
+void gemm_bf16_release(lv_ctx* ctx);
 uint32_t* peer_step_counter(lv_ctx* ctx);
 bool peer_windows(lv_ctx* ctx, float** windows, int* n_ranks, int* rank, uint32_t* capacity);   // the connected peer windows, if any          // device word counting evaluation steps, or null without a peer window
 

@@ -15,4 +15,8 @@ int make_weight_map(CUtensorMap* out, const void* base, uint32_t rows, uint32_t 
 // of 16) belongs to dims[i + 1]; box[i] <= 256.  No swizzle; out-of-range elements read as zero.
 int make_tiled_map(CUtensorMap* out, const void* base, uint32_t rank, const uint64_t* dims, const uint64_t* strides, const uint32_t* box);
 
+// [rows][cols] bfloat16 matrix with ld elements from row to row (a multiple of 8); a box is box_rows rows of 64 columns,
+// stored with the 128-byte swizzle (one 128-byte shared-memory row each).  Out-of-range elements read as zero.
+int make_bf16_map(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows);
+
 }  // namespace lv

@@ -218,18 +218,25 @@ struct hybrid_recorder {
     hybrid_session_state* st;
     lv_ctx* lv;
     u32 T;
+    bool batched;                        // tensor-core products on bfloat16 activations
     const u32* pos;
     const u32* log;
     // residual stream; null until the embedding rows have been read
     float* x = nullptr;
     // the sublayer that the next norm_conv finishes
     const float* y = nullptr;
+    const u32* y_index = nullptr;
+    u32 y_rows = 1;
     const llava_buffer* post = nullptr;
     int finished_run = -1;               // the layer run that ends with it, for traces
 
     static float* f32(const llava_buffer* b) { return b ? static_cast<float*>(b->device_ptr()) : nullptr; }
+    static u32 pad8(u32 n) { return (n + 7) / 8 * 8; }
+    int act_type() const { return batched ? LV_TYPE_BF16 : LV_TYPE_F32; }
 
-    void norm_conv(const llava_buffer* pre, const llava_buffer* conv, llava_buffer* history, const float* step, u32 first = 0) {
+    // rows: destination rows of every token (experts), null for one row per token
+    void norm_conv(const llava_buffer* pre, const llava_buffer* conv, llava_buffer* history, const float* step, const llava_buffer* rows = nullptr,
+                   u32 copies = 1, bool last_only = false) {
         lv_norm_conv_args a{};
         a.x = x;
         a.embed = arch.embed->device_ptr();
@@ -238,7 +245,8 @@ struct hybrid_recorder {
         a.token_log = log;
         a.pos = pos;
         a.y = y;
-        a.y_rows = 1;
+        a.y_index = y_index;
+        a.y_rows = y_rows;
         a.mult = cfg.residual_mult;
         a.eps = cfg.eps;
         a.post_w = f32(post);
@@ -252,28 +260,33 @@ struct hybrid_recorder {
             a.history = f32(history);
         }
         a.out = f32(st->normed);
-        a.out_type = LV_TYPE_F32;
-        a.out_ld = (cfg.width + 7) / 8 * 8;
+        a.out_type = last_only ? LV_TYPE_F32 : act_type();
+        a.out_ld = pad8(cfg.width);
+        a.out_index = rows ? static_cast<const u32*>(rows->device_ptr()) : nullptr;
+        a.out_copies = copies;
         a.width = cfg.width;
-        a.first = first;
+        a.first = last_only ? T - 1 : 0;
         a.batch = T;
         cb->note(lv_norm_conv(lv, &a));
         x = a.x_out;
         y = nullptr;
+        y_index = nullptr;
+        y_rows = 1;
         post = nullptr;
         finished_run = -1;
     }
 
-    void product(llava_buffer* out, u32 out_ld, const llava_buffer* w, llava_buffer* in, u32 in_ld, u32 batch, float factor = 1.0f) {
-        cb->note(lv_gemv_bf16(lv, f32(out), out_ld, w->device_ptr(), w->shape.first, w->leading(), w->shape.second, f32(in), in_ld, batch, factor));
+    void product(llava_buffer* out, const llava_buffer* w, llava_buffer* in, u32 in_ld, float factor = 1.0f) {
+        const u32 rows = w->shape.first;
+        if (batched) cb->note(lv_gemm_bf16(lv, f32(out), LV_TYPE_F32, rows, w->device_ptr(), rows, w->leading(), w->shape.second, f32(in), in_ld, T, factor));
+        else cb->note(lv_gemv_bf16(lv, f32(out), rows, w->device_ptr(), rows, w->leading(), w->shape.second, f32(in), in_ld, T, factor));
     }
 
     void attention(const hybrid_layer& l, const hybrid_mixer& m, const hybrid_run_state& r) {
-        const u32 ld = (cfg.width + 7) / 8 * 8, raw_ld = m.raw_size(), out_ld = (m.out_size() + 7) / 8 * 8;
-        product(st->raw, raw_ld, l.in, st->normed, ld, T);
+        product(st->raw, l.in, st->normed, pad8(cfg.width));
         lv_gqa_args a{};
         a.qkv = f32(st->raw);
-        a.qkv_ld = raw_ld;
+        a.qkv_ld = m.raw_size();
         a.heads = m.heads;
         a.kv_heads = m.kv_heads;
         a.dim = m.dim;
@@ -291,49 +304,57 @@ struct hybrid_recorder {
         a.ctx_rows = s->max_context;
         a.pos = pos;
         a.out = f32(st->mixed);
-        a.out_type = LV_TYPE_F32;
-        a.out_ld = out_ld;
+        a.out_type = act_type();
+        a.out_ld = pad8(m.out_size());
         if (T > 1) cb->note(lv_qk_norm_append(lv, &a, T));
         cb->note(lv_attention_gqa(lv, &a, st->attn_scratch->device_ptr(), st->attn_scratch->byte_size(), T, cb->backlog_size, T == 1));
-        product(st->sub, cfg.width, l.out, st->mixed, out_ld, T);
+        product(st->sub, l.out, st->mixed, a.out_ld);
     }
 
     void mingru(const hybrid_layer& l, const hybrid_mixer& m, const hybrid_run_state& r) {
-        const u32 ld = (cfg.width + 7) / 8 * 8, out_ld = (m.width + 7) / 8 * 8;
         if (T == 1) {
             const u16* w = static_cast<const u16*>(l.in->device_ptr());
             const size_t each = size_t(m.width) * l.in->leading();
             cb->note(lv_gemv_bf16_mingru(lv, f32(st->mixed), w, w + each, w + 2 * each, l.in->leading(), m.width, cfg.width, f32(l.z_bias), f32(l.x_bias),
                                          f32(st->normed), f32(r.gru_state), pos));
         } else {
-            product(st->raw, m.raw_size(), l.in, st->normed, ld, T);
-            cb->note(lv_mingru_scan(lv, f32(st->mixed), LV_TYPE_F32, out_ld, f32(st->raw), m.raw_size(), m.width, f32(l.z_bias), f32(l.x_bias),
+            product(st->raw, l.in, st->normed, pad8(cfg.width));
+            cb->note(lv_mingru_scan(lv, f32(st->mixed), act_type(), pad8(m.width), f32(st->raw), m.raw_size(), m.width, f32(l.z_bias), f32(l.x_bias),
                                     f32(r.gru_state), pos, T));
         }
-        product(st->sub, cfg.width, l.out, st->mixed, out_ld, T);
+        product(st->sub, l.out, st->mixed, pad8(m.width));
     }
 
-    void experts(const hybrid_layer& l, const hybrid_experts& e) {
-        const u32 ld = (cfg.width + 7) / 8 * 8, act_ld = (e.ff + 7) / 8 * 8;
-        lv_expert_args a{};
-        a.w0 = l.gate->device_ptr();
-        a.w1 = l.up->device_ptr();
-        a.ld = l.gate->leading();
-        a.rows = e.ff;
-        a.cols = cfg.width;
-        a.experts = e.experts;
-        a.top = e.top;
-        a.vocab = cfg.vocab;
-        a.table = static_cast<const u32*>(l.table->device_ptr());
-        a.token_log = log;
-        a.pos = pos;
-        cb->note(lv_gemv_bf16_expert_gate_up(lv, f32(st->act), act_ld, &a, f32(st->normed), ld, T));
-        a.w0 = l.down->device_ptr();
-        a.w1 = nullptr;
-        a.ld = l.down->leading();
-        a.rows = cfg.width;
-        a.cols = e.ff;
-        cb->note(lv_gemv_bf16_expert_down(lv, f32(st->sub), cfg.width, &a, f32(st->act), act_ld, T));
+    void experts(u32 layer, const hybrid_layer& l, const hybrid_experts& e) {
+        const u32 ld = pad8(cfg.width), act_ld = pad8(e.ff);
+        lv_expert_args gate_up{}, down{};
+        gate_up.w0 = l.gate->device_ptr();
+        gate_up.w1 = l.up->device_ptr();
+        gate_up.ld = l.gate->leading();
+        gate_up.rows = e.ff;
+        gate_up.cols = cfg.width;
+        gate_up.experts = e.experts;
+        gate_up.top = e.top;
+        gate_up.vocab = cfg.vocab;
+        gate_up.table = static_cast<const u32*>(l.table->device_ptr());
+        gate_up.token_log = log;
+        gate_up.pos = pos;
+        down = gate_up;
+        down.w0 = l.down->device_ptr();
+        down.w1 = nullptr;
+        down.ld = l.down->leading();
+        down.rows = cfg.width;
+        down.cols = e.ff;
+        if (batched) {
+            const auto* tiles = static_cast<const lv_expert_tile*>(st->route_tiles[layer]->device_ptr());
+            cb->note(lv_gemm_bf16_expert_gate_up(lv, f32(st->act), act_ld, &gate_up, tiles, f32(st->normed), ld, T));
+            cb->note(lv_gemm_bf16_expert_down(lv, f32(st->sub), cfg.width, &down, tiles, f32(st->act), act_ld, T));
+            y_index = static_cast<const u32*>(st->route_index[layer]->device_ptr());      // the next norm_conv averages the choices
+            y_rows = e.top;
+        } else {
+            cb->note(lv_gemv_bf16_expert_gate_up(lv, f32(st->act), act_ld, &gate_up, f32(st->normed), ld, T));
+            cb->note(lv_gemv_bf16_expert_down(lv, f32(st->sub), cfg.width, &down, f32(st->act), act_ld, T));
+        }
     }
 
     void finish_sublayer(const llava_buffer* norm) {
@@ -343,31 +364,37 @@ struct hybrid_recorder {
 
     void step() {
         const auto& runs = arch.runs_in_order();
+        if (batched && st->n_route_jobs)
+            cb->note(lv_expert_route(lv, static_cast<const lv_route_job*>(st->route_jobs->device_ptr()), st->n_route_jobs, st->max_experts, log, pos, cfg.vocab, T));
         for (size_t i = 0; i < runs.size(); ++i) {
-            const hybrid_layer& l = arch.layer(runs[i].layer);
-            const hybrid_layer_spec& spec = cfg.layers[runs[i].layer];
+            const u32 layer = runs[i].layer;
+            const hybrid_layer& l = arch.layer(layer);
+            const hybrid_layer_spec& spec = cfg.layers[layer];
             const hybrid_run_state& r = st->runs[i];
             norm_conv(l.norm1, l.canon1, r.history1, runs[i].begins_pass >= 0 ? f32(arch.loop_step) + size_t(runs[i].begins_pass) * cfg.width : nullptr);
             if (spec.mixer.type == hybrid_mixer::kind::attention) attention(l, spec.mixer, r);
             else mingru(l, spec.mixer, r);
             finish_sublayer(l.norm1b);
             if (spec.mlp.experts) {
-                norm_conv(l.norm2, l.canon2, r.history2, nullptr);
-                experts(l, spec.mlp);
+                norm_conv(l.norm2, l.canon2, r.history2, nullptr, batched ? st->route_index[layer] : nullptr, spec.mlp.top);
+                experts(layer, l, spec.mlp);
                 finish_sublayer(l.norm2b);
             }
             finished_run = int(i);
         }
-        const u32 ld = (cfg.width + 7) / 8 * 8;
         if (cb->row_logits) {
             norm_conv(arch.final_norm, nullptr, nullptr, nullptr);
-            product(st->logits_rows, cfg.vocab, arch.head, st->normed, ld, T, cfg.logit_scale);
+            product(st->logits_rows, arch.head, st->normed, pad8(cfg.width), cfg.logit_scale);
         } else if (cb->with_head) {
-            // only the last row's logits are wanted (a trace wants the last layer's stream of every row)
-            const u32 first = st->trace.empty() ? T - 1 : 0;
-            norm_conv(arch.final_norm, nullptr, nullptr, nullptr, first);
+            // only the last row's logits are wanted; a trace wants the last layer's stream of every row as well
+            if (!st->trace.empty() && T > 1) {
+                const hybrid_recorder before = *this;
+                norm_conv(arch.final_norm, nullptr, nullptr, nullptr);
+                x = before.x, y = before.y, y_index = before.y_index, y_rows = before.y_rows, post = before.post;
+            }
+            norm_conv(arch.final_norm, nullptr, nullptr, nullptr, nullptr, 1, true);
             cb->note(lv_gemv_bf16(lv, f32(s->output_probs), cfg.vocab, arch.head->device_ptr(), cfg.vocab, arch.head->leading(), cfg.width,
-                                  f32(st->normed) + size_t(T - 1 - first) * ld, ld, 1, cfg.logit_scale));
+                                  f32(st->normed), pad8(cfg.width), 1, cfg.logit_scale));
         }
         cb->finish_step();
     }
@@ -377,7 +404,7 @@ void hybrid_architecture::record(llava_command_buffer* cb) {
     llava_session* s = cb->session;
     auto* st = static_cast<hybrid_session_state*>(s->state.get());
     if (!cb->expect(st != nullptr && cb->batch_size <= s->max_batch, "session state")) return;
-    hybrid_recorder r{*this, cfg, cb, s, st, s->ctx->lv(), cb->batch_size, static_cast<const u32*>(s->config_buffer->device_ptr()),
+    hybrid_recorder r{*this, cfg, cb, s, st, s->ctx->lv(), cb->batch_size, st->batched(cb->batch_size), static_cast<const u32*>(s->config_buffer->device_ptr()),
                       static_cast<const u32*>(s->token_log->device_ptr())};
     r.step();
 }

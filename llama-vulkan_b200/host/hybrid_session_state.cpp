@@ -47,12 +47,15 @@ hybrid_session_state::~hybrid_session_state() {
 }
 
 void hybrid_session_state::drop_scratch() {
-    for (llava_buffer** b : {&stream_a, &stream_b, &normed, &raw, &mixed, &act, &sub, &attn_scratch, &logits_rows}) {
+    for (llava_buffer** b : {&stream_a, &stream_b, &normed, &raw, &mixed, &act, &sub, &attn_scratch, &logits_rows, &route_jobs}) {
         delete *b;
         *b = nullptr;
     }
-    for (llava_buffer* b : trace) delete b;
-    trace.clear();
+    for (auto* list : {&trace, &route_index, &route_tiles}) {
+        for (llava_buffer* b : *list) delete b;
+        list->clear();
+    }
+    n_route_jobs = max_experts = 0;
     delete scratch;
     scratch = nullptr;
     scratch_batch = 0;
@@ -94,17 +97,50 @@ bool hybrid_session_state::resize() {
     act = new llava_buffer(ctx, F, act_size, B, scratch);
     sub = new llava_buffer(ctx, F, c.width * copies, B, scratch);
     if (attention_bytes) attn_scratch = new llava_buffer(ctx, F, u32((attention_bytes + 3) / 4), 1, scratch);
+    for (const hybrid_layer_spec& l : c.layers) {
+        const hybrid_experts& e = l.mlp;
+        if (f32 || e.experts == 0) {
+            route_index.push_back(nullptr);
+            route_tiles.push_back(nullptr);
+            continue;
+        }
+        u32 tiles = 0;                                         // the tile size follows the batch, every batch must fit
+        for (u32 n = 2; n <= max(B, 2u); ++n) tiles = max(tiles, lv_expert_max_tiles(n, e.top, e.experts));
+        route_index.push_back(new llava_buffer(ctx, F, e.top, B, scratch));
+        route_tiles.push_back(new llava_buffer(ctx, F, u32(sizeof(lv_expert_tile) / 4), tiles, scratch));
+        max_experts = max(max_experts, e.experts);
+        ++n_route_jobs;
+    }
+    if (n_route_jobs) route_jobs = new llava_buffer(ctx, F, u32(sizeof(lv_route_job) / 4), n_route_jobs, scratch);
     if (want_rows) logits_rows = new llava_buffer(ctx, F, c.vocab, B, scratch);
     if (want_trace)
         for (size_t r = 0; r < runs.size(); ++r) {            // numbered so that frames list them in order
             const string n = to_string(r);
             trace.push_back(new llava_buffer(ctx, F, c.width, B, scratch, "run." + string(4 - min<size_t>(4, n.size()), '0') + n + ".residual"));
         }
-    if (!scratch->freeze() || !scratch->zero(0, scratch->get_size())) return false;
+    if (!scratch->freeze() || !scratch->zero(0, scratch->get_size()) || !upload_route_jobs()) return false;
     scratch_batch = B;
     scratch_trace = want_trace;
     scratch_rows = want_rows;
     return true;
+}
+
+bool hybrid_session_state::upload_route_jobs() {
+    if (n_route_jobs == 0) return true;
+    vector<lv_route_job> jobs;
+    for (size_t i = 0; i < route_index.size(); ++i) {
+        if (route_index[i] == nullptr) continue;
+        const hybrid_experts& e = arch->config().layers[i].mlp;
+        lv_route_job j{};
+        j.table = static_cast<const u32*>(arch->layer(u32(i)).table->device_ptr());
+        j.experts = e.experts;
+        j.top = e.top;
+        j.index = static_cast<u32*>(route_index[i]->device_ptr());
+        j.tiles = static_cast<lv_expert_tile*>(route_tiles[i]->device_ptr());
+        j.max_tiles = route_tiles[i]->shape.second;
+        jobs.push_back(j);
+    }
+    return route_jobs->write_raw(0, jobs.data(), jobs.size() * sizeof(lv_route_job));
 }
 
 void hybrid_session_state::dump_frame(int fd) {

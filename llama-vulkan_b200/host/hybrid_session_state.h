@@ -36,9 +36,14 @@ public:
     llava_buffer *act = nullptr;                              // expert activations
     llava_buffer *sub = nullptr;                              // output of a sublayer, f32
     llava_buffer *attn_scratch = nullptr;
+    llava_buffer *route_jobs = nullptr;                       // lv_route_job per layer with experts, in layer order
+    std::vector<llava_buffer*> route_index, route_tiles;      // per layer; null without experts
+    u32 n_route_jobs = 0, max_experts = 0;
     llava_buffer *logits_rows = nullptr;                      // f32 [batch][vocab], only for evaluate_pending
     std::vector<llava_buffer*> trace;                         // per layer run: the residual stream after it, only when tracing
     u32 cache_bytes() const { return f32 ? 4 : 2; }
+    // several tokens go through the tensor-core products (bfloat16 activations), one token through f32 activations
+    bool batched(u32 tokens) const { return !f32 && tokens > 1; }
     bool const f32;                                           // 32-bit arithmetic: activations and caches are f32
 
 private:
@@ -46,6 +51,7 @@ private:
     bool transfer(u8* dst, const u8* src, u32 n);
     llava_device_memory* lasting = nullptr;
     llava_device_memory* scratch = nullptr;
+    bool upload_route_jobs();
     u32 scratch_batch = 0;
     bool scratch_trace = false, scratch_rows = false;
 };
