@@ -7,7 +7,7 @@
 // One CTA serves up to eight query heads of one key/value head for one token and walks its share of the keys in chunks of
 // 128 with an online softmax.  A decoded token spreads the chunks over several CTAs (the last to arrive combines their
 // partial sums through scratch) and its own key and value are normalised and appended to the caches by the same launch;
-// tokens of a prompt are appended first (lv_qk_norm_append).  Caches are [kv head][ctx_rows][padded dim], bfloat16 or f32.
+// tokens of a prompt are appended first (lv_qk_norm_append) and, with bfloat16 caches, go through attention_gqa_tc.cu.  Caches are [kv head][ctx_rows][padded dim], bfloat16 or f32.
 #include <cuda_bf16.h>
 #include <math.h>
 
@@ -341,6 +341,7 @@ extern "C" int lv_attention_gqa(lv_ctx* ctx, const lv_gqa_args* a, void* scratch
     if (const int rc = gqa_check(a, batch)) return rc;
     LV_REQUIRE(a->out && a->out_ld >= a->heads * a->vdim && (a->out_type == LV_TYPE_F32 || a->out_type == LV_TYPE_BF16), "attention: bad output");
     LV_REQUIRE(capacity && capacity <= a->ctx_rows && (!append || batch == 1), "attention: bad capacity");
+    if (!append && gqa_tc_supported(*a, batch)) return gqa_tc_launch(ctx, *a, batch);
     GqaParams p{};
     p.a = *a;
     p.dim_p = pad8(a->dim);

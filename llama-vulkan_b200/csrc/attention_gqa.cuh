@@ -3,9 +3,14 @@
 
 #include <cuda_bf16.h>
 
+#include "../../include/lv_b200.h"
 #include "common.cuh"
 
 namespace lv {
+
+// attention_gqa_tc.cu: the form for several tokens and bfloat16 caches
+bool gqa_tc_supported(const lv_gqa_args& a, uint32_t batch);
+int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch);
 
 // 1 / rms of one head's vector, computed by a warp (every lane gets it)
 __device__ __forceinline__ float gqa_rms_factor(const float* v, uint32_t dim, float eps) {

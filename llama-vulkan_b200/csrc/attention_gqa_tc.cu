@@ -1,0 +1,335 @@
+// The attention of attention_gqa.cu for the tokens of a prompt, on the tcgen05 tensor cores (bfloat16 caches).
+//
+// A CTA takes 128 query rows of one key/value head -- row r is query head r mod group of token r / group, so that grouped
+// heads share the keys -- and walks the keys in blocks of 64:
+//
+//   S = Q K^T      Q normalised, scaled and rounded to bfloat16 in shared memory (128-byte swizzle), K by TMA from the cache
+//   P = exp2(S - bias - m)      four warps, one row per thread; P goes to tensor memory over the scores it came from
+//   O += P V       P is the TMEM operand, V by TMA as an MN-major operand (its rows are keys)
+//
+// Two score buffers let S of the next block run under the softmax of this one.  The distance bias of a block is a small
+// table per head: distances within a block and a tile differ by less than (tokens + 64), so log1p is evaluated once per
+// (head, distance) instead of once per score.  O stays in tensor memory; it is rescaled only when a row's maximum has grown
+// by more than 2^8, which with a sink (maximum >= 0 from the start) is rare.  Everything except the operands is f32.
+//
+// Every wait is bounded (common.cuh); a lost wait sets the error word, the CTA drains and frees its tensor memory.
+#include <cuda.h>
+#include <cuda_bf16.h>
+#include <math.h>
+
+#include "attention_gqa.cuh"
+#include "common.cuh"
+#include "ctx.h"
+#include "tcgen05.cuh"
+#include "tmap.h"
+
+namespace lv {
+
+constexpr int kGtThreads = 192;              // TMA warp, MMA warp, four softmax warps
+constexpr int kGtRows = 128, kGtKeys = 64;
+constexpr uint32_t kGtQChunk = kGtRows * 128, kGtKChunk = kGtKeys * 128;      // 64 columns of Q / of K or V, bytes
+constexpr uint32_t kGtMaxStages = 4;
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr float kGtRescaleStep = 8.f;        // log2
+
+struct GqaTcParams {
+    lv_gqa_args a;
+    uint32_t n_tokens, dim_chunks, dim16, v_chunks, vdim16, stages, tmem_cols, tab_stride, tab_tokens;
+    uint32_t out_bf16;
+    uint32_t* err;
+};
+
+struct GqaTcMaps {
+    CUtensorMap k, v;
+};
+
+// V: rows are keys (the K of the MMA), 64 columns per 128-byte row; 8-key groups 1024 bytes apart, 64-column blocks kGtKChunk apart
+__device__ __forceinline__ uint64_t gt_v_desc(uint32_t smem_addr, uint32_t block_bytes) {
+    return uint64_t((smem_addr >> 4) & 0x3fffu) | (uint64_t(block_bytes >> 4) << 16) | (uint64_t(1024 >> 4) << 32) | (uint64_t(1) << 46) | (uint64_t(2) << 61);
+}
+
+__device__ __forceinline__ uint32_t gt_pack(float lo, float hi) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+__device__ __forceinline__ void gt_store16(uint32_t taddr, const uint32_t (&u)[16]) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+        ::"r"(taddr), "r"(u[0]), "r"(u[1]), "r"(u[2]), "r"(u[3]), "r"(u[4]), "r"(u[5]), "r"(u[6]), "r"(u[7]), "r"(u[8]), "r"(u[9]), "r"(u[10]), "r"(u[11]),
+          "r"(u[12]), "r"(u[13]), "r"(u[14]), "r"(u[15])
+        : "memory");
+}
+__device__ __forceinline__ void gt_wait_store() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+
+__global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p, const __grid_constant__ GqaTcMaps maps) {
+    pdl_launch_dependents();
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023u) & ~uintptr_t(1023));
+    const lv_gqa_args& a = p.a;
+    uint8_t* s_q = smem;
+    uint8_t* s_kv = s_q + p.dim_chunks * kGtQChunk;
+    const uint32_t k_bytes = p.dim_chunks * kGtKChunk, v_bytes = p.v_chunks * kGtKChunk, stage = k_bytes + v_bytes;
+    float* s_tab = reinterpret_cast<float*>(s_kv + p.stages * stage);           // [2][group][tab_stride]
+    __shared__ uint64_t k_full[kGtMaxStages], v_full[kGtMaxStages], kv_empty[kGtMaxStages], s_full[2], p_full[2], pv_done;
+    __shared__ uint32_t s_tmem;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const uint32_t group = a.heads / a.kv_heads, g = blockIdx.y;
+    const uint32_t r0 = blockIdx.x * kGtRows, rows_all = p.n_tokens * group;
+    const uint32_t t_first = r0 / group, t_last = min(rows_all - 1, r0 + kGtRows - 1) / group;
+
+    if (threadIdx.x == 0) {
+        for (uint32_t i = 0; i < kGtMaxStages; ++i) { mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&kv_empty[i], 1); }
+        for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], 4); }
+        mbar_init(&pv_done, 1);
+        fence_mbar_init();
+    }
+    if (warp == 1) tc_alloc(&s_tmem, p.tmem_cols);
+    pdl_wait();
+    const uint32_t P = *a.pos;
+    const bool inside = P + p.n_tokens <= a.ctx_rows;            // (lv_qk_norm_append reports positions beyond the cache)
+    const uint32_t n_keys = P + t_last + 1, n_blocks = inside ? (n_keys + kGtKeys - 1) / kGtKeys : 0;
+    // Q rows: a warp per row, lanes across the head
+    for (uint32_t r = warp; r < uint32_t(kGtRows); r += kGtThreads / 32) {
+        const uint32_t row = r0 + r, t = row / group, h = g * group + (row - t * group);
+        const bool live = row < rows_all;
+        const float* q = a.qkv + size_t(live ? t : 0) * a.qkv_ld + (live ? h : 0) * a.dim;
+        const float f = live ? gqa_rms_factor(q, a.dim, a.eps) * a.scale * kLog2e : 0.f;
+        for (uint32_t c2 = lane; c2 < p.dim_chunks * 32; c2 += 32) {           // pairs of columns
+            const uint32_t c = 2 * c2;
+            const float lo = live && c < a.dim ? q[c] * f * a.q_norm[c] : 0.f, hi = live && c + 1 < a.dim ? q[c + 1] * f * a.q_norm[c + 1] : 0.f;
+            const uint32_t in = c & 63u, off = (r >> 3) * 1024u + (r & 7u) * 128u + (((in >> 3) ^ (r & 7u)) << 4) + (in & 7u) * 2u;
+            *reinterpret_cast<uint32_t*>(s_q + (c >> 6) * kGtQChunk + off) = gt_pack(lo, hi);
+        }
+    }
+    fence_proxy_async();
+    tc_fence_before_sync();
+    __syncthreads();
+    tc_fence_after_sync();
+    const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(&s_tmem);
+    const uint32_t tmem_o = tmem + 2 * kGtKeys;
+    bool ok = true;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            uint32_t s = 0, phase = 1;                           // the first pass over the ring finds it empty
+            for (uint32_t b = 0; b < n_blocks; ++b) {
+                if (b >= p.stages && !mbar_wait(&kv_empty[s], phase, p.err)) break;
+                const int y = int(g * a.ctx_rows + b * kGtKeys);
+                uint8_t* dst = s_kv + s * stage;
+                mbar_expect_tx(&k_full[s], k_bytes);
+                for (uint32_t c = 0; c < p.dim_chunks; ++c) tma_load_2d_plain(dst + c * kGtKChunk, &maps.k, int(c * 64), y, &k_full[s]);
+                mbar_expect_tx(&v_full[s], v_bytes);
+                for (uint32_t c = 0; c < p.v_chunks; ++c) tma_load_2d_plain(dst + k_bytes + c * kGtKChunk, &maps.v, int(c * 64), y, &v_full[s]);
+                if (++s == p.stages) { s = 0; phase ^= 1u; }
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0 && n_blocks != 0) {
+            const uint32_t common = (1u << 4) | (1u << 7) | (1u << 10) | (uint32_t(kGtRows >> 4) << 24);
+            const uint32_t idesc_s = common | (uint32_t(kGtKeys >> 3) << 17);
+            const uint32_t idesc_o = common | (1u << 16) | ((p.vdim16 >> 3) << 17);          // B is MN-major
+            const uint64_t q_desc = tc_smem_desc(smem_u32(s_q)), k_desc0 = tc_smem_desc(smem_u32(s_kv));
+            const uint64_t v_desc0 = gt_v_desc(smem_u32(s_kv) + k_bytes, p.v_chunks > 1 ? kGtKChunk : 1024u);
+            const uint32_t k_steps = p.dim16 / 16;
+            uint32_t ks = 0, k_phase = 0, vs = 0, v_phase = 0;
+            auto scores = [&](uint32_t b) {
+                if (!mbar_wait(&k_full[ks], k_phase, p.err)) return false;
+                tc_fence_after_sync();
+                const uint64_t kd = k_desc0 + ((ks * stage) >> 4);
+                for (uint32_t k = 0; k < k_steps; ++k) {
+                    const uint32_t c = k >> 2, in = (k & 3u) * 2u;
+                    tc_mma_f16(tmem + (b & 1u) * kGtKeys, q_desc + ((c * kGtQChunk) >> 4) + in, kd + ((c * kGtKChunk) >> 4) + in, idesc_s, k != 0 ? 1u : 0u);
+                }
+                tc_commit(&s_full[b & 1u]);
+                if (++ks == p.stages) { ks = 0; k_phase ^= 1u; }
+                return true;
+            };
+            ok = scores(0);
+            if (ok && n_blocks > 1) ok = scores(1);
+            for (uint32_t b = 0; b < n_blocks && ok; ++b) {
+                ok = mbar_wait(&p_full[b & 1u], (b >> 1) & 1u, p.err) && mbar_wait(&v_full[vs], v_phase, p.err);
+                if (!ok) break;
+                tc_fence_after_sync();
+                const uint64_t vd = v_desc0 + ((vs * stage) >> 4);
+                for (uint32_t k = 0; k < kGtKeys / 16; ++k)      // 16 keys: 8 columns of P, two 8-key groups of V
+                    tc_mma_f16_ta(tmem_o, tmem + (b & 1u) * kGtKeys + 8u * k, vd + 128u * k, idesc_o, (b != 0 || k != 0) ? 1u : 0u);
+                tc_commit(&kv_empty[vs]);
+                tc_commit(&pv_done);
+                if (++vs == p.stages) { vs = 0; v_phase ^= 1u; }
+                if (b + 2 < n_blocks) ok = scores(b + 2);        // in order after the P V product that reads this buffer
+            }
+        }
+    } else {
+        // ---- softmax: one row per thread ----------------------------------------------------------
+        const uint32_t quarter = uint32_t(warp) & 3u, tr = quarter * 32u + uint32_t(lane), st = threadIdx.x - 64u;
+        const uint32_t row = r0 + tr, t = min(row, rows_all - 1) / group, hl = min(row, rows_all - 1) - t * group;
+        const uint32_t lanes = quarter * 32u << 16;
+        float m = a.sink ? 0.f : -INFINITY, l = 0.f;
+        uint32_t vs = 0, v_phase = 0;
+        // (after a lost wait the warp goes through the remaining blocks without work: the others wait for it at the barrier)
+        for (uint32_t b = 0; b < n_blocks; ++b) {
+            const uint32_t k0 = b * kGtKeys;
+            // bias table of this block: entry i of a head is distance (P + t_first) - (k0 + 63) + i
+            float* tab = s_tab + (b & 1u) * group * p.tab_stride;
+            const int d0 = int(P + t_first) - int(k0 + kGtKeys - 1);
+            for (uint32_t e = st; e < group * p.tab_tokens; e += 128) {
+                const uint32_t h = e / p.tab_tokens, i = e - h * p.tab_tokens;
+                const float d = float(max(d0 + int(i), 0));
+                tab[h * p.tab_stride + i] = kLog2e * a.r1[g * group + h] * log1pf(a.r2[g * group + h] * d);
+            }
+            asm volatile("bar.sync 1, 128;" ::: "memory");
+            ok = ok && mbar_wait(&s_full[b & 1u], (b >> 1) & 1u, p.err);
+            if (!ok) continue;
+            tc_fence_after_sync();
+            float s[kGtKeys];
+#pragma unroll
+            for (int c = 0; c < kGtKeys; c += 16) {
+                uint32_t u[16];
+                tc_load16(u, tmem + lanes + (b & 1u) * kGtKeys + c);
+                tc_wait_load();
+#pragma unroll
+                for (int i = 0; i < 16; ++i) s[c + i] = __uint_as_float(u[i]);
+            }
+            const float* bias = tab + hl * p.tab_stride + (t - t_first) + (kGtKeys - 1);
+            const int last = int(P + t) - int(k0);               // keys 0 .. last of the block are visible
+            float top = -INFINITY;
+            if (k0 + kGtKeys - 1 <= P + t_first) {
+#pragma unroll
+                for (int j = 0; j < kGtKeys; ++j) {
+                    s[j] -= bias[-j];
+                    top = fmaxf(top, s[j]);
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < kGtKeys; ++j) {
+                    s[j] = j <= last ? s[j] - bias[-j] : -INFINITY;
+                    top = fmaxf(top, s[j]);
+                }
+            }
+            // a new maximum takes effect when it is far above the old one (or there was none)
+            const bool grow = top > m + kGtRescaleStep;
+            float f = 1.f;
+            if (grow) {
+                f = exp2f(m - top);                              // 0 when there was none
+                m = top;
+                l *= f;
+            }
+            if (__any_sync(0xffffffffu, grow) && b != 0) {
+                ok = mbar_wait(&pv_done, (b - 1) & 1u, p.err);
+                if (!ok) continue;
+                tc_fence_after_sync();
+                for (uint32_t c = 0; c < p.vdim16; c += 16) {
+                    uint32_t u[16];
+                    tc_load16(u, tmem_o + lanes + c);
+                    tc_wait_load();
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) u[i] = __float_as_uint(__uint_as_float(u[i]) * f);
+                    gt_store16(tmem_o + lanes + c, u);
+                }
+                gt_wait_store();
+            }
+            const float base = m == -INFINITY ? 0.f : m;
+#pragma unroll
+            for (int c = 0; c < kGtKeys; c += 32) {
+                uint32_t u[16];
+#pragma unroll
+                for (int i = 0; i < 16; ++i) {
+                    const float p0 = exp2f(s[c + 2 * i] - base), p1 = exp2f(s[c + 2 * i + 1] - base);
+                    l += p0;
+                    l += p1;
+                    u[i] = gt_pack(p0, p1);
+                }
+                gt_store16(tmem + lanes + (b & 1u) * kGtKeys + c / 2, u);
+            }
+            gt_wait_store();
+            if (k0 + kGtKeys > P + p.n_tokens) {
+                // rows of V behind the last token hold whatever the cache held: their weights are zero, but zero times NaN is not
+                ok = mbar_wait(&v_full[vs], v_phase, p.err);
+                if (!ok) continue;
+                uint8_t* v = s_kv + vs * stage + k_bytes;
+                const uint32_t first = P + p.n_tokens - k0, n16 = (kGtKeys - first) * 8;
+                for (uint32_t e = st; e < p.v_chunks * n16; e += 128) {
+                    const uint32_t c = e / n16, i = e - c * n16;
+                    *reinterpret_cast<uint4*>(v + c * kGtKChunk + first * 128 + i * 16) = make_uint4(0u, 0u, 0u, 0u);
+                }
+                fence_proxy_async();
+            }
+            if (++vs == p.stages) { vs = 0; v_phase ^= 1u; }
+            tc_fence_before_sync();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&p_full[b & 1u]);
+        }
+        if (ok && n_blocks != 0) {
+            ok = mbar_wait(&pv_done, (n_blocks - 1) & 1u, p.err);
+            tc_fence_after_sync();
+        }
+        if (ok && n_blocks != 0) {
+            const float inv = 1.f / (l + (a.sink ? exp2f(-m) : 0.f));
+            const size_t at = size_t(t) * a.out_ld + (g * group + hl) * a.vdim;
+            for (uint32_t c = 0; c < p.vdim16; c += 16) {
+                uint32_t u[16];
+                tc_load16(u, tmem_o + lanes + c);
+                tc_wait_load();
+                if (row >= rows_all) continue;
+                if (p.out_bf16 && c + 16 <= a.vdim && (at + c) % 8 == 0) {
+                    uint4 w[2];
+                    uint32_t* ww = reinterpret_cast<uint32_t*>(w);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) ww[i] = gt_pack(__uint_as_float(u[2 * i]) * inv, __uint_as_float(u[2 * i + 1]) * inv);
+                    uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.out) + at + c);
+                    dst[0] = w[0];
+                    dst[1] = w[1];
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 16; ++i)
+                        if (c + i < a.vdim) gqa_store_out(a.out, p.out_bf16, at + c + i, __uint_as_float(u[i]) * inv);
+                }
+            }
+        }
+        tc_fence_before_sync();
+    }
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after_sync();
+        tc_free(tmem, p.tmem_cols);
+    }
+}
+
+bool gqa_tc_supported(const lv_gqa_args& a, uint32_t batch) {
+    return a.cache_type == LV_TYPE_BF16 && batch > 1 && a.heads / a.kv_heads <= 64;
+}
+
+int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch) {
+    GqaTcParams p{};
+    p.a = a;
+    p.n_tokens = batch;
+    const uint32_t dim_p = (a.dim + 7) / 8 * 8, vdim_p = (a.vdim + 7) / 8 * 8, group = a.heads / a.kv_heads;
+    p.dim_chunks = (dim_p + 63) / 64;
+    p.dim16 = (dim_p + 15) / 16 * 16;
+    p.v_chunks = (vdim_p + 63) / 64;
+    p.vdim16 = (vdim_p + 15) / 16 * 16;
+    p.out_bf16 = a.out_type == LV_TYPE_BF16;
+    p.err = ctx->d_err;
+    p.tmem_cols = 2 * kGtKeys + p.vdim16 <= 256 ? 256 : 512;
+    // tokens that a tile of 128 rows can touch, plus the keys of a block; heads 32 / group banks apart
+    p.tab_tokens = (kGtRows + group - 1) / group + 1 + kGtKeys;
+    const uint32_t want = group < 32 ? 32 / group : 1;
+    p.tab_stride = p.tab_tokens;
+    while (p.tab_stride % 32 != want % 32) ++p.tab_stride;
+    const uint32_t stage = (p.dim_chunks + p.v_chunks) * kGtKChunk, q_bytes = p.dim_chunks * kGtQChunk, tab = 2 * group * p.tab_stride * 4;
+    p.stages = 2;
+    while (p.stages < kGtMaxStages && q_bytes + (p.stages + 1) * stage + tab + 1024 <= 110 * 1024) ++p.stages;      // two CTAs per SM where they fit
+    const size_t smem = 1024 + size_t(q_bytes) + size_t(p.stages) * stage + tab;
+    LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "attention: head sizes need too much shared memory");
+    GqaTcMaps maps{};
+    const uint64_t rows = uint64_t(a.kv_heads) * a.ctx_rows;
+    LV_REQUIRE(rows <= 0x7fffffffu, "attention: cache too long");
+    if (int rc = make_bf16_map(&maps.k, a.k_cache, rows, dim_p, dim_p, kGtKeys)) return rc;
+    if (int rc = make_bf16_map(&maps.v, a.v_cache, rows, vdim_p, vdim_p, kGtKeys)) return rc;
+    LV_CUDA(cudaFuncSetAttribute(gqa_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    LV_CUDA(launch_pdl(ctx, gqa_tc_kernel, dim3((batch * group + kGtRows - 1) / kGtRows, a.kv_heads), dim3(kGtThreads), smem, p, maps));
+    return LV_OK;
+}
+
+}  // namespace lv
