@@ -396,11 +396,12 @@ int lv_decode_step(lv_ctx* ctx, const lv_step_plan* plan, uint32_t* config, uint
  * already evaluated (config[0] of lv_argmax_advance), token t of a launch is at position *pos + t and its id in
  * token_log[*pos + t]. */
 
-/* The boundary between two sublayers in one launch: residual add of the normalised output of the finished sublayer, an
+/* The boundary between two sublayers (one launch, two for several tokens with a convolution): residual add of the normalised output of the finished sublayer, an
  * optional vector added to the stream, the next norm, and a causal convolution over time on its result.
  *   y_t  = (1 / y_rows) sum_s y[y_index[t * y_rows + s]]   (y[t] without y_index); y null: no sublayer yet
  *   x_t  = x[t] + mult * y_t / rms(y_t) * (1 + post_w)     -> trace[t] (may be null)
- *   x_t += step (may be null)                              -> x_out[t] (may be null; may equal x for batch 1)
+ *   x_t += step (may be null)                              -> x_out[t] (may equal x; may be null without a convolution
+ *                                                             or for one token)
  *   h_t  = x_t / rms(x_t) * (1 + pre_w),  rms(v) = sqrt(mean(v^2) + eps)
  *   out  = h_t + sum_{j < taps} conv_w[j] * h_{t - taps + 1 + j}   (taps 0: out = h_t)
  * for the tokens first .. batch - 1.  history f32 [taps - 1][width] holds h of the last taps - 1 positions, oldest first,
@@ -420,6 +421,7 @@ typedef struct lv_norm_conv_args {
     const float* step;
     float* trace;
     float* x_out;
+    float* row_factor;              /* scratch [batch], for several tokens with a convolution */
     const float* pre_w;
     const float* conv_w;            /* [taps][width] */
     float* history;

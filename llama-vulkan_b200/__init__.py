@@ -37,7 +37,7 @@ _f32 = C.c_float
 class NormConvArgs(C.Structure):
     """lv_norm_conv_args"""
     _fields_ = [("x", _p), ("embed", _p), ("embed_ld", _u32), ("vocab", _u32), ("token_log", _p), ("pos", _p), ("y", _p), ("y_index", _p),
-                ("y_rows", _u32), ("mult", _f32), ("eps", _f32), ("post_w", _p), ("step", _p), ("trace", _p), ("x_out", _p), ("pre_w", _p),
+                ("y_rows", _u32), ("mult", _f32), ("eps", _f32), ("post_w", _p), ("step", _p), ("trace", _p), ("x_out", _p), ("row_factor", _p), ("pre_w", _p),
                 ("conv_w", _p), ("history", _p), ("taps", _u32), ("out", _p), ("out_type", _int), ("out_ld", _u32), ("out_index", _p),
                 ("out_copies", _u32), ("width", _u32), ("first", _u32), ("batch", _u32)]
 

@@ -5,11 +5,13 @@
 //   p_ij = exp(s_ij) / (sink + sum_j exp(s_ij)),     sink = 1 or 0
 //
 // One CTA serves up to eight query heads of one key/value head for one token and walks its share of the keys in chunks of
-// 128 with an online softmax.  A decoded token spreads the chunks over several CTAs (the last to arrive combines their
+// 64 with an online softmax.  A decoded token spreads the chunks over several CTAs (the last to arrive combines their
 // partial sums through scratch) and its own key and value are normalised and appended to the caches by the same launch;
 // tokens of a prompt are appended first (lv_qk_norm_append) and, with bfloat16 caches, go through attention_gqa_tc.cu.  Caches are [kv head][ctx_rows][padded dim], bfloat16 or f32.
 #include <cuda_bf16.h>
 #include <math.h>
+
+#include <algorithm>
 
 #include "attention_gqa.cuh"
 #include "common.cuh"
@@ -18,37 +20,38 @@
 namespace lv {
 
 constexpr size_t kGqaCounterBytes = 4096;   // arrival counters at the start of the scratch (kept zero between launches)
-constexpr int kGqaThreads = 256, kGqaWarps = 8, kGqaChunk = 128, kGqaHeads = 8;
+constexpr int kGqaThreads = 256, kGqaWarps = 8, kGqaChunk = 64, kGqaHeads = 8, kGqaMaxSplits = 128;
 
 struct GqaParams {
     lv_gqa_args a;
     uint32_t dim_p, vdim_p;         // padded to 8
     uint32_t head_blocks;           // CTAs per key/value head
     uint32_t splits;
-    uint32_t out_bf16;
+    uint32_t out_bf16, append;
     float* scratch;                 // splits > 1: [token][head][split][vdim_p + 2]
     uint32_t* counters;             // [token][kv head * head_blocks]
     uint32_t* err;
 };
 
+// eight cache values: as fetched, and widened to f32
 template <typename CT> struct Cache8;
 template <> struct Cache8<__nv_bfloat16> {
-    static __device__ __forceinline__ void load(float (&v)[8], const __nv_bfloat16* p) {
-        const uint4 w = *reinterpret_cast<const uint4*>(p);
+    using raw = uint4;
+    static __device__ __forceinline__ raw fetch(const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); }
+    static __device__ __forceinline__ void widen(float (&v)[8], const raw& w) {
         const uint32_t q[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
         for (int i = 0; i < 4; ++i) { v[2 * i] = __uint_as_float(q[i] << 16); v[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u); }
     }
     static __device__ __forceinline__ __nv_bfloat16 cast(float v) { return __float2bfloat16_rn(v); }
-    static __device__ __forceinline__ float back(__nv_bfloat16 v) { return __bfloat162float(v); }
 };
 template <> struct Cache8<float> {
-    static __device__ __forceinline__ void load(float (&v)[8], const float* p) {
-        const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    struct raw { float4 a, b; };
+    static __device__ __forceinline__ raw fetch(const float* p) { return {*reinterpret_cast<const float4*>(p), *reinterpret_cast<const float4*>(p + 4)}; }
+    static __device__ __forceinline__ void widen(float (&v)[8], const raw& w) {
+        v[0] = w.a.x; v[1] = w.a.y; v[2] = w.a.z; v[3] = w.a.w; v[4] = w.b.x; v[5] = w.b.y; v[6] = w.b.z; v[7] = w.b.w;
     }
     static __device__ __forceinline__ float cast(float v) { return v; }
-    static __device__ __forceinline__ float back(float v) { return v; }
 };
 
 // Appends the normalised key and the value of token t (one warp per key/value head).
@@ -74,8 +77,8 @@ __global__ void __launch_bounds__(128) qk_norm_append_kernel(const GqaParams p, 
     for (uint32_t i = lane; i < p.vdim_p; i += 32) vd[i] = Cache8<CT>::cast(i < a.vdim ? v[i] : 0.f);
 }
 
-// HB: query heads of this CTA, rounded up.  LPK: lanes that share a key, VU: threads that share a value row.
-template <typename CT, int HB, bool APPEND>
+// HB: query heads of this CTA, rounded up.  L: lanes that share a key and threads that share a value row (8 values each).
+template <typename CT, int HB, int L>
 __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -85,26 +88,46 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
     const uint32_t h0 = g * group + hb * kGqaHeads, nh = min(uint32_t(kGqaHeads), group - hb * kGqaHeads);
     const uint32_t t = blockIdx.z;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    uint32_t vu = 1;
-    while (vu * 8 < p.vdim_p) vu *= 2;                     // threads across a value row (power of two, <= 32)
-    uint32_t lpk = 8;
-    while (lpk * 8 < p.dim_p) lpk *= 2;                    // lanes across a key (>= the heads of a CTA)
+    constexpr int kPerWarp = 32 / L, kIters = kGqaChunk / (kGqaWarps * kPerWarp);      // keys of a warp per pass, passes per chunk
+    constexpr int kGroups = kGqaThreads / L;                                             // value rows in flight; kIters each
     float* s_q = reinterpret_cast<float*>(smem_raw);      // [HB][dim_p]
     float* s_sc = s_q + HB * p.dim_p;                      // [HB][chunk]
-    float* s_red = s_sc + HB * kGqaChunk;                  // [warps][HB][vu * 8]
-    float* s_m = s_red + kGqaWarps * HB * vu * 8;          // [HB] running maximum
+    float* s_red = s_sc + HB * kGqaChunk;                  // [warps][HB][L * 8]; the combination reuses it
+    float* s_m = s_red + kGqaWarps * HB * L * 8;           // [HB] running maximum
     float* s_l = s_m + HB;                                 // [HB] running sum
     float* s_c = s_l + HB;                                 // [HB] factor of this chunk
-    CT* s_k = reinterpret_cast<CT*>(s_c + 2 * HB);         // (16-byte aligned) APPEND: the token's own key and value as the cache holds them
+    CT* s_k = reinterpret_cast<CT*>(s_c + 2 * HB);         // append: the token's own key and value as the cache holds them (16-byte aligned)
     CT* s_v = s_k + p.dim_p;
     __shared__ uint32_t s_last;
 
+    const uint32_t sub = lane & (L - 1), key_in_warp = lane / L;
+    const uint32_t vcol = (threadIdx.x & (L - 1)) * 8, vgroup = threadIdx.x / L;
+    const float r1 = sub < nh ? a.r1[h0 + sub] : 0.f, r2 = sub < nh ? a.r2[h0 + sub] : 0.f;
     pdl_wait();
     const uint32_t P = *a.pos + t;
     if (P >= a.ctx_rows) {
         if (threadIdx.x == 0) atomicOr(p.err, ERR_BAD_INDEX);
         return;
     }
+    CT* kc = static_cast<CT*>(a.k_cache) + size_t(g) * a.ctx_rows * p.dim_p;
+    CT* vc = static_cast<CT*>(a.v_cache) + size_t(g) * a.ctx_rows * p.vdim_p;
+    const bool append = p.append != 0;
+    const uint32_t own_chunk = P / kGqaChunk;
+    // a chunk's keys and values are requested before anything waits for them
+    typename Cache8<CT>::raw kr[kIters], vr[kIters];
+    auto fetch = [&](uint32_t k0) {
+#pragma unroll
+        for (int i = 0; i < kIters; ++i) {
+            const uint32_t j = k0 + (i * kGqaWarps + warp) * kPerWarp + key_in_warp;
+            if (sub * 8 < p.dim_p && j <= P && !(append && j == P)) kr[i] = Cache8<CT>::fetch(kc + size_t(j) * p.dim_p + sub * 8);
+        }
+#pragma unroll
+        for (int i = 0; i < kIters; ++i) {
+            const uint32_t j = k0 + i * kGroups + vgroup;
+            if (vcol < p.vdim_p && j <= P && !(append && j == P)) vr[i] = Cache8<CT>::fetch(vc + size_t(j) * p.vdim_p + vcol);
+        }
+    };
+    if (blockIdx.y <= own_chunk) fetch(blockIdx.y * kGqaChunk);
     const float* raw = a.qkv + size_t(t) * a.qkv_ld;
     if (warp < int(nh)) {
         const float* q = raw + (h0 + warp) * a.dim;
@@ -113,11 +136,7 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
     } else if (warp < HB) {
         for (uint32_t i = lane; i < p.dim_p; i += 32) s_q[warp * p.dim_p + i] = 0.f;
     }
-    const uint32_t own_chunk = P / kGqaChunk;
-    const bool own = APPEND && own_chunk % p.splits == blockIdx.y;
-    CT* kc = static_cast<CT*>(a.k_cache) + size_t(g) * a.ctx_rows * p.dim_p;
-    CT* vc = static_cast<CT*>(a.v_cache) + size_t(g) * a.ctx_rows * p.vdim_p;
-    if (own && warp == kGqaWarps - 1) {
+    if (append && own_chunk % p.splits == blockIdx.y && warp == kGqaWarps - 1) {
         const float* k = raw + a.heads * a.dim + g * a.dim;
         const float* v = raw + (a.heads + a.kv_heads) * a.dim + g * a.vdim;
         const float r = gqa_rms_factor(k, a.dim, a.eps);
@@ -133,9 +152,6 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
         }
     }
     if (threadIdx.x < HB) { s_m[threadIdx.x] = -INFINITY; s_l[threadIdx.x] = 0.f; }
-    const uint32_t sub = lane & (lpk - 1), key_in_warp = lane / lpk, keys_per_warp = 32 / lpk;
-    const float r1 = sub < nh ? a.r1[h0 + sub] : 0.f, r2 = sub < nh ? a.r2[h0 + sub] : 0.f;
-    const uint32_t vcol = (threadIdx.x & (vu - 1)) * 8, vgroup = threadIdx.x / vu, vgroups = kGqaThreads / vu;
     float acc[HB][8];
 #pragma unroll
     for (int h = 0; h < HB; ++h)
@@ -144,43 +160,49 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
     __syncthreads();
 
     for (uint32_t c = blockIdx.y; c <= own_chunk; c += p.splits) {
-        const uint32_t k0 = c * kGqaChunk, n = min(uint32_t(kGqaChunk), P + 1 - k0);
-        // scores: lpk lanes share a key
-#pragma unroll 2
-        for (uint32_t kk = warp * keys_per_warp + key_in_warp; kk < kGqaChunk; kk += kGqaWarps * keys_per_warp) {
-            const uint32_t j = k0 + kk;
-            const bool live = kk < n && sub * 8 < p.dim_p;
+        const uint32_t k0 = c * kGqaChunk;
+        if (c != blockIdx.y) fetch(k0);
+        float bias[kIters];
+#pragma unroll
+        for (int i = 0; i < kIters; ++i) {
+            const uint32_t j = k0 + (i * kGqaWarps + warp) * kPerWarp + key_in_warp;
+            bias[i] = j <= P ? r1 * log1pf(r2 * float(P - j)) : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < kIters; ++i) {
+            const uint32_t kk = (i * kGqaWarps + warp) * kPerWarp + key_in_warp, j = k0 + kk;
+            const bool live = j <= P && sub * 8 < p.dim_p;
             float kv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-            if (live) Cache8<CT>::load(kv, (APPEND && j == P) ? s_k + sub * 8 : kc + size_t(j) * p.dim_p + sub * 8);
+            if (live) {
+                if (append && j == P) kr[i] = Cache8<CT>::fetch(s_k + sub * 8);
+                Cache8<CT>::widen(kv, kr[i]);
+            }
             float mine = 0.f;
 #pragma unroll
             for (int h = 0; h < HB; ++h) {
                 float s = 0.f;
                 if (live) {
                     float qv[8];
-                    Cache8<float>::load(qv, s_q + h * p.dim_p + sub * 8);
+                    Cache8<float>::widen(qv, Cache8<float>::fetch(s_q + h * p.dim_p + sub * 8));
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) s = fmaf(qv[i], kv[i], s);
+                    for (int e = 0; e < 8; ++e) s = fmaf(qv[e], kv[e], s);
                 }
-                for (uint32_t o = lpk >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+#pragma unroll
+                for (int o = L / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
                 if (sub == uint32_t(h)) mine = s;
             }
-            if (sub < HB) s_sc[sub * kGqaChunk + kk] = (kk < n && sub < nh) ? mine - r1 * log1pf(r2 * float(P - j)) : -INFINITY;
+            if (sub < HB) s_sc[sub * kGqaChunk + kk] = (j <= P && sub < nh) ? mine - bias[i] : -INFINITY;
         }
         __syncthreads();
         // online softmax: warp h takes head h
         if (warp < HB) {
             float* sc = s_sc + warp * kGqaChunk;
-            float m = -INFINITY;
-            for (int i = lane; i < kGqaChunk; i += 32) m = fmaxf(m, sc[i]);
-            const float m_old = s_m[warp], m_new = fmaxf(m_old, warp_max(m));
-            float l = 0.f;
-            for (int i = lane; i < kGqaChunk; i += 32) {
-                const float e = m_new == -INFINITY ? 0.f : expf(sc[i] - m_new);
-                sc[i] = e;
-                l += e;
-            }
-            l = warp_sum(l);
+            const float a0 = sc[lane], a1 = sc[lane + 32];
+            const float m_old = s_m[warp], m_new = fmaxf(m_old, warp_max(fmaxf(a0, a1)));
+            const float e0 = m_new == -INFINITY ? 0.f : expf(a0 - m_new), e1 = m_new == -INFINITY ? 0.f : expf(a1 - m_new);
+            sc[lane] = e0;
+            sc[lane + 32] = e1;
+            const float l = warp_sum(e0 + e1);
             if (lane == 0) {
                 const float f = m_new == -INFINITY ? 1.f : expf(m_old - m_new);
                 s_c[warp] = f;
@@ -195,38 +217,39 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) acc[h][i] *= f;
         }
-        if (vcol < p.vdim_p) {
-#pragma unroll 4
-            for (uint32_t kk = vgroup; kk < n; kk += vgroups) {
-                const uint32_t j = k0 + kk;
-                float vv[8];
-                Cache8<CT>::load(vv, (APPEND && j == P) ? s_v + vcol : vc + size_t(j) * p.vdim_p + vcol);
 #pragma unroll
-                for (int h = 0; h < HB; ++h) {
-                    const float pr = s_sc[h * kGqaChunk + kk];
+        for (int i = 0; i < kIters; ++i) {
+            const uint32_t kk = i * kGroups + vgroup, j = k0 + kk;
+            if (j > P || vcol >= p.vdim_p) continue;
+            if (append && j == P) vr[i] = Cache8<CT>::fetch(s_v + vcol);
+            float vv[8];
+            Cache8<CT>::widen(vv, vr[i]);
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) acc[h][i] = fmaf(pr, vv[i], acc[h][i]);
-                }
+            for (int h = 0; h < HB; ++h) {
+                const float pr = s_sc[h * kGqaChunk + kk];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) acc[h][e] = fmaf(pr, vv[e], acc[h][e]);
             }
         }
         __syncthreads();
     }
-    // value groups of a warp, then of the CTA, in a fixed order
+    // value rows of a warp, then of the CTA, in a fixed order
 #pragma unroll
     for (int h = 0; h < HB; ++h)
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             float v = acc[h][i];
-            for (uint32_t o = vu; o < 32; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-            if (lane < int(vu)) s_red[(warp * HB + h) * vu * 8 + vcol + i] = v;
+#pragma unroll
+            for (int o = L; o < 32; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+            if (lane < L) s_red[(warp * HB + h) * (L * 8) + vcol + i] = v;
         }
     __syncthreads();
-    const uint32_t vw = vu * 8;
     const uint32_t part = p.vdim_p + 2;
     for (uint32_t e = threadIdx.x; e < nh * p.vdim_p; e += kGqaThreads) {
         const uint32_t h = e / p.vdim_p, col = e - h * p.vdim_p;
         float v = 0.f;
-        for (int w = 0; w < kGqaWarps; ++w) v += s_red[(w * HB + h) * vw + col];
+#pragma unroll
+        for (int w = 0; w < kGqaWarps; ++w) v += s_red[(w * HB + h) * (L * 8) + col];
         const float m = s_m[h], l = s_l[h];
         if (p.splits == 1) {
             if (col < a.vdim) {
@@ -250,18 +273,36 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
     __syncthreads();
     if (!s_last) return;
     __threadfence();
+    // the last CTA weighs the shares: warp h forms exp(m_s - M) / denominator of head h for every share (splits <= kGqaMaxSplits)
+    float* s_w = s_red;                                    // [HB][kGqaMaxSplits]
+    if (warp < int(nh)) {
+        const float* src = p.scratch + (size_t(t) * a.heads + h0 + warp) * p.splits * part;
+        float m[kGqaMaxSplits / 32], l[kGqaMaxSplits / 32], M = a.sink ? 0.f : -INFINITY, den = 0.f;
+#pragma unroll
+        for (int i = 0; i < kGqaMaxSplits / 32; ++i) {
+            const uint32_t s = i * 32 + lane;
+            m[i] = s < p.splits ? __ldcg(src + s * part) : -INFINITY;
+            l[i] = s < p.splits ? __ldcg(src + s * part + 1) : 0.f;
+            M = fmaxf(M, m[i]);
+        }
+        M = warp_max(M);
+#pragma unroll
+        for (int i = 0; i < kGqaMaxSplits / 32; ++i) {
+            m[i] = expf(m[i] - M);
+            den = fmaf(m[i], l[i], den);
+        }
+        const float inv = 1.f / (warp_sum(den) + (a.sink ? expf(-M) : 0.f));
+#pragma unroll
+        for (int i = 0; i < kGqaMaxSplits / 32; ++i) s_w[warp * kGqaMaxSplits + i * 32 + lane] = m[i] * inv;
+    }
+    __syncthreads();
     for (uint32_t e = threadIdx.x; e < nh * a.vdim; e += kGqaThreads) {
         const uint32_t h = e / a.vdim, col = e - h * a.vdim;
-        const float* src = p.scratch + (size_t(t) * a.heads + h0 + h) * p.splits * part;
-        float M = a.sink ? 0.f : -INFINITY;
-        for (uint32_t s = 0; s < p.splits; ++s) M = fmaxf(M, __ldcg(src + s * part));
-        float num = 0.f, den = a.sink ? expf(-M) : 0.f;
-        for (uint32_t s = 0; s < p.splits; ++s) {
-            const float f = expf(__ldcg(src + s * part) - M);
-            num = fmaf(f, __ldcg(src + s * part + 2 + col), num);
-            den = fmaf(f, __ldcg(src + s * part + 1), den);
-        }
-        gqa_store_out(a.out, p.out_bf16, size_t(t) * a.out_ld + (h0 + h) * a.vdim + col, num / den);
+        const float* src = p.scratch + (size_t(t) * a.heads + h0 + h) * p.splits * part + 2 + col;
+        float v = 0.f;
+#pragma unroll 8
+        for (uint32_t s = 0; s < p.splits; ++s) v = fmaf(s_w[h * kGqaMaxSplits + s], __ldcg(src + s * part), v);
+        gqa_store_out(a.out, p.out_bf16, size_t(t) * a.out_ld + (h0 + h) * a.vdim + col, v);
     }
 }
 
@@ -273,7 +314,7 @@ static uint32_t gqa_head_blocks(const lv_gqa_args& a) { return (a.heads / a.kv_h
 static uint32_t gqa_splits(const lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch, uint32_t capacity) {
     const uint32_t ctas = a.kv_heads * gqa_head_blocks(a) * batch, chunks = (capacity + kGqaChunk - 1) / kGqaChunk;
     const uint32_t want = (2u * uint32_t(ctx->sm_count) + ctas - 1) / ctas;
-    return want < 1 ? 1 : (want > chunks ? chunks : want);
+    return std::max(1u, std::min({want, chunks, uint32_t(kGqaMaxSplits)}));
 }
 
 static int gqa_check(const lv_gqa_args* a, uint32_t batch) {
@@ -284,28 +325,32 @@ static int gqa_check(const lv_gqa_args* a, uint32_t batch) {
     return LV_OK;
 }
 
-template <typename CT, bool APPEND>
-static int gqa_launch(lv_ctx* ctx, const GqaParams& p, uint32_t batch) {
-    const lv_gqa_args& a = p.a;
-    const uint32_t group = a.heads / a.kv_heads;
-    const int HB = group >= 5 ? 8 : group >= 3 ? 4 : int(group);
-    uint32_t vu = 1;
-    while (vu * 8 < p.vdim_p) vu *= 2;
-    const size_t smem = sizeof(float) * (size_t(HB) * p.dim_p + HB * kGqaChunk + size_t(kGqaWarps) * HB * vu * 8 + 4 * HB) + sizeof(CT) * (p.dim_p + p.vdim_p) + 16;
+template <typename CT, int HB, int L>
+static int gqa_launch_typed(lv_ctx* ctx, const GqaParams& p, uint32_t batch) {
+    const size_t smem = sizeof(float) * (size_t(HB) * p.dim_p + HB * kGqaChunk + size_t(kGqaWarps) * HB * L * 8 + 5 * HB) + sizeof(CT) * (p.dim_p + p.vdim_p) + 16;
+    static_assert(kGqaWarps * L * 8 >= kGqaMaxSplits, "the combination's weights reuse the reduction buffer");
     LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "attention: head sizes need too much shared memory");
-    const dim3 grid(a.kv_heads * p.head_blocks, p.splits, batch);
-    auto go = [&](auto kernel) -> cudaError_t {
-        if (smem > 48 * 1024) {
-            const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
-            if (e != cudaSuccess) return e;
-        }
-        return launch_pdl(ctx, kernel, grid, dim3(kGqaThreads), smem, p);
-    };
-    if (HB == 8) LV_CUDA(go(gqa_kernel<CT, 8, APPEND>));
-    else if (HB == 4) LV_CUDA(go(gqa_kernel<CT, 4, APPEND>));
-    else if (HB == 2) LV_CUDA(go(gqa_kernel<CT, 2, APPEND>));
-    else LV_CUDA(go(gqa_kernel<CT, 1, APPEND>));
+    auto* kernel = gqa_kernel<CT, HB, L>;
+    if (smem > 48 * 1024) LV_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    LV_CUDA(launch_pdl(ctx, kernel, dim3(p.a.kv_heads * p.head_blocks, p.splits, batch), dim3(kGqaThreads), smem, p));
     return LV_OK;
+}
+
+template <typename CT, int L>
+static int gqa_launch_heads(lv_ctx* ctx, const GqaParams& p, uint32_t batch) {
+    const uint32_t group = p.a.heads / p.a.kv_heads;
+    if (group >= 5) return gqa_launch_typed<CT, 8, L>(ctx, p, batch);
+    if (group >= 3) return gqa_launch_typed<CT, 4, L>(ctx, p, batch);
+    if (group == 2) return gqa_launch_typed<CT, 2, L>(ctx, p, batch);
+    return gqa_launch_typed<CT, 1, L>(ctx, p, batch);
+}
+
+template <typename CT>
+static int gqa_launch(lv_ctx* ctx, const GqaParams& p, uint32_t batch) {
+    const uint32_t widest = std::max(p.dim_p, p.vdim_p);
+    if (widest <= 64) return gqa_launch_heads<CT, 8>(ctx, p, batch);
+    if (widest <= 128) return gqa_launch_heads<CT, 16>(ctx, p, batch);
+    return gqa_launch_heads<CT, 32>(ctx, p, batch);
 }
 
 }  // namespace lv
@@ -358,6 +403,6 @@ extern "C" int lv_attention_gqa(lv_ctx* ctx, const lv_gqa_args* a, void* scratch
         p.counters = static_cast<uint32_t*>(scratch);
         p.scratch = reinterpret_cast<float*>(static_cast<uint8_t*>(scratch) + kGqaCounterBytes);
     }
-    if (a->cache_type == LV_TYPE_F32) return append ? gqa_launch<float, true>(ctx, p, batch) : gqa_launch<float, false>(ctx, p, batch);
-    return append ? gqa_launch<__nv_bfloat16, true>(ctx, p, batch) : gqa_launch<__nv_bfloat16, false>(ctx, p, batch);
+    p.append = append != 0;
+    return a->cache_type == LV_TYPE_F32 ? gqa_launch<float>(ctx, p, batch) : gqa_launch<__nv_bfloat16>(ctx, p, batch);
 }

@@ -171,7 +171,6 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const GemmBf16
                     float* dst = partial + size_t(blockIdx.z) * (kAcc * NT * kBgRows);
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
-                        if (z0 + i >= n_tok) break;
                         dst[(z0 + i) * kBgRows + tr] = v[i];
                         if constexpr (PAIR) dst[(NT + z0 + i) * kBgRows + tr] = g[i];
                     }
@@ -191,11 +190,11 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const GemmBf16
                 __threadfence();
                 for (uint32_t z0 = 0; z0 < NT && z0 < n_tok; z0 += 16) {
                     float v[16] = {}, g[16] = {};
+#pragma unroll 2
                     for (uint32_t s = 0; s < p.splits; ++s) {
                         const float* src = partial + size_t(s) * (kAcc * NT * kBgRows);
 #pragma unroll
                         for (int i = 0; i < 16; ++i) {
-                            if (z0 + i >= n_tok) break;
                             v[i] += __ldcg(src + (z0 + i) * kBgRows + tr);
                             if constexpr (PAIR) g[i] += __ldcg(src + (NT + z0 + i) * kBgRows + tr);
                         }
@@ -323,7 +322,9 @@ extern "C" int lv_gemm_bf16(lv_ctx* ctx, void* out, int out_type, uint32_t out_l
     LV_REQUIRE(ld % 8 == 0 && ld >= cols && x_ld % 8 == 0 && x_ld >= cols && (out_type == LV_TYPE_F32 || out_type == LV_TYPE_BF16), "gemm_bf16: bad strides");
     GemmBf16Params p{};
     p.rows = rows; p.tokens = batch; p.K = cols; p.out = out; p.out_ld = out_ld; p.out_bf16 = out_type == LV_TYPE_BF16; p.factor = factor;
-    const uint32_t nt = batch <= 16 ? 16 : batch <= 32 ? 32 : batch <= 64 ? 64 : 128;
+    uint32_t nt = batch <= 16 ? 16 : batch <= 32 ? 32 : batch <= 64 ? 64 : 128;
+    // narrower token tiles before K splits: partial sums cost more than reading a weight tile twice
+    while (nt > 32 && (rows + kBgRows - 1) / kBgRows * ((batch + nt - 1) / nt) * 2 <= uint32_t(ctx->sm_count) && batch > nt / 2) nt /= 2;
     GemmBf16Maps maps{};
     if (int rc = make_bf16_map(&maps.w, w, rows, cols, ld, kBgRows)) return rc;
     if (int rc = make_bf16_map(&maps.x, x, batch, cols, x_ld, nt)) return rc;

@@ -1,6 +1,6 @@
-// The boundary between two sublayers of a pre- and post-normalised decoder in one launch: residual add of the finished
-// sublayer (its output normalised), an optional vector added to the stream, the norm of the next sublayer and a short
-// causal convolution over time on its result.
+// The boundary between two sublayers of a pre- and post-normalised decoder: residual add of the finished sublayer (its
+// output normalised), an optional vector added to the stream, the norm of the next sublayer and a short causal convolution
+// over time on its result.
 //
 //   y_t   = mean of y_rows rows of the finished sublayer          (experts leave one row per choice)
 //   x'_t  = x_t + mult * y_t / rms(y_t) * (1 + post_w)            rms(v) = sqrt(mean(v^2) + eps)
@@ -10,6 +10,10 @@
 //
 // x may come from the embedding table instead of the stream.  The last taps - 1 values of h are the state that the next
 // step reads; positions before the start of the sequence are masked by the position word, so a state needs no clearing.
+//
+// A CTA per token holds the token's row in registers (all loads are issued before the first sum).  One token is done in
+// that launch.  Several tokens leave x'' and 1 / rms in memory for a second launch that forms h again and convolves: its
+// threads own channels and slide over a few tokens, so it has no sum to wait for.
 #include <cuda_bf16.h>
 
 #include "common.cuh"
@@ -25,210 +29,242 @@ struct NormConvParams {
     uint32_t* err;
 };
 
-__device__ __forceinline__ float nc_load_x(const lv_norm_conv_args& a, uint32_t t, uint32_t i, uint32_t id) {
-    if (a.x != nullptr) return a.x[size_t(t) * a.width + i];
-    return __bfloat162float(static_cast<const __nv_bfloat16*>(a.embed)[size_t(id) * a.embed_ld + i]);
-}
-
-__device__ __forceinline__ float nc_load_y(const lv_norm_conv_args& a, uint32_t t, uint32_t i) {
-    if (a.y_index == nullptr) return a.y[size_t(t) * a.width + i];
-    float v = 0.f;
-    for (uint32_t s = 0; s < a.y_rows; ++s) v += a.y[size_t(a.y_index[t * a.y_rows + s]) * a.width + i];
-    return v / float(a.y_rows);
-}
-
-__device__ __forceinline__ uint32_t nc_token(const lv_norm_conv_args& a, uint32_t pos, uint32_t t, uint32_t* err) {
-    if (a.x != nullptr) return 0u;
-    uint32_t id = a.token_log[pos + t];
-    if (id >= a.vocab) {
-        if (threadIdx.x == 0) atomicOr(err, ERR_BAD_INDEX);
-        id = 0;
+template <int VEC> struct NcVec;
+template <> struct NcVec<1> {
+    float v[1];
+    __device__ __forceinline__ void load(const float* p) { v[0] = *p; }
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { v[0] = __bfloat162float(*p); }
+    __device__ __forceinline__ void store(float* p) const { *p = v[0]; }
+    __device__ __forceinline__ void store(__nv_bfloat16* p) const { *p = __float2bfloat16_rn(v[0]); }
+};
+template <> struct NcVec<4> {
+    float v[4];
+    __device__ __forceinline__ void load(const float* p) {
+        const float4 f = *reinterpret_cast<const float4*>(p);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
     }
-    return id;
-}
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+        v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+    }
+    __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+    __device__ __forceinline__ void store(__nv_bfloat16* p) const {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    }
+};
 
-template <typename OutT> __device__ __forceinline__ OutT nc_cast(float v);
-template <> __device__ __forceinline__ float nc_cast<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 nc_cast<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
-
-template <typename OutT>
-__device__ __forceinline__ void nc_store(const lv_norm_conv_args& a, uint32_t t, uint32_t i, float v) {
+template <int VEC, typename OutT>
+__device__ __forceinline__ void nc_store(const lv_norm_conv_args& a, uint32_t t, uint32_t i, const NcVec<VEC>& v) {
     OutT* out = static_cast<OutT*>(a.out);
     if (a.out_index == nullptr) {
-        out[size_t(t - a.first) * a.out_ld + i] = nc_cast<OutT>(v);
+        v.store(out + size_t(t - a.first) * a.out_ld + i);
     } else {
-        for (uint32_t s = 0; s < a.out_copies; ++s) out[size_t(a.out_index[t * a.out_copies + s]) * a.out_ld + i] = nc_cast<OutT>(v);
+        for (uint32_t s = 0; s < a.out_copies; ++s) v.store(out + size_t(a.out_index[t * a.out_copies + s]) * a.out_ld + i);
     }
 }
 
-// One token: one CTA, a thread keeps its channels in registers.
-template <int NV, typename OutT>
-__global__ void __launch_bounds__(1024) norm_conv_one_kernel(const NormConvParams p) {
+// CTA b: token a.first + b.  A thread holds NV vectors of VEC channels.
+template <int VEC, int NV, typename OutT>
+__global__ void __launch_bounds__(1024) norm_rows_kernel(const NormConvParams p) {
     pdl_launch_dependents();
     const lv_norm_conv_args& a = p.a;
     __shared__ float scratch[64];
-    const uint32_t W = a.width, t = a.first, keep = a.taps ? a.taps - 1 : 0;
-    float pre[NV], post[NV];
+    const uint32_t W = a.width, t = a.first + blockIdx.x, keep = a.taps ? a.taps - 1 : 0;
+    const bool finish = a.taps == 0 || a.batch == 1;      // else the second launch forms h
+    NcVec<VEC> pre[NV], post[NV];
 #pragma unroll
     for (int k = 0; k < NV; ++k) {                        // weights do not depend on the previous kernel
-        const uint32_t i = threadIdx.x + k * blockDim.x;
-        pre[k] = i < W ? a.pre_w[i] : 0.f;
-        post[k] = (a.y != nullptr && i < W) ? a.post_w[i] : 0.f;
+        const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+        if (i < W) {
+            if (finish) pre[k].load(a.pre_w + i);
+            if (a.y != nullptr) post[k].load(a.post_w + i);
+        }
     }
     pdl_wait();
     const uint32_t pos = *a.pos;
-    const uint32_t id = nc_token(a, pos, t, p.err);
-    float x[NV];
-#pragma unroll
-    for (int k = 0; k < NV; ++k) {
-        const uint32_t i = threadIdx.x + k * blockDim.x;
-        x[k] = i < W ? nc_load_x(a, t, i, id) : 0.f;
-    }
-    if (a.y != nullptr) {
-        float y[NV], part = 0.f;
+    NcVec<VEC> x[NV], y[NV];
+    if (a.x == nullptr) {
+        uint32_t id = a.token_log[pos + t];
+        if (id >= a.vocab) {
+            if (threadIdx.x == 0) atomicOr(p.err, ERR_BAD_INDEX);
+            id = 0;
+        }
+        const __nv_bfloat16* row = static_cast<const __nv_bfloat16*>(a.embed) + size_t(id) * a.embed_ld;
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
-            const uint32_t i = threadIdx.x + k * blockDim.x;
-            y[k] = i < W ? nc_load_y(a, t, i) : 0.f;
-            part = fmaf(y[k], y[k], part);
+            const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+            if (i < W) x[k].load(row + i);
         }
+    } else {
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+            if (i < W) x[k].load(a.x + size_t(t) * W + i);
+        }
+    }
+    if (a.y != nullptr) {
+        float part = 0.f;
+        if (a.y_index == nullptr) {
+#pragma unroll
+            for (int k = 0; k < NV; ++k) {
+                const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+                if (i < W) y[k].load(a.y + size_t(t) * W + i);
+            }
+        } else {
+#pragma unroll
+            for (int k = 0; k < NV; ++k)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) y[k].v[e] = 0.f;
+            for (uint32_t s = 0; s < a.y_rows; ++s) {
+                const float* row = a.y + size_t(a.y_index[t * a.y_rows + s]) * W;
+#pragma unroll
+                for (int k = 0; k < NV; ++k) {
+                    const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+                    NcVec<VEC> v;
+                    if (i < W) {
+                        v.load(row + i);
+#pragma unroll
+                        for (int e = 0; e < VEC; ++e) y[k].v[e] += v.v[e];
+                    }
+                }
+            }
+            const float n = float(a.y_rows);
+#pragma unroll
+            for (int k = 0; k < NV; ++k)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) y[k].v[e] /= n;
+        }
+#pragma unroll
+        for (int k = 0; k < NV; ++k)
+            if ((threadIdx.x + k * blockDim.x) * VEC < W)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) part = fmaf(y[k].v[e], y[k].v[e], part);
         const float r = a.mult / sqrtf(block_sum(part, scratch) / float(W) + a.eps);
 #pragma unroll
-        for (int k = 0; k < NV; ++k) x[k] = fmaf(y[k] * r, 1.f + post[k], x[k]);
+        for (int k = 0; k < NV; ++k)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) x[k].v[e] = fmaf(y[k].v[e] * r, 1.f + post[k].v[e], x[k].v[e]);
     }
     float part = 0.f;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
-        const uint32_t i = threadIdx.x + k * blockDim.x;
-        if (i < W) {
-            if (a.trace != nullptr) a.trace[size_t(t) * W + i] = x[k];
-            if (a.step != nullptr) x[k] += a.step[i];
-            if (a.x_out != nullptr) a.x_out[size_t(t) * W + i] = x[k];
-            part = fmaf(x[k], x[k], part);
+        const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+        if (i >= W) continue;
+        if (a.trace != nullptr) x[k].store(a.trace + size_t(t) * W + i);
+        if (a.step != nullptr) {
+            NcVec<VEC> s;
+            s.load(a.step + i);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) x[k].v[e] += s.v[e];
         }
+        if (a.x_out != nullptr) x[k].store(a.x_out + size_t(t) * W + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) part = fmaf(x[k].v[e], x[k].v[e], part);
     }
     const float r = 1.f / sqrtf(block_sum(part, scratch) / float(W) + a.eps);
+    if (!finish) {
+        if (threadIdx.x == 0) a.row_factor[t] = r;
+        return;
+    }
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
-        const uint32_t i = threadIdx.x + k * blockDim.x;
+        const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
         if (i >= W) continue;
-        const float h = x[k] * r * (1.f + pre[k]);
-        float out = h;
+        NcVec<VEC> h, out;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) out.v[e] = h.v[e] = x[k].v[e] * r * (1.f + pre[k].v[e]);
         if (a.taps) {
-            out = fmaf(a.conv_w[size_t(keep) * W + i], h, out);
+            NcVec<VEC> w, old;
+            w.load(a.conv_w + size_t(keep) * W + i);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) out.v[e] = fmaf(w.v[e], h.v[e], out.v[e]);
             for (uint32_t j = 0; j < keep; ++j) {                   // history oldest first; shifted by one as it is read
-                const float old = pos + j >= keep ? a.history[size_t(j) * W + i] : 0.f;
-                out = fmaf(a.conv_w[size_t(j) * W + i], old, out);
-                if (j > 0) a.history[size_t(j - 1) * W + i] = old;
+                w.load(a.conv_w + size_t(j) * W + i);
+                old.load(a.history + size_t(j) * W + i);
+                if (pos + j < keep) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) old.v[e] = 0.f;
+                }
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) out.v[e] = fmaf(w.v[e], old.v[e], out.v[e]);
+                if (j > 0) old.store(a.history + size_t(j - 1) * W + i);
             }
-            if (keep) a.history[size_t(keep - 1) * W + i] = h;
+            if (keep) h.store(a.history + size_t(keep - 1) * W + i);
         }
-        nc_store<OutT>(a, t, i, out);
+        nc_store<VEC, OutT>(a, t, i, out);
     }
 }
 
-// Several tokens: a CTA takes tokens_per_block of them and recomputes the h of the taps - 1 tokens before its first
-// (x and x_out are different buffers).  Block 0 alone reads the state, whose successor it writes at its end.
-template <int MAXT, typename OutT>
-__global__ void __launch_bounds__(512) norm_conv_kernel(const NormConvParams p) {
+// Second launch for several tokens: blockIdx.x = channels, blockIdx.y = tokens_per_block tokens.  A thread owns VEC channels
+// and slides over its tokens with the last MAXT values of h in registers.  Block row 0 alone reads the state, whose
+// successor it writes at its end.
+template <int VEC, int MAXT, typename OutT>
+__global__ void __launch_bounds__(128) conv_rows_kernel(const NormConvParams p) {
     pdl_launch_dependents();
-    pdl_wait();
     const lv_norm_conv_args& a = p.a;
-    extern __shared__ float sm[];                        // per row: mult / rms(y), 1 / rms(x''); then token ids
-    const uint32_t W = a.width, keep = a.taps ? a.taps - 1 : 0, T = a.batch;
-    const uint32_t t0 = a.first + blockIdx.x * p.tokens_per_block, t1 = min(T, t0 + p.tokens_per_block);
-    const uint32_t halo = min(keep, t0);                 // rows before t0 that belong to this step
-    const uint32_t r_first = t0 - halo;
-    const uint32_t n_main = t1 - r_first;
-    const bool keeper = blockIdx.x == 0 && keep != 0;
-    const uint32_t tail_first = T > keep ? T - keep : 0; // tokens whose h becomes the state
-    const uint32_t n_rows = n_main + (keeper ? T - tail_first : 0);
-    float* s_ry = sm;
-    float* s_rx = sm + n_rows;
-    uint32_t* s_id = reinterpret_cast<uint32_t*>(sm + 2 * n_rows);
-    const uint32_t pos = *a.pos;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-    for (uint32_t r = warp; r < n_rows; r += nwarps) {
-        const uint32_t t = r < n_main ? r_first + r : tail_first + (r - n_main);
-        uint32_t id = 0;
-        if (a.x == nullptr) {
-            id = a.token_log[pos + t];
-            if (id >= a.vocab) {
-                if (lane == 0) atomicOr(p.err, ERR_BAD_INDEX);
-                id = 0;
-            }
+    const uint32_t W = a.width, keep = a.taps - 1, T = a.batch;
+    const uint32_t i = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    const uint32_t t0 = blockIdx.y * p.tokens_per_block, t1 = min(T, t0 + p.tokens_per_block);
+    if (i >= W) return;
+    NcVec<VEC> pre, cw[MAXT], win[MAXT];                  // taps right-aligned: index MAXT - 1 is the current token
+    pre.load(a.pre_w + i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) pre.v[e] += 1.f;
+#pragma unroll
+    for (int j = 0; j < MAXT; ++j) {
+        const int s = j - (MAXT - int(a.taps));
+        if (s >= 0) cw[j].load(a.conv_w + size_t(s) * W + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            if (s < 0) cw[j].v[e] = 0.f;
+            win[j].v[e] = 0.f;
         }
-        float ry = 0.f;
-        if (a.y != nullptr) {
-            float part = 0.f;
-            for (uint32_t i = lane; i < W; i += 32) {
-                const float y = nc_load_y(a, t, i);
-                part = fmaf(y, y, part);
-            }
-            ry = a.mult / sqrtf(warp_sum(part) / float(W) + a.eps);
-        }
-        float part = 0.f;
-        for (uint32_t i = lane; i < W; i += 32) {
-            float x = nc_load_x(a, t, i, id);
-            if (a.y != nullptr) x = fmaf(nc_load_y(a, t, i) * ry, 1.f + a.post_w[i], x);
-            if (a.step != nullptr) x += a.step[i];
-            part = fmaf(x, x, part);
-        }
-        const float rx = 1.f / sqrtf(warp_sum(part) / float(W) + a.eps);
-        if (lane == 0) { s_ry[r] = ry; s_rx[r] = rx; s_id[r] = id; }
     }
-    __syncthreads();
-    for (uint32_t i = threadIdx.x; i < W; i += blockDim.x) {
-        const float pre = 1.f + a.pre_w[i], post = a.y != nullptr ? 1.f + a.post_w[i] : 0.f, step = a.step != nullptr ? a.step[i] : 0.f;
-        float cw[MAXT], win[MAXT];                        // taps right-aligned: index MAXT - 1 is the current token
+    pdl_wait();
+    const uint32_t pos = *a.pos;
+    auto h_of = [&](uint32_t t) {
+        NcVec<VEC> h;
+        h.load(a.x_out + size_t(t) * W + i);
+        const float r = a.row_factor[t];
 #pragma unroll
-        for (int j = 0; j < MAXT; ++j) {
-            const int s = j - (MAXT - int(a.taps));
-            cw[j] = s >= 0 ? a.conv_w[size_t(s) * W + i] : 0.f;
-            win[j] = 0.f;
-        }
-        // the window before row r_first; positions before this step come from the state
+        for (int e = 0; e < VEC; ++e) h.v[e] = h.v[e] * r * pre.v[e];
+        return h;
+    };
+    // the window before t0: win[j] is h of the token MAXT - j before t0, from this step or from the state
 #pragma unroll
-        for (int j = 1; j < MAXT; ++j) {
-            // win[j] will be h of the token (MAXT - j) before r_first
-            const int back = MAXT - j;                    // 1 .. MAXT - 1
-            if (blockIdx.x == 0 && back <= int(keep) && pos >= uint32_t(back)) win[j] = a.history[size_t(keep - back) * W + i];
-        }
-        auto stream = [&](uint32_t r, uint32_t t) {
-            float x = nc_load_x(a, t, i, s_id[r]);
-            if (a.y != nullptr) x = fmaf(nc_load_y(a, t, i) * s_ry[r], post, x);
-            return x;
-        };
-        for (uint32_t r = 0; r < n_main; ++r) {
-            const uint32_t t = r_first + r;
-            float x = stream(r, t);
-            const bool mine = r >= halo;
-            if (mine && a.trace != nullptr) a.trace[size_t(t) * W + i] = x;
-            x += step;
-            if (mine && a.x_out != nullptr) a.x_out[size_t(t) * W + i] = x;
-            const float h = x * s_rx[r] * pre;
+    for (int j = 1; j < MAXT; ++j) {
+        const uint32_t back = MAXT - j;                   // 1 .. MAXT - 1
+        if (back > keep) continue;
+        if (t0 >= back) win[j] = h_of(t0 - back);
+        else if (blockIdx.y == 0 && pos >= back) win[j].load(a.history + size_t(keep - back) * W + i);
+    }
+#pragma unroll 2
+    for (uint32_t t = t0; t < t1; ++t) {
 #pragma unroll
-            for (int j = 0; j + 1 < MAXT; ++j) win[j] = win[j + 1];
-            win[MAXT - 1] = h;
-            if (mine) {
-                float out = h;
+        for (int j = 0; j + 1 < MAXT; ++j) win[j] = win[j + 1];
+        win[MAXT - 1] = h_of(t);
+        NcVec<VEC> out = win[MAXT - 1];
 #pragma unroll
-                for (int j = 0; j < MAXT; ++j) out = fmaf(cw[j], win[j], out);
-                nc_store<OutT>(a, t, i, out);
+        for (int j = 0; j < MAXT; ++j)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) out.v[e] = fmaf(cw[j].v[e], win[j].v[e], out.v[e]);
+        nc_store<VEC, OutT>(a, t, i, out);
+    }
+    if (blockIdx.y != 0) return;
+    for (uint32_t j = 0; j < keep; ++j) {                 // ascending: entries that stay move towards lower indexes
+        NcVec<VEC> v;
+        if (j + T < keep) {
+            v.load(a.history + size_t(j + T) * W + i);
+            if (pos + j + T < keep) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v.v[e] = 0.f;
             }
+        } else {
+            v = h_of(j + T - keep);
         }
-        if (keeper) {
-            for (uint32_t j = 0; j < keep; ++j) {         // ascending: entries that stay move towards lower indexes
-                float v;
-                if (j + T < keep) {
-                    v = pos + j + T >= keep ? a.history[size_t(j + T) * W + i] : 0.f;
-                } else {
-                    const uint32_t t = j + T - keep, r = n_main + (t - tail_first);
-                    v = (stream(r, t) + step) * s_rx[r] * pre;
-                }
-                a.history[size_t(j) * W + i] = v;
-            }
-        }
+        v.store(a.history + size_t(j) * W + i);
     }
 }
 
@@ -237,26 +273,35 @@ static int norm_conv_launch(lv_ctx* ctx, const lv_norm_conv_args& a) {
     NormConvParams p{};
     p.a = a;
     p.err = ctx->d_err;
-    const uint32_t count = a.batch - a.first;
-    if (a.batch == 1 || (count == 1 && a.taps == 0)) {
-        const uint32_t threads = a.width >= 1024 ? 1024 : ((a.width + 31) / 32 * 32);
-        const uint32_t nv = (a.width + threads - 1) / threads;
-        auto go = [&](auto kernel) { return launch_pdl(ctx, kernel, dim3(1), dim3(threads), 0, p); };
-        if (nv <= 1) LV_CUDA(go(norm_conv_one_kernel<1, OutT>));
-        else if (nv <= 2) LV_CUDA(go(norm_conv_one_kernel<2, OutT>));
-        else if (nv <= 4) LV_CUDA(go(norm_conv_one_kernel<4, OutT>));
-        else if (nv <= 8) LV_CUDA(go(norm_conv_one_kernel<8, OutT>));
-        else LV_CUDA(go(norm_conv_one_kernel<16, OutT>));
-        return LV_OK;
-    }
-    const uint32_t keep = a.taps ? a.taps - 1 : 0;
-    p.tokens_per_block = keep > 4 ? keep : 4;            // block 0 holds every token that reads the state
-    const uint32_t blocks = (count + p.tokens_per_block - 1) / p.tokens_per_block;
-    const size_t smem = size_t(p.tokens_per_block + 2 * keep) * 12;
-    auto go = [&](auto kernel) { return launch_pdl(ctx, kernel, dim3(blocks), dim3(512), smem, p); };
-    if (a.taps <= 4) LV_CUDA(go(norm_conv_kernel<4, OutT>));
-    else if (a.taps <= 8) LV_CUDA(go(norm_conv_kernel<8, OutT>));
-    else LV_CUDA(go(norm_conv_kernel<16, OutT>));
+    // four channels per access where every row starts on 16 bytes
+    auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
+    bool vec = a.width % 4 == 0 && a.out_ld % 4 == 0 && a.embed_ld % 4 == 0;
+    for (const void* q : {static_cast<const void*>(a.x), a.embed, static_cast<const void*>(a.y), static_cast<const void*>(a.post_w), static_cast<const void*>(a.step),
+                          static_cast<const void*>(a.trace), static_cast<const void*>(a.x_out), static_cast<const void*>(a.pre_w),
+                          static_cast<const void*>(a.conv_w), static_cast<const void*>(a.history), static_cast<const void*>(a.out)})
+        vec = vec && aligned(q);
+    const uint32_t count = a.batch - a.first, units = vec ? a.width / 4 : a.width;
+    uint32_t nv = vec ? (units <= 1024 ? 1 : units <= 2048 ? 2 : 4) : 16;
+    if (vec && units >= 512 && nv == 1) nv = 2;           // fewer warps to sum over
+    const uint32_t threads = ((units + nv - 1) / nv + 31) / 32 * 32;
+    auto rows = [&](auto kernel) { return launch_pdl(ctx, kernel, dim3(count), dim3(threads), 0, p); };
+    if (!vec) LV_CUDA(rows(norm_rows_kernel<1, 16, OutT>));
+    else if (nv == 1) LV_CUDA(rows(norm_rows_kernel<4, 1, OutT>));
+    else if (nv == 2) LV_CUDA(rows(norm_rows_kernel<4, 2, OutT>));
+    else LV_CUDA(rows(norm_rows_kernel<4, 4, OutT>));
+    if (a.taps == 0 || a.batch == 1) return LV_OK;
+    // the blocks of the first tokens read the state alone: every token that needs it lies in block row 0
+    const uint32_t keep = a.taps - 1, cta_columns = (units + 127) / 128;
+    p.tokens_per_block = 16;
+    while (p.tokens_per_block > 4 && cta_columns * ((count + p.tokens_per_block - 1) / p.tokens_per_block) < 4u * uint32_t(ctx->sm_count)) p.tokens_per_block /= 2;
+    if (p.tokens_per_block < keep) p.tokens_per_block = keep;
+    const dim3 grid(cta_columns, (count + p.tokens_per_block - 1) / p.tokens_per_block);
+    auto conv = [&](auto kernel) { return launch_pdl(ctx, kernel, grid, dim3(128), 0, p); };
+    if (vec && a.taps <= 4) LV_CUDA(conv(conv_rows_kernel<4, 4, OutT>));
+    else if (a.taps <= 4) LV_CUDA(conv(conv_rows_kernel<1, 4, OutT>));
+    else if (vec && a.taps <= 8) LV_CUDA(conv(conv_rows_kernel<4, 8, OutT>));
+    else if (vec) LV_CUDA(conv(conv_rows_kernel<4, 16, OutT>));
+    else LV_CUDA(conv(conv_rows_kernel<1, 16, OutT>));
     return LV_OK;
 }
 
@@ -273,7 +318,7 @@ extern "C" int lv_norm_conv(lv_ctx* ctx, const lv_norm_conv_args* args) {
     LV_REQUIRE(a.x != nullptr || (a.embed && a.token_log && a.vocab && a.embed_ld >= a.width), "norm_conv: no input stream");
     LV_REQUIRE(a.y == nullptr || (a.post_w && a.y_rows && (a.y_index || a.y_rows == 1)), "norm_conv: bad sublayer rows");
     LV_REQUIRE(a.taps <= kNormConvMaxTaps && (a.taps == 0 || (a.conv_w && a.first == 0)) && (a.taps < 2 || a.history), "norm_conv: bad taps");
-    LV_REQUIRE(a.x == nullptr || a.x != a.x_out || a.batch == 1, "norm_conv: the stream cannot be updated in place for several tokens");
+    LV_REQUIRE(a.taps == 0 || a.batch == 1 || (a.x_out && a.row_factor), "norm_conv: several tokens need x_out and row_factor");
     LV_REQUIRE(a.out_index == nullptr || a.out_copies, "norm_conv: bad output rows");
     LV_REQUIRE(a.out_type == LV_TYPE_F32 || a.out_type == LV_TYPE_BF16, "norm_conv: output type");
     return a.out_type == LV_TYPE_F32 ? norm_conv_launch<float>(ctx, a) : norm_conv_launch<__nv_bfloat16>(ctx, a);

@@ -26,7 +26,8 @@ template <typename OutT> __device__ __forceinline__ void scan_store(void* out, s
 template <> __device__ __forceinline__ void scan_store<float>(void* out, size_t at, float v) { static_cast<float*>(out)[at] = v; }
 template <> __device__ __forceinline__ void scan_store<__nv_bfloat16>(void* out, size_t at, float v) { static_cast<__nv_bfloat16*>(out)[at] = __float2bfloat16_rn(v); }
 
-template <typename OutT>
+// PER > 0: a segment has at most PER tokens, whose gate and candidate stay in registers between the two walks.
+template <int PER, typename OutT>
 __global__ void __launch_bounds__(1024) mingru_scan_kernel(const MingruScanParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -34,10 +35,27 @@ __global__ void __launch_bounds__(1024) mingru_scan_kernel(const MingruScanParam
     const uint32_t lane = threadIdx.x & 31u, seg = threadIdx.x >> 5;
     const uint32_t c = blockIdx.x * 32u + lane;
     const bool live = c < p.channels;
-    const uint32_t per = (p.T + kScanSegments - 1) / kScanSegments, t0 = min(p.T, seg * per), t1 = min(p.T, t0 + per);
+    const uint32_t per = (p.T + kScanSegments - 1) / kScanSegments, t0 = min(p.T, seg * per), t1 = live ? min(p.T, t0 + per) : t0;
     const float bz = live ? p.bz[c] : 0.f, bx = live ? p.bx[c] : 0.f;
-    float A = 1.f, B = 0.f;
-    if (live) {
+    constexpr int N = PER > 0 ? PER : 1;
+    float z[N], u[N], A = 1.f, B = 0.f;
+    if constexpr (PER > 0) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) {                    // all loads before the first use
+            if (t0 + i >= t1) continue;
+            const float* r = p.raw + size_t(t0 + i) * p.raw_ld + c;
+            z[i] = r[0];
+            u[i] = r[p.channels];
+        }
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            if (t0 + i >= t1) continue;
+            z[i] = sigmoid_f32(z[i] + bz);
+            u[i] = z[i] * mingru_candidate(u[i] + bx);
+            A *= 1.f - z[i];
+            B = fmaf(1.f - z[i], B, u[i]);
+        }
+    } else {
 #pragma unroll 4
         for (uint32_t t = t0; t < t1; ++t) {
             const float* r = p.raw + size_t(t) * p.raw_ld + c;
@@ -58,14 +76,34 @@ __global__ void __launch_bounds__(1024) mingru_scan_kernel(const MingruScanParam
         }
     }
     __syncthreads();
-    if (!live) return;
+    if (t0 >= t1) return;
     float S = s_a[seg][lane];
+    if constexpr (PER > 0) {
+        float g[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) g[i] = t0 + i < t1 ? p.raw[size_t(t0 + i) * p.raw_ld + 2 * p.channels + c] : 0.f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            if (t0 + i >= t1) continue;
+            S = fmaf(1.f - z[i], S, u[i]);
+            scan_store<OutT>(p.out, size_t(t0 + i) * p.out_ld + c, S * silu_f32(g[i]));
+        }
+    } else {
 #pragma unroll 4
-    for (uint32_t t = t0; t < t1; ++t) {
-        const float* r = p.raw + size_t(t) * p.raw_ld + c;
-        scan_store<OutT>(p.out, size_t(t) * p.out_ld + c, mingru_step(r[0] + bz, r[p.channels] + bx, r[2 * p.channels], S, &S));
+        for (uint32_t t = t0; t < t1; ++t) {
+            const float* r = p.raw + size_t(t) * p.raw_ld + c;
+            scan_store<OutT>(p.out, size_t(t) * p.out_ld + c, mingru_step(r[0] + bz, r[p.channels] + bx, r[2 * p.channels], S, &S));
+        }
     }
-    if (t1 == p.T && t0 < t1) p.state[c] = S;           // the segment that holds the last token
+    if (t1 == p.T) p.state[c] = S;                      // the segment that holds the last token
+}
+
+template <typename OutT>
+static cudaError_t mingru_scan_launch(lv_ctx* ctx, const MingruScanParams& p) {
+    const dim3 grid((p.channels + 31) / 32), block(1024);
+    if (p.T <= 4 * kScanSegments) return launch_pdl(ctx, mingru_scan_kernel<4, OutT>, grid, block, 0, p);
+    if (p.T <= 16 * kScanSegments) return launch_pdl(ctx, mingru_scan_kernel<16, OutT>, grid, block, 0, p);
+    return launch_pdl(ctx, mingru_scan_kernel<0, OutT>, grid, block, 0, p);
 }
 
 }  // namespace lv
@@ -78,8 +116,6 @@ extern "C" int lv_mingru_scan(lv_ctx* ctx, void* out, int out_type, uint32_t out
     LV_REQUIRE(out && raw && bz && bx && state && pos && channels && batch, "bad mingru_scan arguments");
     LV_REQUIRE(raw_ld >= 3 * channels && out_ld >= channels && (out_type == LV_TYPE_F32 || out_type == LV_TYPE_BF16), "mingru_scan: bad layout");
     MingruScanParams p{raw, raw_ld, channels, batch, bz, bx, state, pos, out, out_ld};
-    const dim3 grid((channels + 31) / 32), block(1024);
-    if (out_type == LV_TYPE_F32) LV_CUDA(launch_pdl(ctx, mingru_scan_kernel<float>, grid, block, 0, p));
-    else LV_CUDA(launch_pdl(ctx, mingru_scan_kernel<__nv_bfloat16>, grid, block, 0, p));
+    LV_CUDA(out_type == LV_TYPE_F32 ? mingru_scan_launch<float>(ctx, p) : mingru_scan_launch<__nv_bfloat16>(ctx, p));
     return LV_OK;
 }

@@ -252,7 +252,8 @@ struct hybrid_recorder {
         a.post_w = f32(post);
         a.step = step;
         if (finished_run >= 0 && !st->trace.empty()) a.trace = f32(st->trace[finished_run]);
-        a.x_out = (x == f32(st->stream_a) && T > 1) ? f32(st->stream_b) : f32(st->stream_a);
+        a.x_out = f32(st->stream);
+        a.row_factor = f32(st->row_factor);
         a.pre_w = f32(pre);
         if (conv) {
             a.conv_w = f32(conv);
@@ -387,11 +388,7 @@ struct hybrid_recorder {
             product(st->logits_rows, arch.head, st->normed, pad8(cfg.width), cfg.logit_scale);
         } else if (cb->with_head) {
             // only the last row's logits are wanted; a trace wants the last layer's stream of every row as well
-            if (!st->trace.empty() && T > 1) {
-                const hybrid_recorder before = *this;
-                norm_conv(arch.final_norm, nullptr, nullptr, nullptr);
-                x = before.x, y = before.y, y_index = before.y_index, y_rows = before.y_rows, post = before.post;
-            }
+            if (!st->trace.empty() && T > 1) norm_conv(arch.final_norm, nullptr, nullptr, nullptr);      // (finishes the last sublayer for all rows)
             norm_conv(arch.final_norm, nullptr, nullptr, nullptr, nullptr, 1, true);
             cb->note(lv_gemv_bf16(lv, f32(s->output_probs), cfg.vocab, arch.head->device_ptr(), cfg.vocab, arch.head->leading(), cfg.width,
                                   f32(st->normed), pad8(cfg.width), 1, cfg.logit_scale));

@@ -47,7 +47,7 @@ hybrid_session_state::~hybrid_session_state() {
 }
 
 void hybrid_session_state::drop_scratch() {
-    for (llava_buffer** b : {&stream_a, &stream_b, &normed, &raw, &mixed, &act, &sub, &attn_scratch, &logits_rows, &route_jobs}) {
+    for (llava_buffer** b : {&stream, &row_factor, &normed, &raw, &mixed, &act, &sub, &attn_scratch, &logits_rows, &route_jobs}) {
         delete *b;
         *b = nullptr;
     }
@@ -89,8 +89,8 @@ bool hybrid_session_state::resize() {
     }
     const auto F = ggml_value_type::f32;
     scratch = new llava_device_memory(ctx);
-    stream_a = new llava_buffer(ctx, F, c.width, B, scratch);
-    stream_b = new llava_buffer(ctx, F, c.width, B, scratch);
+    stream = new llava_buffer(ctx, F, c.width, B, scratch);
+    row_factor = new llava_buffer(ctx, F, 1, B, scratch);
     normed = new llava_buffer(ctx, F, pad8(c.width) * copies, B, scratch);
     raw = new llava_buffer(ctx, F, raw_size, B, scratch);
     mixed = new llava_buffer(ctx, F, mixed_size, B, scratch);

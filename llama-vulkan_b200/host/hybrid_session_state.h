@@ -29,7 +29,8 @@ public:
     const hybrid_architecture* const arch;
     std::vector<hybrid_run_state> runs;
     // scratch of one step
-    llava_buffer *stream_a = nullptr, *stream_b = nullptr;    // residual stream, f32 [batch][width]
+    llava_buffer *stream = nullptr;                           // residual stream, f32 [batch][width]
+    llava_buffer *row_factor = nullptr;                       // one word per token between the two launches of lv_norm_conv
     llava_buffer *normed = nullptr;                           // input of a sublayer, one row per token or per chosen expert
     llava_buffer *raw = nullptr;                              // input projections, f32
     llava_buffer *mixed = nullptr;                            // mixer output before its output projection

@@ -198,7 +198,7 @@ def test_norm_conv_in_portions(gpu, width, taps, cuts):
             xa, xb, tr = d.zeros(n * width * 4), d.zeros(n * width * 4), d.zeros(n * width * 4)
             out = d.zeros(n * pad8(width) * 4)
             a = pkg.NormConvArgs(embed=emb.value, embed_ld=pad8(width), vocab=vocab, token_log=log.value, pos=pos.value, eps=EPS, mult=mult, step=dstep.value,
-                                 x_out=xa.value, pre_w=dpre.value, conv_w=dconv.value, history=hist.value, taps=taps, out=out.value, out_type=pkg.TYPE_F32,
+                                 x_out=xa.value, row_factor=d.zeros(n * 4).value, pre_w=dpre.value, conv_w=dconv.value, history=hist.value, taps=taps, out=out.value, out_type=pkg.TYPE_F32,
                                  out_ld=pad8(width), width=width, batch=n, y_rows=1)
             d.call("lv_norm_conv", C.byref(a))
             assert rel(d.get(out, (n, pad8(width)))[:, :width], want0[at:at + n]) < 2e-6
@@ -208,7 +208,7 @@ def test_norm_conv_in_portions(gpu, width, taps, cuts):
             rows = rng.permutation(3 * n).reshape(n, 3)
             out16 = d.zeros(3 * n * pad8(width) * 2)
             b = pkg.NormConvArgs(x=xa.value, pos=pos.value, y=y_at.value, y_index=index.value, y_rows=2, post_w=dpost.value, eps=EPS, mult=mult, trace=tr.value,
-                                 x_out=(xa if n == 1 else xb).value, pre_w=dpre2.value, conv_w=dconv2.value, history=hist2.value, taps=taps, out=out16.value,
+                                 x_out=(xa if n == 1 else xb).value, row_factor=d.zeros(n * 4).value, pre_w=dpre2.value, conv_w=dconv2.value, history=hist2.value, taps=taps, out=out16.value,
                                  out_type=pkg.TYPE_BF16, out_ld=pad8(width), out_index=d.u32(rows).value, out_copies=3, width=width, batch=n)
             d.call("lv_norm_conv", C.byref(b))
             assert rel(d.get(tr, (n, width)), x1[at:at + n]) < 1e-6
