@@ -5,8 +5,9 @@
 //   p_ij = exp(s_ij) / (sink + sum_j exp(s_ij)),     sink = 1 or 0
 //
 // One CTA serves up to eight query heads of one key/value head for one token and walks its share of the keys in chunks of
-// 64 with an online softmax.  A decoded token spreads the chunks over several CTAs (the last to arrive combines their
-// partial sums through scratch) and its own key and value are normalised and appended to the caches by the same launch;
+// 64 with an online softmax.  A decoded token spreads the chunks over several CTAs: up to 16 form a thread-block cluster and
+// combine their partial sums through distributed shared memory; beyond that (long contexts) the last to arrive combines
+// them through scratch.  A decoded token's own key and value are normalised and appended to the caches by the same launch;
 // tokens of a prompt are appended first (lv_qk_norm_append) and, with bfloat16 caches, go through attention_gqa_tc.cu.  Caches are [kv head][ctx_rows][padded dim], bfloat16 or f32.
 #include <cuda_bf16.h>
 #include <math.h>
@@ -20,13 +21,14 @@
 namespace lv {
 
 constexpr size_t kGqaCounterBytes = 4096;   // arrival counters at the start of the scratch (kept zero between launches)
-constexpr int kGqaThreads = 256, kGqaWarps = 8, kGqaChunk = 64, kGqaHeads = 8, kGqaMaxSplits = 128;
+constexpr int kGqaThreads = 256, kGqaWarps = 8, kGqaChunk = 64, kGqaHeads = 8, kGqaMaxSplits = 128, kGqaCluster = 16;
 
 struct GqaParams {
     lv_gqa_args a;
     uint32_t dim_p, vdim_p;         // padded to 8
     uint32_t head_blocks;           // CTAs per key/value head
     uint32_t splits;
+    uint32_t clustered;             // the splits of a token are one thread-block cluster
     uint32_t out_bf16, append;
     float* scratch;                 // splits > 1: [token][head][split][vdim_p + 2]
     uint32_t* counters;             // [token][kv head * head_blocks]
@@ -44,6 +46,8 @@ template <> struct Cache8<__nv_bfloat16> {
         for (int i = 0; i < 4; ++i) { v[2 * i] = __uint_as_float(q[i] << 16); v[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u); }
     }
     static __device__ __forceinline__ __nv_bfloat16 cast(float v) { return __float2bfloat16_rn(v); }
+    // (the fast logarithm is good to about 2^-21 here, far below the rounding of the operands)
+    static __device__ __forceinline__ float log_one_plus(float v) { return __logf(1.f + v); }
 };
 template <> struct Cache8<float> {
     struct raw { float4 a, b; };
@@ -52,7 +56,20 @@ template <> struct Cache8<float> {
         v[0] = w.a.x; v[1] = w.a.y; v[2] = w.a.z; v[3] = w.a.w; v[4] = w.b.x; v[5] = w.b.y; v[6] = w.b.z; v[7] = w.b.w;
     }
     static __device__ __forceinline__ float cast(float v) { return v; }
+    static __device__ __forceinline__ float log_one_plus(float v) { return log1pf(v); }
 };
+
+__device__ __forceinline__ void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// a float in the shared memory of another CTA of the cluster
+__device__ __forceinline__ float cluster_load(const float* local, uint32_t rank) {
+    uint32_t at;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"(smem_u32(local)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(at));
+    return v;
+}
 
 // Appends the normalised key and the value of token t (one warp per key/value head).
 template <typename CT>
@@ -102,53 +119,67 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
 
     const uint32_t sub = lane & (L - 1), key_in_warp = lane / L;
     const uint32_t vcol = (threadIdx.x & (L - 1)) * 8, vgroup = threadIdx.x / L;
-    const float r1 = sub < nh ? a.r1[h0 + sub] : 0.f, r2 = sub < nh ? a.r2[h0 + sub] : 0.f;
+    // the lane that ends up with head h's score of a key is lane h * (L / HB) of the key's lanes
+    const uint32_t my_head = sub / (L / HB);
+    const bool score_lane = sub % (L / HB) == 0;
+    const float r1 = my_head < nh ? a.r1[h0 + my_head] : 0.f, r2 = my_head < nh ? a.r2[h0 + my_head] : 0.f;
+    // warp h normalises query head h, the last warp the token's own key
+    const bool own_key = warp == kGqaWarps - 1;
+    float qw[L / 4], kw[L / 4];
+    gqa_head_load<L / 4>(qw, a.q_norm, a.dim, warp < int(nh));
+    gqa_head_load<L / 4>(kw, a.k_norm, a.dim, own_key);
     pdl_wait();
-    const uint32_t P = *a.pos + t;
-    if (P >= a.ctx_rows) {
-        if (threadIdx.x == 0) atomicOr(p.err, ERR_BAD_INDEX);
-        return;
-    }
     CT* kc = static_cast<CT*>(a.k_cache) + size_t(g) * a.ctx_rows * p.dim_p;
     CT* vc = static_cast<CT*>(a.v_cache) + size_t(g) * a.ctx_rows * p.vdim_p;
     const bool append = p.append != 0;
-    const uint32_t own_chunk = P / kGqaChunk;
-    // a chunk's keys and values are requested before anything waits for them
+    // a chunk's keys and values are requested before anything waits for them (rows up to `limit`; the position is not known
+    // yet when the first chunk is requested, so rows behind it come along and are never used)
     typename Cache8<CT>::raw kr[kIters], vr[kIters];
-    auto fetch = [&](uint32_t k0) {
+    auto fetch = [&](uint32_t k0, uint32_t limit) {
 #pragma unroll
         for (int i = 0; i < kIters; ++i) {
             const uint32_t j = k0 + (i * kGqaWarps + warp) * kPerWarp + key_in_warp;
-            if (sub * 8 < p.dim_p && j <= P && !(append && j == P)) kr[i] = Cache8<CT>::fetch(kc + size_t(j) * p.dim_p + sub * 8);
+            if (sub * 8 < p.dim_p && j < limit) kr[i] = Cache8<CT>::fetch(kc + size_t(j) * p.dim_p + sub * 8);
         }
 #pragma unroll
         for (int i = 0; i < kIters; ++i) {
             const uint32_t j = k0 + i * kGroups + vgroup;
-            if (vcol < p.vdim_p && j <= P && !(append && j == P)) vr[i] = Cache8<CT>::fetch(vc + size_t(j) * p.vdim_p + vcol);
+            if (vcol < p.vdim_p && j < limit) vr[i] = Cache8<CT>::fetch(vc + size_t(j) * p.vdim_p + vcol);
         }
     };
-    if (blockIdx.y <= own_chunk) fetch(blockIdx.y * kGqaChunk);
+    const uint32_t P = *a.pos + t;
     const float* raw = a.qkv + size_t(t) * a.qkv_ld;
-    if (warp < int(nh)) {
-        const float* q = raw + (h0 + warp) * a.dim;
-        const float r = gqa_rms_factor(q, a.dim, a.eps) * a.scale;
-        for (uint32_t i = lane; i < p.dim_p; i += 32) s_q[warp * p.dim_p + i] = i < a.dim ? q[i] * r * a.q_norm[i] : 0.f;
-    } else if (warp < HB) {
-        for (uint32_t i = lane; i < p.dim_p; i += 32) s_q[warp * p.dim_p + i] = 0.f;
+    float q[L / 4], k[L / 4], v[L / 4];
+    gqa_head_load<L / 4>(q, raw + (h0 + warp) * a.dim, a.dim, warp < int(nh));
+    gqa_head_load<L / 4>(k, raw + a.heads * a.dim + g * a.dim, a.dim, own_key);
+    gqa_head_load<L / 4>(v, raw + (a.heads + a.kv_heads) * a.dim + g * a.vdim, a.vdim, own_key);
+    fetch(blockIdx.y * kGqaChunk, a.ctx_rows);
+    if (P >= a.ctx_rows) {                                 // (the same for every CTA of a cluster)
+        if (threadIdx.x == 0) atomicOr(p.err, ERR_BAD_INDEX);
+        return;
     }
-    if (append && own_chunk % p.splits == blockIdx.y && warp == kGqaWarps - 1) {
-        const float* k = raw + a.heads * a.dim + g * a.dim;
-        const float* v = raw + (a.heads + a.kv_heads) * a.dim + g * a.vdim;
-        const float r = gqa_rms_factor(k, a.dim, a.eps);
-        for (uint32_t i = lane; i < p.dim_p; i += 32) {
-            const CT e = Cache8<CT>::cast(i < a.dim ? k[i] * r * a.k_norm[i] : 0.f);
-            s_k[i] = e;
-            if (hb == 0) kc[size_t(P) * p.dim_p + i] = e;
-        }
-        for (uint32_t i = lane; i < p.vdim_p; i += 32) {
-            const CT e = Cache8<CT>::cast(i < a.vdim ? v[i] : 0.f);
-            s_v[i] = e;
-            if (hb == 0) vc[size_t(P) * p.vdim_p + i] = e;
+    const uint32_t own_chunk = P / kGqaChunk;
+    if (warp < HB) {
+        const float r = gqa_head_factor<L / 4>(q, a.dim, a.eps) * a.scale;
+#pragma unroll
+        for (int i = 0; i < L / 4; ++i)
+            if (lane + 32 * i < int(p.dim_p)) s_q[warp * p.dim_p + lane + 32 * i] = q[i] * r * qw[i];      // zeros for missing heads and columns
+    }
+    if (append && own_key && own_chunk % p.splits == blockIdx.y) {
+        const float r = gqa_head_factor<L / 4>(k, a.dim, a.eps);
+#pragma unroll
+        for (int i = 0; i < L / 4; ++i) {
+            const uint32_t c = lane + 32 * i;
+            if (c < p.dim_p) {
+                const CT e = Cache8<CT>::cast(k[i] * r * kw[i]);
+                s_k[c] = e;
+                if (hb == 0) kc[size_t(P) * p.dim_p + c] = e;
+            }
+            if (c < p.vdim_p) {
+                const CT e = Cache8<CT>::cast(v[i]);
+                s_v[c] = e;
+                if (hb == 0) vc[size_t(P) * p.vdim_p + c] = e;
+            }
         }
     }
     if (threadIdx.x < HB) { s_m[threadIdx.x] = -INFINITY; s_l[threadIdx.x] = 0.f; }
@@ -161,12 +192,12 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
 
     for (uint32_t c = blockIdx.y; c <= own_chunk; c += p.splits) {
         const uint32_t k0 = c * kGqaChunk;
-        if (c != blockIdx.y) fetch(k0);
+        if (c != blockIdx.y) fetch(k0, P + 1);
         float bias[kIters];
 #pragma unroll
         for (int i = 0; i < kIters; ++i) {
             const uint32_t j = k0 + (i * kGqaWarps + warp) * kPerWarp + key_in_warp;
-            bias[i] = j <= P ? r1 * log1pf(r2 * float(P - j)) : 0.f;
+            bias[i] = j <= P ? r1 * Cache8<CT>::log_one_plus(r2 * float(P - j)) : 0.f;
         }
 #pragma unroll
         for (int i = 0; i < kIters; ++i) {
@@ -177,21 +208,31 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
                 if (append && j == P) kr[i] = Cache8<CT>::fetch(s_k + sub * 8);
                 Cache8<CT>::widen(kv, kr[i]);
             }
-            float mine = 0.f;
+            float sum[HB];
 #pragma unroll
             for (int h = 0; h < HB; ++h) {
-                float s = 0.f;
+                sum[h] = 0.f;
                 if (live) {
                     float qv[8];
                     Cache8<float>::widen(qv, Cache8<float>::fetch(s_q + h * p.dim_p + sub * 8));
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) s = fmaf(qv[e], kv[e], s);
+                    for (int e = 0; e < 8; ++e) sum[h] = fmaf(qv[e], kv[e], sum[h]);
                 }
-#pragma unroll
-                for (int o = L / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-                if (sub == uint32_t(h)) mine = s;
             }
-            if (sub < HB) s_sc[sub * kGqaChunk + kk] = (j <= P && sub < nh) ? mine - bias[i] : -INFINITY;
+            // the key's lanes share the sums of all heads: each exchange halves the heads a lane keeps
+            int o = L / 2;
+#pragma unroll
+            for (int n = HB / 2; n > 0; n /= 2, o /= 2) {
+                const bool upper = (sub & o) != 0;
+#pragma unroll
+                for (int h = 0; h < n; ++h) {
+                    const float keep = upper ? sum[h + n] : sum[h], give = upper ? sum[h] : sum[h + n];
+                    sum[h] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                }
+            }
+#pragma unroll
+            for (; o > 0; o /= 2) sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], o);
+            if (score_lane) s_sc[my_head * kGqaChunk + kk] = (j <= P && my_head < nh) ? sum[0] - bias[i] : -INFINITY;
         }
         __syncthreads();
         // online softmax: warp h takes head h
@@ -245,6 +286,7 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
         }
     __syncthreads();
     const uint32_t part = p.vdim_p + 2;
+    float* s_part = s_red + kGqaWarps * HB * L * 8 + 4 * HB + (p.dim_p + p.vdim_p) * sizeof(CT) / 4;      // behind s_v: [HB][part]
     for (uint32_t e = threadIdx.x; e < nh * p.vdim_p; e += kGqaThreads) {
         const uint32_t h = e / p.vdim_p, col = e - h * p.vdim_p;
         float v = 0.f;
@@ -256,11 +298,44 @@ __global__ void __launch_bounds__(kGqaThreads) gqa_kernel(const GqaParams p) {
                 const float M = a.sink ? fmaxf(m, 0.f) : m, f = expf(m - M);
                 gqa_store_out(a.out, p.out_bf16, size_t(t) * a.out_ld + (h0 + h) * a.vdim + col, v * f / (l * f + (a.sink ? expf(-M) : 0.f)));
             }
+        } else if (p.clustered) {
+            s_part[h * part + 2 + col] = v;
+            if (col == 0) { s_part[h * part] = m; s_part[h * part + 1] = l; }
         } else {
             float* dst = p.scratch + ((size_t(t) * a.heads + h0 + h) * p.splits + blockIdx.y) * part;
             dst[2 + col] = v;
             if (col == 0) { dst[0] = m; dst[1] = l; }
         }
+    }
+    if (p.clustered) {
+        cluster_sync();                                    // every CTA's partial sums are in its shared memory
+        // each CTA combines its slice of the values
+        const uint32_t all = nh * a.vdim, slice = (all + p.splits - 1) / p.splits, e_end = min(all, (blockIdx.y + 1) * slice);
+        for (uint32_t e = blockIdx.y * slice + threadIdx.x; e < e_end; e += kGqaThreads) {
+            const uint32_t h = e / a.vdim, col = e - h * a.vdim;
+            const float* mine = s_part + h * part;
+            float m[kGqaCluster], l[kGqaCluster], v[kGqaCluster];
+#pragma unroll
+            for (int s = 0; s < kGqaCluster; ++s) {        // all loads before the first use
+                const uint32_t rank = min(uint32_t(s), p.splits - 1);
+                m[s] = cluster_load(mine, rank);
+                l[s] = cluster_load(mine + 1, rank);
+                v[s] = cluster_load(mine + 2 + col, rank);
+            }
+            float M = a.sink ? 0.f : -INFINITY, num = 0.f;
+#pragma unroll
+            for (int s = 0; s < kGqaCluster; ++s) M = fmaxf(M, m[s]);
+            float den = a.sink ? expf(-M) : 0.f;
+#pragma unroll
+            for (int s = 0; s < kGqaCluster; ++s) {
+                const float f = uint32_t(s) < p.splits ? expf(m[s] - M) : 0.f;
+                den = fmaf(f, l[s], den);
+                num = fmaf(f, v[s], num);
+            }
+            gqa_store_out(a.out, p.out_bf16, size_t(t) * a.out_ld + (h0 + h) * a.vdim + col, num / den);
+        }
+        cluster_sync();                                    // no CTA leaves while another reads its shared memory
+        return;
     }
     if (p.splits == 1) return;
     __threadfence();
@@ -327,12 +402,32 @@ static int gqa_check(const lv_gqa_args* a, uint32_t batch) {
 
 template <typename CT, int HB, int L>
 static int gqa_launch_typed(lv_ctx* ctx, const GqaParams& p, uint32_t batch) {
-    const size_t smem = sizeof(float) * (size_t(HB) * p.dim_p + HB * kGqaChunk + size_t(kGqaWarps) * HB * L * 8 + 5 * HB) + sizeof(CT) * (p.dim_p + p.vdim_p) + 16;
+    const size_t smem = sizeof(float) * (size_t(HB) * p.dim_p + HB * kGqaChunk + size_t(kGqaWarps) * HB * L * 8 + 4 * HB + size_t(HB) * (p.vdim_p + 2)) + sizeof(CT) * (p.dim_p + p.vdim_p) + 16;
     static_assert(kGqaWarps * L * 8 >= kGqaMaxSplits, "the combination's weights reuse the reduction buffer");
     LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "attention: head sizes need too much shared memory");
     auto* kernel = gqa_kernel<CT, HB, L>;
     if (smem > 48 * 1024) LV_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-    LV_CUDA(launch_pdl(ctx, kernel, dim3(p.a.kv_heads * p.head_blocks, p.splits, batch), dim3(kGqaThreads), smem, p));
+    const dim3 grid(p.a.kv_heads * p.head_blocks, p.splits, batch);
+    if (!p.clustered) {
+        LV_CUDA(launch_pdl(ctx, kernel, grid, dim3(kGqaThreads), smem, p));
+        return LV_OK;
+    }
+    if (p.splits > 8) LV_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(kGqaThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = 1;
+    attr[1].val.clusterDim.y = p.splits;
+    attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
+    LV_CUDA(cudaLaunchKernelEx(&cfg, kernel, p));
     return LV_OK;
 }
 
@@ -393,9 +488,14 @@ extern "C" int lv_attention_gqa(lv_ctx* ctx, const lv_gqa_args* a, void* scratch
     p.vdim_p = pad8(a->vdim);
     p.head_blocks = gqa_head_blocks(*a);
     p.splits = gqa_splits(ctx, *a, batch, capacity);
+    // up to 64 chunks of keys are shared by a cluster of at most 16 CTAs; longer contexts need more CTAs than a cluster has
+    if (p.splits > 1 && capacity <= 64 * kGqaChunk) {
+        p.splits = std::min(p.splits, uint32_t(kGqaCluster));
+        p.clustered = 1;
+    }
     p.out_bf16 = a->out_type == LV_TYPE_BF16;
     p.err = ctx->d_err;
-    if (p.splits > 1) {
+    if (p.splits > 1 && !p.clustered) {
         // fewer than two CTAs per SM would run unsplit, so the counters of a split launch always fit
         LV_REQUIRE(size_t(batch) * a->kv_heads * p.head_blocks * 4 <= kGqaCounterBytes, "attention: too many arrival counters");
         const size_t need = kGqaCounterBytes + size_t(batch) * a->heads * p.splits * (p.vdim_p + 2) * 4;

@@ -19,6 +19,24 @@ __device__ __forceinline__ float gqa_rms_factor(const float* v, uint32_t dim, fl
     return 1.f / sqrtf(warp_sum(part) / float(dim) + eps);
 }
 
+// A head's vector spread over a warp: value lane + 32 i in v[i]; zeros beyond dim and for warps without one
+template <int N>
+__device__ __forceinline__ void gqa_head_load(float (&v)[N], const float* src, uint32_t dim, bool live) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        const uint32_t c = (threadIdx.x & 31u) + 32u * i;
+        v[i] = live && c < dim ? src[c] : 0.f;
+    }
+}
+// 1 / rms of such a vector
+template <int N>
+__device__ __forceinline__ float gqa_head_factor(const float (&v)[N], uint32_t dim, float eps) {
+    float part = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) part = fmaf(v[i], v[i], part);
+    return 1.f / sqrtf(warp_sum(part) / float(dim) + eps);
+}
+
 __device__ __forceinline__ void gqa_store_out(void* out, uint32_t bf16, size_t at, float v) {
     if (bf16) static_cast<__nv_bfloat16*>(out)[at] = __float2bfloat16_rn(v);
     else static_cast<float*>(out)[at] = v;

@@ -4,12 +4,16 @@
 // heads share the keys -- and walks the keys in blocks of 64:
 //
 //   S = Q K^T      Q normalised, scaled and rounded to bfloat16 in shared memory (128-byte swizzle), K by TMA from the cache
-//   P = exp2(S - bias - m)      four warps, one row per thread; P goes to tensor memory over the scores it came from
+//   P = exp2(S - bias - m)      one row per thread; P goes to tensor memory over the scores it came from
 //   O += P V       P is the TMEM operand, V by TMA as an MN-major operand (its rows are keys)
 //
+// Two threads share a row where tensor memory allows (values of up to 192): each takes one half of every key block, with its
+// own running maximum, sum and O, and the halves meet once, at the end.  A prompt has few tiles per SM, so the softmax is
+// bound by the latency of a thread's chain, which this halves.
+//
 // Two score buffers let S of the next block run under the softmax of this one.  The distance bias of a block is a small
-// table per head: distances within a block and a tile differ by less than (tokens + 64), so log1p is evaluated once per
-// (head, distance) instead of once per score.  O stays in tensor memory; it is rescaled only when a row's maximum has grown
+// table per head: distances within a block and a tile differ by less than (tokens + 64), so the logarithm is evaluated
+// once per (head, distance) instead of once per score.  O stays in tensor memory; it is rescaled only when a row's maximum has grown
 // by more than 2^8, which with a sink (maximum >= 0 from the start) is rare.  Everything except the operands is f32.
 //
 // Every wait is bounded (common.cuh); a lost wait sets the error word, the CTA drains and frees its tensor memory.
@@ -25,7 +29,9 @@
 
 namespace lv {
 
-constexpr int kGtThreads = 192;              // TMA warp, MMA warp, four softmax warps
+// warps: TMA, S products, P V products (each issued by one lane: a single lane would spend longer on the instructions and
+// waits of both than the softmax takes), then four softmax warps per half
+constexpr int kGtFirstSoftmax = 3;
 constexpr int kGtRows = 128, kGtKeys = 64;
 constexpr uint32_t kGtQChunk = kGtRows * 128, kGtKChunk = kGtKeys * 128;      // 64 columns of Q / of K or V, bytes
 constexpr uint32_t kGtMaxStages = 4;
@@ -62,7 +68,15 @@ __device__ __forceinline__ void gt_store16(uint32_t taddr, const uint32_t (&u)[1
 }
 __device__ __forceinline__ void gt_wait_store() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-__global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p, const __grid_constant__ GqaTcMaps maps) {
+__device__ __forceinline__ float gt_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// NH: halves a row is split into; PAIRS: 64 PAIRS >= head size
+template <int NH, int PAIRS>
+__global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel(const GqaTcParams p, const __grid_constant__ GqaTcMaps maps) {
     pdl_launch_dependents();
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023u) & ~uintptr_t(1023));
@@ -71,7 +85,9 @@ __global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p,
     uint8_t* s_kv = s_q + p.dim_chunks * kGtQChunk;
     const uint32_t k_bytes = p.dim_chunks * kGtKChunk, v_bytes = p.v_chunks * kGtKChunk, stage = k_bytes + v_bytes;
     float* s_tab = reinterpret_cast<float*>(s_kv + p.stages * stage);           // [2][group][tab_stride]
-    __shared__ uint64_t k_full[kGtMaxStages], v_full[kGtMaxStages], kv_empty[kGtMaxStages], s_full[2], p_full[2], pv_done;
+    constexpr int kThreads = 32 * kGtFirstSoftmax + 128 * NH, kHalfKeys = kGtKeys / NH;
+    __shared__ float s_ml[2][kGtRows];                           // maximum and sum of the second half
+    __shared__ uint64_t k_full[kGtMaxStages], v_full[kGtMaxStages], kv_empty[kGtMaxStages], s_full[2], p_full[2], pv_done[2];
     __shared__ uint32_t s_tmem;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const uint32_t group = a.heads / a.kv_heads, g = blockIdx.y;
@@ -80,8 +96,7 @@ __global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p,
 
     if (threadIdx.x == 0) {
         for (uint32_t i = 0; i < kGtMaxStages; ++i) { mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&kv_empty[i], 1); }
-        for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], 4); }
-        mbar_init(&pv_done, 1);
+        for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], 4 * NH); mbar_init(&pv_done[i], 1); }
         fence_mbar_init();
     }
     if (warp == 1) tc_alloc(&s_tmem, p.tmem_cols);
@@ -89,17 +104,49 @@ __global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p,
     const uint32_t P = *a.pos;
     const bool inside = P + p.n_tokens <= a.ctx_rows;            // (lv_qk_norm_append reports positions beyond the cache)
     const uint32_t n_keys = P + t_last + 1, n_blocks = inside ? (n_keys + kGtKeys - 1) / kGtKeys : 0;
-    // Q rows: a warp per row, lanes across the head
-    for (uint32_t r = warp; r < uint32_t(kGtRows); r += kGtThreads / 32) {
-        const uint32_t row = r0 + r, t = row / group, h = g * group + (row - t * group);
-        const bool live = row < rows_all;
-        const float* q = a.qkv + size_t(live ? t : 0) * a.qkv_ld + (live ? h : 0) * a.dim;
-        const float f = live ? gqa_rms_factor(q, a.dim, a.eps) * a.scale * kLog2e : 0.f;
-        for (uint32_t c2 = lane; c2 < p.dim_chunks * 32; c2 += 32) {           // pairs of columns
-            const uint32_t c = 2 * c2;
-            const float lo = live && c < a.dim ? q[c] * f * a.q_norm[c] : 0.f, hi = live && c + 1 < a.dim ? q[c + 1] * f * a.q_norm[c + 1] : 0.f;
-            const uint32_t in = c & 63u, off = (r >> 3) * 1024u + (r & 7u) * 128u + (((in >> 3) ^ (r & 7u)) << 4) + (in & 7u) * 2u;
-            *reinterpret_cast<uint32_t*>(s_q + (c >> 6) * kGtQChunk + off) = gt_pack(lo, hi);
+    // Q rows: a warp takes several rows at a time, lanes across the head (pairs of columns), all loads before the first sum
+    constexpr int kPairs = PAIRS, kBatch = PAIRS <= 2 ? 16 : 8;
+    float qw[2 * kPairs];
+#pragma unroll
+    for (int c2 = 0; c2 < kPairs; ++c2) {
+        const uint32_t c = 2 * (uint32_t(lane) + 32 * c2);
+        qw[2 * c2] = c < a.dim ? a.q_norm[c] : 0.f;
+        qw[2 * c2 + 1] = c + 1 < a.dim ? a.q_norm[c + 1] : 0.f;
+    }
+    for (uint32_t b0 = uint32_t(warp) * kBatch; b0 < uint32_t(kGtRows); b0 += kThreads / 32 * kBatch) {
+        float v[kBatch][2 * kPairs], part[kBatch];
+#pragma unroll
+        for (int i = 0; i < kBatch; ++i) {
+            const uint32_t row = r0 + b0 + i, t = row / group, h = g * group + (row - t * group);
+            const float* q = a.qkv + size_t(t) * a.qkv_ld + h * a.dim;
+#pragma unroll
+            for (int c2 = 0; c2 < kPairs; ++c2) {
+                const uint32_t c = 2 * (uint32_t(lane) + 32 * c2);
+                v[i][2 * c2] = row < rows_all && c < a.dim ? q[c] : 0.f;
+                v[i][2 * c2 + 1] = row < rows_all && c + 1 < a.dim ? q[c + 1] : 0.f;
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < kBatch; ++i) {
+            part[i] = 0.f;
+#pragma unroll
+            for (int c = 0; c < 2 * kPairs; ++c) part[i] = fmaf(v[i][c], v[i][c], part[i]);
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int i = 0; i < kBatch; ++i) part[i] += __shfl_xor_sync(0xffffffffu, part[i], o);
+#pragma unroll
+        for (int i = 0; i < kBatch; ++i) {
+            const float f = a.scale * kLog2e / sqrtf(part[i] / float(a.dim) + a.eps);
+            const uint32_t r = b0 + i;
+#pragma unroll
+            for (int c2 = 0; c2 < kPairs; ++c2) {
+                const uint32_t c = 2 * (uint32_t(lane) + 32 * c2);
+                if (c >= p.dim_chunks * 64) continue;
+                const uint32_t in = c & 63u, off = (r >> 3) * 1024u + (r & 7u) * 128u + (((in >> 3) ^ (r & 7u)) << 4) + (in & 7u) * 2u;
+                *reinterpret_cast<uint32_t*>(s_q + (c >> 6) * kGtQChunk + off) = gt_pack(v[i][2 * c2] * f * qw[2 * c2], v[i][2 * c2 + 1] * f * qw[2 * c2 + 1]);
+            }
         }
     }
     fence_proxy_async();
@@ -125,88 +172,112 @@ __global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p,
             }
         }
     } else if (warp == 1) {
-        if (lane == 0 && n_blocks != 0) {
-            const uint32_t common = (1u << 4) | (1u << 7) | (1u << 10) | (uint32_t(kGtRows >> 4) << 24);
-            const uint32_t idesc_s = common | (uint32_t(kGtKeys >> 3) << 17);
-            const uint32_t idesc_o = common | (1u << 16) | ((p.vdim16 >> 3) << 17);          // B is MN-major
+        if (lane == 0) {
+            constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (uint32_t(kGtRows >> 4) << 24) | (uint32_t(kGtKeys >> 3) << 17);
             const uint64_t q_desc = tc_smem_desc(smem_u32(s_q)), k_desc0 = tc_smem_desc(smem_u32(s_kv));
-            const uint64_t v_desc0 = gt_v_desc(smem_u32(s_kv) + k_bytes, p.v_chunks > 1 ? kGtKChunk : 1024u);
             const uint32_t k_steps = p.dim16 / 16;
-            uint32_t ks = 0, k_phase = 0, vs = 0, v_phase = 0;
-            auto scores = [&](uint32_t b) {
-                if (!mbar_wait(&k_full[ks], k_phase, p.err)) return false;
+            uint32_t ks = 0, k_phase = 0;
+            for (uint32_t b = 0; b < n_blocks && ok; ++b) {
+                // the buffer held P of block b - 2
+                ok = mbar_wait(&k_full[ks], k_phase, p.err) && (b < 2 || mbar_wait(&pv_done[b & 1u], ((b >> 1) - 1u) & 1u, p.err));
+                if (!ok) break;
                 tc_fence_after_sync();
                 const uint64_t kd = k_desc0 + ((ks * stage) >> 4);
                 for (uint32_t k = 0; k < k_steps; ++k) {
                     const uint32_t c = k >> 2, in = (k & 3u) * 2u;
-                    tc_mma_f16(tmem + (b & 1u) * kGtKeys, q_desc + ((c * kGtQChunk) >> 4) + in, kd + ((c * kGtKChunk) >> 4) + in, idesc_s, k != 0 ? 1u : 0u);
+                    tc_mma_f16(tmem + (b & 1u) * kGtKeys, q_desc + ((c * kGtQChunk) >> 4) + in, kd + ((c * kGtKChunk) >> 4) + in, idesc, k != 0 ? 1u : 0u);
                 }
                 tc_commit(&s_full[b & 1u]);
                 if (++ks == p.stages) { ks = 0; k_phase ^= 1u; }
-                return true;
-            };
-            ok = scores(0);
-            if (ok && n_blocks > 1) ok = scores(1);
+            }
+        }
+    } else if (warp == 2) {
+        if (lane == 0) {
+            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((p.vdim16 >> 3) << 17) | (uint32_t(kGtRows >> 4) << 24);      // B is MN-major
+            const uint64_t v_desc0 = gt_v_desc(smem_u32(s_kv) + k_bytes, p.v_chunks > 1 ? kGtKChunk : 1024u);
+            uint32_t vs = 0, v_phase = 0;
             for (uint32_t b = 0; b < n_blocks && ok; ++b) {
                 ok = mbar_wait(&p_full[b & 1u], (b >> 1) & 1u, p.err) && mbar_wait(&v_full[vs], v_phase, p.err);
                 if (!ok) break;
                 tc_fence_after_sync();
                 const uint64_t vd = v_desc0 + ((vs * stage) >> 4);
-                for (uint32_t k = 0; k < kGtKeys / 16; ++k)      // 16 keys: 8 columns of P, two 8-key groups of V
-                    tc_mma_f16_ta(tmem_o, tmem + (b & 1u) * kGtKeys + 8u * k, vd + 128u * k, idesc_o, (b != 0 || k != 0) ? 1u : 0u);
-                tc_commit(&kv_empty[vs]);
-                tc_commit(&pv_done);
+#pragma unroll
+                for (uint32_t k = 0; k < kGtKeys / 16; ++k) {    // 16 keys: 8 columns of P, two 8-key groups of V
+                    const uint32_t half = k / (kHalfKeys / 16), in = k - half * (kHalfKeys / 16);
+                    tc_mma_f16_ta(tmem_o + half * p.vdim16, tmem + (b & 1u) * kGtKeys + half * kHalfKeys + 8u * in, vd + 128u * k, idesc,
+                                  (b != 0 || in != 0) ? 1u : 0u);
+                }
+                tc_commit(&pv_done[b & 1u]);
+                tc_commit(&kv_empty[vs]);                        // (the S product of the block is older: its softmax has been here)
                 if (++vs == p.stages) { vs = 0; v_phase ^= 1u; }
-                if (b + 2 < n_blocks) ok = scores(b + 2);        // in order after the P V product that reads this buffer
             }
         }
     } else {
-        // ---- softmax: one row per thread ----------------------------------------------------------
-        const uint32_t quarter = uint32_t(warp) & 3u, tr = quarter * 32u + uint32_t(lane), st = threadIdx.x - 64u;
+        // ---- softmax: a row (or half of its keys) per thread ---------------------------------------
+        const uint32_t quarter = uint32_t(warp) & 3u, tr = quarter * 32u + uint32_t(lane), st = threadIdx.x - 32u * kGtFirstSoftmax;
+        const uint32_t half = (uint32_t(warp) - kGtFirstSoftmax) >> 2, key0 = half * kHalfKeys;
         const uint32_t row = r0 + tr, t = min(row, rows_all - 1) / group, hl = min(row, rows_all - 1) - t * group;
-        const uint32_t lanes = quarter * 32u << 16;
+        const uint32_t lanes = quarter * 32u << 16, o_half = tmem_o + lanes + half * p.vdim16;
+        // the bias table's entries: 32 of one head per warp and job; the first jobs of a warp keep their constants in registers
+        constexpr int kJobs = 4;
+        const uint32_t tab_jobs = (p.tab_tokens + 31) / 32, all_jobs = group * tab_jobs;
+        float job_r1[kJobs], job_r2[kJobs];
+        uint32_t job_at[kJobs];
+        int job_d[kJobs];
+#pragma unroll
+        for (int k = 0; k < kJobs; ++k) {
+            const uint32_t job = uint32_t(warp) - kGtFirstSoftmax + k * 4 * NH, h = job / tab_jobs, i = (job - h * tab_jobs) * 32 + lane;
+            const bool live = job < all_jobs && i < p.tab_tokens;
+            job_r1[k] = live ? a.r1[g * group + h] : 0.f;
+            job_r2[k] = live ? a.r2[g * group + h] : 0.f;
+            job_at[k] = live ? h * p.tab_stride + i : ~0u;
+            job_d[k] = int(i);
+        }
         float m = a.sink ? 0.f : -INFINITY, l = 0.f;
         uint32_t vs = 0, v_phase = 0;
         // (after a lost wait the warp goes through the remaining blocks without work: the others wait for it at the barrier)
         for (uint32_t b = 0; b < n_blocks; ++b) {
-            const uint32_t k0 = b * kGtKeys;
+            const uint32_t k0 = b * kGtKeys, s_at = tmem + lanes + (b & 1u) * kGtKeys + key0;
             // bias table of this block: entry i of a head is distance (P + t_first) - (k0 + 63) + i
             float* tab = s_tab + (b & 1u) * group * p.tab_stride;
             const int d0 = int(P + t_first) - int(k0 + kGtKeys - 1);
-            for (uint32_t e = st; e < group * p.tab_tokens; e += 128) {
-                const uint32_t h = e / p.tab_tokens, i = e - h * p.tab_tokens;
-                const float d = float(max(d0 + int(i), 0));
-                tab[h * p.tab_stride + i] = kLog2e * a.r1[g * group + h] * log1pf(a.r2[g * group + h] * d);
+#pragma unroll
+            for (int k = 0; k < kJobs; ++k)
+                if (job_at[k] != ~0u) tab[job_at[k]] = job_r1[k] * __log2f(fmaf(job_r2[k], float(max(d0 + job_d[k], 0)), 1.f));
+            for (uint32_t job = uint32_t(warp) - kGtFirstSoftmax + kJobs * 4 * NH; job < all_jobs; job += 4 * NH) {
+                const uint32_t h = job / tab_jobs, i = (job - h * tab_jobs) * 32 + lane;
+                if (i < p.tab_tokens) tab[h * p.tab_stride + i] = a.r1[g * group + h] * __log2f(fmaf(a.r2[g * group + h], float(max(d0 + int(i), 0)), 1.f));
             }
-            asm volatile("bar.sync 1, 128;" ::: "memory");
-            ok = ok && mbar_wait(&s_full[b & 1u], (b >> 1) & 1u, p.err);
+            asm volatile("bar.sync 1, %0;" ::"n"(128 * NH) : "memory");
+            ok = ok && mbar_wait_warp(&s_full[b & 1u], (b >> 1) & 1u, p.err);
             if (!ok) continue;
             tc_fence_after_sync();
-            float s[kGtKeys];
+            float s[kHalfKeys];
+            {
+                uint32_t u[kHalfKeys / 16][16];
 #pragma unroll
-            for (int c = 0; c < kGtKeys; c += 16) {
-                uint32_t u[16];
-                tc_load16(u, tmem + lanes + (b & 1u) * kGtKeys + c);
+                for (int c = 0; c < kHalfKeys / 16; ++c) tc_load16(u[c], s_at + 16 * c);
                 tc_wait_load();
 #pragma unroll
-                for (int i = 0; i < 16; ++i) s[c + i] = __uint_as_float(u[i]);
+                for (int c = 0; c < kHalfKeys; ++c) s[c] = __uint_as_float(u[c / 16][c % 16]);
             }
-            const float* bias = tab + hl * p.tab_stride + (t - t_first) + (kGtKeys - 1);
-            const int last = int(P + t) - int(k0);               // keys 0 .. last of the block are visible
-            float top = -INFINITY;
+            const float* bias = tab + hl * p.tab_stride + (t - t_first) + (kGtKeys - 1) - key0;
+            const int last = int(P + t) - int(k0 + key0);        // keys 0 .. last of this half are visible
+            float tops[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             if (k0 + kGtKeys - 1 <= P + t_first) {
 #pragma unroll
-                for (int j = 0; j < kGtKeys; ++j) {
+                for (int j = 0; j < kHalfKeys; ++j) {
                     s[j] -= bias[-j];
-                    top = fmaxf(top, s[j]);
+                    tops[j & 3] = fmaxf(tops[j & 3], s[j]);
                 }
             } else {
 #pragma unroll
-                for (int j = 0; j < kGtKeys; ++j) {
+                for (int j = 0; j < kHalfKeys; ++j) {
                     s[j] = j <= last ? s[j] - bias[-j] : -INFINITY;
-                    top = fmaxf(top, s[j]);
+                    tops[j & 3] = fmaxf(tops[j & 3], s[j]);
                 }
             }
+            const float top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
             // a new maximum takes effect when it is far above the old one (or there was none)
             const bool grow = top > m + kGtRescaleStep;
             float f = 1.f;
@@ -216,40 +287,42 @@ __global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p,
                 l *= f;
             }
             if (__any_sync(0xffffffffu, grow) && b != 0) {
-                ok = mbar_wait(&pv_done, (b - 1) & 1u, p.err);
+                ok = mbar_wait_warp(&pv_done[(b - 1) & 1u], ((b - 1) >> 1) & 1u, p.err);
                 if (!ok) continue;
                 tc_fence_after_sync();
                 for (uint32_t c = 0; c < p.vdim16; c += 16) {
                     uint32_t u[16];
-                    tc_load16(u, tmem_o + lanes + c);
+                    tc_load16(u, o_half + c);
                     tc_wait_load();
 #pragma unroll
                     for (int i = 0; i < 16; ++i) u[i] = __float_as_uint(__uint_as_float(u[i]) * f);
-                    gt_store16(tmem_o + lanes + c, u);
+                    gt_store16(o_half + c, u);
                 }
                 gt_wait_store();
             }
             const float base = m == -INFINITY ? 0.f : m;
+            float sums[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-            for (int c = 0; c < kGtKeys; c += 32) {
+            for (int c = 0; c < kHalfKeys; c += 32) {
                 uint32_t u[16];
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
-                    const float p0 = exp2f(s[c + 2 * i] - base), p1 = exp2f(s[c + 2 * i + 1] - base);
-                    l += p0;
-                    l += p1;
+                    const float p0 = gt_exp2(s[c + 2 * i] - base), p1 = gt_exp2(s[c + 2 * i + 1] - base);
+                    sums[(2 * i) & 3] += p0;
+                    sums[(2 * i + 1) & 3] += p1;
                     u[i] = gt_pack(p0, p1);
                 }
-                gt_store16(tmem + lanes + (b & 1u) * kGtKeys + c / 2, u);
+                gt_store16(s_at + c / 2, u);
             }
+            l += (sums[0] + sums[1]) + (sums[2] + sums[3]);
             gt_wait_store();
             if (k0 + kGtKeys > P + p.n_tokens) {
                 // rows of V behind the last token hold whatever the cache held: their weights are zero, but zero times NaN is not
-                ok = mbar_wait(&v_full[vs], v_phase, p.err);
+                ok = mbar_wait_warp(&v_full[vs], v_phase, p.err);
                 if (!ok) continue;
                 uint8_t* v = s_kv + vs * stage + k_bytes;
                 const uint32_t first = P + p.n_tokens - k0, n16 = (kGtKeys - first) * 8;
-                for (uint32_t e = st; e < p.v_chunks * n16; e += 128) {
+                for (uint32_t e = st; e < p.v_chunks * n16; e += 128 * NH) {
                     const uint32_t c = e / n16, i = e - c * n16;
                     *reinterpret_cast<uint4*>(v + c * kGtKChunk + first * 128 + i * 16) = make_uint4(0u, 0u, 0u, 0u);
                 }
@@ -260,30 +333,49 @@ __global__ void __launch_bounds__(kGtThreads) gqa_tc_kernel(const GqaTcParams p,
             __syncwarp();
             if (lane == 0) mbar_arrive(&p_full[b & 1u]);
         }
-        if (ok && n_blocks != 0) {
-            ok = mbar_wait(&pv_done, (n_blocks - 1) & 1u, p.err);
+        if (n_blocks != 0) {
+            ok = ok && mbar_wait_warp(&pv_done[(n_blocks - 1) & 1u], ((n_blocks - 1) >> 1) & 1u, p.err);
             tc_fence_after_sync();
-        }
-        if (ok && n_blocks != 0) {
-            const float inv = 1.f / (l + (a.sink ? exp2f(-m) : 0.f));
-            const size_t at = size_t(t) * a.out_ld + (g * group + hl) * a.vdim;
-            for (uint32_t c = 0; c < p.vdim16; c += 16) {
-                uint32_t u[16];
-                tc_load16(u, tmem_o + lanes + c);
-                tc_wait_load();
-                if (row >= rows_all) continue;
-                if (p.out_bf16 && c + 16 <= a.vdim && (at + c) % 8 == 0) {
-                    uint4 w[2];
-                    uint32_t* ww = reinterpret_cast<uint32_t*>(w);
+            float fa = 1.f, fb = 0.f;                            // weights of the two halves' sums
+            if constexpr (NH == 2) {
+                if (half == 1) { s_ml[0][tr] = m; s_ml[1][tr] = l; }
+                asm volatile("bar.sync 1, %0;" ::"n"(128 * NH) : "memory");
+                if (half == 0) {
+                    const float mb = s_ml[0][tr], lb = s_ml[1][tr], M = fmaxf(m, mb);
+                    fa = exp2f(m - M);
+                    fb = exp2f(mb - M);
+                    l = l * fa + lb * fb;
+                    m = M;
+                }
+            }
+            if (ok && half == 0) {
+                const float inv = 1.f / (l + (a.sink ? exp2f(-m) : 0.f));
+                fa *= inv;
+                fb *= inv;
+                const size_t at = size_t(t) * a.out_ld + (g * group + hl) * a.vdim;
+                for (uint32_t c = 0; c < p.vdim16; c += 16) {
+                    uint32_t u[NH][16];
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) ww[i] = gt_pack(__uint_as_float(u[2 * i]) * inv, __uint_as_float(u[2 * i + 1]) * inv);
-                    uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.out) + at + c);
-                    dst[0] = w[0];
-                    dst[1] = w[1];
-                } else {
+                    for (int h = 0; h < NH; ++h) tc_load16(u[h], o_half + h * p.vdim16 + c);
+                    tc_wait_load();
+                    if (row >= rows_all) continue;
+                    float o[16];
 #pragma unroll
                     for (int i = 0; i < 16; ++i)
-                        if (c + i < a.vdim) gqa_store_out(a.out, p.out_bf16, at + c + i, __uint_as_float(u[i]) * inv);
+                        o[i] = NH == 2 ? fmaf(__uint_as_float(u[NH - 1][i]), fb, __uint_as_float(u[0][i]) * fa) : __uint_as_float(u[0][i]) * fa;
+                    if (p.out_bf16 && c + 16 <= a.vdim && (at + c) % 8 == 0) {
+                        uint4 w[2];
+                        uint32_t* ww = reinterpret_cast<uint32_t*>(w);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) ww[i] = gt_pack(o[2 * i], o[2 * i + 1]);
+                        uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.out) + at + c);
+                        dst[0] = w[0];
+                        dst[1] = w[1];
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i)
+                            if (c + i < a.vdim) gqa_store_out(a.out, p.out_bf16, at + c + i, o[i]);
+                    }
                 }
             }
         }
@@ -311,7 +403,8 @@ int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch) {
     p.vdim16 = (vdim_p + 15) / 16 * 16;
     p.out_bf16 = a.out_type == LV_TYPE_BF16;
     p.err = ctx->d_err;
-    p.tmem_cols = 2 * kGtKeys + p.vdim16 <= 256 ? 256 : 512;
+    const bool halves = 2 * kGtKeys + 2 * p.vdim16 <= 512;
+    p.tmem_cols = 2 * kGtKeys + (halves ? 2 : 1) * p.vdim16 <= 256 ? 256 : 512;
     // tokens that a tile of 128 rows can touch, plus the keys of a block; heads 32 / group banks apart
     p.tab_tokens = (kGtRows + group - 1) / group + 1 + kGtKeys;
     const uint32_t want = group < 32 ? 32 / group : 1;
@@ -319,7 +412,8 @@ int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch) {
     while (p.tab_stride % 32 != want % 32) ++p.tab_stride;
     const uint32_t stage = (p.dim_chunks + p.v_chunks) * kGtKChunk, q_bytes = p.dim_chunks * kGtQChunk, tab = 2 * group * p.tab_stride * 4;
     p.stages = 2;
-    while (p.stages < kGtMaxStages && q_bytes + (p.stages + 1) * stage + tab + 1024 <= 110 * 1024) ++p.stages;      // two CTAs per SM where they fit
+    const uint32_t room = (p.tmem_cols == 512 ? 200 : 110) * 1024;       // two CTAs per SM where their tensor memory fits
+    while (p.stages < kGtMaxStages && q_bytes + (p.stages + 1) * stage + tab + 1024 <= room) ++p.stages;
     const size_t smem = 1024 + size_t(q_bytes) + size_t(p.stages) * stage + tab;
     LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "attention: head sizes need too much shared memory");
     GqaTcMaps maps{};
@@ -327,8 +421,9 @@ int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch) {
     LV_REQUIRE(rows <= 0x7fffffffu, "attention: cache too long");
     if (int rc = make_bf16_map(&maps.k, a.k_cache, rows, dim_p, dim_p, kGtKeys)) return rc;
     if (int rc = make_bf16_map(&maps.v, a.v_cache, rows, vdim_p, vdim_p, kGtKeys)) return rc;
-    LV_CUDA(cudaFuncSetAttribute(gqa_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-    LV_CUDA(launch_pdl(ctx, gqa_tc_kernel, dim3((batch * group + kGtRows - 1) / kGtRows, a.kv_heads), dim3(kGtThreads), smem, p, maps));
+    auto* kernel = halves ? (a.dim <= 128 ? gqa_tc_kernel<2, 2> : gqa_tc_kernel<2, 4>) : (a.dim <= 128 ? gqa_tc_kernel<1, 2> : gqa_tc_kernel<1, 4>);
+    LV_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    LV_CUDA(launch_pdl(ctx, kernel, dim3((batch * group + kGtRows - 1) / kGtRows, a.kv_heads), dim3(32 * kGtFirstSoftmax + (halves ? 256 : 128)), smem, p, maps));
     return LV_OK;
 }
 

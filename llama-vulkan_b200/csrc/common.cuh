@@ -93,6 +93,14 @@ __device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, uint32
     return false;
 }
 
+// The same for a whole warp: one lane polls (32 lanes that poll one barrier take turns at it, about half a microsecond for
+// the eight warps of a softmax).
+__device__ __forceinline__ bool mbar_wait_warp(uint64_t* bar, uint32_t parity, uint32_t* err) {
+    uint32_t ok = 1;
+    if ((threadIdx.x & 31u) == 0) ok = mbar_wait(bar, parity, err) ? 1u : 0u;
+    return __shfl_sync(0xffffffffu, ok, 0) != 0;
+}
+
 // 1-D bulk copy global -> shared, completion counted in bytes on `bar`.
 // Both addresses must be 16-byte aligned and `bytes` a multiple of 16.
 __device__ __forceinline__ void bulk_g2s(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {

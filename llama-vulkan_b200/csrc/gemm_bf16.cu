@@ -140,7 +140,7 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const GemmBf16
         // ---- epilogue: warp w reads lanes 32 (w mod 4) .. + 31 of the accumulator --------------------
         const uint32_t quarter = uint32_t(warp) & 3u, tr = quarter * 32u + uint32_t(lane);
         const uint32_t row = row0 + tr, taddr = tmem + (quarter * 32u << 16);
-        ok = mbar_wait(&acc_full, 0, p.err);
+        ok = mbar_wait_warp(&acc_full, 0, p.err);
         tc_fence_after_sync();
         constexpr int kAcc = PAIR ? 2 : 1;
         const uint32_t tile = blockIdx.y * gridDim.x + blockIdx.x;
