@@ -1,6 +1,6 @@
 """Builds the native libraries of this package in-tree with nvcc / g++.
 
-    python llama-vulkan_b200/build.py [--force]
+    python llama-vulkan_b200/build.py [--force] [--locked] [program ...]
 
 Outputs (next to this file): liblv_b200.so (sm_100a kernels + C ABI),
 libllava_host.so (C++ host surface) and the command-line tools vulkan_llama and trace_run.
@@ -69,7 +69,7 @@ def build_kernels(force=False, verbose_ptxas=False):
     return out
 
 
-def build_host(force=False):
+def build_host(force=False, programs=None):
     if not os.path.isdir(HOST):
         return None
     cpp = [f for f in _glob(HOST, (".cpp",)) if os.path.basename(f) not in [p[0] for p in PROGRAMS]] + _glob(os.path.join(HOST, "server"), (".cpp",))
@@ -83,6 +83,8 @@ def build_host(force=False):
         _run([cxx, "-std=c++20", "-O2", "-fPIC", "-shared", "-pthread", "-Wall", "-o", out] + cpp +
              ["-L" + HERE, "-llv_b200", "-Wl,-rpath,$ORIGIN", "-Wl,-Bsymbolic"])
     for source, program in PROGRAMS:
+        if programs is not None and program not in programs:
+            continue
         main = os.path.join(HOST, source)
         exe = os.path.join(HERE, program)
         if force or _newer(exe, [main, out]):
@@ -91,9 +93,10 @@ def build_host(force=False):
     return out
 
 
-def build_all(force=False):
+def build_all(force=False, programs=None):
+    """programs: the command-line tools to link (all of them when None)."""
     k = build_kernels(force)
-    h = build_host(force)
+    h = build_host(force, programs)
     return k, h
 
 
@@ -103,4 +106,5 @@ if __name__ == "__main__":
         os.makedirs(os.path.join(HERE, "build"), exist_ok=True)
         lock = open(os.path.join(HERE, "build", ".lock"), "w")
         fcntl.flock(lock, fcntl.LOCK_EX)
-    build_all(force="--force" in sys.argv)
+    wanted = [p for _, p in PROGRAMS if p in sys.argv[1:]]
+    build_all(force="--force" in sys.argv, programs=wanted or None)

@@ -87,7 +87,7 @@ def test_gemv_bf16_is_exact_in_f32(gpu, rows, cols, batch):
     assert rel(got, want) < 1e-6
 
 
-@pytest.mark.parametrize("rows,cols,batch", [(64, 64, 2), (7, 24, 3), (200, 72, 17), (576, 256, 40), (128, 328, 64), (1000, 520, 300), (300, 40, 129),
+@pytest.mark.parametrize("rows,cols,batch", [(64, 64, 2), (7, 24, 3), (200, 72, 17), (560, 264, 40), (128, 328, 64), (1000, 520, 300), (300, 40, 129),
                                              (96, 4096, 5)])
 @pytest.mark.parametrize("out_bf16", [False, True])
 def test_gemm_bf16(gpu, rows, cols, batch, out_bf16):
@@ -318,7 +318,7 @@ class Attention:
 
 
 @pytest.mark.parametrize("H,G,dim,vdim,cuts", [
-    (4, 1, 64, 64, [1] * 12), (4, 4, 24, 40, [5, 1, 1, 9]), (6, 2, 48, 80, [130, 1, 2, 1, 127, 1]), (8, 1, 96, 32, [300, 1, 1]), (3, 1, 128, 128, [64, 65, 1]),
+    (4, 1, 72, 64, [1] * 12), (4, 4, 24, 40, [5, 1, 1, 9]), (6, 2, 48, 80, [130, 1, 2, 1, 127, 1]), (8, 1, 96, 32, [300, 1, 1]), (3, 1, 128, 128, [64, 65, 1]),
     (10, 1, 32, 16, [2, 2, 129, 1, 1, 1]), (16, 2, 20, 36, [40, 1, 30]), (2, 1, 256, 256, [20, 1, 3]), (4, 2, 160, 96, [40, 1, 90]), (66, 1, 16, 16, [5, 1, 70])])
 @pytest.mark.parametrize("f32", [True, False])
 def test_attention_in_portions(gpu, H, G, dim, vdim, cuts, f32):
