@@ -162,8 +162,8 @@ def kernel_times(pkg, torch, z, peaks):
         out = gpu.zeros(max(STEP * top * max(W, raw_n, 3 * gru, ff), STEP * VOCAB // 8) * 4)
         for name, r, k in (("input projections (attention)", raw_n, W), ("output projection (attention)", W, H * DIM), ("output projection (recurrent)", W, gru)):
             w, d = ring(r * k * 2)
-            add("sonuzen", "decode", name, t(lambda i: pkg.check(lib.lv_gemv_bf16(h, out, r, w(i), r, k, k, x1, k, 1, 1.0))), r * k * 2)
-            add("sonuzen", f"prompt of {STEP}", name, t(lambda i: pkg.check(lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, r, w(i), r, k, k, xT, k, STEP, 1.0))),
+            add("sonuzen", "decode", name, t(lambda i: pkg.check(lib.lv_gemv_bf16(h, out, r, w(i), r, k, k, x1, k, 1, 1.0, 0))), r * k * 2)
+            add("sonuzen", f"prompt of {STEP}", name, t(lambda i: pkg.check(lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, r, w(i), r, k, k, xT, k, STEP, 1.0, 0))),
                 r * k * 2 + STEP * (k * 2 + r * 4), 2.0 * r * k * STEP)
             gpu.free(d)
         w, d = ring(3 * gru * W * 2)
@@ -171,11 +171,11 @@ def kernel_times(pkg, torch, z, peaks):
         each = gru * W * 2
         add("sonuzen", "decode", "input projections + recurrence", t(lambda i: pkg.check(lib.lv_gemv_bf16_mingru(
             h, out, w(i), pkg.offset(w(i), each), pkg.offset(w(i), 2 * each), W, gru, W, bias, bias, x1, state, pos))), 3 * each)
-        add("sonuzen", f"prompt of {STEP}", "input projections (recurrent)", t(lambda i: pkg.check(lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, 3 * gru, w(i), 3 * gru, W, W, xT, W, STEP, 1.0))),
+        add("sonuzen", f"prompt of {STEP}", "input projections (recurrent)", t(lambda i: pkg.check(lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, 3 * gru, w(i), 3 * gru, W, W, xT, W, STEP, 1.0, 0))),
             3 * each + STEP * (W * 2 + 3 * gru * 4), 6.0 * gru * W * STEP)
         gpu.free(d)
         w, d = ring(VOCAB * W * 2)
-        add("sonuzen", "decode", "output head", t(lambda i: pkg.check(lib.lv_gemv_bf16(h, out, VOCAB, w(i), VOCAB, W, W, x1, W, 1, 1.0))), VOCAB * W * 2)
+        add("sonuzen", "decode", "output head", t(lambda i: pkg.check(lib.lv_gemv_bf16(h, out, VOCAB, w(i), VOCAB, W, W, x1, W, 1, 1.0, 0))), VOCAB * W * 2)
         gpu.free(d)
         # -- experts -------------------------------------------------------------------------
         w, d = ring(E * ff * W * 2 * 3)

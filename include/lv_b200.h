@@ -406,7 +406,9 @@ int lv_decode_step(lv_ctx* ctx, const lv_step_plan* plan, uint32_t* config, uint
  *   out  = h_t + sum_{j < taps} conv_w[j] * h_{t - taps + 1 + j}   (taps 0: out = h_t)
  * for the tokens first .. batch - 1.  history f32 [taps - 1][width] holds h of the last taps - 1 positions, oldest first,
  * and is updated (entries of positions before 0 are never read).  With out_index, out row out_index[t * out_copies + s]
- * is written for every s < out_copies, else row t - first.  x null: rows of the bfloat16 embedding table. */
+ * is written for every s < out_copies, else row t - first.  pre_w null (without a convolution): no norm, h_t = x_t.
+ * x null: embed_scale times the rows of the bfloat16 embedding table, plus -- with pair_embed -- the row
+ * (id_(t-1) * pair_mul_prev + id_t * pair_mul_cur) mod pair_buckets of a table of pairs of ids, row pair_buckets at position 0. */
 typedef struct lv_norm_conv_args {
     const float* x;
     const void* embed;
@@ -432,13 +434,20 @@ typedef struct lv_norm_conv_args {
     const uint32_t* out_index;
     uint32_t out_copies;
     uint32_t width, first, batch;
+    int plain_w;                    /* norms multiply by w instead of 1 + w */
+    float embed_scale;              /* factor of the embedding rows; 0: 1 */
+    const void* pair_embed;         /* null, or a bfloat16 table [pair_buckets + 1][pair_ld] */
+    uint32_t pair_ld, pair_buckets, pair_mul_prev, pair_mul_cur;
 } lv_norm_conv_args;
 int lv_norm_conv(lv_ctx* ctx, const lv_norm_conv_args* args);
 
-/* out[t][r] = factor * sum_k W[r][k] x[t][k] in f32 arithmetic (weights are exact in f32).  One pass over the weights per
+/* What the products below do with a finished sum (times `factor`) before it is stored. */
+enum { LV_ACT_NONE = 0, LV_ACT_RELU2 = 1 /* max(v, 0)^2 */ };
+
+/* out[t][r] = act(factor * sum_k W[r][k] x[t][k]) in f32 arithmetic (weights are exact in f32).  One pass over the weights per
  * token. */
 int lv_gemv_bf16(lv_ctx* ctx, float* out, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols, const float* x,
-                 uint32_t x_ld, uint32_t batch, float factor);
+                 uint32_t x_ld, uint32_t batch, float factor, int act);
 
 /* minGRU for one token: z = sigmoid(Wz x + bz), u = Wx x + bx, c = u + 1/2 (u >= 0) or sigmoid(u),
  * state = (1 - z) state + z c (0 at position 0), out = state * silu(Wg x). */
@@ -466,7 +475,12 @@ int lv_gemv_bf16_expert_down(lv_ctx* ctx, float* out, uint32_t out_ld, const lv_
 /* Products of a batch on the tensor cores: x and W bfloat16, f32 sums, one pass over the weights for up to 128 tokens.
  * x [batch][x_ld] with x_ld a multiple of 8; out f32 or bfloat16 [batch][out_ld]. */
 int lv_gemm_bf16(lv_ctx* ctx, void* out, int out_type, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols,
-                 const void* x, uint32_t x_ld, uint32_t batch, float factor);
+                 const void* x, uint32_t x_ld, uint32_t batch, float factor, int act);
+/* The same for the rows of a cache [x_rows][x_ld] that `batch` tokens at *pos see through a window of `window` positions (0: all):
+ * out row i = W times cache row first + i, first = max(0, *pos + 1 - window), for all rows below *pos + batch.  max_rows: upper
+ * bound of the number of rows, sizes the grid. */
+int lv_gemm_bf16_window(lv_ctx* ctx, void* out, int out_type, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols,
+                        const void* x, uint32_t x_ld, uint32_t x_rows, const uint32_t* pos, uint32_t batch, uint32_t window, uint32_t max_rows);
 /* The experts of a batch.  lv_expert_route sorts the (token, choice) pairs of each job's layer by expert: index[t * top + s] =
  * row of choice s of token t, and lists tiles of up to tile_rows = lv_expert_tile_rows(batch, top, experts) rows of one expert
  * (max_tiles = lv_expert_max_tiles entries, unused ones with rows 0).  The products below read and write rows in that order.
@@ -518,6 +532,79 @@ int lv_qk_norm_append(lv_ctx* ctx, const lv_gqa_args* a, uint32_t batch);
  * batch and capacity used, zero-filled once. */
 size_t lv_gqa_scratch_bytes(lv_ctx* ctx, const lv_gqa_args* a, uint32_t batch, uint32_t capacity);
 int lv_attention_gqa(lv_ctx* ctx, const lv_gqa_args* a, void* scratch, size_t scratch_bytes, uint32_t batch, uint32_t capacity, int append);
+
+/* {cos, sin} of (*pos + t) * freqs[k], times mults[k], for the `pairs` frequencies of a model: out f32 [batch][pairs][2].  The
+ * angle is formed in f64; freqs f64, mults f32. */
+int lv_rotary_table(lv_ctx* ctx, float* out, const double* freqs, const float* mults, uint32_t pairs, const uint32_t* pos, uint32_t batch);
+
+/* Attention over a latent cache: a position keeps one vector c (kv_rank values, RMS-normed) and one rotated key part (rot
+ * values) for all heads; per head the key is [W_uk c | rotated part] and the value W_uv c.
+ *   s_ij = scale * (q_i . W_uk c_j + q'_i . k'_j),  0 <= i - j < window;   p_ij = exp(s_ij) / (exp(sink_h) + sum_j exp(s_ij))
+ *   out_i = sum_j p_ij W_uv c_j
+ * q f32 [batch][q_ld]: per head dim values and rot values (not yet rotated), as projected.  dkv f32 [batch][dkv_ld]: kv_rank + rot
+ * values as projected, normed (weights kv_norm), rotated and appended to the cache before the attention; null when the cache
+ * rows of these tokens are there already (a layer that reads another layer's cache).  Rotation: pair (2 i, 2 i + 1) of the rot
+ * values turns by angles[t * angle_ld + 2 i] = {cos, sin} for i < angle_pairs.  w bfloat16 [heads * dim + heads * vdim][w_ld]: W_uk,
+ * then W_uv.  cache [ctx_rows][kv_rank rounded up to 8 + rot rounded up to 8], bfloat16 or f32.
+ * Two forms.  Absorbed: W_uk^T q is scored against c itself and W_uv is applied to the weighted sum of c (f32 arithmetic on CUDA
+ * cores, any size).  Expanded: keys and values of the visible rows are formed on the tensor cores, then attended to there
+ * (bfloat16 caches, several tokens, dim and vdim multiples of 8, at most 256 values per key and value). */
+enum { LV_LATENT_AUTO = 0, LV_LATENT_ABSORBED = 1, LV_LATENT_EXPANDED = 2 };
+typedef struct lv_latent_args {
+    const float* q;
+    uint32_t q_ld;
+    const float* dkv;
+    uint32_t dkv_ld;
+    uint32_t heads, dim, rot, vdim, kv_rank;
+    float scale, eps;
+    const float* kv_norm;           /* [kv_rank] */
+    const float* angles;
+    uint32_t angle_ld, angle_pairs;
+    const void* w;
+    uint32_t w_ld;
+    const float* sink;              /* [heads]; null: none */
+    uint32_t window;                /* 0: no window */
+    void* cache;
+    int cache_type;
+    uint32_t ctx_rows;
+    const uint32_t* pos;
+    void* out;
+    int out_type;
+    uint32_t out_ld;
+    int form;
+} lv_latent_args;
+/* scratch for the given batch; capacity: upper bound of *pos + batch */
+size_t lv_latent_scratch_bytes(lv_ctx* ctx, const lv_latent_args* a, uint32_t batch, uint32_t capacity);
+int lv_latent_attention(lv_ctx* ctx, const lv_latent_args* a, void* scratch, size_t scratch_bytes, uint32_t batch, uint32_t capacity);
+
+/* A selective state space (Mamba-2) over `batch` tokens, from the input projection to the normed, gated output.
+ * raw f32 [batch][raw_ld] = [z: inner | x: inner | B: groups * state | C: groups * state | dt: heads], inner = heads * vdim.
+ *   x, B, C    pass a causal convolution per channel (conv_w [taps][channels], last row the current token; conv_b) and silu
+ *   dt         softplus(dt + dt_bias)
+ *   S_t        = exp(-exp(A_log_h) dt) S_(t-1) + dt B_t x_t^T,  y_t = C_t S_t + D_h x_t   (head h: group h / (heads / groups))
+ *   out        RMS norm of y * silu(z) in norm_groups equal parts, times norm_w
+ * history f32 [taps][channels]: the convolution's input of position p in row p mod taps.  S f32 [heads][vdim][state rounded up to 16].
+ * Both count as zero before position 0 and need no clearing.  scratch: lv_ssm_scratch_bytes. */
+typedef struct lv_ssm_args {
+    const float* raw;
+    uint32_t raw_ld, heads, vdim, state, groups, taps;
+    const float* conv_w;
+    const float* conv_b;
+    const float* dt_bias;
+    const float* A_log;
+    const float* D;
+    const float* norm_w;            /* [inner] */
+    uint32_t norm_groups;
+    float eps;
+    float* history;
+    float* S;
+    const uint32_t* pos;
+    void* out;
+    int out_type;
+    uint32_t out_ld;
+} lv_ssm_args;
+size_t lv_ssm_scratch_bytes(const lv_ssm_args* a, uint32_t batch);
+int lv_ssm(lv_ctx* ctx, const lv_ssm_args* a, void* scratch, size_t scratch_bytes, uint32_t batch);
 
 /* ---- multi-GPU: one process per GPU, one communicator per context.  The
  *      reference is single-device (llava_context.cpp:264-279 takes one queue of

@@ -39,7 +39,8 @@ class NormConvArgs(C.Structure):
     _fields_ = [("x", _p), ("embed", _p), ("embed_ld", _u32), ("vocab", _u32), ("token_log", _p), ("pos", _p), ("y", _p), ("y_index", _p),
                 ("y_rows", _u32), ("mult", _f32), ("eps", _f32), ("post_w", _p), ("step", _p), ("trace", _p), ("x_out", _p), ("row_factor", _p), ("pre_w", _p),
                 ("conv_w", _p), ("history", _p), ("taps", _u32), ("out", _p), ("out_type", _int), ("out_ld", _u32), ("out_index", _p),
-                ("out_copies", _u32), ("width", _u32), ("first", _u32), ("batch", _u32)]
+                ("out_copies", _u32), ("width", _u32), ("first", _u32), ("batch", _u32), ("plain_w", _int), ("embed_scale", _f32), ("pair_embed", _p),
+                ("pair_ld", _u32), ("pair_buckets", _u32), ("pair_mul_prev", _u32), ("pair_mul_cur", _u32)]
 
 
 class ExpertArgs(C.Structure):
@@ -53,6 +54,22 @@ class GqaArgs(C.Structure):
     _fields_ = [("qkv", _p), ("qkv_ld", _u32), ("heads", _u32), ("kv_heads", _u32), ("dim", _u32), ("vdim", _u32), ("scale", _f32), ("eps", _f32),
                 ("q_norm", _p), ("k_norm", _p), ("r1", _p), ("r2", _p), ("sink", _int), ("k_cache", _p), ("v_cache", _p), ("cache_type", _int),
                 ("ctx_rows", _u32), ("pos", _p), ("out", _p), ("out_type", _int), ("out_ld", _u32)]
+
+
+class LatentArgs(C.Structure):
+    """lv_latent_args"""
+    _fields_ = [("q", _p), ("q_ld", _u32), ("dkv", _p), ("dkv_ld", _u32), ("heads", _u32), ("dim", _u32), ("rot", _u32), ("vdim", _u32), ("kv_rank", _u32),
+                ("scale", _f32), ("eps", _f32), ("kv_norm", _p), ("angles", _p), ("angle_ld", _u32), ("angle_pairs", _u32), ("w", _p), ("w_ld", _u32), ("sink", _p),
+                ("window", _u32), ("cache", _p), ("cache_type", _int), ("ctx_rows", _u32), ("pos", _p), ("out", _p), ("out_type", _int), ("out_ld", _u32),
+                ("form", _int)]
+
+
+class SsmArgs(C.Structure):
+    """lv_ssm_args"""
+    _fields_ = [("raw", _p), ("raw_ld", _u32), ("heads", _u32), ("vdim", _u32), ("state", _u32), ("groups", _u32), ("taps", _u32), ("conv_w", _p), ("conv_b", _p),
+                ("dt_bias", _p), ("A_log", _p), ("D", _p), ("norm_w", _p), ("norm_groups", _u32), ("eps", _f32), ("history", _p), ("S", _p), ("pos", _p), ("out", _p),
+                ("out_type", _int), ("out_ld", _u32)]
+
 
 # name -> (restype, argtypes); mirrors include/lv_b200.h
 KERNEL_API = {
@@ -130,12 +147,13 @@ KERNEL_API = {
     "lv_step_plan_read_trace": (_int, [_p, _p, _sz, _p, _p, _p]),
     "lv_decode_step": (_int, [_p, _p, _p, _p, _u32, _p, _p, _p, _int]),
     "lv_norm_conv": (_int, [_p, C.POINTER(NormConvArgs)]),
-    "lv_gemv_bf16": (_int, [_p, _p, _u32, _p, _u32, _u32, _u32, _p, _u32, _u32, _f32]),
+    "lv_gemv_bf16": (_int, [_p, _p, _u32, _p, _u32, _u32, _u32, _p, _u32, _u32, _f32, _int]),
     "lv_gemv_bf16_mingru": (_int, [_p, _p, _p, _p, _p, _u32, _u32, _u32, _p, _p, _p, _p, _p]),
     "lv_mingru_scan": (_int, [_p, _p, _int, _u32, _p, _u32, _u32, _p, _p, _p, _p, _u32]),
     "lv_gemv_bf16_expert_gate_up": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _u32, _u32]),
     "lv_gemv_bf16_expert_down": (_int, [_p, _p, _u32, C.POINTER(ExpertArgs), _p, _u32, _u32]),
-    "lv_gemm_bf16": (_int, [_p, _p, _int, _u32, _p, _u32, _u32, _u32, _p, _u32, _u32, _f32]),
+    "lv_gemm_bf16": (_int, [_p, _p, _int, _u32, _p, _u32, _u32, _u32, _p, _u32, _u32, _f32, _int]),
+    "lv_gemm_bf16_window": (_int, [_p, _p, _int, _u32, _p, _u32, _u32, _u32, _p, _u32, _u32, _p, _u32, _u32, _u32]),
     "lv_expert_tile_rows": (_u32, [_u32, _u32, _u32]),
     "lv_expert_max_tiles": (_u32, [_u32, _u32, _u32]),
     "lv_expert_route": (_int, [_p, _p, _u32, _u32, _p, _p, _u32, _u32]),
@@ -144,6 +162,11 @@ KERNEL_API = {
     "lv_qk_norm_append": (_int, [_p, C.POINTER(GqaArgs), _u32]),
     "lv_gqa_scratch_bytes": (_sz, [_p, C.POINTER(GqaArgs), _u32, _u32]),
     "lv_attention_gqa": (_int, [_p, C.POINTER(GqaArgs), _p, _sz, _u32, _u32, _int]),
+    "lv_rotary_table": (_int, [_p, _p, _p, _p, _u32, _p, _u32]),
+    "lv_latent_scratch_bytes": (_sz, [_p, C.POINTER(LatentArgs), _u32, _u32]),
+    "lv_latent_attention": (_int, [_p, C.POINTER(LatentArgs), _p, _sz, _u32, _u32]),
+    "lv_ssm_scratch_bytes": (_sz, [C.POINTER(SsmArgs), _u32]),
+    "lv_ssm": (_int, [_p, C.POINTER(SsmArgs), _p, _sz, _u32]),
 }
 
 _kernels = None

@@ -1,4 +1,4 @@
-// Pieces shared by the attention kernels with query/key norm.
+// Pieces shared by the attention kernels with bfloat16 or f32 caches.
 #pragma once
 
 #include <cuda_bf16.h>
@@ -11,6 +11,10 @@ namespace lv {
 // attention_gqa_tc.cu: the form for several tokens and bfloat16 caches
 bool gqa_tc_supported(const lv_gqa_args& a, uint32_t batch);
 int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch);
+// The same for a latent cache: kv holds keys [heads][dim] and, from column v_at on, values [heads][vdim] of the `rows` positions that
+// the step sees, expanded for the heads h0 .. h0 + n - 1, bfloat16 with ld elements per position
+bool latent_tc_supported(const lv_latent_args& a);
+int latent_tc_launch(lv_ctx* ctx, const lv_latent_args& a, uint32_t batch, const void* kv, uint32_t ld, uint32_t v_at, uint32_t rows, uint32_t h0, uint32_t n);
 
 // 1 / rms of one head's vector, computed by a warp (every lane gets it)
 __device__ __forceinline__ float gqa_rms_factor(const float* v, uint32_t dim, float eps) {

@@ -1,4 +1,5 @@
-// The attention of attention_gqa.cu for the tokens of a prompt, on the tcgen05 tensor cores (bfloat16 caches).
+// The attention of attention_gqa.cu and attention_latent.cu for the tokens of a prompt, on the tcgen05 tensor cores (bfloat16
+// caches).
 //
 // A CTA takes 128 query rows of one key/value head -- row r is query head r mod group of token r / group, so that grouped
 // heads share the keys -- and walks the keys in blocks of 64:
@@ -15,6 +16,11 @@
 // table per head: distances within a block and a tile differ by less than (tokens + 64), so the logarithm is evaluated
 // once per (head, distance) instead of once per score.  O stays in tensor memory; it is rescaled only when a row's maximum has grown
 // by more than 2^8, which with a sink (maximum >= 0 from the start) is rare.  Everything except the operands is f32.
+//
+// Latent caches (LATENT): every head has keys and values of its own, expanded from the cache before the launch; a key is the head's
+// part from there and the rotated part from the cache itself, side by side in shared memory.  The query is rotated instead of
+// normalised, there is no distance bias, a row sees a window of positions (a tile begins at the first row's window), and the
+// sink is a logit per head that the running maximum starts from.
 //
 // Every wait is bounded (common.cuh); a lost wait sets the error word, the CTA drains and frees its tensor memory.
 #include <cuda.h>
@@ -42,11 +48,16 @@ struct GqaTcParams {
     lv_gqa_args a;
     uint32_t n_tokens, dim_chunks, dim16, v_chunks, vdim16, stages, tmem_cols, tab_stride, tab_tokens;
     uint32_t out_bf16;
+    // LATENT (heads == kv_heads: the heads of this launch)
+    uint32_t own_chunks, own_steps, steps;       // chunks of the head's own key part; MMA steps of it and of the whole key
+    uint32_t rot, angle_ld, angle_pairs, window, v_at;
+    const float* angles;
+    const float* sinks;
     uint32_t* err;
 };
 
 struct GqaTcMaps {
-    CUtensorMap k, v;
+    CUtensorMap k, v, rot;
 };
 
 // V: rows are keys (the K of the MMA), 64 columns per 128-byte row; 8-key groups 1024 bytes apart, 64-column blocks kGtKChunk apart
@@ -74,8 +85,8 @@ __device__ __forceinline__ float gt_exp2(float x) {
     return y;
 }
 
-// NH: halves a row is split into; PAIRS: 64 PAIRS >= head size
-template <int NH, int PAIRS>
+// NH: halves a row is split into; PAIRS: 64 PAIRS >= head size (chunks of a key for LATENT)
+template <int NH, int PAIRS, bool LATENT>
 __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel(const GqaTcParams p, const __grid_constant__ GqaTcMaps maps) {
     pdl_launch_dependents();
     extern __shared__ uint8_t smem_raw[];
@@ -103,25 +114,49 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
     pdl_wait();
     const uint32_t P = *a.pos;
     const bool inside = P + p.n_tokens <= a.ctx_rows;            // (lv_qk_norm_append reports positions beyond the cache)
-    const uint32_t n_keys = P + t_last + 1, n_blocks = inside ? (n_keys + kGtKeys - 1) / kGtKeys : 0;
+    // first key of the tile, and of the launch
+    const uint32_t tile_first = LATENT && p.window != 0 && P + t_first + 1 > p.window ? P + t_first + 1 - p.window : 0;
+    const uint32_t step_first = LATENT && p.window != 0 && P + 1 > p.window ? P + 1 - p.window : 0;
+    const uint32_t n_keys = P + t_last + 1 - tile_first, n_blocks = inside ? (n_keys + kGtKeys - 1) / kGtKeys : 0;
     // Q rows: a warp takes several rows at a time, lanes across the head (pairs of columns), all loads before the first sum
     constexpr int kPairs = PAIRS, kBatch = PAIRS <= 2 ? 16 : 8;
     float qw[2 * kPairs];
 #pragma unroll
     for (int c2 = 0; c2 < kPairs; ++c2) {
         const uint32_t c = 2 * (uint32_t(lane) + 32 * c2);
-        qw[2 * c2] = c < a.dim ? a.q_norm[c] : 0.f;
-        qw[2 * c2 + 1] = c + 1 < a.dim ? a.q_norm[c + 1] : 0.f;
+        qw[2 * c2] = LATENT ? 1.f : c < a.dim ? a.q_norm[c] : 0.f;
+        qw[2 * c2 + 1] = LATENT ? 1.f : c + 1 < a.dim ? a.q_norm[c + 1] : 0.f;
     }
+    const uint32_t rot_at = LATENT ? p.own_chunks * 64u : 0;     // column of the rotated part
     for (uint32_t b0 = uint32_t(warp) * kBatch; b0 < uint32_t(kGtRows); b0 += kThreads / 32 * kBatch) {
         float v[kBatch][2 * kPairs], part[kBatch];
 #pragma unroll
         for (int i = 0; i < kBatch; ++i) {
             const uint32_t row = r0 + b0 + i, t = row / group, h = g * group + (row - t * group);
-            const float* q = a.qkv + size_t(t) * a.qkv_ld + h * a.dim;
+            const float* q = a.qkv + size_t(t) * a.qkv_ld + h * (LATENT ? a.dim + p.rot : a.dim);
 #pragma unroll
             for (int c2 = 0; c2 < kPairs; ++c2) {
                 const uint32_t c = 2 * (uint32_t(lane) + 32 * c2);
+                if constexpr (LATENT) {
+                    float lo = 0.f, hi = 0.f;
+                    if (row < rows_all && c < rot_at) {
+                        if (c < a.dim) lo = q[c];
+                        if (c + 1 < a.dim) hi = q[c + 1];
+                    } else if (row < rows_all && c - rot_at < p.rot) {
+                        const uint32_t r = c - rot_at;
+                        lo = q[a.dim + r];
+                        hi = r + 1 < p.rot ? q[a.dim + r + 1] : 0.f;
+                        if (r < 2 * p.angle_pairs) {
+                            const float2 cs = *reinterpret_cast<const float2*>(p.angles + size_t(t) * p.angle_ld + r);
+                            const float u = lo;
+                            lo = u * cs.x - hi * cs.y;
+                            hi = hi * cs.x + u * cs.y;
+                        }
+                    }
+                    v[i][2 * c2] = lo;
+                    v[i][2 * c2 + 1] = hi;
+                    continue;
+                }
                 v[i][2 * c2] = row < rows_all && c < a.dim ? q[c] : 0.f;
                 v[i][2 * c2 + 1] = row < rows_all && c + 1 < a.dim ? q[c + 1] : 0.f;
             }
@@ -138,7 +173,7 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
             for (int i = 0; i < kBatch; ++i) part[i] += __shfl_xor_sync(0xffffffffu, part[i], o);
 #pragma unroll
         for (int i = 0; i < kBatch; ++i) {
-            const float f = a.scale * kLog2e / sqrtf(part[i] / float(a.dim) + a.eps);
+            const float f = LATENT ? a.scale * kLog2e : a.scale * kLog2e / sqrtf(part[i] / float(a.dim) + a.eps);
             const uint32_t r = b0 + i;
 #pragma unroll
             for (int c2 = 0; c2 < kPairs; ++c2) {
@@ -162,12 +197,19 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
             uint32_t s = 0, phase = 1;                           // the first pass over the ring finds it empty
             for (uint32_t b = 0; b < n_blocks; ++b) {
                 if (b >= p.stages && !mbar_wait(&kv_empty[s], phase, p.err)) break;
-                const int y = int(g * a.ctx_rows + b * kGtKeys);
+                const int y = LATENT ? int(tile_first - step_first + b * kGtKeys) : int(g * a.ctx_rows + b * kGtKeys);
                 uint8_t* dst = s_kv + s * stage;
                 mbar_expect_tx(&k_full[s], k_bytes);
-                for (uint32_t c = 0; c < p.dim_chunks; ++c) tma_load_2d_plain(dst + c * kGtKChunk, &maps.k, int(c * 64), y, &k_full[s]);
+                if constexpr (LATENT) {
+                    for (uint32_t c = 0; c < p.own_chunks; ++c) tma_load_2d_plain(dst + c * kGtKChunk, &maps.k, int(g * a.dim + c * 64), y, &k_full[s]);
+                    for (uint32_t c = p.own_chunks; c < p.dim_chunks; ++c)
+                        tma_load_2d_plain(dst + c * kGtKChunk, &maps.rot, int((c - p.own_chunks) * 64), int(tile_first + b * kGtKeys), &k_full[s]);
+                } else {
+                    for (uint32_t c = 0; c < p.dim_chunks; ++c) tma_load_2d_plain(dst + c * kGtKChunk, &maps.k, int(c * 64), y, &k_full[s]);
+                }
+                const int vx = LATENT ? int(p.v_at + g * a.vdim) : 0;
                 mbar_expect_tx(&v_full[s], v_bytes);
-                for (uint32_t c = 0; c < p.v_chunks; ++c) tma_load_2d_plain(dst + k_bytes + c * kGtKChunk, &maps.v, int(c * 64), y, &v_full[s]);
+                for (uint32_t c = 0; c < p.v_chunks; ++c) tma_load_2d_plain(dst + k_bytes + c * kGtKChunk, &maps.v, vx + int(c * 64), y, &v_full[s]);
                 if (++s == p.stages) { s = 0; phase ^= 1u; }
             }
         }
@@ -175,7 +217,7 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
         if (lane == 0) {
             constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (uint32_t(kGtRows >> 4) << 24) | (uint32_t(kGtKeys >> 3) << 17);
             const uint64_t q_desc = tc_smem_desc(smem_u32(s_q)), k_desc0 = tc_smem_desc(smem_u32(s_kv));
-            const uint32_t k_steps = p.dim16 / 16;
+            const uint32_t k_steps = LATENT ? p.steps : p.dim16 / 16;
             uint32_t ks = 0, k_phase = 0;
             for (uint32_t b = 0; b < n_blocks && ok; ++b) {
                 // the buffer held P of block b - 2
@@ -184,7 +226,7 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
                 tc_fence_after_sync();
                 const uint64_t kd = k_desc0 + ((ks * stage) >> 4);
                 for (uint32_t k = 0; k < k_steps; ++k) {
-                    const uint32_t c = k >> 2, in = (k & 3u) * 2u;
+                    const uint32_t at = LATENT && k >= p.own_steps ? p.own_chunks * 4 + k - p.own_steps : k, c = at >> 2, in = (at & 3u) * 2u;
                     tc_mma_f16(tmem + (b & 1u) * kGtKeys, q_desc + ((c * kGtQChunk) >> 4) + in, kd + ((c * kGtKChunk) >> 4) + in, idesc, k != 0 ? 1u : 0u);
                 }
                 tc_commit(&s_full[b & 1u]);
@@ -225,7 +267,7 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
         uint32_t job_at[kJobs];
         int job_d[kJobs];
 #pragma unroll
-        for (int k = 0; k < kJobs; ++k) {
+        for (int k = 0; k < (LATENT ? 0 : kJobs); ++k) {
             const uint32_t job = uint32_t(warp) - kGtFirstSoftmax + k * 4 * NH, h = job / tab_jobs, i = (job - h * tab_jobs) * 32 + lane;
             const bool live = job < all_jobs && i < p.tab_tokens;
             job_r1[k] = live ? a.r1[g * group + h] : 0.f;
@@ -233,22 +275,25 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
             job_at[k] = live ? h * p.tab_stride + i : ~0u;
             job_d[k] = int(i);
         }
-        float m = a.sink ? 0.f : -INFINITY, l = 0.f;
+        const float sink = LATENT ? (p.sinks ? p.sinks[g] * kLog2e : -INFINITY) : a.sink ? 0.f : -INFINITY;      // log2 of the sink's share
+        float m = sink, l = 0.f;
         uint32_t vs = 0, v_phase = 0;
         // (after a lost wait the warp goes through the remaining blocks without work: the others wait for it at the barrier)
         for (uint32_t b = 0; b < n_blocks; ++b) {
-            const uint32_t k0 = b * kGtKeys, s_at = tmem + lanes + (b & 1u) * kGtKeys + key0;
-            // bias table of this block: entry i of a head is distance (P + t_first) - (k0 + 63) + i
-            float* tab = s_tab + (b & 1u) * group * p.tab_stride;
-            const int d0 = int(P + t_first) - int(k0 + kGtKeys - 1);
+            const uint32_t k0 = tile_first + b * kGtKeys, s_at = tmem + lanes + (b & 1u) * kGtKeys + key0;
+            [[maybe_unused]] float* tab = s_tab + (b & 1u) * group * p.tab_stride;
+            if constexpr (!LATENT) {
+                // bias table of this block: entry i of a head is distance (P + t_first) - (k0 + 63) + i
+                const int d0 = int(P + t_first) - int(k0 + kGtKeys - 1);
 #pragma unroll
-            for (int k = 0; k < kJobs; ++k)
-                if (job_at[k] != ~0u) tab[job_at[k]] = job_r1[k] * __log2f(fmaf(job_r2[k], float(max(d0 + job_d[k], 0)), 1.f));
-            for (uint32_t job = uint32_t(warp) - kGtFirstSoftmax + kJobs * 4 * NH; job < all_jobs; job += 4 * NH) {
-                const uint32_t h = job / tab_jobs, i = (job - h * tab_jobs) * 32 + lane;
-                if (i < p.tab_tokens) tab[h * p.tab_stride + i] = a.r1[g * group + h] * __log2f(fmaf(a.r2[g * group + h], float(max(d0 + int(i), 0)), 1.f));
+                for (int k = 0; k < kJobs; ++k)
+                    if (job_at[k] != ~0u) tab[job_at[k]] = job_r1[k] * __log2f(fmaf(job_r2[k], float(max(d0 + job_d[k], 0)), 1.f));
+                for (uint32_t job = uint32_t(warp) - kGtFirstSoftmax + kJobs * 4 * NH; job < all_jobs; job += 4 * NH) {
+                    const uint32_t h = job / tab_jobs, i = (job - h * tab_jobs) * 32 + lane;
+                    if (i < p.tab_tokens) tab[h * p.tab_stride + i] = a.r1[g * group + h] * __log2f(fmaf(a.r2[g * group + h], float(max(d0 + int(i), 0)), 1.f));
+                }
+                asm volatile("bar.sync 1, %0;" ::"n"(128 * NH) : "memory");
             }
-            asm volatile("bar.sync 1, %0;" ::"n"(128 * NH) : "memory");
             ok = ok && mbar_wait_warp(&s_full[b & 1u], (b >> 1) & 1u, p.err);
             if (!ok) continue;
             tc_fence_after_sync();
@@ -261,19 +306,21 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
 #pragma unroll
                 for (int c = 0; c < kHalfKeys; ++c) s[c] = __uint_as_float(u[c / 16][c % 16]);
             }
-            const float* bias = tab + hl * p.tab_stride + (t - t_first) + (kGtKeys - 1) - key0;
+            [[maybe_unused]] const float* bias = tab + hl * p.tab_stride + (t - t_first) + (kGtKeys - 1) - key0;
             const int last = int(P + t) - int(k0 + key0);        // keys 0 .. last of this half are visible
             float tops[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-            if (k0 + kGtKeys - 1 <= P + t_first) {
+            const int low = LATENT && p.window != 0 ? last + 1 - int(p.window) : -1;      // keys from `low` on
+            if (k0 + kGtKeys - 1 <= P + t_first && (!LATENT || p.window == 0 || P + t_last - k0 < p.window)) {
 #pragma unroll
                 for (int j = 0; j < kHalfKeys; ++j) {
-                    s[j] -= bias[-j];
+                    if constexpr (!LATENT) s[j] -= bias[-j];
                     tops[j & 3] = fmaxf(tops[j & 3], s[j]);
                 }
             } else {
 #pragma unroll
                 for (int j = 0; j < kHalfKeys; ++j) {
-                    s[j] = j <= last ? s[j] - bias[-j] : -INFINITY;
+                    if constexpr (LATENT) s[j] = j <= last && j >= low ? s[j] : -INFINITY;
+                    else s[j] = j <= last ? s[j] - bias[-j] : -INFINITY;
                     tops[j & 3] = fmaxf(tops[j & 3], s[j]);
                 }
             }
@@ -349,7 +396,7 @@ __global__ void __launch_bounds__(32 * kGtFirstSoftmax + 128 * NH) gqa_tc_kernel
                 }
             }
             if (ok && half == 0) {
-                const float inv = 1.f / (l + (a.sink ? exp2f(-m) : 0.f));
+                const float inv = 1.f / (l + exp2f(sink - m));
                 fa *= inv;
                 fb *= inv;
                 const size_t at = size_t(t) * a.out_ld + (g * group + hl) * a.vdim;
@@ -421,9 +468,66 @@ int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch) {
     LV_REQUIRE(rows <= 0x7fffffffu, "attention: cache too long");
     if (int rc = make_bf16_map(&maps.k, a.k_cache, rows, dim_p, dim_p, kGtKeys)) return rc;
     if (int rc = make_bf16_map(&maps.v, a.v_cache, rows, vdim_p, vdim_p, kGtKeys)) return rc;
-    auto* kernel = halves ? (a.dim <= 128 ? gqa_tc_kernel<2, 2> : gqa_tc_kernel<2, 4>) : (a.dim <= 128 ? gqa_tc_kernel<1, 2> : gqa_tc_kernel<1, 4>);
+    auto* kernel = halves ? (a.dim <= 128 ? gqa_tc_kernel<2, 2, false> : gqa_tc_kernel<2, 4, false>) : (a.dim <= 128 ? gqa_tc_kernel<1, 2, false> : gqa_tc_kernel<1, 4, false>);
     LV_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
     LV_CUDA(launch_pdl(ctx, kernel, dim3((batch * group + kGtRows - 1) / kGtRows, a.kv_heads), dim3(32 * kGtFirstSoftmax + (halves ? 256 : 128)), smem, p, maps));
+    return LV_OK;
+}
+
+bool latent_tc_supported(const lv_latent_args& a) {
+    return a.cache_type == LV_TYPE_BF16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && (a.dim + 63) / 64 + (a.rot + 63) / 64 <= 4 && a.vdim <= 256;
+}
+
+int latent_tc_launch(lv_ctx* ctx, const lv_latent_args& l, uint32_t batch, const void* kv, uint32_t ld, uint32_t v_at, uint32_t rows, uint32_t h0, uint32_t n) {
+    GqaTcParams p{};
+    lv_gqa_args& a = p.a;
+    a.qkv = l.q + size_t(h0) * (l.dim + l.rot);
+    a.qkv_ld = l.q_ld;
+    a.heads = a.kv_heads = n;
+    a.dim = l.dim;
+    a.vdim = l.vdim;
+    a.scale = l.scale;
+    a.ctx_rows = l.ctx_rows;
+    a.pos = l.pos;
+    a.out = static_cast<uint8_t*>(l.out) + size_t(h0) * l.vdim * (l.out_type == LV_TYPE_BF16 ? 2 : 4);
+    a.out_type = l.out_type;
+    a.out_ld = l.out_ld;
+    p.n_tokens = batch;
+    p.own_chunks = (l.dim + 63) / 64;
+    p.dim_chunks = p.own_chunks + (l.rot + 63) / 64;
+    p.own_steps = (l.dim + 15) / 16;
+    p.steps = p.own_steps + (l.rot + 15) / 16;
+    p.v_chunks = (l.vdim + 63) / 64;
+    p.vdim16 = (l.vdim + 15) / 16 * 16;
+    p.out_bf16 = l.out_type == LV_TYPE_BF16;
+    p.rot = l.rot;
+    p.angles = l.angles;
+    p.angle_ld = l.angle_ld;
+    p.angle_pairs = l.angle_pairs;
+    p.window = l.window;
+    p.v_at = v_at;
+    p.sinks = l.sink ? l.sink + h0 : nullptr;
+    p.err = ctx->d_err;
+    const bool halves = 2 * kGtKeys + 2 * p.vdim16 <= 512;
+    p.tmem_cols = 2 * kGtKeys + (halves ? 2 : 1) * p.vdim16 <= 256 ? 256 : 512;
+    const uint32_t stage = (p.dim_chunks + p.v_chunks) * kGtKChunk, q_bytes = p.dim_chunks * kGtQChunk;
+    p.stages = 2;
+    const uint32_t room = (p.tmem_cols == 512 ? 200 : 110) * 1024;
+    while (p.stages < kGtMaxStages && q_bytes + (p.stages + 1) * stage + 1024 <= room) ++p.stages;
+    const size_t smem = 1024 + size_t(q_bytes) + size_t(p.stages) * stage;
+    LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "latent attention: head sizes need too much shared memory");
+    LV_REQUIRE(l.ctx_rows <= 0x7fffffffu && n <= 65535, "latent attention: cache too long");
+    const uint32_t rank_p = (l.kv_rank + 7) / 8 * 8, rot_p = (l.rot + 7) / 8 * 8;
+    GqaTcMaps maps{};
+    if (int rc = make_bf16_map(&maps.k, kv, rows, ld, ld, kGtKeys)) return rc;
+    maps.v = maps.k;
+    maps.rot = maps.k;
+    if (l.rot != 0)
+        if (int rc = make_bf16_map(&maps.rot, static_cast<const uint8_t*>(l.cache) + rank_p * 2, l.ctx_rows, rot_p, rank_p + rot_p, kGtKeys)) return rc;
+    auto* kernel = halves ? (p.dim_chunks <= 2 ? gqa_tc_kernel<2, 2, true> : gqa_tc_kernel<2, 4, true>)
+                          : (p.dim_chunks <= 2 ? gqa_tc_kernel<1, 2, true> : gqa_tc_kernel<1, 4, true>);
+    LV_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    LV_CUDA(launch_pdl(ctx, kernel, dim3((batch + kGtRows - 1) / kGtRows, n), dim3(32 * kGtFirstSoftmax + (halves ? 256 : 128)), smem, p, maps));
     return LV_OK;
 }
 

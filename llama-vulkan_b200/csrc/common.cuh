@@ -212,6 +212,15 @@ __device__ __forceinline__ float half_bits_to_float(uint32_t h16) {
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.f + expf(-z)); }
 
+// Activation of a finished product (LV_ACT_* of lv_b200.h; 1: the square of relu).
+__device__ __forceinline__ float product_act(float v, int act) {
+    if (act == 1) {
+        const float u = fmaxf(v, 0.f);
+        return u * u;
+    }
+    return v;
+}
+
 // One token of one channel of the minGRU recurrence: S = (1 - sigmoid(z)) S + sigmoid(z) c(u) with c(u) = u + 1/2 for
 // u >= 0 and sigmoid(u) below; returns S * silu(gate).
 __device__ __forceinline__ float mingru_candidate(float u) { return u >= 0.f ? u + 0.5f : sigmoid_f32(u); }

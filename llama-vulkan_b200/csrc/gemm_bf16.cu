@@ -1,6 +1,6 @@
 // Products of several tokens with bfloat16 matrices on the tcgen05 tensor cores, dense and per expert.
 //
-//   out[t][r] = factor * sum_k W[r][k] x[t][k]        W and x bfloat16, sums f32
+//   out[t][r] = act(factor * sum_k W[r][k] x[t][k])        W and x bfloat16, sums f32
 //
 // A CTA covers 128 rows of W (the M of the MMA) and NT tokens (its N).  Both operands are K-major and come by TMA in boxes of
 // 64 columns with the 128-byte swizzle, 4 to 8 stages deep; one lane issues the loads, one lane the MMAs, four warps read the
@@ -11,6 +11,9 @@
 // Experts: lv_expert_route sorts the (token, choice) pairs of a step by expert and lists tiles of NT rows; the input rows lie
 // in that order (lv_norm_conv scatters them there), a tile multiplies them with its expert's rows of the stacked matrix.
 // The gated pair keeps two accumulators, so gate and up of a feature meet in one thread.
+//
+// Windows (lv_gemm_bf16_window): x is a cache, and the rows to multiply are those that the step's tokens see; where they begin is
+// only known on the device, so a tile finds its rows from the position word, and tiles behind the last row leave at once.
 //
 // Every wait is bounded (common.cuh); a lost wait sets the error word, the CTA drains and frees its tensor memory.
 #include <cuda.h>
@@ -40,7 +43,10 @@ struct GemmBf16Params {
     float factor;
     float* scratch;
     uint32_t* counters;
+    int act;
     const lv_expert_tile* tiles;
+    const uint32_t* pos;        // windows: the position word, null otherwise
+    uint32_t window, batch;
     uint32_t* err;
 };
 
@@ -65,12 +71,19 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const GemmBf16
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
 
     uint32_t row0 = blockIdx.x * kBgRows, tok0 = blockIdx.y * NT, n_tok;
-    uint32_t w_row0 = row0;
-    if constexpr (GROUPED) {
+    uint32_t w_row0 = row0, x_row0 = tok0;
+    const bool wait_first = GROUPED || p.pos != nullptr;
+    if (!GROUPED && p.pos != nullptr) {
+        pdl_wait();
+        const uint32_t P = *p.pos, first = p.window != 0 && P + 1 > p.window ? P + 1 - p.window : 0, n = min(p.tokens, P + p.batch - first);
+        if (tok0 >= n) return;
+        n_tok = min(uint32_t(NT), n - tok0);
+        x_row0 = first + tok0;
+    } else if constexpr (GROUPED) {
         pdl_wait();
         const lv_expert_tile t = p.tiles[blockIdx.y];
         if (t.rows == 0) return;
-        tok0 = t.row0;
+        tok0 = x_row0 = t.row0;
         n_tok = t.rows;
         w_row0 += t.expert * p.rows;
     } else {
@@ -100,11 +113,11 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const GemmBf16
                 if constexpr (PAIR) tma_load_2d_plain(dst + kBgTile, &maps.w2, int((c0 + c) * kBgK), int(w_row0), &full[s]);
             };
             auto load_x = [&](uint32_t c, uint32_t s) {
-                tma_load_2d_plain(smem + s * kStage + kXAt, &maps.x, int((c0 + c) * kBgK), int(tok0), &full[s]);
+                tma_load_2d_plain(smem + s * kStage + kXAt, &maps.x, int((c0 + c) * kBgK), int(x_row0), &full[s]);
             };
             const uint32_t first = min(p.stages, n_chunks);
             for (uint32_t c = 0; c < first; ++c) load_w(c, c);
-            if constexpr (!GROUPED) pdl_wait();
+            if (!wait_first) pdl_wait();
             for (uint32_t c = 0; c < first; ++c) load_x(c, c);
             uint32_t s = 0, phase = 0;
             for (uint32_t c = first; c < n_chunks; ++c) {
@@ -150,7 +163,7 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const GemmBf16
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
                 if (z0 + i >= n_tok) break;
-                const float r = PAIR ? silu_f32(v[i]) * g[i] : v[i] * p.factor;
+                const float r = PAIR ? silu_f32(v[i]) * g[i] : product_act(v[i] * p.factor, p.act);
                 const size_t at = size_t(tok0 + z0 + i) * p.out_ld + row;
                 if (p.out_bf16) static_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(r);
                 else static_cast<float*>(p.out)[at] = r;
@@ -316,12 +329,13 @@ static bool bg_aligned(const void* p) { return p != nullptr && (reinterpret_cast
 using namespace lv;
 
 extern "C" int lv_gemm_bf16(lv_ctx* ctx, void* out, int out_type, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols,
-                            const void* x, uint32_t x_ld, uint32_t batch, float factor) {
+                            const void* x, uint32_t x_ld, uint32_t batch, float factor, int act) {
     LV_ENTER(ctx);
     LV_REQUIRE(out && bg_aligned(w) && bg_aligned(x) && rows && cols && batch && out_ld >= rows, "bad gemm_bf16 arguments");
     LV_REQUIRE(ld % 8 == 0 && ld >= cols && x_ld % 8 == 0 && x_ld >= cols && (out_type == LV_TYPE_F32 || out_type == LV_TYPE_BF16), "gemm_bf16: bad strides");
+    LV_REQUIRE(act == LV_ACT_NONE || act == LV_ACT_RELU2, "gemm_bf16: unknown activation");
     GemmBf16Params p{};
-    p.rows = rows; p.tokens = batch; p.K = cols; p.out = out; p.out_ld = out_ld; p.out_bf16 = out_type == LV_TYPE_BF16; p.factor = factor;
+    p.rows = rows; p.tokens = batch; p.K = cols; p.out = out; p.out_ld = out_ld; p.out_bf16 = out_type == LV_TYPE_BF16; p.factor = factor; p.act = act;
     uint32_t nt = batch <= 16 ? 16 : batch <= 32 ? 32 : batch <= 64 ? 64 : 128;
     // narrower token tiles before K splits: partial sums cost more than reading a weight tile twice
     while (nt > 32 && (rows + kBgRows - 1) / kBgRows * ((batch + nt - 1) / nt) * 2 <= uint32_t(ctx->sm_count) && batch > nt / 2) nt /= 2;
@@ -330,6 +344,23 @@ extern "C" int lv_gemm_bf16(lv_ctx* ctx, void* out, int out_type, uint32_t out_l
     if (int rc = make_bf16_map(&maps.x, x, batch, cols, x_ld, nt)) return rc;
     maps.w2 = maps.w;
     return gemm_bf16_pick<false, false>(ctx, p, maps, nt, (batch + nt - 1) / nt);
+}
+
+extern "C" int lv_gemm_bf16_window(lv_ctx* ctx, void* out, int out_type, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols,
+                                   const void* x, uint32_t x_ld, uint32_t x_rows, const uint32_t* pos, uint32_t batch, uint32_t window, uint32_t max_rows) {
+    LV_ENTER(ctx);
+    LV_REQUIRE(out && bg_aligned(w) && bg_aligned(x) && rows && cols && batch && pos && max_rows && x_rows && out_ld >= rows, "bad gemm_bf16 arguments");
+    LV_REQUIRE(ld % 8 == 0 && ld >= cols && x_ld % 8 == 0 && x_ld >= cols && (out_type == LV_TYPE_F32 || out_type == LV_TYPE_BF16), "gemm_bf16: bad strides");
+    GemmBf16Params p{};
+    p.rows = rows; p.tokens = max_rows; p.K = cols; p.out = out; p.out_ld = out_ld; p.out_bf16 = out_type == LV_TYPE_BF16; p.factor = 1.0f;
+    p.pos = pos; p.window = window; p.batch = batch;
+    uint32_t nt = max_rows <= 16 ? 16 : max_rows <= 32 ? 32 : max_rows <= 64 ? 64 : 128;
+    while (nt > 32 && (rows + kBgRows - 1) / kBgRows * ((max_rows + nt - 1) / nt) * 2 <= uint32_t(ctx->sm_count)) nt /= 2;
+    GemmBf16Maps maps{};
+    if (int rc = make_bf16_map(&maps.w, w, rows, cols, ld, kBgRows)) return rc;
+    if (int rc = make_bf16_map(&maps.x, x, x_rows, cols, x_ld, nt)) return rc;
+    maps.w2 = maps.w;
+    return gemm_bf16_pick<false, false>(ctx, p, maps, nt, (max_rows + nt - 1) / nt);
 }
 
 extern "C" uint32_t lv_expert_tile_rows(uint32_t batch, uint32_t top, uint32_t experts) {

@@ -1,6 +1,6 @@
 // Matrix-vector products with bfloat16 weights: the decode-side products of models whose weights are not quantised.
 //
-//   lv_gemv_bf16                 one matrix (stacked projections that share an input); optional factor
+//   lv_gemv_bf16                 one matrix (stacked projections that share an input); optional factor and activation
 //   lv_gemv_bf16_mingru          three products per channel and the gated recurrence on them in the epilogue
 //   lv_gemv_bf16_expert_gate_up  silu(gate x) * (up x) of the experts that a table gives a token
 //   lv_gemv_bf16_expert_down     the mean of those experts' down products
@@ -88,6 +88,7 @@ struct GemvBf16Params {
     float* out;
     uint32_t out_ld;
     float factor;
+    int act;
 };
 
 __global__ void __launch_bounds__(kGbThreads) gemv_bf16_kernel(const GemvBf16Params p) {
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(kGbThreads) gemv_bf16_kernel(const GemvBf16Par
     gb_dot<2, true>(acc, row, p.x + size_t(blockIdx.y) * p.x_ld, p.K);
     const float a0 = warp_sum(acc[0]), a1 = warp_sum(acc[1]);
     const uint32_t lane = threadIdx.x & 31u;
-    if (lane < 2 && u + lane < p.rows) p.out[size_t(blockIdx.y) * p.out_ld + u + lane] = (lane ? a1 : a0) * p.factor;
+    if (lane < 2 && u + lane < p.rows) p.out[size_t(blockIdx.y) * p.out_ld + u + lane] = product_act((lane ? a1 : a0) * p.factor, p.act);
 }
 
 __global__ void __launch_bounds__(kGbThreads) gemv_bf16_mingru_kernel(const GemvBf16Params p, const float* __restrict__ bz, const float* __restrict__ bx,
@@ -175,14 +176,15 @@ static bool gb_aligned(const void* p) { return (reinterpret_cast<uintptr_t>(p) &
 using namespace lv;
 
 extern "C" int lv_gemv_bf16(lv_ctx* ctx, float* out, uint32_t out_ld, const void* w, uint32_t rows, uint32_t ld, uint32_t cols, const float* x,
-                            uint32_t x_ld, uint32_t batch, float factor) {
+                            uint32_t x_ld, uint32_t batch, float factor, int act) {
     LV_ENTER(ctx);
     LV_REQUIRE(out && w && rows && x && cols && batch && batch <= 65535 && out_ld >= rows, "bad gemv_bf16 arguments");
     LV_REQUIRE(ld % 8 == 0 && ld >= cols && x_ld >= cols && (batch == 1 || x_ld % 4 == 0) && gb_aligned(x) && gb_aligned(w), "gemv_bf16: bad strides");
+    LV_REQUIRE(act == LV_ACT_NONE || act == LV_ACT_RELU2, "gemv_bf16: unknown activation");
     GemvBf16Params p{};
     p.w[0] = static_cast<const __nv_bfloat16*>(w);
     p.rows = rows;
-    p.ld = ld; p.K = cols; p.x = x; p.x_ld = x_ld; p.out = out; p.out_ld = out_ld; p.factor = factor;
+    p.ld = ld; p.K = cols; p.x = x; p.x_ld = x_ld; p.out = out; p.out_ld = out_ld; p.factor = factor; p.act = act;
     LV_CUDA(launch_pdl(ctx, gemv_bf16_kernel, dim3((rows + 2 * kGbWarps - 1) / (2 * kGbWarps), batch), dim3(kGbThreads), 0, p));
     return LV_OK;
 }

@@ -8,7 +8,8 @@
 //   h_t   = x''_t / rms(x''_t) * (1 + pre_w)
 //   out_t = h_t + sum_j conv_w[j] * h_(t - taps + 1 + j)          h before position 0 is zero
 //
-// x may come from the embedding table instead of the stream.  The last taps - 1 values of h are the state that the next
+// plain_w: the weights themselves instead of 1 + w.  pre_w null: no second norm, h_t = x''_t (designs that norm the output of a
+// sublayer only).  x may come from the embedding table instead of the stream, with a factor and a second table of pairs of ids.  The last taps - 1 values of h are the state that the next
 // step reads; positions before the start of the sequence are masked by the position word, so a state needs no clearing.
 //
 // A CTA per token holds the token's row in registers (all loads are issued before the first sum).  One token is done in
@@ -78,10 +79,11 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormConvParams p)
     for (int k = 0; k < NV; ++k) {                        // weights do not depend on the previous kernel
         const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
         if (i < W) {
-            if (finish) pre[k].load(a.pre_w + i);
+            if (finish && a.pre_w != nullptr) pre[k].load(a.pre_w + i);
             if (a.y != nullptr) post[k].load(a.post_w + i);
         }
     }
+    const float w0 = a.plain_w ? 0.f : 1.f;
     pdl_wait();
     const uint32_t pos = *a.pos;
     NcVec<VEC> x[NV], y[NV];
@@ -96,6 +98,30 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormConvParams p)
         for (int k = 0; k < NV; ++k) {
             const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
             if (i < W) x[k].load(row + i);
+        }
+        if (a.embed_scale != 0.f) {
+#pragma unroll
+            for (int k = 0; k < NV; ++k)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) x[k].v[e] *= a.embed_scale;
+        }
+        if (a.pair_embed != nullptr) {
+            uint32_t bucket = a.pair_buckets;             // position 0 has a row of its own
+            if (pos + t != 0) {
+                const uint64_t n = a.pair_buckets;
+                bucket = uint32_t((uint64_t(a.token_log[pos + t - 1]) * a.pair_mul_prev % n + uint64_t(id) * a.pair_mul_cur % n) % n);
+            }
+            const __nv_bfloat16* pair = static_cast<const __nv_bfloat16*>(a.pair_embed) + size_t(bucket) * a.pair_ld;
+#pragma unroll
+            for (int k = 0; k < NV; ++k) {
+                const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+                NcVec<VEC> v;
+                if (i < W) {
+                    v.load(pair + i);
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) x[k].v[e] += v.v[e];
+                }
+            }
         }
     } else {
 #pragma unroll
@@ -145,7 +171,7 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormConvParams p)
 #pragma unroll
         for (int k = 0; k < NV; ++k)
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) x[k].v[e] = fmaf(y[k].v[e] * r, 1.f + post[k].v[e], x[k].v[e]);
+            for (int e = 0; e < VEC; ++e) x[k].v[e] = fmaf(y[k].v[e] * r, w0 + post[k].v[e], x[k].v[e]);
     }
     float part = 0.f;
 #pragma unroll
@@ -163,6 +189,14 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormConvParams p)
 #pragma unroll
         for (int e = 0; e < VEC; ++e) part = fmaf(x[k].v[e], x[k].v[e], part);
     }
+    if (a.pre_w == nullptr) {
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const uint32_t i = (threadIdx.x + k * blockDim.x) * VEC;
+            if (i < W) nc_store<VEC, OutT>(a, t, i, x[k]);
+        }
+        return;
+    }
     const float r = 1.f / sqrtf(block_sum(part, scratch) / float(W) + a.eps);
     if (!finish) {
         if (threadIdx.x == 0) a.row_factor[t] = r;
@@ -174,7 +208,7 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormConvParams p)
         if (i >= W) continue;
         NcVec<VEC> h, out;
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) out.v[e] = h.v[e] = x[k].v[e] * r * (1.f + pre[k].v[e]);
+        for (int e = 0; e < VEC; ++e) out.v[e] = h.v[e] = x[k].v[e] * r * (w0 + pre[k].v[e]);
         if (a.taps) {
             NcVec<VEC> w, old;
             w.load(a.conv_w + size_t(keep) * W + i);
@@ -211,7 +245,7 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(const NormConvParams p) 
     NcVec<VEC> pre, cw[MAXT], win[MAXT];                  // taps right-aligned: index MAXT - 1 is the current token
     pre.load(a.pre_w + i);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) pre.v[e] += 1.f;
+    for (int e = 0; e < VEC; ++e) pre.v[e] += a.plain_w ? 0.f : 1.f;
 #pragma unroll
     for (int j = 0; j < MAXT; ++j) {
         const int s = j - (MAXT - int(a.taps));
@@ -275,8 +309,8 @@ static int norm_conv_launch(lv_ctx* ctx, const lv_norm_conv_args& a) {
     p.err = ctx->d_err;
     // four channels per access where every row starts on 16 bytes
     auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
-    bool vec = a.width % 4 == 0 && a.out_ld % 4 == 0 && a.embed_ld % 4 == 0;
-    for (const void* q : {static_cast<const void*>(a.x), a.embed, static_cast<const void*>(a.y), static_cast<const void*>(a.post_w), static_cast<const void*>(a.step),
+    bool vec = a.width % 4 == 0 && a.out_ld % 4 == 0 && a.embed_ld % 4 == 0 && a.pair_ld % 4 == 0;
+    for (const void* q : {static_cast<const void*>(a.x), a.embed, a.pair_embed, static_cast<const void*>(a.y), static_cast<const void*>(a.post_w), static_cast<const void*>(a.step),
                           static_cast<const void*>(a.trace), static_cast<const void*>(a.x_out), static_cast<const void*>(a.pre_w),
                           static_cast<const void*>(a.conv_w), static_cast<const void*>(a.history), static_cast<const void*>(a.out)})
         vec = vec && aligned(q);
@@ -313,9 +347,10 @@ extern "C" int lv_norm_conv(lv_ctx* ctx, const lv_norm_conv_args* args) {
     LV_ENTER(ctx);
     LV_REQUIRE(args != nullptr, "null argument");
     const lv_norm_conv_args& a = *args;
-    LV_REQUIRE(a.pos && a.pre_w && a.out && a.width && a.batch && a.first < a.batch, "bad norm_conv arguments");
+    LV_REQUIRE(a.pos && (a.pre_w || a.taps == 0) && a.out && a.width && a.batch && a.first < a.batch, "bad norm_conv arguments");
     LV_REQUIRE(a.width <= 16384, "norm_conv: width above 16384");
     LV_REQUIRE(a.x != nullptr || (a.embed && a.token_log && a.vocab && a.embed_ld >= a.width), "norm_conv: no input stream");
+    LV_REQUIRE(a.pair_embed == nullptr || (a.token_log && a.pair_buckets && a.pair_ld >= a.width), "norm_conv: bad table of pairs");
     LV_REQUIRE(a.y == nullptr || (a.post_w && a.y_rows && (a.y_index || a.y_rows == 1)), "norm_conv: bad sublayer rows");
     LV_REQUIRE(a.taps <= kNormConvMaxTaps && (a.taps == 0 || (a.conv_w && a.first == 0)) && (a.taps < 2 || a.history), "norm_conv: bad taps");
     LV_REQUIRE(a.taps == 0 || a.batch == 1 || (a.x_out && a.row_factor), "norm_conv: several tokens need x_out and row_factor");

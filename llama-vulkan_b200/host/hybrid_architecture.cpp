@@ -1,6 +1,7 @@
 #include "hybrid_architecture.h"
 
 #include <algorithm>
+#include <cmath>
 #include <iostream>
 
 #include "hybrid_session_state.h"
@@ -29,7 +30,40 @@ bool need_float(const json_value* at, const char* key, float* out, string* error
     *error = string(key) + " missing or not a number";
     return false;
 }
+
+bool need_double(const json_value* at, const char* key, double* out, string* error) {
+    const json_value* v = at ? at->find(key) : nullptr;
+    if (v && v->is_number() && isfinite(v->number())) {
+        *out = v->number();
+        return true;
+    }
+    *error = string(key) + " missing or not a number";
+    return false;
+}
+
+bool given(const json_value* v) { return v != nullptr && !v->is_null(); }
+
+const json_value* need_layers(const json_value& config, string* error) {
+    const json_value* layers = config.find("layers");
+    if (layers && layers->is_array() && !layers->items().empty()) return layers;
+    *error = "layers missing";
+    return nullptr;
+}
 }  // namespace
+
+hybrid_rotation make_rotation(u32 dims, double base, const rotary_scaling* s) {
+    hybrid_rotation r;
+    for (u32 i = 0; i < dims / 2; ++i) r.freqs.push_back(pow(base, -2.0 * i / dims));
+    if (s == nullptr) return r;
+    auto pair_of = [&](double turns) { return dims * log(s->original / (2 * M_PI * turns)) / (2 * log(base)); };
+    const double lo = max(floor(pair_of(s->fast)), 0.0), hi = min(ceil(pair_of(s->slow)), double(dims) - 1);
+    for (u32 i = 0; i < dims / 2; ++i) {
+        const double ramp = clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0);
+        r.freqs[i] = r.freqs[i] / s->factor * ramp + r.freqs[i] * (1 - ramp);
+    }
+    r.mult = float(0.1 * log(s->factor) + 1);
+    return r;
+}
 
 bool parse_sonuzen_config(const json_value& config, hybrid_config* out, string* error) {
     hybrid_config& c = *out;
@@ -37,11 +71,8 @@ bool parse_sonuzen_config(const json_value& config, hybrid_config* out, string* 
         !need_float(config.find("norm"), "eps", &c.eps, error) || !need_float(&config, "residual_mult", &c.residual_mult, error) ||
         !need_float(&config, "logit_scale", &c.logit_scale, error) || !need_u32(config.find("canon"), "taps", &c.taps, error))
         return false;
-    const json_value* layers = config.find("layers");
-    if (!layers || !layers->is_array() || layers->items().empty()) {
-        *error = "layers missing";
-        return false;
-    }
+    const json_value* layers = need_layers(config, error);
+    if (!layers) return false;
     for (const json_value& l : layers->items()) {
         hybrid_layer_spec spec;
         const json_value *type = l.find("type"), *mixer = l.find("mixer"), *mlp = l.find("mlp");
@@ -63,7 +94,7 @@ bool parse_sonuzen_config(const json_value& config, hybrid_config* out, string* 
             *error = "unknown layer type";
             return false;
         }
-        if (mlp && !mlp->is_null()) {
+        if (given(mlp)) {
             const json_value* kind = mlp->find("kind");
             if (kind && kind->text() != "moe") {
                 *error = "unknown feed-forward " + kind->text();
@@ -90,10 +121,90 @@ bool parse_sonuzen_config(const json_value& config, hybrid_config* out, string* 
     return true;
 }
 
+// Nuforax: attention over latent caches and Mamba-2 layers with dense feed-forwards, norms on the outputs of the sublayers only,
+// an embedding of token pairs, the embedding table as the output matrix.
+bool parse_nuforax_config(const json_value& config, hybrid_config* out, string* error) {
+    hybrid_config& c = *out;
+    c.pre_norm = false;
+    c.plain_norm = c.tied_head = true;
+    const json_value *embedding = config.find("embedding"), *bigram = embedding ? embedding->find("bigram") : nullptr;
+    if (!need_u32(&config, "width", &c.width, error) || !need_u32(&config, "vocab", &c.vocab, error) ||
+        !need_float(config.find("norm"), "eps", &c.eps, error) || !need_float(embedding, "scale", &c.embed_scale, error) ||
+        !need_u32(bigram, "buckets", &c.pair_buckets, error) || !need_u32(bigram, "mul_prev", &c.pair_mul_prev, error, 0) ||
+        !need_u32(bigram, "mul_cur", &c.pair_mul_cur, error, 0))
+        return false;
+    const json_value* layers = need_layers(config, error);
+    if (!layers) return false;
+    auto bad = [&](const char* why) {
+        *error = why;
+        return false;
+    };
+    for (const json_value& l : layers->items()) {
+        hybrid_layer_spec spec;
+        const json_value *type = l.find("type"), *mixer = l.find("mixer"), *mlp = l.find("mlp");
+        hybrid_mixer& m = spec.mixer;
+        if (type && type->text() == "latent_attention") {
+            m.type = hybrid_mixer::kind::latent;
+            m.sink = true;
+            const json_value *rot = mixer ? mixer->find("rot") : nullptr, *scaling = rot ? rot->find("scaling") : nullptr, *from = mixer ? mixer->find("kv_from") : nullptr;
+            u32 dims = 0;
+            double base = 0;
+            if (!need_u32(mixer, "heads", &m.heads, error) || !need_u32(mixer, "dim", &m.dim, error) || !need_u32(mixer, "rot_dim", &m.rot, error) ||
+                !need_u32(mixer, "vdim", &m.vdim, error) || !need_u32(mixer, "kv_rank", &m.kv_rank, error) || !need_float(mixer, "scale", &m.scale, error) ||
+                !need_u32(mixer->find("mask"), "size", &m.window, error) || !need_u32(rot, "dims", &dims, error) || !need_double(rot, "base", &base, error))
+                return false;
+            if (dims % 2 != 0 || dims > m.rot || base <= 0) return bad("rot.dims must be even and at most rot_dim");
+            rotary_scaling s{};
+            if (given(scaling)) {
+                if (!need_double(scaling, "factor", &s.factor, error) || !need_double(scaling, "original", &s.original, error) ||
+                    !need_double(scaling, "fast", &s.fast, error) || !need_double(scaling, "slow", &s.slow, error))
+                    return false;
+                if (s.factor <= 0 || s.original <= 0 || s.fast <= 0 || s.slow <= 0 || base == 1) return bad("rot.scaling out of range");
+            }
+            hybrid_rotation r = make_rotation(dims, base, given(scaling) ? &s : nullptr);
+            m.rot_pairs = dims / 2;
+            while (m.rotation < c.rotations.size() && (c.rotations[m.rotation].freqs != r.freqs || c.rotations[m.rotation].mult != r.mult)) ++m.rotation;
+            if (m.rotation == c.rotations.size()) {
+                r.first = c.rotation_pairs();
+                c.rotations.push_back(r);
+            }
+            if (given(from)) {
+                u32 source = 0;
+                if (!from->as_u32(&source) || source >= c.layers.size()) return bad("kv_from is not an earlier layer");
+                const hybrid_mixer& o = c.layers[source].mixer;
+                if (!o.has_own_cache() || o.kv_rank != m.kv_rank || o.rot != m.rot || o.rotation != m.rotation) return bad("kv_from names a layer without such a cache");
+                m.kv_from = int(source);
+            }
+        } else if (type && type->text() == "mamba2") {
+            m.type = hybrid_mixer::kind::ssm;
+            if (!need_u32(mixer, "heads", &m.heads, error) || !need_u32(mixer, "vdim", &m.vdim, error) || !need_u32(mixer, "state", &m.state, error) ||
+                !need_u32(mixer, "groups", &m.groups, error) || !need_u32(mixer, "conv", &m.taps, error) || !need_u32(mixer, "norm_groups", &m.norm_groups, error))
+                return false;
+            if (m.heads % m.groups != 0) return bad("heads must be a multiple of groups");
+            if (u64(m.heads) * m.vdim % m.norm_groups != 0) return bad("norm_groups must divide the inner width");
+        } else {
+            return bad("unknown layer type");
+        }
+        if (given(mlp)) {
+            const json_value* kind = mlp->find("kind");
+            if (kind && kind->text() != "dense") {
+                *error = "unknown feed-forward " + kind->text();
+                return false;
+            }
+            if (!need_u32(mlp, "ff", &spec.dense.ff, error)) return false;
+            spec.dense.act = LV_ACT_RELU2;
+        }
+        c.layers.push_back(spec);
+    }
+    return true;
+}
+
 // ---- model -----------------------------------------------------------------------------------
 
 hybrid_architecture::~hybrid_architecture() {
     for (llava_buffer* b : tensors) delete b;
+    delete rot_freqs;
+    delete rot_mults;
 }
 
 bool hybrid_architecture::check(const model_file& model, u32 n_ranks) {
@@ -107,11 +218,17 @@ bool hybrid_architecture::check(const model_file& model, u32 n_ranks) {
         cerr << "[!] " << name_ << " models run on one GPU" << endl;
         return false;
     }
-    for (const hybrid_layer_spec& l : cfg.layers)
-        if (l.mixer.type == hybrid_mixer::kind::attention && (l.mixer.dim > 256 || l.mixer.vdim > 256)) {
-            cerr << "[!] " << name_ << ": heads of more than 256 values are not supported" << endl;
+    for (const hybrid_layer_spec& l : cfg.layers) {
+        const hybrid_mixer& m = l.mixer;
+        const char* why = nullptr;
+        if (m.type == hybrid_mixer::kind::attention && (m.dim > 256 || m.vdim > 256)) why = "heads of more than 256 values";
+        if (m.type == hybrid_mixer::kind::latent && m.kv_rank > 1024) why = "latents of more than 1024 values";
+        if (m.type == hybrid_mixer::kind::ssm && (m.state > 256 || m.taps > 16)) why = "states of more than 256 rows or convolutions of more than 16 taps";
+        if (why) {
+            cerr << "[!] " << name_ << ": " << why << " are not supported" << endl;
             return false;
         }
+    }
     if (cfg.width > 16384 || cfg.taps > 16) {
         cerr << "[!] " << name_ << ": width above 16384 or more than 16 taps" << endl;
         return false;
@@ -122,6 +239,12 @@ bool hybrid_architecture::check(const model_file& model, u32 n_ranks) {
     for (u32 t = 0; t < cfg.loop_times; ++t)
         for (u32 i = first; i < last; ++i) runs.push_back({i, i == first ? int(t) : -1});
     for (u32 i = last; i < n; ++i) runs.push_back({i, -1});
+    vector<u32> latest(n, 0);            // last run of each layer so far
+    for (u32 r = 0; r < runs.size(); ++r) {
+        const hybrid_mixer& m = cfg.layers[runs[r].layer].mixer;
+        runs[r].cache_run = m.kv_from < 0 ? r : latest[m.kv_from];
+        latest[runs[r].layer] = r;
+    }
     return true;
 }
 
@@ -150,34 +273,68 @@ bool hybrid_architecture::build(llava_context* ctx) {
     auto values = [&](const string& name, u32 rows, u32 cols = 1) { return stack({{name, rows}}, cols, weight_form::vector_f32); };
 
     embed = matrix("embed", cfg.vocab, cfg.width);
-    head = matrix("head", cfg.vocab, cfg.width);
+    head = cfg.tied_head ? embed : matrix("head", cfg.vocab, cfg.width);
+    if (cfg.pair_buckets) pair_embed = matrix("bigram", cfg.pair_buckets + 1, cfg.width);
     final_norm = values("final.norm", cfg.width);
     if (cfg.loop_times) loop_step = values("loop.step", cfg.loop_times, cfg.width);
+    if (const u32 pairs = cfg.rotation_pairs()) {
+        rot_freqs = new llava_buffer(ctx, ggml_value_type::f32, 2, pairs, ctx->weights_memory());
+        rot_mults = new llava_buffer(ctx, ggml_value_type::f32, pairs, 1, ctx->weights_memory());
+    }
     for (u32 i = 0; i < cfg.layers.size(); ++i) {
         const hybrid_layer_spec& spec = cfg.layers[i];
         const hybrid_mixer& m = spec.mixer;
         const string p = "l" + to_string(i) + ".", mix = p + "mix.", mlp = p + "mlp.";
         hybrid_layer l;
-        auto taps = [&](const string& name) { return stack({{name, cfg.width}}, cfg.taps, weight_form::columns_f32); };
-        l.norm1 = values(p + "norm1", cfg.width);
-        l.norm1b = values(p + "norm1b", cfg.width);
-        l.canon1 = taps(p + "canon1");
+        auto taps = [&](const string& name, u32 channels, u32 n) { return stack({{name, channels}}, n, weight_form::columns_f32); };
+        // "norm1" is the norm in front where there are two, and the one on the output where that is all
+        auto sublayer = [&](const string& n, llava_buffer** pre, llava_buffer** post, llava_buffer** conv) {
+            if (cfg.pre_norm) *pre = values(p + "norm" + n, cfg.width);
+            *post = values(p + "norm" + n + (cfg.pre_norm ? "b" : ""), cfg.width);
+            if (cfg.taps) *conv = taps(p + "canon" + n, cfg.width, cfg.taps);
+        };
+        sublayer("1", &l.pre1, &l.post1, &l.canon1);
         l.out = matrix(mix + "o", cfg.width, m.out_size());
-        if (m.type == hybrid_mixer::kind::attention) {
-            l.in = stack({{mix + "q", m.heads * m.dim}, {mix + "k", m.kv_heads * m.dim}, {mix + "v", m.kv_heads * m.vdim}}, cfg.width, weight_form::rows_bf16);
-            l.q_norm = values(mix + "q.norm", m.dim);
-            l.k_norm = values(mix + "k.norm", m.dim);
-            l.r1 = values(mix + "r1", m.heads);
-            l.r2 = values(mix + "r2", m.heads);
-        } else {
-            l.in = stack({{mix + "z", m.width}, {mix + "x", m.width}, {mix + "g", m.width}}, cfg.width, weight_form::rows_bf16);
-            l.z_bias = values(mix + "z.b", m.width);
-            l.x_bias = values(mix + "x.b", m.width);
+        switch (m.type) {
+            case hybrid_mixer::kind::attention:
+                l.in = stack({{mix + "q", m.heads * m.dim}, {mix + "k", m.kv_heads * m.dim}, {mix + "v", m.kv_heads * m.vdim}}, cfg.width, weight_form::rows_bf16);
+                l.q_norm = values(mix + "q.norm", m.dim);
+                l.k_norm = values(mix + "k.norm", m.dim);
+                l.r1 = values(mix + "r1", m.heads);
+                l.r2 = values(mix + "r2", m.heads);
+                break;
+            case hybrid_mixer::kind::mingru:
+                l.in = stack({{mix + "z", m.width}, {mix + "x", m.width}, {mix + "g", m.width}}, cfg.width, weight_form::rows_bf16);
+                l.z_bias = values(mix + "z.b", m.width);
+                l.x_bias = values(mix + "x.b", m.width);
+                break;
+            case hybrid_mixer::kind::latent: {
+                vector<pair<string, u32>> in = {{mix + "q", m.heads * (m.dim + m.rot)}};
+                if (m.has_own_cache()) {
+                    in.emplace_back(mix + "dkv", m.kv_rank + m.rot);
+                    l.kv_norm = values(mix + "dkv.norm", m.kv_rank);
+                }
+                l.in = stack(in, cfg.width, weight_form::rows_bf16);
+                l.kv_up = stack({{mix + "uk", m.heads * m.dim}, {mix + "uv", m.heads * m.vdim}}, m.kv_rank, weight_form::rows_bf16);
+                l.sink = values(mix + "sink", m.heads);
+                break;
+            }
+            case hybrid_mixer::kind::ssm:
+                l.in = matrix(mix + "in", m.raw_size(), cfg.width);
+                l.conv_w = taps(mix + "conv", m.conv_channels(), m.taps);
+                l.conv_b = values(mix + "conv.b", m.conv_channels());
+                l.dt_bias = values(mix + "dt_bias", m.heads);
+                l.A_log = values(mix + "A_log", m.heads);
+                l.D = values(mix + "D", m.heads);
+                l.norm = values(mix + "norm", m.out_size());
+                break;
+        }
+        if (spec.has_feed_forward()) sublayer("2", &l.pre2, &l.post2, &l.canon2);
+        if (spec.dense.ff) {
+            l.up = matrix(mlp + "up", spec.dense.ff, cfg.width);
+            l.down = matrix(mlp + "down", cfg.width, spec.dense.ff);
         }
         if (spec.mlp.experts) {
-            l.norm2 = values(p + "norm2", cfg.width);
-            l.norm2b = values(p + "norm2b", cfg.width);
-            l.canon2 = taps(p + "canon2");
             vector<pair<string, u32>> gate, up, down;
             for (u32 e = 0; e < spec.mlp.experts; ++e) {
                 const string x = mlp + "e" + to_string(e) + ".";
@@ -201,7 +358,14 @@ bool hybrid_architecture::upload(llava_context* ctx) {
             cerr << "[!] cannot upload " << b->backing_buffer_name << ": " << lv_last_error_string() << endl;
             return false;
         }
-    return true;
+    if (rot_freqs == nullptr) return true;
+    vector<double> freqs;
+    vector<float> mults;
+    for (const hybrid_rotation& r : cfg.rotations) {
+        freqs.insert(freqs.end(), r.freqs.begin(), r.freqs.end());
+        mults.insert(mults.end(), r.freqs.size(), r.mult);
+    }
+    return rot_freqs->write_raw(0, freqs.data(), freqs.size() * sizeof(double)) && rot_mults->write_raw(0, mults.data(), mults.size() * sizeof(float));
 }
 
 unique_ptr<session_state> hybrid_architecture::make_session_state(llava_session* session) { return make_unique<hybrid_session_state>(session, this); }
@@ -265,6 +429,15 @@ struct hybrid_recorder {
         a.out_ld = pad8(cfg.width);
         a.out_index = rows ? static_cast<const u32*>(rows->device_ptr()) : nullptr;
         a.out_copies = copies;
+        a.plain_w = cfg.plain_norm;
+        a.embed_scale = cfg.embed_scale;
+        if (arch.pair_embed) {
+            a.pair_embed = arch.pair_embed->device_ptr();
+            a.pair_ld = arch.pair_embed->leading();
+            a.pair_buckets = cfg.pair_buckets;
+            a.pair_mul_prev = cfg.pair_mul_prev;
+            a.pair_mul_cur = cfg.pair_mul_cur;
+        }
         a.width = cfg.width;
         a.first = last_only ? T - 1 : 0;
         a.batch = T;
@@ -279,8 +452,60 @@ struct hybrid_recorder {
 
     void product(llava_buffer* out, const llava_buffer* w, llava_buffer* in, u32 in_ld, float factor = 1.0f) {
         const u32 rows = w->shape.first;
-        if (batched) cb->note(lv_gemm_bf16(lv, f32(out), LV_TYPE_F32, rows, w->device_ptr(), rows, w->leading(), w->shape.second, f32(in), in_ld, T, factor));
-        else cb->note(lv_gemv_bf16(lv, f32(out), rows, w->device_ptr(), rows, w->leading(), w->shape.second, f32(in), in_ld, T, factor));
+        if (batched) cb->note(lv_gemm_bf16(lv, f32(out), LV_TYPE_F32, rows, w->device_ptr(), rows, w->leading(), w->shape.second, f32(in), in_ld, T, factor, LV_ACT_NONE));
+        else cb->note(lv_gemv_bf16(lv, f32(out), rows, w->device_ptr(), rows, w->leading(), w->shape.second, f32(in), in_ld, T, factor, LV_ACT_NONE));
+    }
+
+    void dense(const hybrid_layer& l, const hybrid_dense& d) {
+        const u32 ld = pad8(cfg.width), act_ld = pad8(d.ff);
+        if (batched) cb->note(lv_gemm_bf16(lv, f32(st->act), LV_TYPE_BF16, act_ld, l.up->device_ptr(), d.ff, l.up->leading(), cfg.width, f32(st->normed), ld, T, 1.0f, d.act));
+        else cb->note(lv_gemv_bf16(lv, f32(st->act), act_ld, l.up->device_ptr(), d.ff, l.up->leading(), cfg.width, f32(st->normed), ld, T, 1.0f, d.act));
+        product(st->sub, l.down, st->act, act_ld);
+    }
+
+    void latent(const hybrid_layer& l, const hybrid_mixer& m, const hybrid_run& run) {
+        product(st->raw, l.in, st->normed, pad8(cfg.width));
+        lv_latent_args a = st->latent_args(m);
+        a.q = f32(st->raw);
+        a.q_ld = m.raw_size();
+        if (m.has_own_cache()) {
+            a.dkv = a.q + m.heads * (m.dim + m.rot);
+            a.dkv_ld = a.q_ld;
+            a.kv_norm = f32(l.kv_norm);
+        }
+        a.angles = f32(st->angles) + 2 * cfg.rotations[m.rotation].first;
+        a.angle_ld = 2 * cfg.rotation_pairs();
+        a.w = l.kv_up->device_ptr();
+        a.w_ld = l.kv_up->leading();
+        a.sink = f32(l.sink);
+        a.cache = st->runs[run.cache_run].latent_cache->device_ptr();
+        a.pos = pos;
+        a.out = f32(st->mixed);
+        a.out_type = act_type();
+        a.out_ld = pad8(m.out_size());
+        cb->note(lv_latent_attention(lv, &a, st->mix_scratch->device_ptr(), st->mix_scratch->byte_size(), T, cb->backlog_size));
+        product(st->sub, l.out, st->mixed, a.out_ld);
+    }
+
+    void ssm(const hybrid_layer& l, const hybrid_mixer& m, const hybrid_run_state& r) {
+        product(st->raw, l.in, st->normed, pad8(cfg.width));
+        lv_ssm_args a = st->ssm_args(m);
+        a.raw = f32(st->raw);
+        a.raw_ld = m.raw_size();
+        a.conv_w = f32(l.conv_w);
+        a.conv_b = f32(l.conv_b);
+        a.dt_bias = f32(l.dt_bias);
+        a.A_log = f32(l.A_log);
+        a.D = f32(l.D);
+        a.norm_w = f32(l.norm);
+        a.history = f32(r.conv_history);
+        a.S = f32(r.ssm_state);
+        a.pos = pos;
+        a.out = f32(st->mixed);
+        a.out_type = act_type();
+        a.out_ld = pad8(m.out_size());
+        cb->note(lv_ssm(lv, &a, st->mix_scratch->device_ptr(), st->mix_scratch->byte_size(), T));
+        product(st->sub, l.out, st->mixed, a.out_ld);
     }
 
     void attention(const hybrid_layer& l, const hybrid_mixer& m, const hybrid_run_state& r) {
@@ -367,19 +592,29 @@ struct hybrid_recorder {
         const auto& runs = arch.runs_in_order();
         if (batched && st->n_route_jobs)
             cb->note(lv_expert_route(lv, static_cast<const lv_route_job*>(st->route_jobs->device_ptr()), st->n_route_jobs, st->max_experts, log, pos, cfg.vocab, T));
+        if (st->angles)
+            cb->note(lv_rotary_table(lv, f32(st->angles), static_cast<const double*>(arch.rot_freqs->device_ptr()), f32(arch.rot_mults), cfg.rotation_pairs(), pos, T));
         for (size_t i = 0; i < runs.size(); ++i) {
             const u32 layer = runs[i].layer;
             const hybrid_layer& l = arch.layer(layer);
             const hybrid_layer_spec& spec = cfg.layers[layer];
             const hybrid_run_state& r = st->runs[i];
-            norm_conv(l.norm1, l.canon1, r.history1, runs[i].begins_pass >= 0 ? f32(arch.loop_step) + size_t(runs[i].begins_pass) * cfg.width : nullptr);
-            if (spec.mixer.type == hybrid_mixer::kind::attention) attention(l, spec.mixer, r);
-            else mingru(l, spec.mixer, r);
-            finish_sublayer(l.norm1b);
-            if (spec.mlp.experts) {
-                norm_conv(l.norm2, l.canon2, r.history2, nullptr, batched ? st->route_index[layer] : nullptr, spec.mlp.top);
+            norm_conv(l.pre1, l.canon1, r.history1, runs[i].begins_pass >= 0 ? f32(arch.loop_step) + size_t(runs[i].begins_pass) * cfg.width : nullptr);
+            switch (spec.mixer.type) {
+                case hybrid_mixer::kind::attention: attention(l, spec.mixer, r); break;
+                case hybrid_mixer::kind::mingru: mingru(l, spec.mixer, r); break;
+                case hybrid_mixer::kind::latent: latent(l, spec.mixer, runs[i]); break;
+                case hybrid_mixer::kind::ssm: ssm(l, spec.mixer, r); break;
+            }
+            finish_sublayer(l.post1);
+            if (spec.dense.ff) {
+                norm_conv(l.pre2, l.canon2, r.history2, nullptr);
+                dense(l, spec.dense);
+                finish_sublayer(l.post2);
+            } else if (spec.mlp.experts) {
+                norm_conv(l.pre2, l.canon2, r.history2, nullptr, batched ? st->route_index[layer] : nullptr, spec.mlp.top);
                 experts(layer, l, spec.mlp);
-                finish_sublayer(l.norm2b);
+                finish_sublayer(l.post2);
             }
             finished_run = int(i);
         }
@@ -391,7 +626,7 @@ struct hybrid_recorder {
             if (!st->trace.empty() && T > 1) norm_conv(arch.final_norm, nullptr, nullptr, nullptr);      // (finishes the last sublayer for all rows)
             norm_conv(arch.final_norm, nullptr, nullptr, nullptr, nullptr, 1, true);
             cb->note(lv_gemv_bf16(lv, f32(s->output_probs), cfg.vocab, arch.head->device_ptr(), cfg.vocab, arch.head->leading(), cfg.width,
-                                  f32(st->normed), pad8(cfg.width), 1, cfg.logit_scale));
+                                  f32(st->normed), pad8(cfg.width), 1, cfg.logit_scale, LV_ACT_NONE));
         }
         cb->finish_step();
     }

@@ -24,15 +24,26 @@ hybrid_session_state::hybrid_session_state(llava_session* _session, const hybrid
     for (const hybrid_run& r : arch->runs_in_order()) {
         const hybrid_layer_spec& spec = c.layers[r.layer];
         hybrid_run_state s;
-        if (spec.mixer.type == hybrid_mixer::kind::attention) {
-            s.k_cache = new llava_buffer(ctx, C, spec.mixer.kv_heads * session->max_context, pad8(spec.mixer.dim), lasting, "k_cache");
-            s.v_cache = new llava_buffer(ctx, C, spec.mixer.kv_heads * session->max_context, pad8(spec.mixer.vdim), lasting, "v_cache");
-        } else {
-            s.gru_state = new llava_buffer(ctx, F, spec.mixer.width, 1, lasting, "gru_state");
+        const hybrid_mixer& m = spec.mixer;
+        switch (m.type) {
+            case hybrid_mixer::kind::attention:
+                s.k_cache = new llava_buffer(ctx, C, m.kv_heads * session->max_context, pad8(m.dim), lasting, "k_cache");
+                s.v_cache = new llava_buffer(ctx, C, m.kv_heads * session->max_context, pad8(m.vdim), lasting, "v_cache");
+                break;
+            case hybrid_mixer::kind::mingru:
+                s.gru_state = new llava_buffer(ctx, F, m.width, 1, lasting, "gru_state");
+                break;
+            case hybrid_mixer::kind::latent:
+                if (m.has_own_cache()) s.latent_cache = new llava_buffer(ctx, C, session->max_context, pad8(m.kv_rank) + pad8(m.rot), lasting, "latent_cache");
+                break;
+            case hybrid_mixer::kind::ssm:
+                s.ssm_state = new llava_buffer(ctx, F, m.heads * m.vdim, (m.state + 15) / 16 * 16, lasting, "ssm_state");
+                s.conv_history = new llava_buffer(ctx, F, m.conv_channels(), m.taps, lasting, "conv_history");
+                break;
         }
         if (c.taps > 1) {
             s.history1 = new llava_buffer(ctx, F, c.width, c.taps - 1, lasting, "history1");
-            if (spec.mlp.experts) s.history2 = new llava_buffer(ctx, F, c.width, c.taps - 1, lasting, "history2");
+            if (spec.has_feed_forward()) s.history2 = new llava_buffer(ctx, F, c.width, c.taps - 1, lasting, "history2");
         }
         runs.push_back(s);
     }
@@ -42,12 +53,12 @@ hybrid_session_state::hybrid_session_state(llava_session* _session, const hybrid
 hybrid_session_state::~hybrid_session_state() {
     drop_scratch();
     for (hybrid_run_state& s : runs)
-        for (llava_buffer* b : {s.k_cache, s.v_cache, s.gru_state, s.history1, s.history2}) delete b;
+        for (llava_buffer* b : {s.k_cache, s.v_cache, s.latent_cache, s.gru_state, s.ssm_state, s.conv_history, s.history1, s.history2}) delete b;
     delete lasting;
 }
 
 void hybrid_session_state::drop_scratch() {
-    for (llava_buffer** b : {&stream, &row_factor, &normed, &raw, &mixed, &act, &sub, &attn_scratch, &logits_rows, &route_jobs}) {
+    for (llava_buffer** b : {&stream, &row_factor, &normed, &raw, &mixed, &act, &sub, &attn_scratch, &mix_scratch, &angles, &logits_rows, &route_jobs}) {
         delete *b;
         *b = nullptr;
     }
@@ -61,6 +72,35 @@ void hybrid_session_state::drop_scratch() {
     scratch_batch = 0;
 }
 
+lv_latent_args hybrid_session_state::latent_args(const hybrid_mixer& m) const {
+    lv_latent_args a{};
+    a.heads = m.heads;
+    a.dim = m.dim;
+    a.rot = m.rot;
+    a.vdim = m.vdim;
+    a.kv_rank = m.kv_rank;
+    a.angle_pairs = m.rot_pairs;
+    a.scale = m.scale;
+    a.eps = arch->config().eps;
+    a.window = m.window;
+    a.cache_type = f32 ? LV_TYPE_F32 : LV_TYPE_BF16;
+    a.ctx_rows = session->max_context;
+    a.form = LV_LATENT_AUTO;
+    return a;
+}
+
+lv_ssm_args hybrid_session_state::ssm_args(const hybrid_mixer& m) const {
+    lv_ssm_args a{};
+    a.heads = m.heads;
+    a.vdim = m.vdim;
+    a.state = m.state;
+    a.groups = m.groups;
+    a.taps = m.taps;
+    a.norm_groups = m.norm_groups;
+    a.eps = arch->config().eps;
+    return a;
+}
+
 bool hybrid_session_state::resize() {
     if (!lasting->is_frozen()) return false;
     const u32 B = session->max_batch;
@@ -70,13 +110,22 @@ bool hybrid_session_state::resize() {
     const hybrid_config& c = arch->config();
     llava_context* ctx = session->ctx;
     u32 raw_size = 8, mixed_size = 8, act_size = 8, copies = 1;
-    size_t attention_bytes = 0;
+    size_t attention_bytes = 0, mix_bytes = 0;
     for (const hybrid_layer_spec& l : c.layers) {
         raw_size = max(raw_size, l.mixer.raw_size());
         mixed_size = max(mixed_size, pad8(l.mixer.out_size()));
         if (l.mlp.experts) {
             act_size = max(act_size, l.mlp.top * pad8(l.mlp.ff));
             copies = max(copies, l.mlp.top);
+        }
+        act_size = max(act_size, pad8(l.dense.ff));
+        if (l.mixer.type == hybrid_mixer::kind::latent) {
+            const lv_latent_args a = latent_args(l.mixer);         // its form follows the batch, every batch must fit
+            for (u32 n = 1; n <= B; ++n) mix_bytes = max(mix_bytes, lv_latent_scratch_bytes(ctx->lv(), &a, n, session->max_context));
+        }
+        if (l.mixer.type == hybrid_mixer::kind::ssm) {
+            const lv_ssm_args a = ssm_args(l.mixer);
+            mix_bytes = max(mix_bytes, lv_ssm_scratch_bytes(&a, B));
         }
         if (l.mixer.type == hybrid_mixer::kind::attention) {
             lv_gqa_args a{};
@@ -97,6 +146,8 @@ bool hybrid_session_state::resize() {
     act = new llava_buffer(ctx, F, act_size, B, scratch);
     sub = new llava_buffer(ctx, F, c.width * copies, B, scratch);
     if (attention_bytes) attn_scratch = new llava_buffer(ctx, F, u32((attention_bytes + 3) / 4), 1, scratch);
+    if (mix_bytes) mix_scratch = new llava_buffer(ctx, F, u32((mix_bytes + 3) / 4), 1, scratch);
+    if (c.rotation_pairs()) angles = new llava_buffer(ctx, F, 2 * c.rotation_pairs(), B, scratch);
     for (const hybrid_layer_spec& l : c.layers) {
         const hybrid_experts& e = l.mlp;
         if (f32 || e.experts == 0) {
@@ -147,13 +198,14 @@ void hybrid_session_state::dump_frame(int fd) {
     if (scratch) scratch->dump_buffers(fd, "step");
 }
 
-// Per layer run: the first n rows of every key head, then of every value head, or the recurrent state; then the histories.
+// Per layer run: the first n rows of every key head, then of every value head, or of the latent cache, or the recurrent state; then
+// the histories.
 size_t hybrid_session_state::snapshot_bytes(u32 n) const {
     size_t total = 0;
     for (const hybrid_run_state& s : runs) {
-        for (const llava_buffer* b : {s.k_cache, s.v_cache})
+        for (const llava_buffer* b : {s.k_cache, s.v_cache, s.latent_cache})
             if (b) total += size_t(b->shape.first / session->max_context) * n * b->shape.second * cache_bytes();
-        for (const llava_buffer* b : {s.gru_state, s.history1, s.history2})
+        for (const llava_buffer* b : {s.gru_state, s.ssm_state, s.conv_history, s.history1, s.history2})
             if (b) total += b->byte_size();
     }
     return total;
@@ -167,12 +219,12 @@ bool hybrid_session_state::transfer(u8* dst, const u8* src, u32 n) {
         at += bytes;
     };
     for (hybrid_run_state& s : runs) {
-        for (llava_buffer* b : {s.k_cache, s.v_cache}) {
+        for (llava_buffer* b : {s.k_cache, s.v_cache, s.latent_cache}) {
             if (b == nullptr) continue;
             const size_t row = size_t(b->shape.second) * cache_bytes();
             for (u32 g = 0; g < b->shape.first / session->max_context; ++g) move(b, size_t(g) * session->max_context * row, n * row);
         }
-        for (llava_buffer* b : {s.gru_state, s.history1, s.history2})
+        for (llava_buffer* b : {s.gru_state, s.ssm_state, s.conv_history, s.history1, s.history2})
             if (b) move(b, 0, b->byte_size());
     }
     return ok;

@@ -142,6 +142,7 @@ bool llava_session::recreate_buffers() {
     sampler_state_dirty = true;
     if (!m->freeze() || !m->zero(0, m->get_size())) return false;
     device_pos = ~0U;
+    token_log_complete = false;
     if (!state && ctx->architecture()->has_session_state()) state = ctx->architecture()->make_session_state(this);
     return !state || state->resize();
 }
@@ -210,6 +211,11 @@ llava_command_buffer* llava_session::get_command_buffer(u32 batch, bool with_hea
 }
 
 bool llava_session::upload_pending_tokens(u32 first, u32 count) {
+    if (!token_log_complete) {          // a new log (other options, a restored session): the evaluated tokens as well
+        count += first;
+        first = 0;
+        token_log_complete = true;
+    }
     memcpy(pinned + first, token_buffer.data() + first, size_t(count) * 4);
     return lv_upload_async(ctx->lv(), static_cast<u32*>(token_log->device_ptr()) + first, pinned + first, size_t(count) * 4) == LV_OK;
 }
@@ -647,5 +653,6 @@ ReturnCode llava_session::restore(const string& path) {
     ::close(fd);
     token_buffer = toks;
     current_tokens_in_gpu = n;
+    token_log_complete = false;
     return ReturnCode::ok;
 }

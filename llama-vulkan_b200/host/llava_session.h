@@ -164,6 +164,7 @@ private:
     u32 device_pos = ~0U;         // value of config_buffer on the device as far as the host knows
     u32* pinned = nullptr;        // [max_context] token staging + [8] config/argmax words
     bool upload_pending_tokens(u32 first, u32 count);
+    bool token_log_complete = false;   // the device's token log holds every evaluated token (steps may read earlier ones)
     bool sync_device_position(u32 pos);
 
     // one-launch token step (lv_decode_step): weights of the context + caches of this session; null when

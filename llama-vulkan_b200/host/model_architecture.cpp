@@ -13,6 +13,7 @@ struct entry {
 const entry kRegistry[] = {
     {"ggjt", []() -> unique_ptr<model_architecture> { return make_unique<llama_architecture>(); }},
     {"Sonuzen", []() -> unique_ptr<model_architecture> { return make_unique<hybrid_architecture>("Sonuzen", parse_sonuzen_config); }},
+    {"Nuforax", []() -> unique_ptr<model_architecture> { return make_unique<hybrid_architecture>("Nuforax", parse_nuforax_config); }},
 };
 }  // namespace
 

@@ -81,7 +81,7 @@ def test_gemv_bf16_is_exact_in_f32(gpu, rows, cols, batch):
     w, x = weights(rng, rows, cols), rng.standard_normal((batch, pad8(cols))).astype(np.float32)
     with Dev(gpu) as d:
         out = d.zeros(batch * rows * 4)
-        d.call("lv_gemv_bf16", out, rows, d.bf16(w), rows, pad8(cols), cols, d.f32(x), pad8(cols), batch, 0.75)
+        d.call("lv_gemv_bf16", out, rows, d.bf16(w), rows, pad8(cols), cols, d.f32(x), pad8(cols), batch, 0.75, 0)
         got = d.get(out, (batch, rows))
     want = 0.75 * x[:, :cols].astype(np.float64) @ w.T.astype(np.float64)
     assert rel(got, want) < 1e-6
@@ -95,7 +95,7 @@ def test_gemm_bf16(gpu, rows, cols, batch, out_bf16):
     w, x = weights(rng, rows, cols), weights(rng, batch, cols, scale=1.0)
     with Dev(gpu) as d:
         out = d.zeros(batch * rows * 4)
-        d.call("lv_gemm_bf16", out, pkg.TYPE_BF16 if out_bf16 else pkg.TYPE_F32, rows, d.bf16(w), rows, pad8(cols), cols, d.bf16(x), pad8(cols), batch, 0.5)
+        d.call("lv_gemm_bf16", out, pkg.TYPE_BF16 if out_bf16 else pkg.TYPE_F32, rows, d.bf16(w), rows, pad8(cols), cols, d.bf16(x), pad8(cols), batch, 0.5, 0)
         got = d.get(out, (batch, rows), out_bf16)
     want = 0.5 * x.astype(np.float64) @ w.T.astype(np.float64)
     assert rel(got, want) < (3e-3 if out_bf16 else 2e-5)
@@ -259,7 +259,7 @@ def test_min_gru_steps_and_scan(gpu, width, channels, cuts):
                 d.call("lv_gemv_bf16_mingru", out, dw, pkg.offset(dw, each), pkg.offset(dw, 2 * each), ld, channels, width, dbz, dbx, x, state, pos)
             else:
                 raw = d.zeros(n * 3 * channels * 4)
-                d.call("lv_gemv_bf16", raw, 3 * channels, dw, 3 * channels, ld, width, x, ld, n, 1.0)
+                d.call("lv_gemv_bf16", raw, 3 * channels, dw, 3 * channels, ld, width, x, ld, n, 1.0, 0)
                 d.call("lv_mingru_scan", out, pkg.TYPE_F32, pad8(channels), raw, 3 * channels, channels, dbz, dbx, state, pos, n)
             assert rel(d.get(out, (n, pad8(channels)))[:, :channels], want[at:at + n]) < 1e-5
             at += n
@@ -382,8 +382,8 @@ def test_bad_arguments_are_refused(gpu):
     bad = pkg.LV_ERR_BAD_ARGUMENTS
     with Dev(gpu) as d:
         b = d.zeros(1 << 16)
-        assert lib.lv_gemm_bf16(h, b, pkg.TYPE_F32, 8, b, 8, 12, 12, b, 16, 2, 1.0) == bad          # ld not a multiple of 8
-        assert lib.lv_gemv_bf16(h, b, 4, b, 8, 16, 16, b, 16, 1, 1.0) == bad                        # out_ld below the rows
+        assert lib.lv_gemm_bf16(h, b, pkg.TYPE_F32, 8, b, 8, 12, 12, b, 16, 2, 1.0, 0) == bad          # ld not a multiple of 8
+        assert lib.lv_gemv_bf16(h, b, 4, b, 8, 16, 16, b, 16, 1, 1.0, 0) == bad                        # out_ld below the rows
         a = pkg.NormConvArgs(pos=b.value, pre_w=b.value, out=b.value, width=8, batch=1, out_type=pkg.TYPE_F32)
         assert lib.lv_norm_conv(h, C.byref(a)) == bad                                               # no stream
         g = pkg.GqaArgs(qkv=b.value, qkv_ld=4096, heads=3, kv_heads=2, dim=16, vdim=16)
