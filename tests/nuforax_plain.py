@@ -103,8 +103,9 @@ def relu_squared(z):
 # ---- the model -----------------------------------------------------------------------------
 
 class Plain:
-    def __init__(self, config, tensors, dtype=np.float64):
-        self.c, self.dtype = config, dtype
+    def __init__(self, config, tensors, dtype=np.float64, operands=lambda a: a):
+        """operands: applied to what enters a matrix product and to what a cache holds (rounding, to see what it causes)."""
+        self.c, self.dtype, self.op = config, dtype, operands
         self.w = {k: (a if np.issubdtype(a.dtype, np.integer) else a.astype(dtype)) for k, a in tensors.items()}
         self.eps = config["norm"]["eps"]
 
@@ -121,16 +122,17 @@ class Plain:
 
     def attention(self, i, h, kept):
         w, m, p = self.w, self.c["layers"][i]["mixer"], f"l{i}.mix."
-        T, H, pos = h.shape[0], m["heads"], np.arange(h.shape[0]).astype(self.dtype)
+        op, T, H, pos = self.op, h.shape[0], m["heads"], np.arange(h.shape[0]).astype(self.dtype)
         freqs, mult = yarn(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
         freqs = freqs.astype(self.dtype)
         q = (h @ w[p + "q"].T).reshape(T, H, m["dim"] + m["rot_dim"])
         q = np.concatenate([q[..., :m["dim"]], rotate(q[..., m["dim"]:], pos, freqs, mult)], axis=-1)
         if m.get("kv_from") is None:
             d = h @ w[p + "dkv"].T
-            kept[i] = norm_plain(d[:, :m["kv_rank"]], w[p + "dkv.norm"], self.eps), rotate(d[:, m["kv_rank"]:], pos, freqs, mult)
+            kept[i] = op(norm_plain(d[:, :m["kv_rank"]], w[p + "dkv.norm"], self.eps)), op(rotate(d[:, m["kv_rank"]:], pos, freqs, mult))
         c, k_rot = kept[m.get("kv_from") if m.get("kv_from") is not None else i]
-        return latent_attention(q, c, k_rot, w[p + "uk"], w[p + "uv"], w[p + "sink"], m["scale"], m["mask"]["size"]) @ w[p + "o"].T
+        y = latent_attention(op(q), c, k_rot, w[p + "uk"], w[p + "uv"], w[p + "sink"], m["scale"], m["mask"]["size"])
+        return op(y) @ w[p + "o"].T
 
     def mamba2(self, i, h):
         w, m, p = self.w, self.c["layers"][i]["mixer"], f"l{i}.mix."
@@ -140,14 +142,15 @@ class Plain:
         xbc = silu(causal_conv(xbc, w[p + "conv"]) + w[p + "conv.b"])
         x, B, C = np.split(xbc, [inner, inner + G * N], axis=1)
         y = state_space(x.reshape(T, H, P), B.reshape(T, G, N), C.reshape(T, G, N), softplus(dt + w[p + "dt_bias"]), w[p + "A_log"], w[p + "D"])
-        return gated_group_norm(y.reshape(T, inner), z, w[p + "norm"], m["norm_groups"], self.eps) @ w[p + "o"].T
+        return self.op(gated_group_norm(y.reshape(T, inner), z, w[p + "norm"], m["norm_groups"], self.eps)) @ w[p + "o"].T
 
     def layer(self, i, x, kept):
         w, spec = self.w, self.c["layers"][i]
-        y = self.attention(i, x, kept) if spec["type"] == "latent_attention" else self.mamba2(i, x)
+        h = self.op(x)
+        y = self.attention(i, h, kept) if spec["type"] == "latent_attention" else self.mamba2(i, h)
         x = x + norm_plain(y, w[f"l{i}.norm1"], self.eps)
         if spec["mlp"] is not None:
-            y = relu_squared(x @ w[f"l{i}.mlp.up"].T) @ w[f"l{i}.mlp.down"].T
+            y = self.op(relu_squared(self.op(x) @ w[f"l{i}.mlp.up"].T)) @ w[f"l{i}.mlp.down"].T
             x = x + norm_plain(y, w[f"l{i}.norm2"], self.eps)
         return x
 
@@ -158,4 +161,4 @@ class Plain:
             x = self.layer(i, x, kept)
             if layers is not None:
                 layers.append(x.copy())
-        return norm_plain(x, self.w["final.norm"], self.eps) @ self.w["embed"].T
+        return self.op(norm_plain(x, self.w["final.norm"], self.eps)) @ self.w["embed"].T

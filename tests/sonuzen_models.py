@@ -95,3 +95,7 @@ def distance(got, want):
     d -= d.mean(axis=-1, keepdims=True)
     w = want - want.mean(axis=-1, keepdims=True)
     return np.sqrt((d ** 2).mean(axis=-1) / (w ** 2).mean())
+
+
+def plain(cfg, t):
+    return sp.Plain(cfg, t)

@@ -11,58 +11,15 @@ import pytest
 import sonuzen_models as sm
 import sonuzen_plain as sp
 from conftest import ROOT, load_pkg
+from hybrid_harness import LIMIT, Model, cached_models, feed, frame_records, greedy
 
 pytestmark = pytest.mark.gpu
 pkg = load_pkg()
-LIMIT = {"float32": 3e-5, "bfloat16": 3e-2}
-
-
-class Model:
-    def __init__(self, folder, name, seed=1):
-        self.path = str(folder)
-        self.cfg, t = sm.write(self.path, name, seed)
-        self.vocab = self.cfg["vocab"]
-        self.plain = sp.Plain(self.cfg, t)
-        self.open = {}
-
-    def ctx(self, dtype):
-        if dtype not in self.open:
-            self.open[dtype] = pkg.HostContext(self.path, 0, dtype=dtype)
-        return self.open[dtype]
-
-    def tokens(self, n, seed=0):
-        return [int(x) for x in np.random.default_rng(seed).integers(0, self.vocab, n)]
-
-    def session(self, dtype, max_context=0):
-        s = self.ctx(dtype).session(max_context)
-        s.set_deterministic(True)
-        return s
 
 
 @pytest.fixture(scope="module")
 def models(tmp_path_factory):
-    made = {}
-
-    def get(name):
-        if name not in made:
-            made[name] = Model(tmp_path_factory.mktemp(name), name)
-        return made[name]
-    yield get
-    for m in made.values():
-        for c in m.open.values():
-            c.close()
-
-
-def feed(s, m, tokens, cuts):
-    """Evaluates `tokens` in portions; logits of every token."""
-    out, at = [], 0
-    for n in cuts:
-        for t in tokens[at:at + n]:
-            assert s.push_token(t)
-        out.append(s.evaluate_pending(range(at, at + n), m.vocab))
-        at += n
-    assert at == len(tokens)
-    return np.concatenate(out)
+    yield from cached_models(sm, tmp_path_factory)
 
 
 CUTS = {"whole": [150], "token by token": [1] * 150, "pairs": [2] * 75, "sizes": [1, 2, 3, 61, 1, 1, 2, 64, 5, 10], "prompt and decoding": [131] + [1] * 19}
@@ -143,17 +100,6 @@ def test_rewound_sessions_start_over(models, dtype):
     s.close()
 
 
-def greedy(plain, prompt, n):
-    """Greedy tokens of the plain implementation and how far each winner is ahead of the runner-up."""
-    tokens, lead = list(prompt), []
-    for _ in range(n):
-        z = plain.forward(tokens)[-1]
-        top = np.sort(z)[-2:]
-        lead.append((top[1] - top[0]) / np.abs(z).max())
-        tokens.append(int(z.argmax()))
-    return tokens[len(prompt):], min(lead)
-
-
 def test_greedy_generation_three_ways(models):
     m = models("no_loop")
     prompt = m.tokens(23, 8)
@@ -209,7 +155,7 @@ def test_long_decoding(models, dtype):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_a_session_longer_than_the_default(tmp_path, dtype):
     cfg = sm.config(64, 40, [sm.attention(4, 2, 32, 32, mlp=sm.moe(32, 2, 1)), sm.mingru(32)], taps=4)
-    m = Model(tmp_path, cfg)
+    m = Model(tmp_path, cfg, sm)
     tokens = m.tokens(2500)
     want = m.plain.forward(tokens)
     s = m.session(dtype, 2600)
@@ -223,7 +169,7 @@ def test_a_session_longer_than_the_default(tmp_path, dtype):
         assert s.push_token(t)
     assert not s.push_token(tokens[2048])
     s.close()
-    m.open[dtype].close()
+    m.close()
 
 
 def test_sampled_generation_is_reproducible(models):
@@ -280,13 +226,7 @@ def test_frames_hold_the_stream_after_every_layer_run(models, dtype, n, tmp_path
     path = str(tmp_path / "frame")
     assert s.save_frame(path) == 0
     s.close()
-    data, at, seen = open(path, "rb").read(), 0, []
-    while at < len(data):
-        cols, rows, _ = struct.unpack_from("<III", data, at)
-        name = data[at + 12:data.index(b"\0", at + 12)].decode()
-        at += (12 + len(name) + 1 + 31) & ~31
-        seen.append((name, np.frombuffer(data, np.float32, cols * rows, at).reshape(rows, cols)))
-        at += 4 * cols * rows
+    seen = frame_records(path)
     assert [k for k, _ in seen] == [f"step.run.{i:04d}.residual" for i in range(len(layers))]
     for (name, got), want in zip(seen, layers):
         err = np.linalg.norm(got[:n] - want) / np.linalg.norm(want)
