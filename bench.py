@@ -658,8 +658,8 @@ def main():
     ap.add_argument("--steps", type=int, default=256)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="7b-q4_0", choices=sorted(WORKLOADS) + ["sonuzen-1024", "sonuzen-2048", "sonuzen-4096"],
-                    help="sonuzen-*: that design beside LLaMA models of equal size on one GPU (bench_sonuzen.py)")
+    ap.add_argument("--workload", default="7b-q4_0", choices=sorted(WORKLOADS) + [f"{d}-{n}" for d in ("sonuzen", "nuforax") for n in (1024, 2048, 4096)],
+                    help="sonuzen-*: that design beside LLaMA models of equal size, nuforax-*: that design beside Sonuzen models, on one GPU (bench_<design>.py)")
     ap.add_argument("--repeats", type=int, default=5, help="timed regions per figure; the median is reported")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-parity", action="store_true", help="skip the oracle comparison that precedes the timed runs")
@@ -682,14 +682,15 @@ def main():
         return run_reference(args, rank, world)
 
     pkg = load_pkg()
-    if args.workload.startswith("sonuzen-"):
-        import bench_sonuzen
+    design = args.workload.split("-")[0]
+    if design in ("sonuzen", "nuforax"):
+        import importlib
         if world != 1:
-            raise SystemExit("sonuzen workloads run on one GPU")
+            raise SystemExit(f"{design} workloads run on one GPU")
         peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}           # used when nothing was measured
         if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
             peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
-        return bench_sonuzen.run(pkg, args, MODEL_DIR, peaks, ClockSampler(0), RESULT_OUT)
+        return importlib.import_module(f"bench_{design}").run(pkg, args, MODEL_DIR, peaks, ClockSampler(0), RESULT_OUT)
     w = WORKLOADS[args.workload]
     dim, heads, ff, n_layers = model_geometry(pkg, w)
     n_prompt = w["prompt"]

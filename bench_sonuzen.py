@@ -14,13 +14,16 @@ import time
 
 import numpy as np
 
+import bench_models
+from bench_models import CONTEXT, STEP, VOCAB
+
 SIZES = {
     # width, query heads of 128, key/value heads, recurrent width, experts, expert width, experts of a token, layers
     "sonuzen-1024": dict(width=1024, heads=8, kv_heads=2, gru=1536, experts=16, ff=512, top=4, layers=8),
     "sonuzen-2048": dict(width=2048, heads=16, kv_heads=4, gru=2560, experts=16, ff=1408, top=4, layers=8),
     "sonuzen-4096": dict(width=4096, heads=32, kv_heads=8, gru=4096, experts=8, ff=5504, top=2, layers=4),
 }
-VOCAB, DIM, TAPS, CONTEXT, PROMPT, STEP = 32000, 128, 4, 1024, 2048, 512
+DIM, TAPS = 128, 4
 
 
 def config(z):
@@ -55,32 +58,8 @@ def write_folder(path, z):
             shapes[f"{p}mlp.e{e}.gate"] = shapes[f"{p}mlp.e{e}.up"] = (z["ff"], W)
             shapes[f"{p}mlp.e{e}.down"] = (W, z["ff"])
         shapes[p + "mlp.table"] = (VOCAB, z["top"])
-    head, at = {}, 0
-    for name, s in shapes.items():
-        table = name.endswith("table")
-        n = int(np.prod(s)) * (4 if table else 2)
-        head[name] = {"dtype": "I32" if table else "BF16", "shape": list(s), "data_offsets": [at, at + n]}
-        at += n
-    text = json.dumps(head).encode()
-    slab = (rng.standard_normal(1 << 22).astype(np.float32) * 0.02).view(np.uint32) >> 16
-    slab = slab.astype(np.uint16)
-    os.makedirs(path, exist_ok=True)
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(cfg, f)
-    with open(os.path.join(path, "model.safetensors"), "wb") as f:
-        f.write(len(text).to_bytes(8, "little") + text)
-        for name, s in shapes.items():
-            n = int(np.prod(s))
-            if name.endswith("table"):
-                t = rng.random((s[0], z["experts"])).argsort(axis=1)[:, :z["top"]].astype(np.int32)
-                f.write(t.tobytes())
-                continue
-            off = int(rng.integers(0, 1 << 20))
-            while n:
-                k = min(n, slab.size - off)
-                f.write(slab[off:off + k].tobytes())
-                n -= k
-                off = 0
+    tables = {n: rng.random((VOCAB, z["experts"])).argsort(axis=1)[:, :z["top"]] for n in shapes if n.endswith("table")}
+    bench_models.write_folder(path, cfg, shapes, tables)
 
 
 def active_bytes(z, layers):
@@ -95,62 +74,12 @@ def active_bytes(z, layers):
     return total
 
 
-class Timer:
-    def __init__(self, pkg, gpu, torch):
-        self.pkg, self.gpu, self.torch, self.lib, self.h = pkg, gpu, torch, gpu.lib, gpu.handle
-        self.stream = torch.cuda.ExternalStream(self.lib.lv_ctx_stream(self.h), device=0)
-
-    def __call__(self, launch, iters=40):
-        """Seconds per launch; launch(i) enqueues the i-th one."""
-        pkg, lib, h, torch = self.pkg, self.lib, self.h, self.torch
-        for i in range(3):
-            launch(i)
-        self.gpu.sync()
-        graph = C.c_void_p()
-        pkg.check(lib.lv_graph_begin_capture(h))
-        for i in range(iters):
-            launch(i)
-        pkg.check(lib.lv_graph_end_capture(h, C.byref(graph)))
-        best = []
-        for _ in range(4):
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record(self.stream)
-            pkg.check(lib.lv_graph_launch(h, graph))
-            e1.record(self.stream)
-            self.gpu.sync()
-            best.append(e0.elapsed_time(e1) * 1e-3 / iters)
-        pkg.check(lib.lv_graph_destroy(graph))
-        return sorted(best[1:])[1]
-
-
-def kernel_times(pkg, torch, z, peaks):
-    """Every kernel of a layer alone, new design and its LLaMA counterpart of equal size -> list of rows."""
-    hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+def kernel_times(pkg, torch, z, peaks, llama=True):
+    """Every kernel of a layer alone and, with `llama`, its LLaMA counterpart of equal size -> list of rows."""
     W, H, G, gru, ff, top, E = z["width"], z["heads"], z["kv_heads"], z["gru"], z["ff"], z["top"], z["experts"]
-    rows = []
     with pkg.Context(0) as gpu:
-        lib, h = gpu.lib, gpu.handle
-        t = Timer(pkg, gpu, torch)
-        rng = np.random.default_rng(3)
-
-        def ring(nbytes):
-            """copies of a random block of nbytes, more than 400 MB together"""
-            n = max(3, int(400e6 // nbytes) + 1)
-            stride = (nbytes + 255) // 256 * 256
-            d = gpu.alloc(n * stride)
-            slab = ((rng.standard_normal(1 << 20).astype(np.float32) * 0.02).view(np.uint32) >> 16).astype(np.uint16)
-            host = np.resize(slab, nbytes // 2 + 1)
-            for i in range(n):
-                pkg.check(lib.lv_upload(h, pkg.offset(d, i * stride), host.ctypes.data_as(C.c_void_p), nbytes))
-            return lambda i: pkg.offset(d, (i % n) * stride), d
-
-        def add(model, phase, name, sec, nbytes, flops=0.0):
-            roof = max(nbytes / hbm, flops / tflops)
-            rows.append({"model": model, "phase": phase, "kernel": name, "us": round(sec * 1e6, 2), "GB/s": round(nbytes / sec / 1e9),
-                         "TFLOP/s": round(flops / sec / 1e12, 1), "frac": round(roof / sec, 3)})
-
-        f32 = lambda *s: gpu.upload(rng.standard_normal(s).astype(np.float32))
-        b16 = lambda *s: gpu.upload(((rng.standard_normal(s).astype(np.float32)).view(np.uint32) >> 16).astype(np.uint16))
+        bench = bench_models.Kernels(pkg, torch, gpu, peaks)
+        lib, h, rng, ring, f32, b16, add = bench.lib, bench.h, bench.rng, bench.ring, bench.f32, bench.b16, bench.add
         pos = gpu.upload(np.array([CONTEXT - 1] * 4, np.uint32))
         pos_prompt = gpu.upload(np.array([CONTEXT - STEP] * 4, np.uint32))
         zero = gpu.upload(np.zeros(4, np.uint32))
@@ -162,20 +91,20 @@ def kernel_times(pkg, torch, z, peaks):
         out = gpu.zeros(max(STEP * top * max(W, raw_n, 3 * gru, ff), STEP * VOCAB // 8) * 4)
         for name, r, k in (("input projections (attention)", raw_n, W), ("output projection (attention)", W, H * DIM), ("output projection (recurrent)", W, gru)):
             w, d = ring(r * k * 2)
-            add("sonuzen", "decode", name, t(lambda i: pkg.check(lib.lv_gemv_bf16(h, out, r, w(i), r, k, k, x1, k, 1, 1.0, 0))), r * k * 2)
-            add("sonuzen", f"prompt of {STEP}", name, t(lambda i: pkg.check(lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, r, w(i), r, k, k, xT, k, STEP, 1.0, 0))),
+            add("sonuzen", "decode", name, lambda i: lib.lv_gemv_bf16(h, out, r, w(i), r, k, k, x1, k, 1, 1.0, 0), r * k * 2)
+            add("sonuzen", f"prompt of {STEP}", name, lambda i: lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, r, w(i), r, k, k, xT, k, STEP, 1.0, 0),
                 r * k * 2 + STEP * (k * 2 + r * 4), 2.0 * r * k * STEP)
             gpu.free(d)
         w, d = ring(3 * gru * W * 2)
         bias, state = f32(gru), f32(gru)
         each = gru * W * 2
-        add("sonuzen", "decode", "input projections + recurrence", t(lambda i: pkg.check(lib.lv_gemv_bf16_mingru(
-            h, out, w(i), pkg.offset(w(i), each), pkg.offset(w(i), 2 * each), W, gru, W, bias, bias, x1, state, pos))), 3 * each)
-        add("sonuzen", f"prompt of {STEP}", "input projections (recurrent)", t(lambda i: pkg.check(lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, 3 * gru, w(i), 3 * gru, W, W, xT, W, STEP, 1.0, 0))),
+        add("sonuzen", "decode", "input projections + recurrence", lambda i: lib.lv_gemv_bf16_mingru(
+            h, out, w(i), pkg.offset(w(i), each), pkg.offset(w(i), 2 * each), W, gru, W, bias, bias, x1, state, pos), 3 * each)
+        add("sonuzen", f"prompt of {STEP}", "input projections (recurrent)", lambda i: lib.lv_gemm_bf16(h, out, pkg.TYPE_F32, 3 * gru, w(i), 3 * gru, W, W, xT, W, STEP, 1.0, 0),
             3 * each + STEP * (W * 2 + 3 * gru * 4), 6.0 * gru * W * STEP)
         gpu.free(d)
         w, d = ring(VOCAB * W * 2)
-        add("sonuzen", "decode", "output head", t(lambda i: pkg.check(lib.lv_gemv_bf16(h, out, VOCAB, w(i), VOCAB, W, W, x1, W, 1, 1.0, 0))), VOCAB * W * 2)
+        add("sonuzen", "decode", "output head", lambda i: lib.lv_gemv_bf16(h, out, VOCAB, w(i), VOCAB, W, W, x1, W, 1, 1.0, 0), VOCAB * W * 2)
         gpu.free(d)
         # -- experts -------------------------------------------------------------------------
         w, d = ring(E * ff * W * 2 * 3)
@@ -189,17 +118,17 @@ def kernel_times(pkg, torch, z, peaks):
                 a.w0, a.w1, a.ld, a.rows, a.cols = w(i).value, pkg.offset(w(i), mat).value, W, ff, W
             return C.byref(a)
         act = f32(top, ff)
-        add("sonuzen", "decode", "expert gate/up + SiLU", t(lambda i: pkg.check(lib.lv_gemv_bf16_expert_gate_up(h, out, ff, expert(i, 0), x1, W, 1))), 2 * top * ff * W * 2)
-        add("sonuzen", "decode", "expert down", t(lambda i: pkg.check(lib.lv_gemv_bf16_expert_down(h, out, W, expert(i, 1), act, ff, 1))), top * ff * W * 2)
+        add("sonuzen", "decode", "expert gate/up + SiLU", lambda i: lib.lv_gemv_bf16_expert_gate_up(h, out, ff, expert(i, 0), x1, W, 1), 2 * top * ff * W * 2)
+        add("sonuzen", "decode", "expert down", lambda i: lib.lv_gemv_bf16_expert_down(h, out, W, expert(i, 1), act, ff, 1), top * ff * W * 2)
         max_tiles = lib.lv_expert_max_tiles(STEP, top, E)
         index, tiles = gpu.zeros(STEP * top * 4), gpu.zeros(max_tiles * 12)
         job = np.zeros(1, np.dtype([("table", "u8"), ("experts", "u4"), ("top", "u4"), ("index", "u8"), ("tiles", "u8"), ("max_tiles", "u4"), ("unused", "u4")]))
         job[0] = (table.value, E, top, index.value, tiles.value, max_tiles, 0)
         dj = gpu.upload(job)
-        add("sonuzen", f"prompt of {STEP}", "expert routing", t(lambda i: pkg.check(lib.lv_expert_route(h, dj, 1, E, ids, zero, VOCAB, STEP))), STEP * top * 12)
-        add("sonuzen", f"prompt of {STEP}", "expert gate/up + SiLU", t(lambda i: pkg.check(lib.lv_gemm_bf16_expert_gate_up(h, out, ff, expert(i, 0), tiles, xT, W, STEP))),
+        add("sonuzen", f"prompt of {STEP}", "expert routing", lambda i: lib.lv_expert_route(h, dj, 1, E, ids, zero, VOCAB, STEP), STEP * top * 12)
+        add("sonuzen", f"prompt of {STEP}", "expert gate/up + SiLU", lambda i: lib.lv_gemm_bf16_expert_gate_up(h, out, ff, expert(i, 0), tiles, xT, W, STEP),
             2 * mat + STEP * top * (W + ff) * 2, 4.0 * STEP * top * ff * W)
-        add("sonuzen", f"prompt of {STEP}", "expert down", t(lambda i: pkg.check(lib.lv_gemm_bf16_expert_down(h, out, W, expert(i, 1), tiles, xT, ff, STEP))),
+        add("sonuzen", f"prompt of {STEP}", "expert down", lambda i: lib.lv_gemm_bf16_expert_down(h, out, W, expert(i, 1), tiles, xT, ff, STEP),
             mat + STEP * top * (ff * 2 + W * 4), 2.0 * STEP * top * ff * W)
         gpu.free(d)
         # -- norm / residual / convolution ------------------------------------------------------
@@ -211,9 +140,9 @@ def kernel_times(pkg, torch, z, peaks):
                                  post_w=vec.value, x_out=xb.value, row_factor=factor.value, pre_w=vec.value, conv_w=conv.value, history=hist.value, taps=TAPS, out=out.value,
                                  out_type=pkg.TYPE_F32 if n == 1 else pkg.TYPE_BF16, out_ld=W, width=W, batch=n)
             return C.byref(a)
-        add("sonuzen", "decode", "norm, residual, norm, convolution", t(lambda i: pkg.check(lib.lv_norm_conv(h, nc(1, 1)))), (4 * W + 2 * TAPS * W + 4 * W) * 4)
-        add("sonuzen", f"prompt of {STEP}", "norm, residual, norm, convolution", t(lambda i: pkg.check(lib.lv_norm_conv(h, nc(STEP, 1)))), STEP * W * 14)
-        add("sonuzen", f"prompt of {STEP}", "the same after experts", t(lambda i: pkg.check(lib.lv_norm_conv(h, nc(STEP, top)))), STEP * W * (10 + 4 * top))
+        add("sonuzen", "decode", "norm, residual, norm, convolution", lambda i: lib.lv_norm_conv(h, nc(1, 1)), (4 * W + 2 * TAPS * W + 4 * W) * 4)
+        add("sonuzen", f"prompt of {STEP}", "norm, residual, norm, convolution", lambda i: lib.lv_norm_conv(h, nc(STEP, 1)), STEP * W * 14)
+        add("sonuzen", f"prompt of {STEP}", "the same after experts", lambda i: lib.lv_norm_conv(h, nc(STEP, top)), STEP * W * (10 + 4 * top))
         # -- attention and recurrence over a prompt ------------------------------------------------
         kc, vc = b16(G * 2048, DIM), b16(G * 2048, DIM)
         hv, qn = f32(H), f32(DIM)
@@ -227,13 +156,15 @@ def kernel_times(pkg, torch, z, peaks):
         habs = gpu.upload(np.abs(rng.standard_normal(H)).astype(np.float32) * 0.3)
         nbytes = lib.lv_gqa_scratch_bytes(h, C.byref(gqa(1)), STEP, 2048)
         scratch = gpu.zeros(nbytes)
-        add("sonuzen", "decode", f"attention, {CONTEXT} keys", t(lambda i: pkg.check(lib.lv_attention_gqa(h, C.byref(gqa(1)), scratch, nbytes, 1, CONTEXT, 1))), 2 * CONTEXT * G * DIM * 2)
-        add("sonuzen", f"prompt of {STEP}", "key norm + append", t(lambda i: pkg.check(lib.lv_qk_norm_append(h, C.byref(gqa(STEP)), STEP))), STEP * 2 * G * DIM * 6)
+        add("sonuzen", "decode", f"attention, {CONTEXT} keys", lambda i: lib.lv_attention_gqa(h, C.byref(gqa(1)), scratch, nbytes, 1, CONTEXT, 1), 2 * CONTEXT * G * DIM * 2)
+        add("sonuzen", f"prompt of {STEP}", "key norm + append", lambda i: lib.lv_qk_norm_append(h, C.byref(gqa(STEP)), STEP), STEP * 2 * G * DIM * 6)
         pairs = STEP * (CONTEXT - STEP) + STEP * STEP / 2
-        add("sonuzen", f"prompt of {STEP}", f"attention, {CONTEXT} keys", t(lambda i: pkg.check(lib.lv_attention_gqa(h, C.byref(gqa(STEP)), scratch, nbytes, STEP, CONTEXT, 0))),
+        add("sonuzen", f"prompt of {STEP}", f"attention, {CONTEXT} keys", lambda i: lib.lv_attention_gqa(h, C.byref(gqa(STEP)), scratch, nbytes, STEP, CONTEXT, 0),
             2 * CONTEXT * G * DIM * 2 + STEP * H * DIM * 6, 4.0 * DIM * H * pairs)
         rawz = f32(STEP, 3 * gru)
-        add("sonuzen", f"prompt of {STEP}", "recurrence scan", t(lambda i: pkg.check(lib.lv_mingru_scan(h, out, pkg.TYPE_BF16, gru, rawz, 3 * gru, gru, bias, bias, state, pos, STEP))), STEP * gru * 14)
+        add("sonuzen", f"prompt of {STEP}", "recurrence scan", lambda i: lib.lv_mingru_scan(h, out, pkg.TYPE_BF16, gru, rawz, 3 * gru, gru, bias, bias, state, pos, STEP), STEP * gru * 14)
+        if not llama:
+            return bench.rows
         # -- LLaMA of equal size ----------------------------------------------------------------
         act_ff = ff * top
         llama_ff = (act_ff + 255) // 256 * 256
@@ -266,74 +197,18 @@ def kernel_times(pkg, torch, z, peaks):
                 else:
                     one = lambda i: lib.lv_gemv(h, out, w(i), wt, x64, r, k, 1, 1)
                     many = lambda i: lib.lv_gemm_tc(h, out, w(i), wt, split, r, k, 64, 1)
-                add(name, "decode", label, t(lambda i: pkg.check(one(i))), n * s)
+                add(name, "decode", label, lambda i: one(i), n * s)
                 if many:
                     pkg.check(lib.lv_act_split_f16(h, split, x64, None, k, 64))
-                    add(name, "prompt of 64", label, t(lambda i: pkg.check(many(i))), n * s + 64 * (k + n * r) * 4, 2.0 * n * r * k * 64)
+                    add(name, "prompt of 64", label, lambda i: many(i), n * s + 64 * (k + n * r) * 4, 2.0 * n * r * k * 64)
                 gpu.free(d)
-        add("llama", "decode", f"attention, {CONTEXT} keys", t(lambda i: pkg.check(lib.lv_attention_fused(h, out, x64, lk, lv_, pos, rope, lscratch, W // DIM, DIM, 1024, 1))), 2 * CONTEXT * W * 2)
+        add("llama", "decode", f"attention, {CONTEXT} keys", lambda i: lib.lv_attention_fused(h, out, x64, lk, lv_, pos, rope, lscratch, W // DIM, DIM, 1024, 1), 2 * CONTEXT * W * 2)
         pos64 = gpu.upload(np.array([CONTEXT - 64] * 4, np.uint32))
-        add("llama", "prompt of 64", f"attention, {CONTEXT} keys", t(lambda i: pkg.check(lib.lv_attention_fused(h, out, x64, lk, lv_, pos64, rope, lscratch, W // DIM, DIM, 1024, 64))),
+        add("llama", "prompt of 64", f"attention, {CONTEXT} keys", lambda i: lib.lv_attention_fused(h, out, x64, lk, lv_, pos64, rope, lscratch, W // DIM, DIM, 1024, 64),
             2 * CONTEXT * W * 2 + 64 * W * 8, 4.0 * W * 64 * (CONTEXT - 32))
-        add("llama", "decode", "norm", t(lambda i: pkg.check(lib.lv_norm_f32(h, out, x64, norm, W, 1))), 3 * W * 4)
-        add("llama", "prompt of 64", "norm + activation split", t(lambda i: pkg.check(lib.lv_act_split_f16(h, split, x64, norm, W, 64))), 64 * W * 8)
-    return rows
-
-
-def model_times(pkg, torch, path, max_context, prompt_step, args, kernels):
-    """Decoding and prompt throughput of one model."""
-    ctx = pkg.HostContext(path, 0)
-    lv = C.c_void_p(ctx.lib.llava_context_lv(ctx.handle))
-    stream = torch.cuda.ExternalStream(kernels.lv_ctx_stream(lv), device=0)
-    tokens = [int(x) for x in np.random.default_rng(4321).integers(3, VOCAB, PROMPT)]
-
-    def timed_prompt(n):
-        s = ctx.session(max_context)
-        s.set_deterministic(True)
-        assert s.set_max_batch(prompt_step)
-        best = []
-        for _ in range(4):                                        # the first pass records the steps
-            s.rewind(0)
-            for x in tokens[:n]:
-                assert s.push_token(x)
-            pkg.check(kernels.lv_stream_sync(lv, 0))
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record(stream)
-            assert s.start_next_token_prediction()
-            e1.record(stream)
-            tok = s.finish_next_token_prediction()
-            best.append(e0.elapsed_time(e1) * 1e-3)
-        return s, tok, sorted(best[1:])[1]
-
-    s, _, sec = timed_prompt(PROMPT if max_context > PROMPT else 1984)
-    s.close()
-    n_prompt = PROMPT if max_context > PROMPT else 1984
-    prompt = {"tokens": n_prompt, "step": prompt_step, "ms": sec * 1e3, "tokens_per_s": n_prompt / sec}
-    s, tok, _ = timed_prompt(CONTEXT - args.steps // 2 - args.warmup - 2)
-    assert s.push_token(tok)
-    s.generate_greedy_on_device(args.warmup)
-    runs = []
-    start = len(s.tokens())
-    e2e = []
-    for _ in range(3):
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        e0.record(stream)
-        s.enqueue_greedy_on_device(args.steps)
-        e1.record(stream)
-        s.collect_greedy_on_device()
-        runs.append(e0.elapsed_time(e1) * 1e-3 / args.steps)
-    launches = s.step_kernel_launches()
-    for _ in range(2):                                            # through the public calls, host in the loop
-        t0 = time.perf_counter()
-        for _ in range(args.steps):
-            tok = s.predict_next_token()
-            assert s.push_token(tok)
-        e2e.append((time.perf_counter() - t0) / args.steps)
-    sec = sorted(runs)[1]
-    decode = {"context": [start, start + 3 * args.steps], "ms_per_token": sec * 1e3, "tokens_per_s": 1 / sec, "e2e_tokens_per_s": 1 / min(e2e), "launches_per_token": launches}
-    s.close()
-    ctx.close()
-    return {"prompt": prompt, "decode": decode}
+        add("llama", "decode", "norm", lambda i: lib.lv_norm_f32(h, out, x64, norm, W, 1), 3 * W * 4)
+        add("llama", "prompt of 64", "norm + activation split", lambda i: lib.lv_act_split_f16(h, split, x64, norm, W, 64), 64 * W * 8)
+    return bench.rows
 
 
 def run(pkg, args, model_dir, peaks, clocks, out):
@@ -351,7 +226,7 @@ def run(pkg, args, model_dir, peaks, clocks, out):
     clocks.start()
     line = {"metric": "sonuzen decode tokens/s", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "higher_is_better": True,
             "data": "synthetic", "dtype": "bf16", "config": dict(z, model=args.workload, vocab=VOCAB, head_dim=DIM, taps=TAPS, l2="weights of a token and kernel rings exceed L2")}
-    ours = model_times(pkg, torch, path, 4096, STEP, args, kernels)
+    ours = bench_models.model_times(pkg, torch, path, 4096, STEP, args, kernels)
     nbytes = active_bytes(z, config(z)["layers"])
     sec = ours["decode"]["ms_per_token"] * 1e-3
     ours["decode"]["weight_bytes_per_token"] = nbytes
@@ -365,7 +240,7 @@ def run(pkg, args, model_dir, peaks, clocks, out):
         if not os.path.exists(p):
             if not pkg.load_host().llava_synth_write(os.fsencode(p), z["width"], z["width"] // DIM, z["layers"], ff, VOCAB, wt, 1234, 0):
                 raise RuntimeError("cannot write " + p)
-        m = model_times(pkg, torch, p, 0, 64, args, kernels)
+        m = bench_models.model_times(pkg, torch, p, 0, 64, args, kernels)
         b = (z["layers"] * (4 * z["width"] ** 2 + 3 * ff * z["width"]) + VOCAB * z["width"]) * bpb // 32
         m["decode"]["weight_bytes_per_token"] = b
         m["decode"]["frac_of_hbm"] = b / (m["decode"]["ms_per_token"] * 1e-3) / (peaks["hbm_gbs"] * 1e9)
