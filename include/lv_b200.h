@@ -583,7 +583,7 @@ int lv_latent_attention(lv_ctx* ctx, const lv_latent_args* a, void* scratch, siz
  *   dt         softplus(dt + dt_bias)
  *   S_t        = exp(-exp(A_log_h) dt) S_(t-1) + dt B_t x_t^T,  y_t = C_t S_t + D_h x_t   (head h: group h / (heads / groups))
  *   out        RMS norm of y * silu(z) in norm_groups equal parts, times norm_w
- * history f32 [taps][channels]: the convolution's input of position p in row p mod taps.  S f32 [heads][vdim][state rounded up to 16].
+ * history f32 [taps][channels]: the convolution's input of position p in row p mod taps.  S f32 [heads][vdim][lv_ssm_state_rows].
  * Both count as zero before position 0 and need no clearing.  scratch: lv_ssm_scratch_bytes. */
 typedef struct lv_ssm_args {
     const float* raw;
@@ -603,6 +603,8 @@ typedef struct lv_ssm_args {
     int out_type;
     uint32_t out_ld;
 } lv_ssm_args;
+/* state rounded up to a power of two, at least 16 */
+uint32_t lv_ssm_state_rows(uint32_t state);
 size_t lv_ssm_scratch_bytes(const lv_ssm_args* a, uint32_t batch);
 int lv_ssm(lv_ctx* ctx, const lv_ssm_args* a, void* scratch, size_t scratch_bytes, uint32_t batch);
 

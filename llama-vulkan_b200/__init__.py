@@ -165,6 +165,7 @@ KERNEL_API = {
     "lv_rotary_table": (_int, [_p, _p, _p, _p, _u32, _p, _u32]),
     "lv_latent_scratch_bytes": (_sz, [_p, C.POINTER(LatentArgs), _u32, _u32]),
     "lv_latent_attention": (_int, [_p, C.POINTER(LatentArgs), _p, _sz, _u32, _u32]),
+    "lv_ssm_state_rows": (_u32, [_u32]),
     "lv_ssm_scratch_bytes": (_sz, [C.POINTER(SsmArgs), _u32]),
     "lv_ssm": (_int, [_p, C.POINTER(SsmArgs), _p, _sz, _u32]),
 }

@@ -59,18 +59,6 @@ template <> struct Cache8<float> {
     static __device__ __forceinline__ float log_one_plus(float v) { return log1pf(v); }
 };
 
-__device__ __forceinline__ void cluster_sync() {
-    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-// a float in the shared memory of another CTA of the cluster
-__device__ __forceinline__ float cluster_load(const float* local, uint32_t rank) {
-    uint32_t at;
-    float v;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"(smem_u32(local)), "r"(rank));
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(at));
-    return v;
-}
-
 // Appends the normalised key and the value of token t (one warp per key/value head).
 template <typename CT>
 __global__ void __launch_bounds__(128) qk_norm_append_kernel(const GqaParams p, uint32_t n_tokens) {
@@ -413,21 +401,7 @@ static int gqa_launch_typed(lv_ctx* ctx, const GqaParams& p, uint32_t batch) {
         return LV_OK;
     }
     if (p.splits > 8) LV_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
-    cudaLaunchConfig_t cfg{};
-    cfg.gridDim = grid;
-    cfg.blockDim = dim3(kGqaThreads);
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = ctx->stream;
-    cudaLaunchAttribute attr[2];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    attr[1].id = cudaLaunchAttributeClusterDimension;
-    attr[1].val.clusterDim.x = 1;
-    attr[1].val.clusterDim.y = p.splits;
-    attr[1].val.clusterDim.z = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = 2;
-    LV_CUDA(cudaLaunchKernelEx(&cfg, kernel, p));
+    LV_CUDA(launch_pdl_cluster(ctx, kernel, grid, dim3(kGqaThreads), dim3(1, p.splits), smem, p));
     return LV_OK;
 }
 

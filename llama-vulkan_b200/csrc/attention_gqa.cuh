@@ -16,6 +16,18 @@ int gqa_tc_launch(lv_ctx* ctx, const lv_gqa_args& a, uint32_t batch);
 bool latent_tc_supported(const lv_latent_args& a);
 int latent_tc_launch(lv_ctx* ctx, const lv_latent_args& a, uint32_t batch, const void* kv, uint32_t ld, uint32_t v_at, uint32_t rows, uint32_t h0, uint32_t n);
 
+__device__ __forceinline__ void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// a float in the shared memory of another CTA of the cluster
+__device__ __forceinline__ float cluster_load(const float* local, uint32_t rank) {
+    uint32_t at;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"(smem_u32(local)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(at));
+    return v;
+}
+
 // 1 / rms of one head's vector, computed by a warp (every lane gets it)
 __device__ __forceinline__ float gqa_rms_factor(const float* v, uint32_t dim, float eps) {
     float part = 0.f;

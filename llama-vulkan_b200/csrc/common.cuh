@@ -191,6 +191,27 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// Sums V values over groups of NL consecutive lanes: each exchange halves the values a lane keeps.  With V >= NL, lane i of a
+// group ends with the values i * V / NL .. in v[0 ..]; with V < NL, with the value i / (NL / V) in v[0].
+template <int NL, int V>
+__device__ __forceinline__ void lanes_reduce(float (&v)[V]) {
+    if constexpr (NL > 1 && V > 1) {
+        const bool upper = (threadIdx.x & (NL / 2)) != 0;
+        float half[V / 2];
+#pragma unroll
+        for (int i = 0; i < V / 2; ++i) {
+            const float keep = upper ? v[i + V / 2] : v[i], give = upper ? v[i] : v[i + V / 2];
+            half[i] = keep + __shfl_xor_sync(0xffffffffu, give, NL / 2);
+        }
+        lanes_reduce<NL / 2, V / 2>(half);
+#pragma unroll
+        for (int i = 0; i < V / 2; ++i) v[i] = half[i];
+    } else {
+#pragma unroll
+        for (int o = NL / 2; o > 0; o /= 2) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+    }
+}
+
 // Block-wide sums over up to 32 warps with a single barrier; `scratch` holds 64 floats of
 // shared memory that must not be in use by another reduction.  Every thread adds the warp
 // totals itself in warp order, so every thread gets the same, reproducible result.

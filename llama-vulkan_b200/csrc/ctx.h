@@ -86,4 +86,24 @@ inline cudaError_t launch_pdl(lv_ctx* ctx, void (*kernel)(KArgs...), dim3 grid, 
     return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
 }
 
+// The same with thread-block clusters.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_pdl_cluster(lv_ctx* ctx, void (*kernel)(KArgs...), dim3 grid, dim3 block, dim3 cluster, size_t smem, Args... args) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = cluster.x;
+    attr[1].val.clusterDim.y = cluster.y;
+    attr[1].val.clusterDim.z = cluster.z;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
+    return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
+}
+
 }  // namespace lv

@@ -37,7 +37,7 @@ hybrid_session_state::hybrid_session_state(llava_session* _session, const hybrid
                 if (m.has_own_cache()) s.latent_cache = new llava_buffer(ctx, C, session->max_context, pad8(m.kv_rank) + pad8(m.rot), lasting, "latent_cache");
                 break;
             case hybrid_mixer::kind::ssm:
-                s.ssm_state = new llava_buffer(ctx, F, m.heads * m.vdim, (m.state + 15) / 16 * 16, lasting, "ssm_state");
+                s.ssm_state = new llava_buffer(ctx, F, m.heads * m.vdim, lv_ssm_state_rows(m.state), lasting, "ssm_state");
                 s.conv_history = new llava_buffer(ctx, F, m.conv_channels(), m.taps, lasting, "conv_history");
                 break;
         }

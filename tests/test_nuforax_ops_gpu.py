@@ -171,7 +171,7 @@ def test_latent_attention_in_portions(gpu, H, dim, rot, vdim, rank, window, f32)
 @pytest.mark.parametrize("H,dim,rot,vdim,rank,window", [(3, 24, 8, 40, 48, 20), (6, 64, 16, 48, 128, 130), (2, 128, 64, 128, 512, 0)])
 def test_both_forms_take_any_portion(gpu, form, H, dim, rot, vdim, rank, window):
     rng = np.random.default_rng(form)
-    cuts = [2, 3, 5, 128, 2, 129, 4, 3]
+    cuts = [2, 3, 5, 128, 2, 129, 4, 3] if form == EXPANDED else [1, 2, 3, 1, 128, 1, 1, 129, 4, 3]
     with Dev(gpu) as d:
         at = Latent(d, rng, H, dim, rot, vdim, rank, window, 320, False)
         q, dkv = at.draw(rng, sum(cuts))
@@ -179,6 +179,33 @@ def test_both_forms_take_any_portion(gpu, form, H, dim, rot, vdim, rank, window)
         for n in cuts:
             assert rel(at.run(q[done:done + n], dkv[done:done + n], done, form), want[done:done + n]) < 1.2e-2, (done, n)
             done += n
+
+
+@pytest.mark.parametrize("f32", [True, False])
+@pytest.mark.parametrize("window,form", [(0, 0), (1500, 0), (0, ABSORBED), (1100, ABSORBED)])
+@pytest.mark.parametrize("H,rank", [(3, 40), (11, 520), (35, 72)])
+def test_decoding_far_into_a_sequence(gpu, f32, window, form, H, rank):
+    """More visible rows than shared memory holds at a time, and a step's own row in any place of a chunk."""
+    rng = np.random.default_rng(H)
+    T, steps = 2100, 34
+    with Dev(gpu) as d:
+        at = Latent(d, rng, H, 16, 8, 16, rank, window, 2200, f32)
+        q, dkv = at.draw(rng, T)
+        for first in range(0, T - steps, 512):
+            last = min(first + 512, T - steps)
+            at.run(q[first:last], dkv[first:last], first)
+        got = np.concatenate([at.run(q[i:i + 1], dkv[i:i + 1], i, form) for i in range(T - steps, T)])
+        # plain, for the decoded positions only
+        pos = np.arange(T).astype(np.float64)
+        c = sp.norm_plain(dkv[:, :rank].astype(np.float64), at.norm.astype(np.float64), EPS)
+        kr = npl.rotate(dkv[:, rank:].astype(np.float64), pos, at.freqs, at.mult)
+        qq = q[T - steps:].astype(np.float64).reshape(steps, H, 24)
+        qr = npl.rotate(qq[..., 16:], pos[T - steps:], at.freqs, at.mult)
+        k, v = (c @ at.uk.T.astype(np.float64)).reshape(T, H, 16), (c @ at.uv.T.astype(np.float64)).reshape(T, H, 16)
+        s = (np.einsum("ihd,jhd->hij", qq[..., :16], k) + np.einsum("ihd,jd->hij", qr, kr)) * at.scale
+        p = npl.sink_weights(s, npl.window_mask(T, window or T + 1)[T - steps:], at.sink.astype(np.float64))
+        want = np.einsum("hij,jhd->ihd", p, v).reshape(steps, -1)
+    assert rel(got, want) < (5e-6 if f32 else 1.2e-2)
 
 
 @pytest.mark.parametrize("f32", [True, False])
@@ -285,7 +312,7 @@ class StateSpace:
         self.conv, self.conv_b, self.D, self.norm = f(self.channels, taps, spread=0.6), f(self.channels), f(H), f(self.inner, mean=1.0)
         self.A_log, self.dt_bias = f(H, mean=A_mean, spread=1.5), f(H, mean=dt_mean, spread=1.0)
         self.dev = [d.f32(np.ascontiguousarray(v)) for v in (self.conv.T, self.conv_b, self.dt_bias, self.A_log, self.D, self.norm)]
-        self.history, self.S = nans(d, taps * self.channels * 4), nans(d, H * P * ((N + 15) // 16 * 16) * 4)      # no clearing needed
+        self.history, self.S = nans(d, taps * self.channels * 4), nans(d, H * P * d.gpu.lib.lv_ssm_state_rows(N) * 4)      # no clearing needed
 
     def draw(self, rng, T):
         return rng.standard_normal((T, 2 * self.inner + 2 * self.G * self.N + self.H)).astype(np.float32)
