@@ -584,7 +584,10 @@ int lv_latent_attention(lv_ctx* ctx, const lv_latent_args* a, void* scratch, siz
  *   S_t        = exp(-exp(A_log_h) dt) S_(t-1) + dt B_t x_t^T,  y_t = C_t S_t + D_h x_t   (head h: group h / (heads / groups))
  *   out        RMS norm of y * silu(z) in norm_groups equal parts, times norm_w
  * history f32 [taps][channels]: the convolution's input of position p in row p mod taps.  S f32 [heads][vdim][lv_ssm_state_rows].
- * Both count as zero before position 0 and need no clearing.  scratch: lv_ssm_scratch_bytes. */
+ * Both count as zero before position 0 and need no clearing.  scratch: lv_ssm_scratch_bytes.
+ * Several tokens: a scan in f32, or -- by default for bfloat16 output, vdim a multiple of 8 -- chunks of tokens as matrix products
+ * with x, B and C in bfloat16 and everything else in f32. */
+enum { LV_SSM_AUTO = 0, LV_SSM_SCAN = 1, LV_SSM_TENSOR = 2 };
 typedef struct lv_ssm_args {
     const float* raw;
     uint32_t raw_ld, heads, vdim, state, groups, taps;
@@ -602,6 +605,7 @@ typedef struct lv_ssm_args {
     void* out;
     int out_type;
     uint32_t out_ld;
+    int form;
 } lv_ssm_args;
 /* state rounded up to a power of two, at least 16 */
 uint32_t lv_ssm_state_rows(uint32_t state);

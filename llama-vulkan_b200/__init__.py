@@ -68,7 +68,7 @@ class SsmArgs(C.Structure):
     """lv_ssm_args"""
     _fields_ = [("raw", _p), ("raw_ld", _u32), ("heads", _u32), ("vdim", _u32), ("state", _u32), ("groups", _u32), ("taps", _u32), ("conv_w", _p), ("conv_b", _p),
                 ("dt_bias", _p), ("A_log", _p), ("D", _p), ("norm_w", _p), ("norm_groups", _u32), ("eps", _f32), ("history", _p), ("S", _p), ("pos", _p), ("out", _p),
-                ("out_type", _int), ("out_ld", _u32)]
+                ("out_type", _int), ("out_ld", _u32), ("form", _int)]
 
 
 # name -> (restype, argtypes); mirrors include/lv_b200.h

@@ -2,7 +2,8 @@
 // grouped norm.
 //
 //   several tokens   ssm_conv_kernel   convolution, silu, step sizes and logarithms of the decays
-//                    ssm_scan_kernel   the recurrence, D x and the gate
+//                    ssm_scan_kernel   the recurrence, D x and the gate; for bfloat16 models chunks of tokens as matrix products
+//                                      instead (state_space_tc.cu)
 //   one token        ssm_step_kernel   all of that
 //   both             ssm_norm_kernel   RMS norm of each part
 //
@@ -17,10 +18,10 @@
 
 #include "common.cuh"
 #include "ctx.h"
+#include "state_space.cuh"
 
 namespace lv {
 
-constexpr uint32_t kSsMaxTaps = 16, kSsMaxState = 256;
 constexpr int kSsThreads = 128;              // of the convolution; at most of the others
 // columns of a head per CTA and threads of it when NL lanes share a column
 __host__ __device__ constexpr int ss_columns(int NL) { return NL <= 4 ? 64 : 256 / NL; }
@@ -28,15 +29,6 @@ __host__ __device__ constexpr int ss_threads(int NL) { return ss_columns(NL) / 2
 constexpr int kSsChunk = 32;                 // tokens
 constexpr double kSsReference = 32.0;
 constexpr int kSsConvTokens = 16;            // tokens of a block of the convolution; at least the taps - 1 before them
-constexpr float kSsMinLog = -200.f;          // a decay below e^-200 is zero in f32
-
-struct SsmParams {
-    lv_ssm_args a;
-    uint32_t batch, inner, channels, state_p;    // state_p: state rounded up to a power of two, at least 16
-    uint32_t x_at, b_at, c_at, dt_at, log_at, conv_ld;      // columns of `conv`: x, B and C (state_p per group), dt and log a per head
-    float* conv;                                 // [batch][conv_ld]
-    float* gated;                                // [batch][inner]
-};
 
 __device__ __forceinline__ float softplus_f32(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float ss_log_decay(float A_log, float dt) { return fmaxf(-expf(A_log) * dt, kSsMinLog); }
@@ -60,62 +52,69 @@ __device__ __forceinline__ uint64_t ss_add2(uint64_t a, uint64_t b) {
 }
 __device__ __forceinline__ float ss_sum2(uint64_t v) { return __uint_as_float(uint32_t(v)) + __uint_as_float(uint32_t(v >> 32)); }
 
-// Columns of `conv`: a thread owns one and kSsConvTokens tokens, all loads before the first use.  Block row 0 alone reads the history,
-// whose successor it writes.
-template <int MAXT>
+// Columns of `conv`, then dt and log a of the heads: a thread owns one column and kSsConvTokens tokens, all loads before the first use.
+// Block row 0 alone reads the history, whose successor it writes.
+template <typename OutT, int MAXT>
 __global__ void __launch_bounds__(kSsThreads) ssm_conv_kernel(const SsmParams p) {
     pdl_launch_dependents();
     const lv_ssm_args& a = p.a;
     const uint32_t col = blockIdx.x * kSsThreads + threadIdx.x, T = p.batch, t0 = blockIdx.y * kSsConvTokens;
-    if (col >= p.conv_ld) return;
-    uint32_t channel = ~0u, source = ~0u;        // of the convolution; column of `raw` behind z
-    const bool is_dt = col >= p.dt_at && col < p.dt_at + a.heads, is_log = col >= p.log_at && col < p.log_at + a.heads;
-    const uint32_t h = is_dt ? col - p.dt_at : is_log ? col - p.log_at : 0;
+    if (col >= p.conv_ld + 2 * a.heads) return;
+    const bool rate = col >= p.conv_ld;
+    const uint32_t h = rate ? (col - p.conv_ld) >> 1 : 0;
+    uint32_t channel = ~0u;                      // of the convolution; none: padding, or a rate
     if (col < p.inner) {
         channel = col;
-    } else if (col >= p.b_at && col < p.dt_at) {
+    } else if (!rate && col >= p.b_at) {
         const bool second = col >= p.c_at;
         const uint32_t g = (col - (second ? p.c_at : p.b_at)) / p.state_p, n = (col - (second ? p.c_at : p.b_at)) - g * p.state_p;
-        if (n < a.state) channel = p.inner + (second ? a.groups * a.state : 0) + g * a.state + n;
+        if (g < a.groups && n < a.state) channel = p.inner + (second ? a.groups * a.state : 0) + g * a.state + n;
     }
-    source = channel != ~0u ? channel : is_dt || is_log ? p.channels + h : ~0u;
-    float w[MAXT], bias = 0.f, rate = 0.f;       // taps right-aligned: index MAXT - 1 is the current token
+    const bool conv = channel != ~0u;
+    float w[MAXT], bias = 0.f, A_log = 0.f;      // taps right-aligned: index MAXT - 1 is the current token
 #pragma unroll
     for (int j = 0; j < MAXT; ++j) {
         const int s = j - (MAXT - int(a.taps));
-        w[j] = channel != ~0u && s >= 0 ? a.conv_w[size_t(s) * p.channels + channel] : 0.f;
+        w[j] = conv && s >= 0 ? a.conv_w[size_t(s) * p.channels + channel] : 0.f;
     }
-    if (channel != ~0u) bias = a.conv_b[channel];
-    else if (source != ~0u) bias = a.dt_bias[h];
-    if (is_log) rate = a.A_log[h];
+    if (conv) bias = a.conv_b[channel];
+    if (rate) {
+        bias = a.dt_bias[h];
+        A_log = a.A_log[h];
+    }
     pdl_wait();
     const uint32_t pos = *a.pos;
-    const float* raw = a.raw + p.inner + (source != ~0u ? source : 0);
+    const float* raw = a.raw + p.inner + (conv ? channel : p.channels + h);
     float* history = a.history + channel;
     float v[MAXT - 1 + kSsConvTokens];           // v[MAXT - 1 + i]: token t0 + i
 #pragma unroll
     for (int i = 0; i < MAXT - 1 + kSsConvTokens; ++i) {
         const int t = int(t0) + i - (MAXT - 1), back = -t;
         v[i] = 0.f;
-        if (t >= 0 && t < int(T) && source != ~0u && (i >= MAXT - 1 || channel != ~0u)) v[i] = raw[size_t(t) * a.raw_ld];
-        else if (t < 0 && channel != ~0u && back < int(a.taps) && pos >= uint32_t(back)) v[i] = history[size_t((pos - back) % a.taps) * p.channels];
+        if (t >= 0 && t < int(T) && (conv || (rate && i >= MAXT - 1))) v[i] = raw[size_t(t) * a.raw_ld];
+        else if (t < 0 && conv && back < int(a.taps) && pos >= uint32_t(back)) v[i] = history[size_t((pos - back) % a.taps) * p.channels];
     }
-    float* out = p.conv + size_t(t0) * p.conv_ld + col;
+    if (rate) {
+        float* out = p.rates + size_t(t0) * a.heads * 2 + (col - p.conv_ld);
+#pragma unroll
+        for (int i = 0; i < kSsConvTokens; ++i) {
+            const float dt = softplus_f32(v[MAXT - 1 + i] + bias);
+            if (t0 + i < T) out[size_t(i) * a.heads * 2] = (col - p.conv_ld) & 1u ? ss_log_decay(A_log, dt) : dt;
+        }
+        return;
+    }
+    OutT* out = static_cast<OutT*>(p.conv) + size_t(t0) * p.conv_ld + col;
 #pragma unroll
     for (int i = 0; i < kSsConvTokens; ++i) {
-        if (t0 + i >= T) continue;
         float y = bias;
-        if (channel != ~0u) {
 #pragma unroll
-            for (int j = 0; j < MAXT; ++j) y = fmaf(w[j], v[i + j], y);
-            y = silu_f32(y);
-        } else if (source != ~0u) {
-            y = softplus_f32(v[MAXT - 1 + i] + bias);
-            if (is_log) y = ss_log_decay(rate, y);
-        }
-        out[size_t(i) * p.conv_ld] = y;          // (padding: zero)
+        for (int j = 0; j < MAXT; ++j) y = fmaf(w[j], v[i + j], y);
+        y = silu_f32(y);                         // (padding: zero)
+        if (t0 + i >= T) continue;
+        if constexpr (sizeof(OutT) == 2) out[size_t(i) * p.conv_ld] = __float2bfloat16_rn(y);
+        else out[size_t(i) * p.conv_ld] = y;
     }
-    if (blockIdx.y != 0 || channel == ~0u) return;
+    if (blockIdx.y != 0 || !conv) return;
     for (uint32_t t = T > a.taps ? T - a.taps : 0; t < T; ++t) history[size_t((pos + t) % a.taps) * p.channels] = raw[size_t(t) * a.raw_ld];
 }
 
@@ -152,7 +151,7 @@ __global__ void __launch_bounds__(ss_threads(NL)) ssm_scan_kernel(const SsmParam
     auto copy4 = [](const float* dst, const float* src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory"); };
     auto fetch = [&](uint32_t chunk, uint32_t buffer) {
         const uint32_t t0 = chunk * kSsChunk, n = min(uint32_t(kSsChunk), T - t0);
-        const float* src = p.conv + size_t(t0) * p.conv_ld;
+        const float* src = static_cast<const float*>(p.conv) + size_t(t0) * p.conv_ld;
         const float* z = a.raw + size_t(t0) * a.raw_ld + h * a.vdim + c0;
 #pragma unroll 4
         for (uint32_t i = threadIdx.x; i < n * (N / 4); i += kThreads) {
@@ -170,7 +169,7 @@ __global__ void __launch_bounds__(ss_threads(NL)) ssm_scan_kernel(const SsmParam
         }
         // the rows that complete the last group of tokens
         for (uint32_t i = n * N + threadIdx.x; i < (n + kGroup - 1) / kGroup * kGroup * N; i += kThreads) s_b[buffer * kSsChunk * N + i] = 0.f;
-        for (uint32_t i = threadIdx.x; i < n * 2; i += kThreads) copy4(s_raw + buffer * kSsChunk * 2 + i, src + size_t(i >> 1) * p.conv_ld + ((i & 1u) ? p.log_at : p.dt_at) + h);
+        for (uint32_t i = threadIdx.x; i < n * 2; i += kThreads) copy4(s_raw + buffer * kSsChunk * 2 + i, p.rates + (size_t(t0 + (i >> 1)) * a.heads + h) * 2 + (i & 1u));
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(0, 0);
@@ -445,18 +444,27 @@ __global__ void __launch_bounds__(256) ssm_norm_kernel(const SsmParams p) {
     for (uint32_t i = (threadIdx.x + kPer * blockDim.x) * VEC; i < n; i += blockDim.x * VEC) store(i, value(i), weight(i));
 }
 
+static bool ssm_tc(const lv_ssm_args& a, uint32_t batch) {
+    return batch > 1 && a.form != LV_SSM_SCAN && (a.form == LV_SSM_TENSOR || a.out_type == LV_TYPE_BF16) && ssm_tc_supported(a);
+}
+
 static void ssm_layout(SsmParams& p) {
     const lv_ssm_args& a = p.a;
-    auto pad = [](uint32_t n, uint32_t to) { return (n + to - 1) / to * to; };
+    auto pad8 = [](uint32_t n) { return (n + 7) / 8 * 8; };
     p.inner = a.heads * a.vdim;
     p.channels = p.inner + 2 * a.groups * a.state;
     p.state_p = lv_ssm_state_rows(a.state);
-    p.x_at = 0;
-    p.b_at = pad(p.inner, 4);
+    p.b_at = pad8(p.inner);
     p.c_at = p.b_at + a.groups * p.state_p;
-    p.dt_at = p.c_at + a.groups * p.state_p;
-    p.log_at = p.dt_at + a.heads;
-    p.conv_ld = pad(p.log_at + a.heads, 4);
+    p.conv_ld = p.c_at + a.groups * p.state_p;
+}
+
+template <typename OutT>
+static int ssm_conv_launch(lv_ctx* ctx, const SsmParams& p) {
+    const dim3 grid((p.conv_ld + 2 * p.a.heads + kSsThreads - 1) / kSsThreads, (p.batch + kSsConvTokens - 1) / kSsConvTokens);
+    auto* conv = p.a.taps <= 4 ? ssm_conv_kernel<OutT, 4> : p.a.taps <= 8 ? ssm_conv_kernel<OutT, 8> : ssm_conv_kernel<OutT, 16>;
+    LV_CUDA(launch_pdl(ctx, conv, grid, dim3(kSsThreads), 0, p));
+    return LV_OK;
 }
 
 template <int NL>
@@ -501,7 +509,7 @@ extern "C" size_t lv_ssm_scratch_bytes(const lv_ssm_args* a, uint32_t batch) {
     SsmParams p{};
     p.a = *a;
     ssm_layout(p);
-    return sizeof(float) * size_t(batch) * (p.conv_ld + (p.inner + 3) / 4 * 4);
+    return sizeof(float) * size_t(batch) * (p.conv_ld + (p.inner + 3) / 4 * 4 + 2 * a->heads);
 }
 
 extern "C" int lv_ssm(lv_ctx* ctx, const lv_ssm_args* a, void* scratch, size_t scratch_bytes, uint32_t batch) {
@@ -517,16 +525,17 @@ extern "C" int lv_ssm(lv_ctx* ctx, const lv_ssm_args* a, void* scratch, size_t s
     LV_REQUIRE(a->raw_ld >= p.inner + p.channels + a->heads && a->out_ld >= p.inner && (a->out_type == LV_TYPE_F32 || a->out_type == LV_TYPE_BF16), "ssm: bad strides");
     LV_REQUIRE((reinterpret_cast<uintptr_t>(a->S) & 15u) == 0 && scratch && (reinterpret_cast<uintptr_t>(scratch) & 15u) == 0 &&
                scratch_bytes >= lv_ssm_scratch_bytes(a, batch), "ssm: bad scratch or state");
-    p.conv = static_cast<float*>(scratch);
-    p.gated = p.conv + size_t(batch) * p.conv_ld;
-    if (batch > 1) {
-        const dim3 grid((p.conv_ld + kSsThreads - 1) / kSsThreads, (batch + kSsConvTokens - 1) / kSsConvTokens);
-        auto* conv = a->taps <= 4 ? ssm_conv_kernel<4> : a->taps <= 8 ? ssm_conv_kernel<8> : ssm_conv_kernel<16>;
-        LV_CUDA(launch_pdl(ctx, conv, grid, dim3(kSsThreads), 0, p));
-    }
-    // lanes that share a column: sixteen state rows each
+    LV_REQUIRE(a->form != LV_SSM_TENSOR || batch == 1 || ssm_tc_supported(*a), "ssm: the tensor-core form does not take these sizes");
+    p.conv = scratch;
+    p.gated = static_cast<float*>(scratch) + size_t(batch) * p.conv_ld;
+    p.rates = p.gated + size_t(batch) * ((p.inner + 3) / 4 * 4);
+    const bool tensor = ssm_tc(*a, batch);
     int rc = LV_OK;
-    if (p.state_p <= 16) rc = ssm_launch<1>(ctx, p);
+    if (batch > 1) rc = tensor ? ssm_conv_launch<__nv_bfloat16>(ctx, p) : ssm_conv_launch<float>(ctx, p);
+    if (rc != LV_OK) return rc;
+    // lanes that share a column: sixteen state rows each
+    if (tensor) rc = ssm_tc_launch(ctx, p);
+    else if (p.state_p <= 16) rc = ssm_launch<1>(ctx, p);
     else if (p.state_p <= 32) rc = ssm_launch<2>(ctx, p);
     else if (p.state_p <= 64) rc = ssm_launch<4>(ctx, p);
     else if (p.state_p <= 128) rc = ssm_launch<8>(ctx, p);

@@ -317,22 +317,25 @@ class StateSpace:
     def draw(self, rng, T):
         return rng.standard_normal((T, 2 * self.inner + 2 * self.G * self.N + self.H)).astype(np.float32)
 
-    def run(self, raw, at, bf16=False):
+    def run(self, raw, at, bf16=False, form=0):
         d, n = self.d, raw.shape[0]
         ld = pad8(self.inner)
         out = nans(d, n * ld * 4)
         conv, conv_b, dt_bias, A_log, D, norm = self.dev
         a = pkg.SsmArgs(raw=d.f32(raw).value, raw_ld=raw.shape[1], heads=self.H, vdim=self.P, state=self.N, groups=self.G, taps=self.taps, conv_w=conv.value, conv_b=conv_b.value,
                         dt_bias=dt_bias.value, A_log=A_log.value, D=D.value, norm_w=norm.value, norm_groups=self.parts, eps=EPS, history=self.history.value, S=self.S.value,
-                        pos=d.u32([at] * 4).value, out=out.value, out_type=pkg.TYPE_BF16 if bf16 else pkg.TYPE_F32, out_ld=ld)
+                        pos=d.u32([at] * 4).value, out=out.value, out_type=pkg.TYPE_BF16 if bf16 else pkg.TYPE_F32, out_ld=ld, form=form)
         nbytes = d.gpu.lib.lv_ssm_scratch_bytes(C.byref(a), n)
         d.call("lv_ssm", C.byref(a), nans(d, nbytes), nbytes, n)
         return d.get(out, (n, ld), bf16)[:, :self.inner]
 
-    def plain(self, raw):
+    def plain(self, raw, rounded=False):
+        """rounded: x, B and C in bfloat16"""
         T = raw.shape[0]
         z, xbc, dt = np.split(raw.astype(np.float64), [self.inner, self.inner + self.channels], axis=1)
         xbc = sp.silu(sp.causal_conv(xbc, self.conv.astype(np.float64)) + self.conv_b)
+        if rounded:
+            xbc = sp.bf16_round(xbc.astype(np.float32)).astype(np.float64)
         x, B, K = np.split(xbc, [self.inner, self.inner + self.G * self.N], axis=1)
         y = npl.state_space(x.reshape(T, self.H, self.P), B.reshape(T, self.G, self.N), K.reshape(T, self.G, self.N), npl.softplus(dt + self.dt_bias),
                             self.A_log.astype(np.float64), self.D.astype(np.float64))
@@ -343,7 +346,7 @@ SIZES = [(6, 20, 24, 2, 3, 3), (4, 32, 16, 4, 5, 1), (3, 40, 130, 1, 2, 1), (8, 
 
 
 @pytest.mark.parametrize("H,P,N,G,taps,parts", SIZES)
-@pytest.mark.parametrize("cuts", [[1] * 40, [140], [33, 1, 1, 2, 31, 64, 3, 1, 1, 2], [2] * 20, [32, 32, 1]])
+@pytest.mark.parametrize("cuts", [[1] * 40, [140], [33, 1, 1, 2, 31, 64, 3, 1, 1, 2], [2] * 20, [32, 32, 1], [640, 1, 131]])
 def test_state_space_in_portions(gpu, H, P, N, G, taps, parts, cuts):
     rng = np.random.default_rng(H * P + N)
     with Dev(gpu) as d:
@@ -352,6 +355,39 @@ def test_state_space_in_portions(gpu, H, P, N, G, taps, parts, cuts):
         want, at = s.plain(raw), 0
         for n in cuts:
             assert rel(s.run(raw[at:at + n], at), want[at:at + n]) < 5e-6, (at, n)
+            at += n
+
+
+TENSOR = 2
+
+
+@pytest.mark.parametrize("H,P,N,G,taps,parts", [(4, 32, 16, 4, 5, 1), (3, 40, 130, 1, 2, 1), (8, 64, 128, 2, 4, 8), (6, 8, 11, 3, 7, 3), (2, 304, 8, 1, 1, 2), (10, 16, 64, 5, 16, 5),
+                                                (1, 24, 256, 1, 4, 1), (5, 48, 33, 1, 3, 1)])
+@pytest.mark.parametrize("cuts", [[140], [33, 2, 31, 64, 3, 2], [2] * 20, [64, 64, 65], [63, 700]])
+def test_chunks_of_tokens_as_matrix_products(gpu, H, P, N, G, taps, parts, cuts):
+    """Everything but x, B and C is as exact as in f32."""
+    rng = np.random.default_rng(H * P + N)
+    with Dev(gpu) as d:
+        s = StateSpace(d, rng, H, P, N, G, taps, parts)
+        raw = s.draw(rng, sum(cuts))
+        want, at = s.plain(raw, rounded=True), 0
+        for n in cuts:
+            far = rel(s.run(raw[at:at + n], at, form=TENSOR), want[at:at + n])
+            assert far < 4e-4, (at, n)                            # (a convolution's output at the middle between two bfloat16 numbers rounds either way)
+            at += n
+
+
+@pytest.mark.parametrize("A_mean,dt_mean", [(-6.0, -5.0), (-9.0, 0.5), (2.0, 3.0), (5.0, 6.0), (1.0, -1.0)])
+def test_matrix_products_and_scan_take_turns(gpu, A_mean, dt_mean):
+    """Weak to complete decays; the state that one form leaves is what the other (and a single token) continues from."""
+    rng = np.random.default_rng(4)
+    with Dev(gpu) as d:
+        s = StateSpace(d, rng, 6, 24, 32, 2, 4, 2, A_mean, dt_mean)
+        raw = s.draw(rng, 400)
+        raw[:, -6:] *= 3
+        want, at = s.plain(raw), 0
+        for n, form in ((100, TENSOR), (70, 1), (1, 0), (129, TENSOR), (1, 0), (99, TENSOR)):
+            assert rel(s.run(raw[at:at + n], at, form=form), want[at:at + n]) < 1e-2, (at, n)
             at += n
 
 
