@@ -232,6 +232,8 @@ __device__ __forceinline__ float half_bits_to_float(uint32_t h16) {
 
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.f + expf(-z)); }
+// (for values that are rounded to bfloat16)
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
 // Activation of a finished product (LV_ACT_* of lv_b200.h; 1: the square of relu).
 __device__ __forceinline__ float product_act(float v, int act) {

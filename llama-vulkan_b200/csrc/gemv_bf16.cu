@@ -9,7 +9,8 @@
 // f32 throughout: a bfloat16 weight is exact in f32, so the same kernels serve a 32-bit evaluation.  The bound is HBM: two
 // bytes per multiply-add, each weight read once.  A warp computes two or three rows, lanes taking 16 bytes of every row per
 // step with four steps in flight (up to 6 KB per warp); the first weights are requested before the previous kernel has
-// finished.  Lanes are combined by shuffles in a fixed order, so a result does not depend on the launch.
+// finished.  Lanes are combined by shuffles in a fixed order, so a result does not depend on the launch.  Matrices with few rows
+// are cut along K over the warps of a CTA, so that enough loads are in flight.
 //
 // gridDim.y = tokens: every token has its own pass over the weights.  Prompts use gemm_bf16.cu instead.
 #include <cuda_bf16.h>
@@ -91,15 +92,32 @@ struct GemvBf16Params {
     int act;
 };
 
+// SPLIT: warps that share two rows
+template <int SPLIT>
 __global__ void __launch_bounds__(kGbThreads) gemv_bf16_kernel(const GemvBf16Params p) {
     pdl_launch_dependents();
-    const uint32_t u = 2u * (blockIdx.x * kGbWarps + (threadIdx.x >> 5));
-    if (u >= p.rows) return;
-    const __nv_bfloat16* row[2] = {p.w[0] + size_t(u) * p.ld, p.w[0] + size_t(min(u + 1, p.rows - 1)) * p.ld};
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
+    const uint32_t u = 2u * (blockIdx.x * (kGbWarps / SPLIT) + warp / SPLIT);
     float acc[2] = {0.f, 0.f};
-    gb_dot<2, true>(acc, row, p.x + size_t(blockIdx.y) * p.x_ld, p.K);
-    const float a0 = warp_sum(acc[0]), a1 = warp_sum(acc[1]);
-    const uint32_t lane = threadIdx.x & 31u;
+    if constexpr (SPLIT == 1) {
+        if (u >= p.rows) return;
+        const __nv_bfloat16* row[2] = {p.w[0] + size_t(u) * p.ld, p.w[0] + size_t(min(u + 1, p.rows - 1)) * p.ld};
+        gb_dot<2, true>(acc, row, p.x + size_t(blockIdx.y) * p.x_ld, p.K);
+    } else {
+        const uint32_t per = (p.K + SPLIT * 256 - 1) / (SPLIT * 256) * 256, first = warp % SPLIT * per, count = u < p.rows && first < p.K ? min(per, p.K - first) : 0;
+        const __nv_bfloat16* row[2] = {p.w[0] + size_t(min(u, p.rows - 1)) * p.ld + first, p.w[0] + size_t(min(u + 1, p.rows - 1)) * p.ld + first};
+        gb_dot<2, true>(acc, row, p.x + size_t(blockIdx.y) * p.x_ld + first, count);
+    }
+    float a0 = warp_sum(acc[0]), a1 = warp_sum(acc[1]);
+    if constexpr (SPLIT > 1) {
+        __shared__ float s_part[kGbWarps][2];
+        if (lane == 0) { s_part[warp][0] = a0; s_part[warp][1] = a1; }
+        __syncthreads();
+        if (warp % SPLIT != 0) return;
+        a0 = a1 = 0.f;
+#pragma unroll
+        for (int k = 0; k < SPLIT; ++k) { a0 += s_part[warp + k][0]; a1 += s_part[warp + k][1]; }
+    }
     if (lane < 2 && u + lane < p.rows) p.out[size_t(blockIdx.y) * p.out_ld + u + lane] = product_act((lane ? a1 : a0) * p.factor, p.act);
 }
 
@@ -185,7 +203,12 @@ extern "C" int lv_gemv_bf16(lv_ctx* ctx, float* out, uint32_t out_ld, const void
     p.w[0] = static_cast<const __nv_bfloat16*>(w);
     p.rows = rows;
     p.ld = ld; p.K = cols; p.x = x; p.x_ld = x_ld; p.out = out; p.out_ld = out_ld; p.factor = factor; p.act = act;
-    LV_CUDA(launch_pdl(ctx, gemv_bf16_kernel, dim3((rows + 2 * kGbWarps - 1) / (2 * kGbWarps), batch), dim3(kGbThreads), 0, p));
+    // three or more CTAs per SM, at least 512 columns per warp
+    uint32_t split = 1;
+    while (split < 8 && uint64_t(rows) * batch * split < uint64_t(48) * uint32_t(ctx->sm_count) && cols >= 512 * 2 * split) split *= 2;
+    const uint32_t per_cta = 2 * kGbWarps / split;
+    auto* kernel = split == 1 ? gemv_bf16_kernel<1> : split == 2 ? gemv_bf16_kernel<2> : split == 4 ? gemv_bf16_kernel<4> : gemv_bf16_kernel<8>;
+    LV_CUDA(launch_pdl(ctx, kernel, dim3((rows + per_cta - 1) / per_cta, batch), dim3(kGbThreads), 0, p));
     return LV_OK;
 }
 

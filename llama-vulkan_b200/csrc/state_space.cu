@@ -109,10 +109,9 @@ __global__ void __launch_bounds__(kSsThreads) ssm_conv_kernel(const SsmParams p)
         float y = bias;
 #pragma unroll
         for (int j = 0; j < MAXT; ++j) y = fmaf(w[j], v[i + j], y);
-        y = silu_f32(y);                         // (padding: zero)
-        if (t0 + i >= T) continue;
-        if constexpr (sizeof(OutT) == 2) out[size_t(i) * p.conv_ld] = __float2bfloat16_rn(y);
-        else out[size_t(i) * p.conv_ld] = y;
+        if (t0 + i >= T) continue;               // (padding: zero)
+        if constexpr (sizeof(OutT) == 2) out[size_t(i) * p.conv_ld] = __float2bfloat16_rn(silu_fast(y));
+        else out[size_t(i) * p.conv_ld] = silu_f32(y);
     }
     if (blockIdx.y != 0 || !conv) return;
     for (uint32_t t = T > a.taps ? T - a.taps : 0; t < T; ++t) history[size_t((pos + t) % a.taps) * p.channels] = raw[size_t(t) * a.raw_ld];

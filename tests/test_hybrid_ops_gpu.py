@@ -15,7 +15,7 @@ pkg = load_pkg()
 
 # ---- products --------------------------------------------------------------------------------
 
-@pytest.mark.parametrize("rows,cols,batch", [(8, 8, 1), (7, 24, 1), (192, 256, 3), (333, 76, 1), (1000, 1544, 2)])
+@pytest.mark.parametrize("rows,cols,batch", [(8, 8, 1), (7, 24, 1), (192, 256, 3), (333, 76, 1), (1000, 1544, 2), (333, 1032, 1), (35, 2200, 1), (7, 8456, 2), (64, 4300, 1), (1, 5000, 1)])
 def test_gemv_bf16_is_exact_in_f32(gpu, rows, cols, batch):
     rng = np.random.default_rng(rows)
     w, x = weights(rng, rows, cols), rng.standard_normal((batch, pad8(cols))).astype(np.float32)
