@@ -9,8 +9,8 @@
 // enters S' as three bfloat16 terms that add up to the f32 value, M and S enter y, which ends in bfloat16, as two terms (16 bits).
 // L is summed in f64 and kept as two f32 terms, in units of log 2, so that differences of large sums stay exact.
 //
-// A CTA has 32 columns of one head and walks its chunks in order, S in the accumulators of its sixteen warps (a warp: sixteen
-// state rows and columns).  For y a warp has sixteen tokens and eight columns.  The tiles are small and the chain from chunk to chunk
+// A CTA has 32 or 64 columns of one head and walks its chunks in order, S in the accumulators of its sixteen warps (a warp: sixteen
+// state rows, half of the columns).  For y a warp has sixteen tokens and a quarter of the columns.  The tiles are small and the chain from chunk to chunk
 // is serial and bound by latency, so the products are warp-level (mma.sync).  A chunk has three phases: {C S, G, L}, {M, weighted x},
 // {M x, S'}; the terms of M lie where those of S were.
 #include <cuda_bf16.h>
@@ -22,9 +22,8 @@
 
 namespace lv {
 
-constexpr int kStThreads = 512, kStWarps = kStThreads / 32, kStTokens = 64, kStCols = 32;
+constexpr int kStThreads = 512, kStWarps = kStThreads / 32, kStTokens = 64;
 constexpr int kStAhead = 8;                 // chunks whose sums of log a are formed together, a warp each
-constexpr int kStXLd = kStCols + 8;          // row strides of tiles in shared memory: an odd multiple of 16 bytes
 
 __device__ __forceinline__ void st_ldmatrix(uint32_t (&r)[4], const __nv_bfloat16* at) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(at)) : "memory");
@@ -56,33 +55,39 @@ __device__ __forceinline__ float st_exp2(float x) {
     return y;
 }
 
+// row strides of tiles in shared memory: odd multiples of 16 bytes
 constexpr int kStMLd = kStTokens + 8;
-template <int NP> __host__ __device__ constexpr uint32_t st_terms_elems() { return 2 * (NP * kStXLd > kStTokens * kStMLd ? NP * kStXLd : kStTokens * kStMLd); }
-template <int NP> constexpr size_t st_smem_bytes() {
-    return size_t(3 * kStTokens * (NP + 8) + 2 * kStTokens * kStXLd + 3 * kStTokens * kStXLd + st_terms_elems<NP>()) * 2 +
+__host__ __device__ constexpr int st_x_ld(int cols) { return cols + 8; }
+template <int NP, int COLS> __host__ __device__ constexpr uint32_t st_terms_elems() {
+    return 2 * (NP * st_x_ld(COLS) > kStTokens * kStMLd ? NP * st_x_ld(COLS) : kStTokens * kStMLd);
+}
+template <int NP, int COLS> constexpr size_t st_smem_bytes() {
+    return size_t(3 * kStTokens * (NP + 8) + 5 * kStTokens * st_x_ld(COLS) + st_terms_elems<NP, COLS>()) * 2 +
            size_t(kStAhead) * (5 * kStTokens + 4) * 4;
 }
 
-// NP: state rows, padded
-template <int NP>
+// NP: state rows, padded; COLS: columns of a head per CTA
+template <int NP, int COLS>
 __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) uint8_t smem_raw[];
     const lv_ssm_args& a = p.a;
+    constexpr uint32_t kStCols = COLS, kStXLd = st_x_ld(COLS);
+    constexpr int kYTiles = COLS / 32, kSTiles = COLS / 16;      // column tiles of a warp
     constexpr uint32_t kLd = NP + 8, kTile = kStTokens * kLd, kXTile = kStTokens * kStXLd, kSTile = NP * kStXLd, kMTile = kStTokens * kStMLd;
     const uint32_t blocks = (a.vdim + kStCols - 1) / kStCols, h = blockIdx.x / blocks, c0 = (blockIdx.x - h * blocks) * kStCols;
-    const uint32_t cols = min(uint32_t(kStCols), a.vdim - c0), g = h / (a.heads / a.groups);
+    const uint32_t cols = min(kStCols, a.vdim - c0), g = h / (a.heads / a.groups);
     __nv_bfloat16* s_c = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [tokens][NP]
     __nv_bfloat16* s_b = s_c + kTile;                                      // [2][tokens][NP]
     __nv_bfloat16* s_x = s_b + 2 * kTile;                                  // [2][tokens][columns]
     __nv_bfloat16* s_wx = s_x + 2 * kXTile;                                // [3][tokens][columns]: terms of the weighted x
     __nv_bfloat16* s_s = s_wx + 3 * kXTile;                                // [2][NP][columns]: terms of S
     __nv_bfloat16* s_m = s_s;                                              // [2][tokens][tokens]: terms of M, later in a chunk
-    float* s_rates = reinterpret_cast<float*>(s_s + st_terms_elems<NP>());        // [ahead][5][tokens]: see `rates`; then [ahead] exp(L_63)
+    float* s_rates = reinterpret_cast<float*>(s_s + st_terms_elems<NP, COLS>());  // [ahead][5][tokens]: see `rates`; then [ahead] exp(L_63)
     const uint32_t lane = threadIdx.x & 31u, warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0);
     const uint32_t gi = lane >> 2, ti = lane & 3u;                          // row and column pair of an accumulator
-    const uint32_t mt = warp >> 2, ph = (warp & 3u) * 8u;                   // tokens 16 mt .., columns ph .. of y
-    const uint32_t st = warp >> 1, sh = (warp & 1u) * 16u;                  // state rows 16 st .., columns sh .. of S
+    const uint32_t mt = warp >> 2, ph = (warp & 3u) * (COLS / 4);           // tokens 16 mt .., columns ph .. of y
+    const uint32_t st = warp >> 1, sh = (warp & 1u) * (COLS / 2);           // state rows 16 st .., columns sh .. of S
     const float Dh = a.D[h];
     pdl_wait();
     const uint32_t T = p.batch, chunks = (T + kStTokens - 1) / kStTokens;
@@ -105,7 +110,7 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
     fetch_bx(0);
     fetch(s_c, kLd, NP, p.state_p, 0, p.c_at + g * p.state_p);
     constexpr int kTiles = NP / 16, kHalf = kStWarps / 2, kPer = (kTiles + kHalf - 1) / kHalf;
-    float S[kPer][2][4];
+    float S[kPer][kSTiles][4];
     float* state = a.S + (size_t(h) * a.vdim + c0) * p.state_p;
     const bool fresh = *a.pos == 0;
     auto element = [&](int m, int n, int e, uint32_t& row, uint32_t& col) {        // of S[m][n][e]
@@ -115,7 +120,7 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
 #pragma unroll
     for (int m = 0; m < kPer; ++m)
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
+        for (int n = 0; n < kSTiles; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 uint32_t row, col;
@@ -127,7 +132,7 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
         for (int m = 0; m < kPer; ++m) {
             if (st + kHalf * m >= uint32_t(kTiles)) continue;
 #pragma unroll
-            for (int n = 0; n < 2; ++n)
+            for (int n = 0; n < kSTiles; ++n)
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
                     uint32_t row, col, u[2];
@@ -187,27 +192,31 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
         __syncthreads();
         if (chunk + 1 < chunks) fetch_bx(chunk + 1);
         // z of this warp's outputs, requested early
-        float2 z[2];
+        float2 z[kYTiles][2];
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const uint32_t t = t0 + i0 + 8 * r, col = ph + ti * 2;
-            const float* at = a.raw + size_t(t) * a.raw_ld + h * a.vdim + c0 + col;
-            z[r] = t < T && col < cols ? make_float2(at[0], at[1]) : make_float2(0.f, 0.f);
-        }
+        for (int n = 0; n < kYTiles; ++n)
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                const uint32_t t = t0 + i0 + 8 * r, col = ph + n * 8 + ti * 2;
+                const float* at = a.raw + size_t(t) * a.raw_ld + h * a.vdim + c0 + col;
+                z[n][r] = t < T && col < cols ? make_float2(at[0], at[1]) : make_float2(0.f, 0.f);
+            }
         // C S; a term's two steps of sixteen state rows come with one ldmatrix
-        float o[2][4] = {};                                                 // a sum per term
+        float o[kYTiles][2][4] = {};                                        // a sum per term
 #pragma unroll
         for (int k = 0; k < NP / 32; ++k) {
             uint32_t ca[2][4];
 #pragma unroll
             for (int i = 0; i < 2; ++i) st_ldmatrix(ca[i], s_c + (mt * 16 + r_a) * kLd + (2 * k + i) * 16 + k_a);
 #pragma unroll
-            for (int s = 0; s < 2; ++s) {
-                uint32_t sb[4];
-                st_ldmatrix_t(sb, s_s + s * kSTile + (k * 32 + lane) * kStXLd + ph);
-                st_mma(o[s], ca[0], sb[0], sb[1]);
-                st_mma(o[s], ca[1], sb[2], sb[3]);
-            }
+            for (int s = 0; s < 2; ++s)
+#pragma unroll
+                for (int n = 0; n < kYTiles; ++n) {
+                    uint32_t sb[4];
+                    st_ldmatrix_t(sb, s_s + s * kSTile + (k * 32 + lane) * kStXLd + ph + n * 8);
+                    st_mma(o[n][s], ca[0], sb[0], sb[1]);
+                    st_mma(o[n][s], ca[1], sb[2], sb[3]);
+                }
         }
         // this warp's tile of G
         float G[2][4] = {};
@@ -244,7 +253,7 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
         }
         // terms of the weighted x
 #pragma unroll
-        for (uint32_t k4 = 0; k4 < kStTokens * kStCols / 4 / kStThreads; ++k4) {
+        for (int k4 = 0; k4 < kStTokens * COLS / 4 / kStThreads; ++k4) {
             const uint32_t i = threadIdx.x + k4 * kStThreads, t = i / (kStCols / 4), q = i % (kStCols / 4) * 4;
             const uint2 v = *reinterpret_cast<const uint2*>(x + t * kStXLd + q);
             const float w = s_w[t];
@@ -256,12 +265,13 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
         }
         __syncthreads();
         // M x
-        float y[2][4] = {};                                                 // a sum per term
+        float y[kYTiles][2][4] = {};                                        // a sum per term
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
             if (uint32_t(2 * j) > mt) continue;
-            uint32_t xb[4];
-            st_ldmatrix_t(xb, x + (j * 32 + lane) * kStXLd + ph);
+            uint32_t xb[kYTiles][4];
+#pragma unroll
+            for (int n = 0; n < kYTiles; ++n) st_ldmatrix_t(xb[n], x + (j * 32 + lane) * kStXLd + ph + n * 8);
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 if (uint32_t(2 * j + i) > mt) continue;
@@ -269,7 +279,8 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
                 for (int k = 0; k < 2; ++k) {
                     uint32_t m[4];
                     st_ldmatrix(m, s_m + k * kMTile + (mt * 16 + r_a) * kStMLd + (2 * j + i) * 16 + k_a);
-                    st_mma(y[k], m, xb[2 * i], xb[2 * i + 1]);
+#pragma unroll
+                    for (int n = 0; n < kYTiles; ++n) st_mma(y[n][k], m, xb[n][2 * i], xb[n][2 * i + 1]);
                 }
             }
         }
@@ -279,7 +290,7 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
         for (int m = 0; m < kPer; ++m) {
             if (st + kHalf * m >= uint32_t(kTiles)) continue;
 #pragma unroll
-            for (int n = 0; n < 2; ++n)
+            for (int n = 0; n < kSTiles; ++n)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) S[m][n][e] *= total;
 #pragma unroll
@@ -287,25 +298,29 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
                 uint32_t ba[4];
                 st_ldmatrix_t(ba, b + (k * 16 + r_b) * kLd + (st + kHalf * m) * 16 + k_b);
 #pragma unroll
-                for (int s = 0; s < 3; ++s) {
-                    uint32_t xb[4];
-                    st_ldmatrix_t(xb, s_wx + s * kXTile + (k * 16 + r_a) * kStXLd + sh + k_a);
-                    st_mma(S[m][0], ba, xb[0], xb[1]);
-                    st_mma(S[m][1], ba, xb[2], xb[3]);
-                }
+                for (int s = 0; s < 3; ++s)
+#pragma unroll
+                    for (int n = 0; n < kSTiles / 2; ++n) {
+                        uint32_t xb[4];
+                        st_ldmatrix_t(xb, s_wx + s * kXTile + (k * 16 + r_a) * kStXLd + sh + n * 16 + k_a);
+                        st_mma(S[m][2 * n], ba, xb[0], xb[1]);
+                        st_mma(S[m][2 * n + 1], ba, xb[2], xb[3]);
+                    }
             }
         }
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const uint32_t t = t0 + i0 + 8 * r, col = ph + ti * 2;
-            const uint32_t v = *reinterpret_cast<const uint32_t*>(x + (i0 + 8 * r) * kStXLd + col);
-            const float el = s_el[i0 + 8 * r];
-            const float y0 = fmaf(Dh, __uint_as_float(v << 16), fmaf(el, o[0][2 * r] + o[1][2 * r], y[0][2 * r] + y[1][2 * r]));
-            const float y1 = fmaf(Dh, __uint_as_float(v & 0xffff0000u), fmaf(el, o[0][2 * r + 1] + o[1][2 * r + 1], y[0][2 * r + 1] + y[1][2 * r + 1]));
-            float* out = p.gated + size_t(t) * p.inner + h * a.vdim + c0 + col;
-            if (t < T && col < cols)                                        // (cols is even)
-                *reinterpret_cast<float2*>(out) = make_float2(y0 * silu_fast(z[r].x), y1 * silu_fast(z[r].y));
-        }
+        for (int n = 0; n < kYTiles; ++n)
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                const uint32_t t = t0 + i0 + 8 * r, col = ph + n * 8 + ti * 2;
+                const uint32_t v = *reinterpret_cast<const uint32_t*>(x + (i0 + 8 * r) * kStXLd + col);
+                const float el = s_el[i0 + 8 * r];
+                const float y0 = fmaf(Dh, __uint_as_float(v << 16), fmaf(el, o[n][0][2 * r] + o[n][1][2 * r], y[n][0][2 * r] + y[n][1][2 * r]));
+                const float y1 = fmaf(Dh, __uint_as_float(v & 0xffff0000u), fmaf(el, o[n][0][2 * r + 1] + o[n][1][2 * r + 1], y[n][0][2 * r + 1] + y[n][1][2 * r + 1]));
+                float* out = p.gated + size_t(t) * p.inner + h * a.vdim + c0 + col;
+                if (t < T && col < cols)                                    // (cols is even)
+                    *reinterpret_cast<float2*>(out) = make_float2(y0 * silu_fast(z[n][r].x), y1 * silu_fast(z[n][r].y));
+            }
         if (chunk + 1 == chunks) break;
         __syncthreads();                                                    // the terms of M have been read
         spread();
@@ -313,7 +328,7 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
 #pragma unroll
     for (int m = 0; m < kPer; ++m)
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
+        for (int n = 0; n < kSTiles; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 uint32_t row, col;
@@ -324,13 +339,21 @@ __global__ void __launch_bounds__(kStThreads, 1) ssm_tc_kernel(const SsmParams p
 
 bool ssm_tc_supported(const lv_ssm_args& a) { return a.vdim % 8 == 0 && a.state <= kSsMaxState; }
 
+template <int NP, int COLS>
+static int ssm_tc_launch_sized(lv_ctx* ctx, const SsmParams& p) {
+    constexpr size_t smem = st_smem_bytes<NP, COLS>();
+    LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "ssm: state needs too much shared memory");
+    LV_CUDA(cudaFuncSetAttribute(ssm_tc_kernel<NP, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    LV_CUDA(launch_pdl(ctx, ssm_tc_kernel<NP, COLS>, dim3(p.a.heads * ((p.a.vdim + COLS - 1) / COLS)), dim3(kStThreads), smem, p));
+    return LV_OK;
+}
+
 template <int NP>
 static int ssm_tc_launch_rows(lv_ctx* ctx, const SsmParams& p) {
-    constexpr size_t smem = st_smem_bytes<NP>();
-    LV_REQUIRE(smem <= size_t(ctx->max_smem_optin), "ssm: state needs too much shared memory");
-    LV_CUDA(cudaFuncSetAttribute(ssm_tc_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-    LV_CUDA(launch_pdl(ctx, ssm_tc_kernel<NP>, dim3(p.a.heads * ((p.a.vdim + kStCols - 1) / kStCols)), dim3(kStThreads), smem, p));
-    return LV_OK;
+    // narrow CTAs while all of them run at a time
+    if constexpr (NP <= 128)
+        if (p.a.vdim > 32 && p.a.heads * ((p.a.vdim + 31) / 32) > uint32_t(ctx->sm_count)) return ssm_tc_launch_sized<NP, 64>(ctx, p);
+    return ssm_tc_launch_sized<NP, 32>(ctx, p);
 }
 
 int ssm_tc_launch(lv_ctx* ctx, const SsmParams& p) {

@@ -362,7 +362,7 @@ TENSOR = 2
 
 
 @pytest.mark.parametrize("H,P,N,G,taps,parts", [(4, 32, 16, 4, 5, 1), (3, 40, 130, 1, 2, 1), (8, 64, 128, 2, 4, 8), (6, 8, 11, 3, 7, 3), (2, 304, 8, 1, 1, 2), (10, 16, 64, 5, 16, 5),
-                                                (1, 24, 256, 1, 4, 1), (5, 48, 33, 1, 3, 1)])
+                                                (1, 24, 256, 1, 4, 1), (5, 48, 33, 1, 3, 1), (80, 64, 16, 2, 2, 4), (76, 40, 72, 1, 3, 1)])
 @pytest.mark.parametrize("cuts", [[140], [33, 2, 31, 64, 3, 2], [2] * 20, [64, 64, 65], [63, 700]])
 def test_chunks_of_tokens_as_matrix_products(gpu, H, P, N, G, taps, parts, cuts):
     """Everything but x, B and C is as exact as in f32."""
