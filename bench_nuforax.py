@@ -40,7 +40,7 @@ def config(z):
             m["kv_from"] = i - 1
         layers.append({"type": "latent_attention", "mlp": mlp, "mixer": m})
     return {"architecture": "Nuforax", "width": z["width"], "vocab": VOCAB, "layers": layers, "norm": {"eps": 1e-5},
-            "embedding": {"scale": z["width"] ** 0.5, "bigram": {"buckets": 20011, "mul_prev": 127, "mul_cur": 7}}}
+            "embedding": {"scale": z["width"] ** 0.5, "bigram": {"buckets": 20011, "mul_prev": 41, "mul_cur": 13}}}
 
 
 def tensor_shapes(cfg):
@@ -104,7 +104,7 @@ def kernel_times(pkg, torch, z, peaks):
             a = pkg.NormConvArgs(pos=pos.value, eps=1e-5, mult=1.0, x_out=xb.value, out=out.value, out_type=pkg.TYPE_F32 if n == 1 else pkg.TYPE_BF16, out_ld=W, width=W, batch=n, plain_w=1)
             if first:
                 a.embed, a.embed_ld, a.vocab, a.token_log, a.embed_scale, a.pos = d.value, W, VOCAB, ids.value, 3.0, pos_prompt.value
-                a.pair_embed, a.pair_ld, a.pair_buckets, a.pair_mul_prev, a.pair_mul_cur = d.value, W, 20011, 127, 7
+                a.pair_embed, a.pair_ld, a.pair_buckets, a.pair_mul_prev, a.pair_mul_cur = d.value, W, 20011, 41, 13
             else:
                 a.x, a.y, a.y_rows, a.post_w = xa.value, y.value, 1, vec.value
             return C.byref(a)

@@ -26,7 +26,7 @@ def mamba2(heads, vdim, state, groups, conv, norm_groups, ff=None):
             "mlp": {"kind": "dense", "ff": ff} if ff else None}
 
 
-def config(width, vocab, layers, buckets=97, mul_prev=31, mul_cur=7, spread=2.0, eps=1e-5):
+def config(width, vocab, layers, buckets=97, mul_prev=31, mul_cur=11, spread=2.0, eps=1e-5):
     """spread: of the logits, roughly"""
     scale = round(width ** 0.5 / spread, 3)
     return {"architecture": "Nuforax", "width": width, "vocab": vocab, "layers": layers, "norm": {"eps": eps},

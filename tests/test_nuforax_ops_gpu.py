@@ -19,7 +19,7 @@ def nans(d, nbytes):
 
 # ---- embedding and norms ---------------------------------------------------------------------
 
-@pytest.mark.parametrize("width,buckets,mul_prev,mul_cur,cuts", [(64, 97, 31, 7, [9]), (72, 5, 4000000007, 4294967295, [1] * 6), (76, 1, 0, 3, [2, 1, 4]),
+@pytest.mark.parametrize("width,buckets,mul_prev,mul_cur,cuts", [(64, 97, 31, 11, [9]), (72, 5, 4000000007, 4294967295, [1] * 6), (76, 1, 0, 3, [2, 1, 4]),
                                                                  (2056, 1000, 1, 1, [3, 3]), (30, 12, 5, 0, [1, 5])])
 def test_pairs_of_tokens_and_norms_behind_sublayers(gpu, width, buckets, mul_prev, mul_cur, cuts):
     rng = np.random.default_rng(width)
@@ -88,7 +88,7 @@ def test_products_of_the_rows_in_a_window(gpu, window, pos, batch):
 
 @pytest.mark.parametrize("pos,batch", [(0, 1), (0, 70), (1000003, 3)])
 def test_rotary_table(gpu, pos, batch):
-    parts = [npl.yarn(16, 1e6, {"factor": 3.0, "original": 100, "fast": 16.0, "slow": 1.0}), npl.yarn(6, 500.0)]
+    parts = [npl.yarn(16, 2e5, {"factor": 3.0, "original": 100, "fast": 16.0, "slow": 1.0}), npl.yarn(6, 500.0)]
     freqs, mults = np.concatenate([p[0] for p in parts]), np.concatenate([np.full(len(p[0]), p[1]) for p in parts]).astype(np.float32)
     with Dev(gpu) as d:
         out = d.zeros(batch * len(freqs) * 8)
